@@ -64,7 +64,7 @@ __device__ __forceinline__ float block_sum_256(float v, float* red) {
     return tot;
 }
 
-// grid (T, 2): y == 0 the query latent, y == 1 the key / value row
+// grid (T, 2): y == 0 the query latent, y == 1 the key / value row; grid (T, 1) without a query latent
 template <typename KT>
 __global__ void __launch_bounds__(256) latent_prep_kernel(float* __restrict__ cq, int q_rank, const float* __restrict__ q_gain, const float* __restrict__ dkv,
                                                           int kv_rank, int rot_dim, const float* __restrict__ kv_gain, float eps, KT* __restrict__ cache,
@@ -73,7 +73,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(float* __restrict__ cq
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
-    if (blockIdx.y == 0) {
+    if (cq && blockIdx.y == 0) {
         float* r = cq + (size_t)t * q_rank;
         float ss = 0.f;
         for (int i = threadIdx.x; i < q_rank; i += 256) ss = fmaf(r[i], r[i], ss);
@@ -261,7 +261,7 @@ template <> struct RowVec<__nv_bfloat16> {
 // part [tokens, slices, heads, vdim + 2].  dim, row multiples of RowVec::N; vdim even.
 template <typename KT>
 __global__ void __launch_bounds__(256) latent_shared_attn_kernel(float* __restrict__ part, const float* __restrict__ Q, const KT* __restrict__ rows,
-                                                                 const int* __restrict__ pos_dev, int p0, int heads, int dim, int vdim, int row, float scale) {
+                                                                 const int* __restrict__ pos_dev, int p0, int heads, int dim, int vdim, int row, float scale, int window) {
     constexpr int VN = RowVec<KT>::N;
     extern __shared__ __align__(16) unsigned char ls_raw[];
     float* qs = reinterpret_cast<float*>(ls_raw);                              // [heads][dim]
@@ -273,6 +273,7 @@ __global__ void __launch_bounds__(256) latent_shared_attn_kernel(float* __restri
     const int t = blockIdx.x, slice = blockIdx.y, n_slices = gridDim.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, key = lane & 15, half = lane >> 4;
     const int n_keys = (pos_dev ? *pos_dev : p0) + t + 1;
+    const int lo = window > 0 ? max(0, n_keys - window) : 0;      // the visible rows are lo .. n_keys - 1
     const float* q = Q + (size_t)t * heads * dim;
     for (int e = threadIdx.x * 4; e < heads * dim; e += 1024) *reinterpret_cast<float4*>(qs + e) = *reinterpret_cast<const float4*>(q + e);
     float m[LS_HB], l[LS_HB], acc[LS_HB][LS_CC][2];
@@ -283,7 +284,7 @@ __global__ void __launch_bounds__(256) latent_shared_attn_kernel(float* __restri
         for (int c = 0; c < LS_CC; c++) acc[i][c][0] = acc[i][c][1] = 0.f;
     }
     const int n_chunks = dim / VN;
-    for (int k0 = slice * LS_KEYS; k0 < n_keys; k0 += n_slices * LS_KEYS) {
+    for (int k0 = lo + slice * LS_KEYS; k0 < n_keys; k0 += n_slices * LS_KEYS) {
         __syncthreads();                                   // the previous tile is consumed (first pass: qs is written)
         for (int e = threadIdx.x; e < LS_KEYS * n_chunks; e += 256) {
             const int r = e / n_chunks, c = e - r * n_chunks;
@@ -400,25 +401,25 @@ __global__ void __launch_bounds__(256) latent_shared_merge_kernel(float* __restr
 }  // namespace
 
 void latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache,
-                 DType cache_dt, int rot_dims, bool interleaved, float rot_base, int T, const int* pos_dev, int p0, cudaStream_t s) {
+                 DType cache_dt, int rot_dims, bool interleaved, double rot_base, int T, const int* pos_dev, int p0, cudaStream_t s) {
     if (T <= 0) return;
     NT_CHECK(cache_dt == DType::F32 || cache_dt == DType::BF16, "latent_prep: F32 or BF16 cache");
-    const double l2b = std::log2((double)rot_base);
+    const double l2b = std::log2(rot_base);
     if (cache_dt == DType::F32)
-        launch_k(latent_prep_kernel<float>, dim3(T, 2), dim3(256), 0, s, cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps, static_cast<float*>(cache),
+        launch_k(latent_prep_kernel<float>, dim3(T, cq ? 2 : 1), dim3(256), 0, s, cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps, static_cast<float*>(cache),
                  rot_dims, interleaved ? 1 : 0, l2b, pos_dev, p0);
     else
-        launch_k(latent_prep_kernel<__nv_bfloat16>, dim3(T, 2), dim3(256), 0, s, cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps,
+        launch_k(latent_prep_kernel<__nv_bfloat16>, dim3(T, cq ? 2 : 1), dim3(256), 0, s, cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps,
                  static_cast<__nv_bfloat16*>(cache), rot_dims, interleaved ? 1 : 0, l2b, pos_dev, p0);
     count_launch();
 }
 
 void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, int rot_dims,
-                     bool interleaved, float rot_base, const int* pos_dev, int p0, cudaStream_t s) {
+                     bool interleaved, double rot_base, const int* pos_dev, int p0, cudaStream_t s) {
     if (T <= 0) return;
     const size_t smem = sizeof(float) * (LT * (size_t)(dim + rot_dim) + 4 * 64 * LT);
     NT_CHECK(smem <= 48 * 1024, "latent_q_absorb: query heads wider than 1280 are not covered");
-    const double l2b = std::log2((double)rot_base);
+    const double l2b = std::log2(rot_base);
     const dim3 grid((T + LT - 1) / LT, heads, (kv_rank + 63) / 64);
 #define NT_QA(TY) launch_k(latent_q_absorb_kernel<TY>, grid, dim3(256), smem, s, qa, q, static_cast<const TY*>(W_uk), T, heads, dim, rot_dim, kv_rank, rot_dims, \
                            interleaved ? 1 : 0, l2b, pos_dev, p0)
@@ -458,10 +459,10 @@ void latent_expand_pack(void* kfull, void* vfull, const float* ku, const float* 
     count_launch();
 }
 
-void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, int rot_dims, bool interleaved, float rot_base, int p0,
+void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, int rot_dims, bool interleaved, double rot_base, int p0,
                       cudaStream_t s) {
     if (T <= 0) return;
-    launch_k(latent_q_rot_pad_kernel, dim3(T, heads), dim3(256), 0, s, qp, q, heads, dim, rot_dim, kw, rot_dims, interleaved ? 1 : 0, std::log2((double)rot_base), p0);
+    launch_k(latent_q_rot_pad_kernel, dim3(T, heads), dim3(256), 0, s, qp, q, heads, dim, rot_dim, kw, rot_dims, interleaved ? 1 : 0, std::log2(rot_base), p0);
     count_launch();
 }
 
@@ -483,7 +484,8 @@ bool attention_shared_rows_supported(int heads, int dim, int vdim, int row, DTyp
     return heads >= 1 && heads <= 8 * LS_HB && dim % vn == 0 && row % vn == 0 && dim <= row && vdim <= row && vdim % 2 == 0 && vdim <= 64 * LS_CC &&
            (reinterpret_cast<uintptr_t>(cache) & 15) == 0 && smem <= 200 * 1024;
 }
-int attention_shared_rows_slices(int tokens, int max_seq) {
+int attention_shared_rows_slices(int tokens, int max_seq, int window) {
+    if (window > 0) max_seq = std::min(max_seq, window);
     return std::max(1, std::min({(max_seq + LS_KEYS - 1) / LS_KEYS, LS_MAX_PARTS / std::max(1, tokens), 128}));      // one query: up to 128 CTAs
 }
 size_t attention_shared_rows_scratch_floats(int heads, int vdim) { return (size_t)LS_MAX_PARTS * heads * ((size_t)vdim + 2); }
@@ -491,7 +493,7 @@ size_t attention_shared_rows_scratch_floats(int heads, int vdim) { return (size_
 // out [tokens, heads, vdim]; Q [tokens, heads, dim]; scratch >= attention_shared_rows_scratch_floats.  The grid depends on tokens and
 // max_seq only, never on the position: the captured decode step replays it unchanged.
 void attention_shared_rows(float* out, const float* Q, const void* cache, DType cache_dt, int tokens, const int* pos_dev, int p0, int max_seq, int heads, int dim,
-                           int vdim, int row, float scale, float* scratch, cudaStream_t s) {
+                           int vdim, int row, float scale, float* scratch, cudaStream_t s, int window) {
     if (tokens <= 0) return;
     NT_CHECK(attention_shared_rows_supported(heads, dim, vdim, row, cache_dt, cache), "attention_shared_rows: shape not covered");
     const bool f32 = cache_dt == DType::F32;
@@ -499,16 +501,16 @@ void attention_shared_rows(float* out, const float* Q, const void* cache, DType 
     const size_t smem = sizeof(float) * ((size_t)heads * dim + (size_t)heads * LS_KEYS) + (size_t)LS_KEYS * (dim + vn) * (f32 ? 4 : 2);
     for (int t0 = 0; t0 < tokens; t0 += LS_MAX_PARTS) {           // long portions (exact mode): blocks of queries with one slice each
         const int nt = std::min(LS_MAX_PARTS, tokens - t0);
-        const int slices = attention_shared_rows_slices(nt, max_seq);
+        const int slices = attention_shared_rows_slices(nt, max_seq, window);
         static unsigned long long cfg_f = 0, cfg_b = 0;
         if (f32) {
             opt_in_dynamic_smem(latent_shared_attn_kernel<float>, 200 * 1024, cfg_f);
             launch_k(latent_shared_attn_kernel<float>, dim3(nt, slices), dim3(256), smem, s, scratch, Q + (size_t)t0 * heads * dim, static_cast<const float*>(cache), pos_dev,
-                     p0 + t0, heads, dim, vdim, row, scale);
+                     p0 + t0, heads, dim, vdim, row, scale, window);
         } else {
             opt_in_dynamic_smem(latent_shared_attn_kernel<__nv_bfloat16>, 200 * 1024, cfg_b);
             launch_k(latent_shared_attn_kernel<__nv_bfloat16>, dim3(nt, slices), dim3(256), smem, s, scratch, Q + (size_t)t0 * heads * dim,
-                     static_cast<const __nv_bfloat16*>(cache), pos_dev, p0 + t0, heads, dim, vdim, row, scale);
+                     static_cast<const __nv_bfloat16*>(cache), pos_dev, p0 + t0, heads, dim, vdim, row, scale, window);
         }
         count_launch();
         launch_k(latent_shared_merge_kernel, dim3(nt, heads, (vdim + 63) / 64), dim3(256), sizeof(float) * slices, s, out + (size_t)t0 * heads * vdim, (const float*)scratch, slices, heads, vdim);

@@ -265,7 +265,7 @@ void attention_window_mma(float* out, const float* Q, const void* kc, const void
 }
 
 // Per-head 16-bit operands built for the call (latent attention's expanded keys / values): key width 64, 128 or 192, value width 64
-// or 128, every head its own key / value head, full causal mask.
+// or 128, every head its own key / value head, causal or windowed mask.
 bool attention_heads_mma_widths(int key_dim, int value_dim, int* kw, int* vw) {
     if (key_dim <= 0 || value_dim <= 0 || key_dim > 192 || value_dim > 128) return false;
     *kw = key_dim <= 64 ? 64 : key_dim <= 128 ? 128 : 192;
@@ -273,10 +273,10 @@ bool attention_heads_mma_widths(int key_dim, int value_dim, int* kw, int* vw) {
     return true;
 }
 void attention_heads_mma(float* out, const float* Q, const void* kc, const void* vc, int tokens, int p0, int rows, int heads, int kw, int vw, float scale,
-                         cudaStream_t s) {
+                         cudaStream_t s, int window) {
     const __half* k = static_cast<const __half*>(kc);
     const __half* v = static_cast<const __half*>(vc);
-#define NT_AH(D, V) launch<D, V, true>(out, Q, k, v, tokens, p0, heads, heads, rows, scale, 0, 0, 0.f, s)
+#define NT_AH(D, V) launch<D, V, true>(out, Q, k, v, tokens, p0, heads, heads, rows, scale, window, 0, 0.f, s)
     if (kw == 64 && vw == 64) NT_AH(64, 64);
     else if (kw == 64 && vw == 128) NT_AH(64, 128);
     else if (kw == 128 && vw == 64) NT_AH(128, 64);

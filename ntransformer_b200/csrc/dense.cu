@@ -4,10 +4,14 @@
 //   gemv_dense   decode: up to 3 matrices share one activation vector staged once per CTA in shared memory; a warp streams one
 //                output row with 16-byte loads; the prologue can RMS-normalise the staged vector; epilogues fuse the residual (+ per-channel gain) and the gated activations, so a
 //                decode step needs no separate add / scale / activation launch.
+//   gemv_multi   decode: several matrices with an input vector each (and an activation on their rows) in one launch
+//   gemv_sum     decode: y (+)= the sum of several matrix-vector products with inputs of their own, routed experts among them: the last
+//                products of a block whose mixer and feed-forward join the residual together
 //   gemm_dense   prompt tokens on CUDA cores: 64x64x16 tiles, 4x4 outputs per thread, true FP32 FMA.  It serves the exact
 //                32-bit mode and shapes the tcgen05 tiles of prefill_gemm.cu do not cover (rows % 128, cols % 64).
 // This file is compiled WITHOUT --use_fast_math (tanh / exp / division at full precision): the 32-bit mode depends on it.
 #include "kernels_internal.h"
+#include "bf16_split.cuh"
 #include "ring.cuh"
 #include <cuda_bf16.h>
 #include <cuda_fp16.h>
@@ -21,6 +25,9 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+// z > 0: a z^2 + z / 2;  z <= 0: (1/2 + b)(e^z - 1 - z) + z / 2   (a, b: softplus of the layer's two numbers)
+__device__ __forceinline__ float xielu_f(float z, float a, float b) { return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(0.5f + b, expm1f(z) - z, 0.5f * z); }
 
 template <typename T> struct Elem;
 template <> struct Elem<float> {
@@ -82,9 +89,9 @@ struct DenseMats {
 
 constexpr int DV_WARPS = 8;
 
-// <row, xs> for one row; vec: row base and pitch 16-byte aligned and K a multiple of PER16
+// <row, xs> for one row, this lane's share; vec: row base and pitch 16-byte aligned and K a multiple of PER16
 template <typename T>
-__device__ __forceinline__ float dense_row_dot(const unsigned char* row, const float* xs, int K, int lane, bool vec) {
+__device__ __forceinline__ float dense_row_part(const unsigned char* row, const float* xs, int K, int lane, bool vec) {
     float acc = 0.f;
     constexpr int P = Elem<T>::PER16;
     if (vec) {
@@ -113,17 +120,25 @@ __device__ __forceinline__ float dense_row_dot(const unsigned char* row, const f
     } else {
         for (int i = lane; i < K; i += 32) acc = fmaf(Elem<T>::one(row, i), xs[i], acc);
     }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xFFFFFFFFu, acc, o);
     return acc;
+}
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+    return v;
+}
+template <typename T>
+__device__ __forceinline__ float dense_row_dot(const unsigned char* row, const float* xs, int K, int lane, bool vec) {
+    return warp_sum(dense_row_part<T>(row, xs, K, lane, vec));
 }
 
 template <typename T>
 __global__ void __launch_bounds__(DV_WARPS * 32) gemv_dense_kernel(DenseMats m, const float* __restrict__ x, int K, int ep,
                                                                    const float* __restrict__ row_scale, float alpha, int vec,
-                                                                   const float* __restrict__ norm_w, float eps, StreamsIO sio) {
+                                                                   const float* __restrict__ norm_w, float eps, StreamsIO sio, int norm_groups) {
     extern __shared__ __align__(16) float xs[];
     __shared__ float red[DV_WARPS];
+    __shared__ float inv_g[DENSE_MAX_NORM_GROUPS];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_launch_dependents();
     pdl_wait();
@@ -136,7 +151,18 @@ __global__ void __launch_bounds__(DV_WARPS * 32) gemv_dense_kernel(DenseMats m, 
         } else v = x[i];
         xs[i] = v; ss = fmaf(v, v, ss);
     }
-    if (norm_w) {
+    if (norm_w && norm_groups > 1) {        // every run of K / norm_groups channels has its own root mean square: a warp per run
+        __syncthreads();
+        const int per = K / norm_groups;
+        for (int g = warp; g < norm_groups; g += DV_WARPS) {
+            float s2 = 0.f;
+            for (int i = lane; i < per; i += 32) { const float v = xs[g * per + i]; s2 = fmaf(v, v, s2); }
+            s2 = warp_sum(s2);
+            if (lane == 0) inv_g[g] = 1.0f / sqrtf(s2 / (float)per + eps);
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < K; i += DV_WARPS * 32) xs[i] = xs[i] * inv_g[i / per] * norm_w[i];
+    } else if (norm_w) {
         // RMS norm of the staged vector: every CTA sums the squares in the same order, so all CTAs (and every launch that reads the
         // same x) derive the bit-identical normalised vector
 #pragma unroll
@@ -171,6 +197,86 @@ __global__ void __launch_bounds__(DV_WARPS * 32) gemv_dense_kernel(DenseMats m, 
             else *y = v;
         }
     }
+}
+
+// ---- several matrices, each with its own input vector ----
+struct MultiDev {
+    struct One { const unsigned char* W; size_t pitch; const float* x; float* y; const float* act_p; int out, K, act, f32, vec, cta_end; };
+    One m[DENSE_MAX_MATS];
+    int n;
+};
+// A CTA serves rows of one matrix: it stages that matrix's input, then a warp per row.
+template <typename T>
+__global__ void __launch_bounds__(DV_WARPS * 32) gemv_multi_kernel(const __grid_constant__ MultiDev md) {
+    extern __shared__ __align__(16) float xs[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    int mi = 0, first = 0;
+    while (mi + 1 < md.n && (int)blockIdx.x >= md.m[mi].cta_end) { first = md.m[mi].cta_end; mi++; }
+    const MultiDev::One& m = md.m[mi];
+    const int ctas = m.cta_end - first, r0 = ((int)blockIdx.x - first) * DV_WARPS + warp;
+    pdl_launch_dependents();
+    pdl_wait();
+    for (int i = threadIdx.x; i < m.K; i += DV_WARPS * 32) xs[i] = m.x[i];
+    __syncthreads();
+    float a = 0.f, b = 0.f;
+    if (m.act == GEMV_ACT_XIELU) { a = softplus_f(m.act_p[0]); b = softplus_f(m.act_p[1]); }
+    for (int r = r0; r < m.out; r += ctas * DV_WARPS) {
+        const unsigned char* row = m.W + (size_t)r * m.pitch;
+        float v = m.f32 ? dense_row_dot<float>(row, xs, m.K, lane, m.vec) : dense_row_dot<T>(row, xs, m.K, lane, m.vec);
+        if (lane == 0) {
+            if (m.act == GEMV_ACT_TANH) v = tanhf(v);
+            else if (m.act == GEMV_ACT_XIELU) v = xielu_f(v, a, b);
+            m.y[r] = v;
+        }
+    }
+}
+
+// ---- y[r] (+)= sum over terms of <W[r], x> (routed term: sum_k wt[k] <table[sel[k]][r], x_k>) ----
+struct SumDev {
+    struct One { const unsigned char* W; const void* const* table; const int* sel; const float* wt; const float* x; int K, top, vec, at; };
+    One t[GEMV_SUM_MAX_TERMS];
+    int n, out, add;
+    float* y;
+};
+template <typename T>
+__global__ void __launch_bounds__(DV_WARPS * 32) gemv_sum_kernel(const __grid_constant__ SumDev sd) {
+    extern __shared__ __align__(16) float xs[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    pdl_launch_dependents();
+    pdl_wait();
+    for (int q = 0; q < sd.n; q++) {
+        const int total = sd.t[q].K * max(1, sd.t[q].top);
+        for (int i = threadIdx.x; i < total; i += DV_WARPS * 32) xs[sd.t[q].at + i] = sd.t[q].x[i];
+    }
+    __syncthreads();
+    for (int r = blockIdx.x * DV_WARPS + warp; r < sd.out; r += gridDim.x * DV_WARPS) {
+        float acc = 0.f;
+        for (int q = 0; q < sd.n; q++) {
+            const SumDev::One& t = sd.t[q];
+            const size_t off = (size_t)r * t.K * sizeof(T);
+            if (!t.table) acc += dense_row_part<T>(t.W + off, xs + t.at, t.K, lane, t.vec);
+            else for (int k = 0; k < t.top; k++)
+                acc = fmaf(t.wt[k], dense_row_part<T>(static_cast<const unsigned char*>(t.table[t.sel[k]]) + off, xs + t.at + k * t.K, t.K, lane, t.vec), acc);
+        }
+        acc = warp_sum(acc);
+        if (lane == 0) sd.y[r] = sd.add ? sd.y[r] + acc : acc;
+    }
+}
+
+template <bool VEC>
+__global__ void __launch_bounds__(256) xielu_kernel(float* __restrict__ out, __nv_bfloat16* __restrict__ hi, size_t lo, const float* __restrict__ in, const float* __restrict__ act_p, size_t n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    constexpr int V = VEC ? 4 : 1;
+    const size_t i = ((size_t)blockIdx.x * 256 + threadIdx.x) * V;
+    if (i >= n) return;
+    const float a = softplus_f(act_p[0]), b = softplus_f(act_p[1]);
+    float v[V];
+    if constexpr (VEC) { const float4 f = *reinterpret_cast<const float4*>(in + i); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; } else v[0] = in[i];
+#pragma unroll
+    for (int e = 0; e < V; e++) v[e] = xielu_f(v[e], a, b);
+    if (out) { if constexpr (VEC) *reinterpret_cast<float4*>(out + i) = make_float4(v[0], v[1], v[2], v[3]); else out[i] = v[0]; }
+    if (hi) { if constexpr (VEC) split_store4(hi, hi + lo, i, v); else split_store1(hi, hi + lo, i, v[0]); }
 }
 
 // ---- C[T,N] (ep)= A[T,K] . W[N,K]^T on CUDA cores ----
@@ -243,7 +349,8 @@ __global__ void to_f32_kernel(float* __restrict__ out, const T* __restrict__ in,
 bool dense_dtype(DType dt) { return dt == DType::F32 || dt == DType::F16 || dt == DType::BF16; }
 
 void gemv_dense(const GemvMat* mats, int n_mat, int K, const float* x, DenseEpilogue ep, const float* row_scale, float alpha, cudaStream_t s,
-                const float* norm_w, float eps, const StreamsIO* sio_p) {
+                const float* norm_w, float eps, const StreamsIO* sio_p, int norm_groups) {
+    NT_CHECK(norm_groups >= 1 && norm_groups <= DENSE_MAX_NORM_GROUPS && K % norm_groups == 0, "gemv_dense: norm groups must be equal parts, at most 256");
     NT_CHECK(n_mat >= 1 && n_mat <= DENSE_MAX_MATS, "gemv_dense: too many matrices for one launch");
     const StreamsIO sio = sio_p ? *sio_p : StreamsIO();
     NT_CHECK(ep != DENSE_STREAMS || (n_mat == 1 && sio.X_out && sio.M && sio.b && sio.S >= 1 && sio.S <= 16), "gemv_dense: the streams epilogue takes one matrix and the stream tables");
@@ -271,9 +378,82 @@ void gemv_dense(const GemvMat* mats, int n_mat, int K, const float* x, DenseEpil
     const int resident = (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)(220 * 1024) / (smem + 1024))) * 148;
     grid = std::min(grid, resident);
 #define NT_DV(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(gemv_dense_kernel<TY>, 200 * 1024, done); \
-                    launch_k(gemv_dense_kernel<TY>, dim3(grid), dim3(DV_WARPS * 32), smem, s, m, x, K, (int)ep, row_scale, alpha, vec, norm_w, eps, sio); }
+                    launch_k(gemv_dense_kernel<TY>, dim3(grid), dim3(DV_WARPS * 32), smem, s, m, x, K, (int)ep, row_scale, alpha, vec, norm_w, eps, sio, norm_groups); }
     if (dt == DType::F32) NT_DV(float) else if (dt == DType::F16) NT_DV(__half) else NT_DV(__nv_bfloat16)
 #undef NT_DV
+    count_launch();
+}
+
+void gemv_multi(const MultiMat* mats, int n_mat, cudaStream_t s) {
+    NT_CHECK(n_mat >= 1 && n_mat <= DENSE_MAX_MATS, "gemv_multi: too many matrices for one launch");
+    MultiDev md{};
+    md.n = n_mat;
+    DType dt = DType::F32;
+    for (int i = 0; i < n_mat; i++) if (mats[i].dtype != DType::F32) dt = mats[i].dtype;
+    size_t bytes[DENSE_MAX_MATS], total = 0;
+    int K = 0, rows = 0;
+    for (int i = 0; i < n_mat; i++) {
+        const MultiMat& a = mats[i];
+        NT_CHECK(dense_dtype(a.dtype) && (a.dtype == dt || a.dtype == DType::F32), "gemv_multi: one 16-bit dtype per launch (beside F32 tables)");
+        NT_CHECK(a.act != GEMV_ACT_XIELU || a.act_p, "gemv_multi: the activation's two numbers are missing");
+        MultiDev::One& o = md.m[i];
+        o.W = static_cast<const unsigned char*>(a.W); o.pitch = a.row_pitch ? a.row_pitch : dtype_row_size(a.dtype, (size_t)a.K);
+        o.x = a.x; o.y = a.y; o.act_p = a.act_p; o.out = a.out; o.K = a.K; o.act = a.act; o.f32 = a.dtype == DType::F32 ? 1 : 0;
+        o.vec = a.K % (o.f32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(a.W) & 15) == 0 && (o.pitch & 15) == 0;
+        bytes[i] = (size_t)a.out * o.pitch; total += bytes[i];
+        K = std::max(K, a.K); rows += a.out;
+    }
+    if (rows <= 0) return;
+    const size_t smem = (size_t)K * sizeof(float);
+    NT_CHECK(smem <= 200 * 1024, "gemv_multi: the activation vector does not fit in shared memory");
+    // CTAs by share of the bytes, no more than resident at once: a warp's rows follow each other without a second wave
+    const int resident = (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)(220 * 1024) / (smem + 1024))) * 148;
+    int end = 0;
+    for (int i = 0; i < n_mat; i++) {
+        const int full = (mats[i].out + DV_WARPS - 1) / DV_WARPS;
+        const int share = (int)((double)resident * (double)bytes[i] / (double)std::max<size_t>(1, total));
+        end += std::max(1, std::min(full, share));
+        md.m[i].cta_end = end;
+    }
+#define NT_MV(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(gemv_multi_kernel<TY>, 200 * 1024, done); \
+                    launch_k(gemv_multi_kernel<TY>, dim3(end), dim3(DV_WARPS * 32), smem, s, md); }
+    if (dt == DType::F32) NT_MV(float) else if (dt == DType::F16) NT_MV(__half) else NT_MV(__nv_bfloat16)
+#undef NT_MV
+    count_launch();
+}
+
+void gemv_sum(float* y, const SumTerm* terms, int n, int out, DType dt, bool add, cudaStream_t s) {
+    NT_CHECK(n >= 1 && n <= GEMV_SUM_MAX_TERMS && dense_dtype(dt), "gemv_sum: 1..4 terms of a dense dtype");
+    if (out <= 0) return;
+    SumDev sd{};
+    sd.n = n; sd.out = out; sd.add = add ? 1 : 0; sd.y = y;
+    int at = 0;
+    for (int i = 0; i < n; i++) {
+        const SumTerm& t = terms[i];
+        SumDev::One& o = sd.t[i];
+        o.W = static_cast<const unsigned char*>(t.W); o.table = t.table; o.sel = t.sel; o.wt = t.wt; o.x = t.x; o.K = t.K; o.top = t.table ? t.top : 1; o.at = at;
+        o.vec = t.K % (dt == DType::F32 ? 4 : 8) == 0 && (t.table ? t.table_aligned : (reinterpret_cast<uintptr_t>(t.W) & 15) == 0);
+        at += (t.K * o.top + 3) & ~3;
+    }
+    const size_t smem = (size_t)at * sizeof(float);
+    NT_CHECK(smem <= 200 * 1024, "gemv_sum: the input vectors do not fit in shared memory");
+    const int resident = (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)(220 * 1024) / (smem + 1024))) * 148;
+    const int grid = std::min((out + DV_WARPS - 1) / DV_WARPS, resident);
+#define NT_SV(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(gemv_sum_kernel<TY>, 200 * 1024, done); \
+                    launch_k(gemv_sum_kernel<TY>, dim3(grid), dim3(DV_WARPS * 32), smem, s, sd); }
+    if (dt == DType::F32) NT_SV(float) else if (dt == DType::F16) NT_SV(__half) else NT_SV(__nv_bfloat16)
+#undef NT_SV
+    count_launch();
+}
+
+void xielu_rows(float* out, void* split, const float* in, const float* act_p, int T, int cols, cudaStream_t s) {
+    const size_t n = (size_t)T * cols;
+    if (!n) return;
+    const bool vec = n % 4 == 0 && cols % 4 == 0 && ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(split)) & 15) == 0;
+    const dim3 grid((unsigned)((n + (vec ? 1023 : 255)) / (vec ? 1024 : 256)));
+    __nv_bfloat16* hi = static_cast<__nv_bfloat16*>(split);
+    if (vec) launch_k(xielu_kernel<true>, grid, dim3(256), 0, s, out, hi, split_lo_offset(T, cols), in, act_p, n);
+    else launch_k(xielu_kernel<false>, grid, dim3(256), 0, s, out, hi, split_lo_offset(T, cols), in, act_p, n);
     count_launch();
 }
 

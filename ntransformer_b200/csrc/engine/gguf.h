@@ -32,6 +32,11 @@ struct ModelConfig {                       // reference src/model/config.h:16-58
     int side_dim = 0;                      // > 0: after every layer the token's own slice [layer * side_dim, +side_dim) of a second embedding table,
                                            // gated by gelu(W_g x), projected back and RMS-normed, is added to the residual (POST_NORM form)
     float skip_scale = 1.0f;               // a of the SUM_NORM block form
+    int norm_groups = 1;                   // block and final norms: every one of this many equal runs of channels has its own root mean square
+    bool depth_average = false;            // after layer i: x <- sum_j w_i[j] X_j over the embedding X_0 and the results X_1 .. X_(i+1) (PARALLEL form)
+    int bigram_buckets = 0;                // > 0: the row (previous token * bigram_prev + token * bigram_cur) mod buckets of a second table joins the
+    long long bigram_prev = 0, bigram_cur = 0;   // embedding (row `buckets` for a sequence's first token); the previous token is sequence state
+    bool tied_head = false;                // logits = embedding table . x
     bool layer_spec() const { return !layers.empty(); }
     void print() const;
 };

@@ -15,13 +15,17 @@ enum class MixerKind { ATTN_ROPE_CAUSAL = 0,     // rotary positions, full causa
                                                  // a fixed-size state per sequence instead
                        DELTA_RULE = 4,           // gated delta-rule recurrence (DeltaSpec): a matrix state per head that is decayed per key channel,
                                                  // corrected towards the new value along the new key and read with the query; no cache rows
-                       BRANCHES = 5 };           // several mixers side by side reading the same input; their outputs are summed with fixed weights
+                       BRANCHES = 5,           // several mixers side by side reading the same input; their outputs are summed with fixed weights
                                                  // (LayerSpec::branches / branch_scale); each branch keeps its own cache rows or state
+                       WKV = 6 };                // token-shifted linear recurrence with a data-dependent decay per key channel (WkvSpec): a matrix state
+                                                 // per head; no cache rows
 enum class QKNorm { NONE = 0, WHOLE = 1,         // WHOLE: one RMS norm across ALL heads of the projection (gain vector of that length)
                     PER_HEAD = 2 };              // every head is RMS-normed on its own with one gain vector of the head's width shared by all heads
-enum class GluAct { SILU = 0, GELU_TANH = 1, RELU = 2 };
+enum class GluAct { SILU = 0, GELU_TANH = 1, RELU = 2,
+                    XIELU = 3 };             // two learned numbers (p, q) per layer: z > 0: softplus(p) z^2 + z / 2; z <= 0: (1/2 + softplus(q))(e^z - 1 - z) + z / 2
 enum class BlockForm { SEQUENTIAL = 0,           // x += mixer(norm1 x) ; x += ff(norm2 x)
-                       PARALLEL = 1,             // h = norm1 x ; x += m * (ls1 * mixer(h) + ls2 * ff(h))
+                       PARALLEL = 1,             // h = norm1 x ; x += m * (ls1 * mixer(h) + ls2 * ff(h)); with ModelConfig::depth_average the next layer reads
+                                                 // a learned average of the embedding and of every layer's result so far
                        STREAMS = 2,              // SEQUENTIAL over several residual streams: a sublayer reads a learned blend of the streams and
                                                  // its output enters every stream through a learned stream-mixing matrix (ModelConfig::streams)
                        POST_NORM = 3,            // x += norm1(mixer(x)) ; x += norm2(ff(x)): the sublayers read x itself, the norm sits on their output
@@ -29,7 +33,8 @@ enum class BlockForm { SEQUENTIAL = 0,           // x += mixer(norm1 x) ; x += f
                                                  // skip path is multiplied by a = ModelConfig::skip_scale
 enum class FfKind { GLU = 0,                     // W_down (act(W_gate h) * W_up h)
                     MOE_RELU2 = 1,               // routed experts W_down relu(W_up h)^2, top-k softmax over the chosen logits, optional gated shared expert
-                    MOE_GLU = 2 };               // routed gated experts W_down (act(W_gate h) * W_up h); how they are chosen and weighted: RouteSpec
+                    MOE_GLU = 2,               // routed gated experts W_down (act(W_gate h) * W_up h); how they are chosen and weighted: RouteSpec
+                    MLP = 3 };                   // W_down act(W_up h)
 
 
 // Rotary positions of one attention layer.  dims == 0: none.  The first `dims` channels of a head rotate, the rest pass.
@@ -38,13 +43,13 @@ enum class FfKind { GLU = 0,                     // W_down (act(W_gate h) * W_up
 // cos and sin are then multiplied by 0.1 * ln(factor) + 1.
 struct RotarySpec {
     int dims = 0;
-    float base = 10000.f;
+    double base = 10000.0;
     bool interleaved = true;     // pairs (2i, 2i+1); false: (i, i + dims/2)
     float factor = 0.f, original = 0.f, fast = 0.f, slow = 0.f;
     float divide = 1.f;          // linear position scaling: every angular frequency is divided by this
 };
 
-// Low-rank attention.  q = W_uq rms(W_dq h): per head [dim unrotated | rot_dim rotated].  W_dkv h = [kv_rank | rot_dim]: the first part,
+// Low-rank attention.  q = W_uq rms(W_dq h), or (q_rank == 0) q = W_q h: per head [dim unrotated | rot_dim rotated].  W_dkv h = [kv_rank | rot_dim]: the first part,
 // RMS-normed, is the latent c; the second, rotated, is a key part common to all heads.  Head h's keys are [W_uk,h c | that part],
 // its values W_uv,h c.  The cache row of a position is [c | rotated part]: kv_rank + rot_dim numbers whatever the head count.
 struct LatentSpec {
@@ -60,9 +65,12 @@ struct ScanSpec {
 // How a mixture of experts chooses and weights.  sigmoid: scores are sigmoid(logit) (else softmax over the chosen logits);
 // correction: a per-expert vector added to the scores for the CHOICE only; groups > 0: experts form `groups` equal runs of
 // neighbours, a run scores the sum of its two largest choice scores and only the best `keep` runs can be chosen from.
+// all: scores are the softmax over ALL experts; the chosen experts' scores times `scale` are the weights, not renormalized.
 struct RouteSpec {
     bool sigmoid = false, correction = false;
     int groups = 0, keep = 0;
+    bool all = false;
+    float scale = 1.f;
 };
 
 // Gated delta rule.  q, k [kv_heads, dim] and v [heads, vdim] come from projections followed by a short causal convolution
@@ -73,6 +81,14 @@ struct RouteSpec {
 // The sequence's state is S plus the last taps - 1 inputs of the three convolutions.
 struct DeltaSpec {
     int decay_rank = 0, gate_rank = 0;
+};
+
+// WKV time mixer.  h' is the previous token's mixer input (zeros for the first token); r, k, v, gate and decay read h + (h' - h) mu_s with a
+// blend vector each: r, k, v = W m_s (heads x dim), gate = silu(W_g m_g), w = exp(-exp(W_w2 tanh(W_w1 m_w) + w0)) per head and key channel
+// (decay_rank = rows of W_w1).  Per head with a matrix state S [dim, dim] in F32: o = (S + diag(u) k v^T)^T r; S <- diag(w) S + k v^T.  o is
+// divided by its root mean square per head, times a gain over all heads, times the gate, then W_o.  The sequence's state is S and h'.
+struct WkvSpec {
+    int decay_rank = 0;
 };
 
 struct LayerSpec {
@@ -99,7 +115,7 @@ struct LayerSpec {
     int kv_from = -1;            // >= 0: no key / value projections; reads that layer's cache rows (rotated keys, values)
     FfKind ff_kind = FfKind::GLU;
     int experts = 0, top = 0;    // MOE_RELU2: routed experts of width ff, experts used per token
-    int shared_ff = 0;           // MOE_RELU2: width of the shared expert (0 = none); its output is scaled by sigmoid(<w_sg, h>)
+    int shared_ff = 0;           // MOE_RELU2, MOE_GLU: width of the shared expert (0 = none); its output is scaled by sigmoid(<w_sg, h>)
     // ---- mechanisms added with the Tanolorn family ----
     LatentSpec latent;           // ATTN_LATENT (heads, dim, vdim, scale, rot and kv_from above apply too)
     ScanSpec scan;               // SSM_SCAN (heads and vdim above apply too)
@@ -119,6 +135,9 @@ struct LayerSpec {
     DeltaSpec delta;             // DELTA_RULE (heads, kv_heads, dim, vdim and conv above apply too)
     std::vector<LayerSpec> branches;     // BRANCHES: the mixers (their form, ff and token_shift are unused)
     std::vector<float> branch_scale;     // BRANCHES: the weight of each branch's output in the sum
+    // ---- mechanisms added with the Fuvozen family ----
+    WkvSpec wkv;                 // WKV (heads and dim above apply too; vdim == dim)
+    bool shared_glu = false;     // MOE_GLU: the shared expert (shared_ff) is a gated unit added as it is, without a sigmoid weight
     int cache_slot = -1;         // set when the model is finalized: which entry of the model's per-mixer cache table holds this mixer's rows
 };
 

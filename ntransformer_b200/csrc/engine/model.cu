@@ -17,7 +17,7 @@ namespace nt { namespace b200 {
 
 namespace {
 
-__global__ void set_step_kernel(int* step, int token, int pos) { step[0] = token; step[1] = pos; }
+__global__ void set_step_kernel(int* step, int token, int pos) { step[2] = step[0]; step[0] = token; step[1] = pos; }
 __global__ void iota_kernel(int* out, int first, int n) {
     int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i < n) out[i] = first + i;
@@ -83,13 +83,16 @@ Model::~Model() {
     if (moe_offsets_host_) cudaFreeHost(moe_offsets_host_);
     auto free_layer = [](LayerWeights& L) {
         for (void* p : {(void*)L.e_up_tab, (void*)L.e_down_tab, (void*)L.rot_freq, (void*)L.e_gate_tab, (void*)L.conv_state, (void*)L.ssm_state, (void*)L.shift_state,
-                        (void*)L.q_conv_state, (void*)L.k_conv_state, (void*)L.v_conv_state, (void*)L.delta_state}) if (p) cudaFree(p);
+                        (void*)L.q_conv_state, (void*)L.k_conv_state, (void*)L.v_conv_state, (void*)L.delta_state, (void*)L.wkv_state}) if (p) cudaFree(p);
     };
     for (LayerWeights& L : layers_) {
         free_layer(L);
         for (LayerWeights& b : L.branch) free_layer(b);
     }
-    for (void* p : {(void*)dec_.y, (void*)dec_.t[0], (void*)dec_.t[1], (void*)dec_.t[2], (void*)dec_.t[3], (void*)dec_.t[4], (void*)dec_.wide, (void*)pf_.wide}) if (p) cudaFree(p);
+    for (void* p : {(void*)dec_.y, (void*)dec_.t[0], (void*)dec_.t[1], (void*)dec_.t[2], (void*)dec_.t[3], (void*)dec_.t[4], (void*)dec_.wide, (void*)pf_.wide,
+                    (void*)par_dec_.slots, (void*)par_dec_.h, (void*)par_dec_.wide, (void*)par_.slots, (void*)par_.h, (void*)par_.wide, par_.hs, par_.mix_s[0], par_.mix_s[1],
+                    par_.mix_s[2], par_.mix_s[3], par_.mix_s[4], (void*)par_dec_.mix[0], (void*)par_dec_.mix[1], (void*)par_dec_.mix[2], (void*)par_dec_.mix[3],
+                    (void*)par_dec_.mix[4]}) if (p) cudaFree(p);
     if (argmax_host_) cudaFreeHost(argmax_host_);
     if (stream_) cudaStreamDestroy(stream_);
 }
@@ -404,7 +407,8 @@ bool Model::finalize() {
     NT_CUDA_CHECK(cudaMemset(kc_, 0, kv_elems * 2));
     NT_CUDA_CHECK(cudaMemset(vc_, 0, kv_elems * 2));
     NT_CUDA_CHECK(cudaMemset(logits_, 0, sizeof(float) * (size_t)vocab_l_ * tp_size_));
-    step_dev_ = dmalloc<int>(2);
+    step_dev_ = dmalloc<int>(3);
+    NT_CUDA_CHECK(cudaMemset(step_dev_, 0, 3 * sizeof(int)));
     argmax_dev_ = dmalloc<int>(1);
     NT_CUDA_CHECK(cudaMallocHost(&argmax_host_, sizeof(int)));
     finalized_ = true;
@@ -437,11 +441,13 @@ size_t Model::weight_bytes() const {
             const LayerWeights& L = layer_weights(i);
             b += L.wq.bytes() + L.wk.bytes() + L.wv.bytes() + L.wo.bytes() + L.gate.bytes() + L.up.bytes() + L.down.bytes();
             b += L.w_dq.bytes() + L.w_uq.bytes() + L.w_dkv.bytes() + L.w_uk.bytes() + L.w_uv.bytes() + L.ssm_in.bytes() + L.side_gate.bytes() + L.side_proj.bytes();
+            b += L.wkv_g.bytes() + L.wkv_w1.bytes() + L.wkv_w2.bytes();
             for (const LayerWeights& m : L.branch)
                 b += m.wq.bytes() + m.wk.bytes() + m.wv.bytes() + m.wo.bytes() + m.d_beta.bytes() + m.d_a1.bytes() + m.d_a2.bytes() + m.d_g1.bytes() + m.d_g2.bytes();
             if (cfg_.layers[(size_t)i].ff_kind == FfKind::MOE_GLU && cfg_.layers[(size_t)i].ff > 0)
                 b += (size_t)cfg_.layers[(size_t)i].experts * cfg_.hidden_size * 4 +
-                     (size_t)cfg_.layers[(size_t)i].top * (L.e_gate[0].bytes() + L.e_up[0].bytes() + L.e_down[0].bytes());
+                     (size_t)cfg_.layers[(size_t)i].top * (L.e_gate[0].bytes() + L.e_up[0].bytes() + L.e_down[0].bytes()) +
+                     L.sh_glu.bytes() + L.sh_up.bytes() + L.sh_down.bytes();
             // a decoded token reads the router, `top` of the experts and the shared expert
             const LayerSpec& S = cfg_.layers[(size_t)i];
             if (S.ff_kind == FfKind::MOE_RELU2 && S.ff > 0)
@@ -461,6 +467,7 @@ size_t Model::bytes_per_token(int ctx) const {
             size_t kw = 0, vw = 0;
             cache_row_widths(L.kv_from >= 0 ? L.kv_from : i, kw, vw);
             b += (size_t)std::min(ctx, L.chunk > 0 ? L.chunk : (L.window > 0 ? L.window + L.keep_first : ctx)) * (kw + vw) * dtype_size(cache_dt_);
+            if (L.mixer == MixerKind::WKV) b += (size_t)2 * L.heads * L.dim * L.dim * 4;
             if (L.mixer == MixerKind::SSM_SCAN) b += (size_t)2 * L.heads * L.vdim * L.scan.state * 4;      // the state is read and written
             for (const LayerSpec& m : L.branches) {
                 if (m.mixer == MixerKind::DELTA_RULE) b += (size_t)2 * m.heads * m.vdim * m.dim * 4;

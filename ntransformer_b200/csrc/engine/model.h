@@ -85,6 +85,16 @@ struct LayerWeights {
     Weight d_beta, d_a1, d_a2, d_g1, d_g2;
     const float *d_dt_bias = nullptr, *d_a_log = nullptr, *d_norm = nullptr;
     float* delta_state = nullptr;
+    // WKV mixer (WkvSpec; r, k, v are wq, wk, wv): blend vectors of r, k, v, gate, decay [width], gate projection, the low-rank pair of the
+    // decay, its offset [heads * dim], bonus [heads, dim], output gain [heads * dim]; the sequence's matrix state [heads, dim (value), dim
+    // (key)] in F32 (owned; shift_state is the previous token's mixer input)
+    const float* wkv_mu[5] = {nullptr, nullptr, nullptr, nullptr, nullptr};
+    Weight wkv_g, wkv_w1, wkv_w2;
+    const float *wkv_w0 = nullptr, *wkv_u = nullptr, *wkv_norm = nullptr;
+    float* wkv_state = nullptr;
+    // weights of the average over depth [layer + 2], the activation's two numbers, gate matrix of a gated shared expert
+    const float *depth_w = nullptr, *ff_act = nullptr;
+    Weight sh_glu;
     // MixerKind::BRANCHES: each branch's tensors and state
     std::vector<LayerWeights> branch;
 };
@@ -175,6 +185,23 @@ private:
     struct MixerBufs;
     void mixer_attention_rows(int layer, const LayerSpec& S, const LayerWeights& L, const MixerBufs& b, float* y, int T, const int* pos_dev, int p0, cudaStream_t s);
     void mixer_delta_rows(const LayerSpec& S, const LayerWeights& L, const MixerBufs& b, float* y, int T, const int* pos_dev, int p0, cudaStream_t s);
+    // PARALLEL block form with rows of its own kind (latent attention / WKV mixers, average over depth, grouped norms): engine/model_parallel.cu
+    bool parallel_rows() const;               // the model's layers are of that kind (not the windowed-attention form of step_body_spec)
+    bool finalize_parallel_layer(int i);
+    void finalize_parallel_decode();
+    size_t parallel_scratch_width() const;    // floats per row of the layers' intermediates
+    bool parallel_split_ok(const Weight& w) const;      // prompt rows of this matrix take the tensor-core GEMM (its input must be split)
+    void parallel_gemm(float* C, const float* A, const void* A_split, const Weight& w, int T, bool add, cudaStream_t s);
+    void step_parallel(cudaStream_t s);       // one decoded token: embedding, all layers -> hidden_
+    void layer_parallel_token(int i, cudaStream_t s);
+    void prefill_parallel(int T, int p0, cudaStream_t s);   // T prompt rows: embedding, all layers -> pf_.x
+    void layer_parallel_rows(int i, int T, int p0, cudaStream_t s);
+    MoeWeights parallel_moe(int i) const;
+    void ensure_parallel_buffers(size_t T);
+    struct ParDec { float *slots = nullptr, *h = nullptr, *mix[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}, *wide = nullptr; size_t slot = 0; } par_dec_;   // decode: stable addresses
+    struct ParRows { float *slots = nullptr, *h = nullptr, *wide = nullptr; void *hs = nullptr, *mix_s[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}; size_t slot = 0; } par_;
+    void latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s);
+    Weight bigram_;                           // second embedding over token pairs [buckets + 1, width]
     const LayerSpec& slot_spec(int slot) const { return *slot_spec_[(size_t)slot]; }
     std::vector<const LayerSpec*> slot_spec_;   // the mixer behind every entry of kcs_ / vcs_: the layers first, then the branches that keep rows
     void layer_postnorm(int i, int T, const int* tok_dev, const int* pos_dev, int p0, const RowBufs& B, cudaStream_t s);
@@ -261,7 +288,7 @@ private:
     unsigned* attn_tickets_ = nullptr;   // last-arriver tickets of the one-launch attention (zero between launches)
     int fuse_mask_ = 1;                  // bit 0: norm + quantiser in the GEMV prologues (default), bit 1: one-launch attention (opt-in: measured slower, profiles/r02_*), bit 2: RoPE + KV write inside the decode kernel, merge separate (NT_B200_FUSE)
     void *kc_ = nullptr, *vc_ = nullptr;
-    int* step_dev_ = nullptr;            // [0] token, [1] position
+    int* step_dev_ = nullptr;            // [0] token, [1] position, [2] the token before it (sequence state of the pair embedding)
     int* argmax_dev_ = nullptr;
     int* argmax_host_ = nullptr;
     int* recent_dev_ = nullptr;          // repeat-penalty window for the GPU sampler

@@ -22,14 +22,17 @@ enum class TensorSlot { EMBED, HEAD, OUT_NORM, NORM1, NORM2, WQ, WK, WV, WO, Q_N
                         SHIFT_MU,                                                         // token shift: per-channel blend with the previous token's input
                         Q_BIAS, K_BIAS, V_BIAS, O_BIAS, Q_CONV, K_CONV, V_CONV,           // biased projections; short convolutions [channels, taps] on q, k, v
                         HEAD_TEMP, TALK, SINK, V_MIX,                                     // per-head score multiplier, head-mixing matrix [heads, heads], sink, lambda
-                        DELTA_BETA, DELTA_A1, DELTA_A2, DELTA_DT_BIAS, DELTA_A_LOG, DELTA_NORM, DELTA_G1, DELTA_G2 };   // gated delta rule
+                        DELTA_BETA, DELTA_A1, DELTA_A2, DELTA_DT_BIAS, DELTA_A_LOG, DELTA_NORM, DELTA_G1, DELTA_G2,   // gated delta rule
+                        BIGRAM, DEPTH_AVG,                                                // second embedding over token pairs; weights of the average over depth
+                        WKV_MU, WKV_G, WKV_W1, WKV_W2, WKV_W0, WKV_U, WKV_NORM,           // WKV mixer (WKV_MU: index r, k, v, g, w; r, k, v are WQ, WK, WV)
+                        FF_ACT, SHARED_GLU };                                             // the activation's numbers; gate matrix of a gated shared expert
 
 struct TensorBinding {
     std::string name;      // in the checkpoint
     TensorSlot slot;
     int layer;             // -1 for model-level tensors
     int rows, cols;        // expected shape (vectors: rows == 1)
-    int index = 0;         // which expert (EXPERT_UP / EXPERT_DOWN)
+    int index = 0;         // which expert (EXPERT_UP / EXPERT_DOWN), which blend (WKV_MU)
     int branch = -1;       // >= 0: the tensor belongs to that branch of a BRANCHES mixer
 };
 // Slots kept as F32 vectors / small F32 tables whatever the checkpoint stores (gains, lambda vectors, stream tables, router rows).
@@ -56,5 +59,6 @@ const ModelFamily* zelunex_family();      // engine/zelunex.cpp
 const ModelFamily* vebotar_family();      // engine/vebotar.cpp
 const ModelFamily* tanolorn_family();     // engine/tanolorn.cpp
 const ModelFamily* savidra_family();      // engine/savidra.cpp
+const ModelFamily* fuvozen_family();      // engine/fuvozen.cpp
 
 }}  // namespace nt::b200

@@ -3,7 +3,7 @@
 // mechanisms (windowed / soft-capped attention, whole-projection q/k norm, parallel block with layer scale, GELU-gated unit,
 // layers sharing tensors) combine freely.  Same buffers, stream, CUDA-graph replay, logits and sampler as the GGUF families
 // (engine/model.cu); the KV cache is per layer because layers may differ in width.  Layers of BlockForm::SUM_NORM live in
-// engine/model_sumnorm.cu.
+// engine/model_sumnorm.cu, layers of the PARALLEL form with latent-attention or WKV mixers in engine/model_parallel.cu.
 //
 // Arithmetic: the residual stream, norms, softmax and every accumulation are F32.  Weights stay in their stored dtype (BF16)
 // and are widened in registers, or — exact 32-bit mode — are widened once at load.  The cache stores BF16 (F32 in exact mode).
@@ -53,6 +53,7 @@ bool Model::bind_slot(TensorSlot slot, int layer, const void* ptr, DType dt, int
     if (slot == TensorSlot::HEAD) return W(head_);
     if (slot == TensorSlot::OUT_NORM) return V(out_norm_);
     if (slot == TensorSlot::SIDE_EMBED) return W(side_embd_);
+    if (slot == TensorSlot::BIGRAM) return W(bigram_);
     if (layer < 0 || layer >= cfg_.n_layers) return false;
     LayerWeights* Lp = &layers_[(size_t)layer];
     if (branch >= 0) {                      // a tensor of one of the mixers that sit side by side
@@ -64,6 +65,16 @@ bool Model::bind_slot(TensorSlot slot, int layer, const void* ptr, DType dt, int
     LayerWeights& L = *Lp;
     switch (slot) {
         case TensorSlot::SHIFT_MU: return V(L.shift_mu);
+        case TensorSlot::WKV_MU: return index >= 0 && index < 5 && V(L.wkv_mu[index]);
+        case TensorSlot::WKV_G: return W(L.wkv_g);
+        case TensorSlot::WKV_W1: return W(L.wkv_w1);
+        case TensorSlot::WKV_W2: return W(L.wkv_w2);
+        case TensorSlot::WKV_W0: return V(L.wkv_w0);
+        case TensorSlot::WKV_U: return V(L.wkv_u);
+        case TensorSlot::WKV_NORM: return V(L.wkv_norm);
+        case TensorSlot::DEPTH_AVG: return V(L.depth_w);
+        case TensorSlot::FF_ACT: return V(L.ff_act);
+        case TensorSlot::SHARED_GLU: return W(L.sh_glu);
         case TensorSlot::Q_BIAS: return V(L.q_bias);
         case TensorSlot::K_BIAS: return V(L.k_bias);
         case TensorSlot::V_BIAS: return V(L.v_bias);
@@ -218,11 +229,17 @@ bool Model::load_dir(const std::string& dir, int max_context) {
 
 bool Model::finalize_spec() {
     const int hidden = cfg_.hidden_size, max_seq = cfg_.max_seq_len;
+    if (cfg_.tied_head && !head_.ptr) { head_ = embd_; head_.owned = false; }
     if (!embd_.ptr || !out_norm_ || !head_.ptr) { fprintf(stderr, "model: embedding / final norm / head missing\n"); return false; }
     int qmax = 1, kmax = 1, vmax = 1, omax = 1, ffmax = 1, mapmax = 1, moe_act = 1, topmax = 1;
     for (int i = 0; i < cfg_.n_layers; i++) {
         const LayerSpec& S = cfg_.layers[(size_t)i];
         const LayerWeights& L = layer_weights(i);
+        if (parallel_rows()) {
+            if (!finalize_parallel_layer(i)) return false;
+            if (S.ff > 0 && S.ff_kind == FfKind::MOE_GLU) topmax = std::max(topmax, S.top);
+            continue;
+        }
         if (S.form == BlockForm::SUM_NORM) {
             if (!finalize_sumnorm_layer(i)) return false;
             ffmax = std::max(ffmax, S.ff);
@@ -334,6 +351,10 @@ bool Model::finalize_spec() {
         fold(out_norm_);
         for (LayerWeights& L : layers_) { fold(L.attn_norm); fold(L.ffn_norm); }
     }
+    if (parallel_rows()) {
+        finalize_parallel_decode();
+        moe_sel_ = dmalloc<int>(topmax); moe_wt_ = dmalloc<float>(topmax);
+    }
     if (cfg_.layers[0].form == BlockForm::SUM_NORM) {
         const size_t m1 = row_scratch_width();
         dec_.y = dmalloc<float>(m1);
@@ -345,6 +366,8 @@ bool Model::finalize_spec() {
         dec_.y = dmalloc<float>(m1);
         for (float*& t : dec_.t) t = dmalloc<float>(m1);
         moe_sel_ = dmalloc<int>(topmax); moe_wt_ = dmalloc<float>(topmax); moe_act_ = dmalloc<float>(moe_act);
+    }
+    {
         size_t parts = 0;                          // per-slice partial results of the attention that serves all heads from one copy of the rows
         for (const LayerSpec& S : cfg_.layers)
             if (S.mixer == MixerKind::ATTN_LATENT) parts = std::max(parts, attention_shared_rows_scratch_floats(S.heads, S.latent.kv_rank));
@@ -393,7 +416,8 @@ bool Model::finalize_spec() {
         NT_CUDA_CHECK(cudaMemset(kcs_[(size_t)i], 0, std::max<size_t>(kb, 16)));
         NT_CUDA_CHECK(cudaMemset(vcs_[(size_t)i], 0, std::max<size_t>(vb, 16)));
     }
-    step_dev_ = dmalloc<int>(2);
+    step_dev_ = dmalloc<int>(3);
+    NT_CUDA_CHECK(cudaMemset(step_dev_, 0, 3 * sizeof(int)));
     argmax_dev_ = dmalloc<int>(1);
     NT_CUDA_CHECK(cudaMallocHost(&argmax_host_, sizeof(int)));
     prefill_min_tokens_ = 16;
@@ -412,6 +436,7 @@ void Model::step_body_spec(cudaStream_t s) {
     const int hidden = cfg_.hidden_size;
     const int* pos_dev = step_dev_ + 1;
     const float m = cfg_.residual_mult;
+    if (parallel_rows()) { step_parallel(s); return; }
     embed_rows(hidden_, embd_.ptr, embd_.dtype, step_dev_, 1, hidden, s);
     if (cfg_.layers[0].form == BlockForm::POST_NORM) {
         RowBufs B = dec_;
@@ -457,7 +482,7 @@ void Model::step_body_spec(cudaStream_t s) {
 
 void Model::step_head_spec(cudaStream_t s) {
     GemvMat h = mat_of(head_, logits_);
-    gemv_dense(&h, 1, cfg_.hidden_size, hidden_, DENSE_STORE, nullptr, 1.f, s, out_norm_, cfg_.norm_eps);       // final norm in the prologue
+    gemv_dense(&h, 1, cfg_.hidden_size, hidden_, DENSE_STORE, nullptr, 1.f, s, out_norm_, cfg_.norm_eps, nullptr, cfg_.norm_groups);       // final norm in the prologue
 }
 
 void Model::ensure_prefill_buffers_spec(int tokens) {
@@ -471,12 +496,13 @@ void Model::ensure_prefill_buffers_spec(int tokens) {
     pf_.xs = pf_.maps = pf_.wt = pf_.sgate = pf_.act_rows = pf_.y_rows = pf_.g2 = pf_.gate_rows = nullptr; pf_.sel = pf_.work = nullptr; pf_.moe_ws = nullptr;
     const size_t T = (size_t)((tokens + 127) / 128 * 128), hidden = (size_t)cfg_.hidden_size;
     size_t qmax = 1, kmax = 1, vmax = 1, omax = 1, ffmax = 1, mapmax = 1, topmax = 0, emax = 1, effmax = 1;
+    const bool par_form = parallel_rows();
     const bool sum_form = cfg_.layers[0].form == BlockForm::SUM_NORM;
-    const bool post_form = cfg_.layers[0].form == BlockForm::POST_NORM || sum_form;       // both keep five scratch rows of the widest intermediate
+    const bool post_form = cfg_.layers[0].form == BlockForm::POST_NORM || sum_form || par_form;       // the first two keep five scratch rows of the widest intermediate
     if (sum_form) pf_.wide = dmalloc<float>(T * sumnorm_scratch_width());
     for (const LayerSpec& S : cfg_.layers) {
         if (post_form) {                  // five scratch rows of the widest intermediate; routed experts as below
-            qmax = kmax = vmax = omax = ffmax = row_scratch_width();
+            if (!par_form) qmax = kmax = vmax = omax = ffmax = row_scratch_width();
             if (S.ff_kind == FfKind::MOE_GLU && S.ff > 0) { topmax = std::max(topmax, (size_t)S.top); emax = std::max(emax, (size_t)S.experts); effmax = std::max(effmax, (size_t)S.ff); }
             continue;
         }
@@ -510,8 +536,9 @@ void Model::ensure_prefill_buffers_spec(int tokens) {
     bool any_tc = false;
     for (int i = 0; i < cfg_.n_layers; i++) {
         const LayerWeights& L = layer_weights(i);
-        for (const Weight* w : {&L.wq, &L.wk, &L.wv, &L.wo, &L.gate, &L.up, &L.down, &L.sh_up, &L.sh_down, &L.w_dq, &L.w_uq, &L.w_dkv, &L.ssm_in, &L.side_gate, &L.side_proj})
-            any_tc = any_tc || (w->ptr && spec_tc_ok(*w));
+        for (const Weight* w : {&L.wq, &L.wk, &L.wv, &L.wo, &L.gate, &L.up, &L.down, &L.sh_up, &L.sh_down, &L.w_dq, &L.w_uq, &L.w_dkv, &L.ssm_in, &L.side_gate, &L.side_proj, &L.wkv_g, &L.wkv_w1,
+                                &L.wkv_w2, &L.sh_glu})
+            any_tc = any_tc || (w->ptr && (spec_tc_ok(*w) || w->tc_ptr));
         for (const LayerWeights& b : L.branch)
             for (const Weight* w : {&b.wq, &b.wk, &b.wv, &b.wo, &b.d_beta, &b.d_a1, &b.d_a2, &b.d_g1, &b.d_g2}) {
                 any_tc = any_tc || (w->ptr && spec_tc_ok(*w));
@@ -519,9 +546,13 @@ void Model::ensure_prefill_buffers_spec(int tokens) {
             }
         ffmax = std::max(ffmax, (size_t)L.wo.cols);
     }
-    if (sum_form && any_tc) {             // the gated feed-forward's fused gate / up GEMM writes the down GEMM's split input here
+    if (par_form) {
+        ensure_parallel_buffers(T);
+        if (any_tc) for (const LayerSpec& S : cfg_.layers) ffmax = std::max({ffmax, (size_t)S.shared_ff, (size_t)S.wkv.decay_rank});
+    }
+    if ((sum_form || par_form) && any_tc) {             // the gated feed-forward's fused gate / up GEMM writes the down GEMM's split input here
         size_t ffw = 1;
-        for (const LayerSpec& S : cfg_.layers) ffw = std::max(ffw, (size_t)S.ff);
+        for (const LayerSpec& S : cfg_.layers) ffw = std::max({ffw, (size_t)S.ff, (size_t)S.shared_ff});
         pf_.ws2 = dmalloc<uint8_t>(gemm_f16_tc_workspace_bytes((int)T, (int)ffw));
     }
     if (post_form && any_tc) {            // one split workspace: rows_matmul splits its input right before the GEMM
@@ -569,6 +600,11 @@ void Model::prefill_spec(const int* tokens, int seq_len, int start_pos) {
         const int T = std::min(SPEC_PREFILL_CHUNK, seq_len - c0), p0 = start_pos + c0;
         last_rows = T;
         NT_CUDA_CHECK(cudaMemcpyAsync(pf_.tok, tokens + c0, sizeof(int) * (size_t)T, cudaMemcpyHostToDevice, s));
+        if (parallel_rows()) {
+            prefill_parallel(T, p0, s);
+            if (!want_.empty()) emit_wanted(pf_.x, c0, T, s);
+            continue;
+        }
         embed_rows(pf_.x, embd_.ptr, embd_.dtype, pf_.tok, T, hidden, s);
         const bool streams_form = cfg_.layers[0].form == BlockForm::STREAMS, post_form = cfg_.layers[0].form == BlockForm::POST_NORM;
         const bool sum_form = cfg_.layers[0].form == BlockForm::SUM_NORM;
@@ -757,7 +793,7 @@ void Model::layer_streams_rows(int i, int T, int p0, cudaStream_t s) {
 
 void Model::cache_row_widths(int i, size_t& k, size_t& v) const {
     const LayerSpec& S = slot_spec(i);
-    if (S.mixer == MixerKind::SSM_SCAN || S.mixer == MixerKind::DELTA_RULE || S.mixer == MixerKind::BRANCHES) { k = v = 0; return; }      // a state, no rows (branches own theirs)
+    if (S.mixer == MixerKind::SSM_SCAN || S.mixer == MixerKind::DELTA_RULE || S.mixer == MixerKind::BRANCHES || S.mixer == MixerKind::WKV) { k = v = 0; return; }      // a state, no rows (branches own theirs)
     if (S.mixer == MixerKind::ATTN_LATENT) { k = (size_t)S.latent.kv_rank + S.latent.rot_dim; v = 0; return; }   // [latent | rotated key part]
     k = (size_t)S.kv_heads * S.maps * S.dim;
     v = (size_t)S.kv_heads * S.vdim;
@@ -851,27 +887,30 @@ void Model::ensure_latent_scratch(const LayerSpec& S, size_t rows, size_t tokens
     lat_.ku = dmalloc<float>((size_t)LATENT_ROW_BLOCK * lat_.stage_w); lat_.vu = dmalloc<float>((size_t)LATENT_ROW_BLOCK * lat_.stage_w);
 }
 
-// q [T, heads, dim + rot_dim] (unrotated) at positions p0..; the layer's cache rows 0 .. p0 + T - 1 are written.  out [T, heads * vdim].
+// q [T, heads, dim + rot_dim] (unrotated) at positions p0..; the layer's visible cache rows up to p0 + T - 1 are written.  out [T, heads * vdim].
 void Model::latent_attention_rows(int i, int T, int p0, const float* q, float* out, cudaStream_t s) {
     const LayerSpec& S = cfg_.layers[(size_t)i];
     const LayerWeights& L = layer_weights(i);
     const LatentSpec& A = S.latent;
     int kw = 0, vw = 0;
     attention_heads_mma_widths(S.dim + A.rot_dim, S.vdim, &kw, &vw);
-    const int P = p0 + T, row = A.kv_rank + A.rot_dim;
+    const int row = A.kv_rank + A.rot_dim;
+    // a sliding window: only the rows the portion's first query can still see are expanded, and positions count from there
+    const int lo = S.window > 0 ? std::max(0, p0 - S.window + 1) : 0, P = p0 + T - lo;
+    const uint8_t* rows = static_cast<const uint8_t*>(kcs_[(size_t)i]) + (size_t)lo * row * dtype_size(cache_dt_);
     ensure_latent_scratch(S, (size_t)P, (size_t)T);
     const bool tk = spec_tc_ok(L.w_uk), tv = spec_tc_ok(L.w_uv);
     for (int r0 = 0; r0 < P; r0 += LATENT_ROW_BLOCK) {
         const int n = std::min(LATENT_ROW_BLOCK, P - r0);
-        latent_rows_f32(lat_.c32, kcs_[(size_t)i], cache_dt_, row, A.kv_rank, r0, n, s);
+        latent_rows_f32(lat_.c32, rows, cache_dt_, row, A.kv_rank, r0, n, s);
         if (tk || tv) split_activations(lat_.ws, lat_.c32, n, A.kv_rank, s, true);
-        spec_gemm(lat_.ku, lat_.c32, tk ? lat_.ws : nullptr, L.w_uk, n, DENSE_STORE, nullptr, 1.f, s);
+        if (S.dim > 0) spec_gemm(lat_.ku, lat_.c32, tk ? lat_.ws : nullptr, L.w_uk, n, DENSE_STORE, nullptr, 1.f, s);
         spec_gemm(lat_.vu, lat_.c32, tv ? lat_.ws : nullptr, L.w_uv, n, DENSE_STORE, nullptr, 1.f, s);
-        latent_expand_pack(lat_.k, lat_.v, lat_.ku, lat_.vu, kcs_[(size_t)i], cache_dt_, A.kv_rank, r0, n, S.heads, S.dim, A.rot_dim, S.vdim, kw, vw, s);
+        latent_expand_pack(lat_.k, lat_.v, lat_.ku, lat_.vu, rows, cache_dt_, A.kv_rank, r0, n, S.heads, S.dim, A.rot_dim, S.vdim, kw, vw, s);
     }
     latent_q_rot_pad(lat_.q, q, T, S.heads, S.dim, A.rot_dim, kw, S.rot.dims, S.rot.interleaved, S.rot.base, p0, s);
     float* o = vw == S.vdim ? out : lat_.o;
-    attention_heads_mma(o, lat_.q, lat_.k, lat_.v, T, p0, P, S.heads, kw, vw, S.scale, s);
+    attention_heads_mma(o, lat_.q, lat_.k, lat_.v, T, p0 - lo, P, S.heads, kw, vw, S.scale, s, S.window);
     if (o != out) latent_unpad(out, lat_.o, T, S.heads, S.vdim, vw, s);
 }
 
@@ -903,6 +942,25 @@ bool Model::moe_glu_rows_tc(int i, int T, const float* x, cudaStream_t s) {
     return true;
 }
 
+// Scores and values of T rows behind the query projection and the cache write: expanded per-head form for prompt portions, absorbed form on
+// the cached rows otherwise.  q [T, heads, dim + rot_dim]; qa, ol: scratch [T, heads, kv_rank + rot_dim], [T, heads, kv_rank]; o (may be q) [T, heads * vdim].
+void Model::latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s) {
+    const LayerSpec& S = cfg_.layers[(size_t)i];
+    const LayerWeights& L = layer_weights(i);
+    const LatentSpec& A = S.latent;
+    const int row = A.kv_rank + A.rot_dim;
+    if (!pos_dev && latent_expand_ok(S, T)) { latent_attention_rows(i, T, p0, q, o, s); return; }
+    latent_q_absorb(qa, q, L.w_uk.ptr, L.w_uv.dtype, T, S.heads, S.dim, A.rot_dim, A.kv_rank, S.rot.dims, S.rot.interleaved, S.rot.base, pos_dev, p0, s);
+    if (lat_part_ && attention_shared_rows_supported(S.heads, row, A.kv_rank, row, cache_dt_, kcs_[(size_t)i])) {
+        attention_shared_rows(ol, qa, kcs_[(size_t)i], cache_dt_, T, pos_dev, p0, cfg_.max_seq_len, S.heads, row, A.kv_rank, row, S.scale, lat_part_, s, S.window);
+    } else {
+        WindowAttn a;                       // one key / value head: keys are the whole cache rows, values their first kv_rank numbers
+        a.heads = S.heads; a.kv_heads = 1; a.dim = row; a.vdim = A.kv_rank; a.scale = S.scale; a.k_stride = row; a.v_stride = row; a.window = S.window;
+        attention_window(ol, qa, kcs_[(size_t)i], kcs_[(size_t)i], cache_dt_, T, pos_dev, p0, cfg_.max_seq_len, a, s);
+    }
+    latent_v_up(o, ol, L.w_uv.ptr, L.w_uv.dtype, T, S.heads, S.vdim, A.kv_rank, s);
+}
+
 // One layer over T rows: x += norm1(mixer(x)); x += norm2(ff(x)); x += side(x, token).  The sublayers read x itself.
 void Model::layer_postnorm(int i, int T, const int* tok_dev, const int* pos_dev, int p0, const RowBufs& B, cudaStream_t s) {
     const LayerSpec& S = cfg_.layers[(size_t)i];
@@ -912,7 +970,6 @@ void Model::layer_postnorm(int i, int T, const int* tok_dev, const int* pos_dev,
     const float eps = cfg_.norm_eps;
     if (S.mixer == MixerKind::ATTN_LATENT) {
         const LatentSpec& A = S.latent;
-        const int row = A.kv_rank + A.rot_dim;
         float *cq = B.t[0], *dkv = B.t[1], *q = B.t[2], *qa = B.t[3], *ol = B.t[4], *o = B.t[2];
         if (T == 1 && S.kv_from < 0) {                  // one decoded token: both down-projections read x, one launch
             GemvMat two[2] = {mat_of(L.w_dq, cq), mat_of(L.w_dkv, dkv)};
@@ -924,20 +981,8 @@ void Model::layer_postnorm(int i, int T, const int* tok_dev, const int* pos_dev,
         latent_prep(cq, A.q_rank, L.dq_norm, S.kv_from < 0 ? dkv : nullptr, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, S.rot.dims,
                     S.rot.interleaved, S.rot.base, T, pos_dev, p0, s);
         rows_matmul(q, cq, L.w_uq, T, s);
-        if (!pos_dev && latent_expand_ok(S, T)) {
-            latent_attention_rows(i, T, p0, q, o, s);
-            rows_matmul(B.y, o, L.wo, T, s);
-        } else {
-        latent_q_absorb(qa, q, L.w_uk.ptr, L.w_uk.dtype, T, S.heads, S.dim, A.rot_dim, A.kv_rank, S.rot.dims, S.rot.interleaved, S.rot.base, pos_dev, p0, s);
-        WindowAttn a;                       // one key / value head: keys are the whole cache rows, values their first kv_rank numbers
-        a.heads = S.heads; a.kv_heads = 1; a.dim = row; a.vdim = A.kv_rank; a.scale = S.scale; a.k_stride = row; a.v_stride = row;
-        if (lat_part_ && attention_shared_rows_supported(S.heads, row, A.kv_rank, row, cache_dt_, kcs_[(size_t)i]))
-            attention_shared_rows(ol, qa, kcs_[(size_t)i], cache_dt_, T, pos_dev, p0, cfg_.max_seq_len, S.heads, row, A.kv_rank, row, S.scale, lat_part_, s);
-        else
-            attention_window(ol, qa, kcs_[(size_t)i], kcs_[(size_t)i], cache_dt_, T, pos_dev, p0, cfg_.max_seq_len, a, s);
-        latent_v_up(o, ol, L.w_uv.ptr, L.w_uv.dtype, T, S.heads, S.vdim, A.kv_rank, s);
+        latent_mixer_core(i, T, pos_dev, p0, q, qa, ol, o, s);
         rows_matmul(B.y, o, L.wo, T, s);
-        }
     } else {
         const ScanSpec& C = S.scan;
         const int inner = S.heads * S.vdim, ch = inner + 2 * C.groups * C.state, ld = inner + ch + S.heads;

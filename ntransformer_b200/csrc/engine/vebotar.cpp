@@ -18,10 +18,10 @@ bool need_int(const Json& o, const char* key, int& out, std::string& err, const 
     out = (int)v.int_or(0);
     return true;
 }
-bool need_float(const Json& o, const char* key, float& out, std::string& err, const std::string& where) {
+template <typename F> bool need_float(const Json& o, const char* key, F& out, std::string& err, const std::string& where) {
     const Json& v = o.at(key);
     if (!v.is_number()) { err = where + ": \"" + key + "\" is missing or not a number"; return false; }
-    out = (float)v.number_or(0.0);
+    out = (F)v.number_or(0.0);
     return true;
 }
 

@@ -145,7 +145,31 @@ bool dense_dtype(DType dt);
 // Up to DENSE_MAX_MATS matrices of one dense dtype sharing the activation vector x[K] (GemvMat::y: each matrix's output rows).
 // norm_w: the kernel's prologue first replaces x by x / sqrt(mean(x^2) + eps) * norm_w (the block's RMS norm, recomputed per CTA).
 void gemv_dense(const GemvMat* mats, int n_mat, int K, const float* x, DenseEpilogue ep, const float* row_scale, float alpha, cudaStream_t s,
-                const float* norm_w = nullptr, float eps = 0.f, const StreamsIO* sio = nullptr);
+                const float* norm_w = nullptr, float eps = 0.f, const StreamsIO* sio = nullptr, int norm_groups = 1);
+constexpr int DENSE_MAX_NORM_GROUPS = 256;
+// Several matrices with an input vector each, one launch; act is applied to a matrix's own rows.  One 16-bit dtype per launch, F32 matrices
+// (router tables) may stand beside it.
+enum GemvAct { GEMV_ACT_NONE = 0, GEMV_ACT_TANH = 1, GEMV_ACT_XIELU = 2 /* two learned numbers: act_p */ };
+struct MultiMat {
+    const void* W = nullptr; DType dtype = DType::F32; size_t row_pitch = 0;
+    const float* x = nullptr; float* y = nullptr;
+    int out = 0, K = 0;
+    GemvAct act = GEMV_ACT_NONE; const float* act_p = nullptr;
+};
+void gemv_multi(const MultiMat* mats, int n_mat, cudaStream_t s);
+// y[out] (+)= the sum of up to GEMV_SUM_MAX_TERMS matrix-vector products.  A term is one matrix W [out, K] with x [K], or `top` routed ones:
+// sum_k wt[k] table[sel[k]] x[k * K ..] (sel, wt, table on the device).  Rows packed, one dtype.
+constexpr int GEMV_SUM_MAX_TERMS = 4;
+struct SumTerm {
+    const void* W = nullptr;
+    const void* const* table = nullptr; const int* sel = nullptr; const float* wt = nullptr; int top = 0;
+    bool table_aligned = false;        // every matrix of the table starts on 16 bytes
+    const float* x = nullptr; int K = 0;
+};
+void gemv_sum(float* y, const SumTerm* terms, int n, int out, DType dt, bool add, cudaStream_t s);
+// a [T, cols] -> xIELU, z > 0: softplus(p) z^2 + z / 2, z <= 0: (1/2 + softplus(q))(e^z - 1 - z) + z / 2, (p, q) = act_p; as F32 rows (in place is
+// fine) and / or as the BF16 split of a tensor-core GEMM's input
+void xielu_rows(float* out, void* split, const float* in, const float* act_p, int T, int cols, cudaStream_t s);
 // C[T,N] (ep)= A[T,K] . W[N,K]^T in true FP32 on CUDA cores (store / add / scaled-add; row_scale indexes N).
 void gemm_dense(float* C, const float* A, const void* W, DType dt, size_t row_pitch, int T, int N, int K, DenseEpilogue ep,
                 const float* row_scale, float alpha, cudaStream_t s);
@@ -216,6 +240,10 @@ struct MoeWeights {
     bool sigmoid = false;
     const float* correction = nullptr;
     int groups = 0, keep = 0;
+    // all: scores are the softmax over ALL experts, weight = the chosen experts' scores times scale (not renormalized)
+    bool all = false;
+    float scale = 1.f;
+    const void* shared_gatew = nullptr;  // [shared_ff, width]: the shared expert is a gated unit too (decode kernels; sgate null: added as it is)
 };
 // Router: logits in F32, the `top` largest (lowest index on ties), softmax over the chosen -> sel [tokens, top], wt [tokens, top];
 // sgate [tokens] = sigmoid(<shared_gate, h>) when shared_gate is given.
@@ -224,7 +252,9 @@ struct MoeWeights {
 void moe_route(int* sel, float* wt, float* sgate, const float* h, const MoeWeights& w, int tokens, cudaStream_t s,
                const StreamsIO* sio = nullptr, const float* norm_w = nullptr, float eps = 0.f, float* h_out = nullptr);
 // One token (decode): act [top * ff + shared_ff] = relu(W_up[sel] h)^2 ; y [width] = sum_k wt[k] * W_down[sel[k]] act[k] + sgate * shared part.
-void moe_expert_up_token(float* act, const float* h, const int* sel, const MoeWeights& w, cudaStream_t s);
+// logits given (RouteSpec::all): the choice is made here from the router's logits [experts] and written to sel_out / wt_out; sel is not read.
+void moe_expert_up_token(float* act, const float* h, const int* sel, const MoeWeights& w, cudaStream_t s, const float* logits = nullptr, int* sel_out = nullptr,
+                         float* wt_out = nullptr);
 // sio->X_out: the result enters the residual streams (StreamsIO) instead of y.
 void moe_expert_down_token(float* y, const float* act, const int* sel, const float* wt, const float* sgate, const float* shared_y,
                            const MoeWeights& w, cudaStream_t s, const StreamsIO* sio = nullptr);
@@ -236,21 +266,21 @@ void moe_group(int* work, const int* sel, int tokens, int experts, int top, cuda
 void moe_expert_up_rows(float* act_rows, const float* h, const int* work, const MoeWeights& w, int tokens, cudaStream_t s);
 void moe_expert_gate_rows(float* gate_rows, const float* h, const int* work, const MoeWeights& w, int tokens, cudaStream_t s);
 void moe_expert_down_rows(float* y_rows, const float* act_rows, const int* work, const MoeWeights& w, int tokens, cudaStream_t s); // [tokens*top, width]
-// y [tokens, width] = sum_k wt[t, k] * y_rows[row(t, k)] (+ sgate[t] * shared_y[t])
+// y [tokens, width] = sum_k wt[t, k] * y_rows[row(t, k)] (+ sgate[t] * shared_y[t]; sgate null: + shared_y[t]); add: y += that
 void moe_combine(float* y, const float* y_rows, const int* work, const float* wt, const float* sgate, const float* shared_y, int tokens,
-                 int experts, int top, int width, cudaStream_t s);
+                 int experts, int top, int width, cudaStream_t s, bool add = false);
 // h rows in the grouped order (the tensor-core path splits them per expert): out [tokens*top, width]
 void moe_gather_rows(float* out, const float* h, const int* work, int tokens, int experts, int top, int width, cudaStream_t s);
 void relu2(float* x, size_t n, cudaStream_t s);
 
 // ---- attention_latent.cu / ssm_scan.cu / postnorm.cu: mechanisms added with the third layer-spec family ----
 // Latent attention (engine/layer_spec.h LatentSpec).  cq [T, q_rank]: RMS-normed in place (gain).  dkv [T, kv_rank + rot_dim] (null: the layer
-// reads another layer's rows): [RMS-normed first part | rotated rest] -> cache row base + t of `cache` ([max_seq, kv_rank + rot_dim]).
+// reads another layer's rows; cq null: the queries have no latent): [RMS-normed first part | rotated rest] -> cache row base + t of `cache` ([max_seq, kv_rank + rot_dim]).
 void latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache,
-                 DType cache_dt, int rot_dims, bool interleaved, float rot_base, int T, const int* pos_dev, int p0, cudaStream_t s);
+                 DType cache_dt, int rot_dims, bool interleaved, double rot_base, int T, const int* pos_dev, int p0, cudaStream_t s);
 // q [T, heads, dim + rot_dim] -> qa [T, heads, kv_rank + rot_dim] = [W_uk,h^T q_unrotated | rot(q_rotated)];  W_uk [heads * dim, kv_rank]
 void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, int rot_dims,
-                     bool interleaved, float rot_base, const int* pos_dev, int p0, cudaStream_t s);
+                     bool interleaved, double rot_base, const int* pos_dev, int p0, cudaStream_t s);
 // ol [T, heads, kv_rank] -> out [T, heads * vdim] = W_uv,h ol_h;  W_uv [heads * vdim, kv_rank]
 void latent_v_up(float* out, const float* ol, const void* W_uv, DType dt, int T, int heads, int vdim, int kv_rank, cudaStream_t s);
 // Prompt portions: F32 latents of cache rows r0.. (input of the two up-projection GEMMs); their results packed with the rotated key part
@@ -259,20 +289,21 @@ void latent_v_up(float* out, const float* ol, const void* W_uv, DType dt, int T,
 void latent_rows_f32(float* out, const void* cache, DType cache_dt, int row, int kv_rank, int r0, int n, cudaStream_t s);
 void latent_expand_pack(void* kfull, void* vfull, const float* ku, const float* vu, const void* cache, DType cache_dt, int kv_rank, int r0, int n, int heads,
                         int dim, int rot_dim, int vdim, int kw, int vw, cudaStream_t s);
-void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, int rot_dims, bool interleaved, float rot_base, int p0,
+void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, int rot_dims, bool interleaved, double rot_base, int p0,
                       cudaStream_t s);
 void latent_unpad(float* out, const float* o, int T, int heads, int vdim, int vw, cudaStream_t s);
 // Attention of a few queries over ONE key / value head stored as rows (keys: the first dim numbers of a row, values: the first vdim),
-// every head served from one shared-memory copy of the rows; key slices merged by a second launch.  Full causal mask.
+// every head served from one shared-memory copy of the rows; key slices merged by a second launch.  Causal mask, with window > 0 only
+// the last `window` positions up to the query's own.
 bool attention_shared_rows_supported(int heads, int dim, int vdim, int row, DType cache_dt, const void* cache);
 size_t attention_shared_rows_scratch_floats(int heads, int vdim);
 void attention_shared_rows(float* out, const float* Q, const void* cache, DType cache_dt, int tokens, const int* pos_dev, int p0, int max_seq, int heads, int dim,
-                           int vdim, int row, float scale, float* scratch, cudaStream_t s);
-// attention_prefill_mma.cu: full causal attention of `tokens` queries [tokens, heads, kw] at positions p0.. over BF16 per-head keys
+                           int vdim, int row, float scale, float* scratch, cudaStream_t s, int window = 0);
+// attention_prefill_mma.cu: causal (window > 0: the last `window` positions) attention of `tokens` queries [tokens, heads, kw] at positions p0.. over BF16 per-head keys
 // [rows, heads, kw] and values [rows, heads, vw]; (kw, vw) from attention_heads_mma_widths.  out [tokens, heads, vw].
 bool attention_heads_mma_widths(int key_dim, int value_dim, int* kw, int* vw);
 void attention_heads_mma(float* out, const float* Q, const void* k, const void* v, int tokens, int p0, int rows, int heads, int kw, int vw, float scale,
-                         cudaStream_t s);
+                         cudaStream_t s, int window = 0);
 // State-space scan (ScanSpec).  u [T, ld]: the input projection's rows; channels of interest start at a column offset.
 // conv_state [taps - 1, ch], state [heads, vdim, N]: the sequence's state, read unless the step starts at position 0, updated in place.
 void ssm_conv(float* out, const float* u, int ld, int col0, float* conv_state, const float* w, const float* b, int T, int ch, int taps,
@@ -332,6 +363,45 @@ void head_prep(float* Q, const float* K, const float* V, const HeadPrep& p, void
 // out [T, heads, vdim] = sum_g M[h, g] A(t, g, kv(h), :), A addressed as A + t * t_stride + g * g_stride + c * c_stride.
 void talk_mix(float* out, const float* A, const float* M, int tokens, int heads, int kv_heads, int vdim, size_t t_stride, size_t g_stride, size_t c_stride,
               cudaStream_t s);
+
+// ---- depth_rows.cu / wkv.cu: mechanisms added with the fifth layer-spec family ----
+// x0[t] (and x1[t] when given) = E[token_t] + B[(token_{t-1} mul_prev + token_t mul_cur) mod buckets]; a sequence's first token reads row `buckets`.
+// prev_dev: the token before the step's first row (unused when the step starts at position 0).  B == null: the plain embedding.
+void embed_bigram_rows(float* x0, float* x1, const void* E, DType edt, const void* B, DType bdt, const int* tokens_dev, const int* prev_dev, int T, int width,
+                       long long buckets, long long mul_prev, long long mul_cur, const int* pos_dev, int p0, cudaStream_t s);
+// x = sum_j coef[j] X_j over n slots (X + j * slot, each [T, width]; coef null: the last slot) -> x_out; h = x / rms(its group) * gain -> h_out
+// and / or the BF16 split (lo half split_lo words behind).  n_mix > 0 (one row): mix_out[s] = h + (carried - h) mu[s] (carried reads as zeros when
+// the step starts at position 0), then carried <- h.
+struct DepthNorm {
+    static constexpr int MAX_MIX = 5;
+    const float* X = nullptr; size_t slot = 0; int n = 1; const float* coef = nullptr;
+    float* x_out = nullptr; float* h_out = nullptr; void* split = nullptr; size_t split_lo = 0;
+    const float* gain = nullptr;       // null: no norm, x_out only
+    float eps = 0.f; int width = 0, groups = 1;
+    int n_mix = 0; const float* mu[MAX_MIX] = {nullptr, nullptr, nullptr, nullptr, nullptr}; float* mix_out[MAX_MIX] = {nullptr, nullptr, nullptr, nullptr, nullptr};
+    float* carried = nullptr; const int* pos_dev = nullptr; int p0 = 0;
+};
+void depth_norm_rows(const DepthNorm& p, int T, cudaStream_t s);
+// WKV time mixer (engine/layer_spec.h WkvSpec).  shift_mix_rows: out[s] and / or split[s] (lo half split_lo words behind) = h + (h_prev - h) mu[s]
+// for every row, h_prev of the first row = carried (zeros at position 0); carried <- the last row.
+struct ShiftMix {
+    static constexpr int MAX = 5;
+    int n = 0; const float* mu[MAX] = {nullptr, nullptr, nullptr, nullptr, nullptr}; float* out[MAX] = {nullptr, nullptr, nullptr, nullptr, nullptr};
+    void* split[MAX] = {nullptr, nullptr, nullptr, nullptr, nullptr}; size_t split_lo = 0;
+};
+constexpr int WKV_MAX_DIM = 256;
+void shift_mix_rows(const ShiftMix& p, const float* h, float* carried, int T, int width, const int* pos_dev, int p0, cudaStream_t s);
+void tanh_rows(float* x, size_t n, cudaStream_t s);
+// a [T, heads * dim] <- exp(-exp(a + w0));  ruk [T, heads] = sum_d r u k
+void wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int T, int heads, int dim, cudaStream_t s);
+// out [T, heads * dim] from the recurrence over the step's rows; state [heads, dim (value), dim (key)] read unless the step starts at position 0, written back
+void wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int T, int heads, int dim, const int* pos_dev, int p0,
+              cudaStream_t s);
+// o / rms(head) * norm * silu(gate), as F32 rows and / or a BF16 split
+void wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int T, int heads, int dim, cudaStream_t s);
+// One token: decay from a1 [rank] (behind the tanh) and W2 [heads * dim, rank], recurrence, head norm and gate -> out [heads * dim]
+void wkv_token(float* out, const float* r, const float* k, const float* v, const float* gate, const float* a1, const void* W2, DType dt, const float* w0, const float* u,
+               const float* norm, float* state, float eps, int rank, int heads, int dim, const int* pos_dev, int p0, cudaStream_t s);
 
 // Programmatic dependent launch (PDL): when enabled, kernels are launched with
 // cudaLaunchAttributeProgrammaticStreamSerialization so that a kernel's prologue (barrier init, TMA weight

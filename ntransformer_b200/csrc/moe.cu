@@ -10,7 +10,7 @@
 //                            result does not depend on which other tokens share its tile.
 // Variants (MoeWeights): gated experts W_down (silu(W_gate h) * W_up h) through a third pointer table; a router that scores by
 // sigmoid, adds a correction vector for the choice only, restricts the choice to the best runs of neighbouring experts and weights
-// by the plain scores.
+// by the plain scores; a router that weights by the softmax over all experts; a gated shared expert.
 // Expert matrices: F32, F16 or BF16 rows.  Compiled WITHOUT --use_fast_math.
 #include "kernels_internal.h"
 #include "ring.cuh"
@@ -92,10 +92,41 @@ __device__ __forceinline__ float warp_dot(const unsigned char* row, const float*
 constexpr int RT_WARPS = 8;
 constexpr int MAX_EXPERTS = 256;
 
+// One warp: softmax over all experts of z, the `top` largest (lowest index on ties) with their share times `scale`, largest first.
+__device__ __forceinline__ void choose_of_all(const float* z, int experts, int top, float scale, int lane, int* sel, float* wt) {
+    float v[MAX_EXPERTS / 32], mx = -INFINITY, den = 0.f;
+#pragma unroll
+    for (int i = 0; i < MAX_EXPERTS / 32; i++) { const int e = lane + 32 * i; v[i] = e < experts ? z[e] : -INFINITY; mx = fmaxf(mx, v[i]); }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, o));
+#pragma unroll
+    for (int i = 0; i < MAX_EXPERTS / 32; i++) den += lane + 32 * i < experts ? expf(v[i] - mx) : 0.f;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xFFFFFFFFu, den, o);
+    unsigned taken = 0;                            // bit i: this lane's expert lane + 32 i is chosen
+    for (int k = 0; k < top; k++) {
+        float bv = -INFINITY;
+        int be = MAX_EXPERTS;
+#pragma unroll
+        for (int i = 0; i < MAX_EXPERTS / 32; i++) {
+            const int e = lane + 32 * i;
+            if (e < experts && !(taken >> i & 1u) && (v[i] > bv || be == MAX_EXPERTS)) { bv = v[i]; be = e; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xFFFFFFFFu, bv, o);
+            const int oe = __shfl_xor_sync(0xFFFFFFFFu, be, o);
+            if (oe < MAX_EXPERTS && (be == MAX_EXPERTS || ov > bv || (ov == bv && oe < be))) { bv = ov; be = oe; }
+        }
+        if ((be & 31) == lane) taken |= 1u << (be >> 5);
+        if (lane == 0) { sel[k] = be; wt[k] = expf(bv - mx) / den * scale; }
+    }
+}
+
 __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(int* __restrict__ sel, float* __restrict__ wt, float* __restrict__ sgate,
                                                                   const float* __restrict__ h, const float* __restrict__ router,
                                                                   const float* __restrict__ shared_gate, int experts, int top, int width,
-                                                                  int sigmoid, const float* __restrict__ correction, int groups, int keep, StreamsIO sio, const float* __restrict__ norm_w, float eps, float* __restrict__ h_out) {
+                                                                  int sigmoid, const float* __restrict__ correction, int groups, int keep, int all, float scale, StreamsIO sio, const float* __restrict__ norm_w, float eps, float* __restrict__ h_out) {
     extern __shared__ __align__(16) float hs[];
     __shared__ float z[MAX_EXPERTS + 1];
     __shared__ float sc[MAX_EXPERTS];
@@ -134,6 +165,11 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(int* __restric
         if (lane == 0) z[e] = d;
     }
     __syncthreads();
+    if (all) {
+        if (threadIdx.x == 0 && shared_gate) sgate[t] = 1.0f / (1.0f + expf(-z[experts]));
+        if (warp == 0) choose_of_all(z, experts, top, scale, lane, sel + (size_t)t * top, wt + (size_t)t * top);
+        return;
+    }
     if (threadIdx.x != 0) return;
     if (shared_gate) sgate[t] = 1.0f / (1.0f + expf(-z[experts]));
     if (sigmoid) {
@@ -189,32 +225,40 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(int* __restric
 struct MoeDev {
     const void* const* gate;       // null: squared-ReLU experts
     const void* const* up; const void* const* down;
-    const void* shared_up; const void* shared_down;
-    int top, ff, width, shared_ff;
+    const void* shared_up; const void* shared_down; const void* shared_gatew;
+    int top, ff, width, shared_ff, experts;
+    float scale;
 };
 
 constexpr int TK_WARPS = 8;
 // act [top * ff + shared_ff]: slot k < top is expert sel[k], the last slot the shared expert
 template <typename T>
-__global__ void __launch_bounds__(TK_WARPS * 32) moe_up_token_kernel(float* __restrict__ act, const float* __restrict__ h, const int* __restrict__ sel, MoeDev m) {
+__global__ void __launch_bounds__(TK_WARPS * 32) moe_up_token_kernel(float* __restrict__ act, const float* __restrict__ h, const int* __restrict__ sel, MoeDev m,
+                                                                     const float* __restrict__ logits, int* __restrict__ sel_out, float* __restrict__ wt_out) {
     extern __shared__ __align__(16) float hs[];
+    __shared__ int sel_s[MAX_EXPERTS];
+    __shared__ float wt_s[MAX_EXPERTS];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_launch_dependents();
     pdl_wait();
     for (int i = threadIdx.x; i < m.width; i += TK_WARPS * 32) hs[i] = h[i];
+    if (logits) {                                  // every CTA makes the same choice from the router's logits; the first one publishes it
+        if (warp == 0) choose_of_all(logits, m.experts, m.top, m.scale, lane, sel_s, wt_s);
+    } else for (int k = threadIdx.x; k < m.top; k += TK_WARPS * 32) sel_s[k] = sel[k];
     __syncthreads();
+    if (logits && blockIdx.x == 0) for (int k = threadIdx.x; k < m.top; k += TK_WARPS * 32) { sel_out[k] = sel_s[k]; wt_out[k] = wt_s[k]; }
     const int total = m.top * m.ff + m.shared_ff;
     const size_t pitch = (size_t)m.width * sizeof(T);
     const bool kvec = m.width % El<T>::P == 0;
     for (int r = blockIdx.x * TK_WARPS + warp; r < total; r += gridDim.x * TK_WARPS) {
         const unsigned char* base;
         int row;
-        if (r < m.top * m.ff) { base = static_cast<const unsigned char*>(m.up[sel[r / m.ff]]); row = r % m.ff; }
+        if (r < m.top * m.ff) { base = static_cast<const unsigned char*>(m.up[sel_s[r / m.ff]]); row = r % m.ff; }
         else { base = static_cast<const unsigned char*>(m.shared_up); row = r - m.top * m.ff; }
         const unsigned char* wr = base + (size_t)row * pitch;
         const float d = warp_dot<T>(wr, hs, m.width, lane, kvec && (reinterpret_cast<uintptr_t>(wr) & 15) == 0);
-        if (m.gate && r < m.top * m.ff) {       // gated unit: silu(<gate row, h>) * <up row, h>
-            const unsigned char* gr = static_cast<const unsigned char*>(m.gate[sel[r / m.ff]]) + (size_t)row * pitch;
+        if (r < m.top * m.ff ? m.gate != nullptr : m.shared_gatew != nullptr) {       // gated unit: silu(<gate row, h>) * <up row, h>
+            const unsigned char* gr = static_cast<const unsigned char*>(r < m.top * m.ff ? m.gate[sel_s[r / m.ff]] : m.shared_gatew) + (size_t)row * pitch;
             const float g = warp_dot<T>(gr, hs, m.width, lane, kvec && (reinterpret_cast<uintptr_t>(gr) & 15) == 0);
             if (lane == 0) act[r] = g / (1.0f + expf(-g)) * d;
             continue;
@@ -241,7 +285,7 @@ __global__ void __launch_bounds__(TK_WARPS * 32) moe_down_token_kernel(float* __
         }
         if (m.shared_ff > 0) {
             const unsigned char* wr = static_cast<const unsigned char*>(m.shared_down) + (size_t)r * m.shared_ff * sizeof(T);
-            acc = fmaf(sgate[0], warp_dot<T>(wr, as + (size_t)m.top * m.ff, m.shared_ff, lane, svec && (reinterpret_cast<uintptr_t>(wr) & 15) == 0 && (((size_t)m.top * m.ff) & 3) == 0), acc);
+            acc = fmaf(sgate ? sgate[0] : 1.f, warp_dot<T>(wr, as + (size_t)m.top * m.ff, m.shared_ff, lane, svec && (reinterpret_cast<uintptr_t>(wr) & 15) == 0 && (((size_t)m.top * m.ff) & 3) == 0), acc);
         }
         if (lane == 0) {
             if (!sio.X_out) y[r] = acc;
@@ -380,7 +424,7 @@ __global__ void moe_gather_rows_kernel(float* __restrict__ out, const float* __r
     out[i] = h[(size_t)row_token[r] * width + c];
 }
 __global__ void moe_combine_kernel(float* __restrict__ y, const float* __restrict__ y_rows, const int* __restrict__ assign_row, const float* __restrict__ wt,
-                                   const float* __restrict__ sgate, const float* __restrict__ shared_y, size_t n, int top, int width) {
+                                   const float* __restrict__ sgate, const float* __restrict__ shared_y, size_t n, int top, int width, int add) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -388,8 +432,8 @@ __global__ void moe_combine_kernel(float* __restrict__ y, const float* __restric
     const size_t t = i / width, c = i % width;
     float acc = 0.f;
     for (int k = 0; k < top; k++) acc = fmaf(wt[t * top + k], y_rows[(size_t)assign_row[t * top + k] * width + c], acc);
-    if (shared_y) acc = fmaf(sgate[t], shared_y[i], acc);
-    y[i] = acc;
+    if (shared_y) acc = fmaf(sgate ? sgate[t] : 1.f, shared_y[i], acc);
+    y[i] = add ? y[i] + acc : acc;
 }
 __global__ void relu2_kernel(float* __restrict__ x, size_t n) {
     pdl_launch_dependents();
@@ -398,7 +442,7 @@ __global__ void relu2_kernel(float* __restrict__ x, size_t n) {
     if (i < n) { const float z = fmaxf(x[i], 0.f); x[i] = z * z; }
 }
 
-MoeDev dev_of(const MoeWeights& w) { return MoeDev{w.gate, w.up, w.down, w.shared_up, w.shared_down, w.top, w.ff, w.width, w.shared_up ? w.shared_ff : 0}; }
+MoeDev dev_of(const MoeWeights& w) { return MoeDev{w.gate, w.up, w.down, w.shared_up, w.shared_down, w.shared_gatew, w.top, w.ff, w.width, w.shared_up ? w.shared_ff : 0, w.experts, w.scale}; }
 
 }  // namespace
 
@@ -414,7 +458,7 @@ void moe_route(int* sel, float* wt, float* sgate, const float* h, const MoeWeigh
     static unsigned long long done = 0;
     if (smem > 40 * 1024) opt_in_dynamic_smem(moe_route_kernel, 160 * 1024, done);
     launch_k(moe_route_kernel, dim3(tokens), dim3(RT_WARPS * 32), smem, s, sel, wt, sgate, h, w.router, w.shared_gate, w.experts, w.top, w.width,
-             w.sigmoid ? 1 : 0, w.correction, w.groups, w.keep, sio, norm_w, eps, h_out);
+             w.sigmoid ? 1 : 0, w.correction, w.groups, w.keep, w.all ? 1 : 0, w.scale, sio, norm_w, eps, h_out);
     count_launch();
 }
 
@@ -422,14 +466,15 @@ void moe_route(int* sel, float* wt, float* sgate, const float* h, const MoeWeigh
     if (w.dtype == DType::F32) { CALL(float) } else if (w.dtype == DType::F16) { CALL(__half) } else if (w.dtype == DType::BF16) { CALL(__nv_bfloat16) } \
     else NT_CHECK(false, "moe: dense expert dtypes only");
 
-void moe_expert_up_token(float* act, const float* h, const int* sel, const MoeWeights& w, cudaStream_t s) {
+void moe_expert_up_token(float* act, const float* h, const int* sel, const MoeWeights& w, cudaStream_t s, const float* logits, int* sel_out, float* wt_out) {
+    NT_CHECK(!logits || (w.all && sel_out && wt_out && w.experts <= MAX_EXPERTS && w.top <= w.experts), "moe_expert_up_token: a choice from logits is the softmax over all experts");
     const MoeDev m = dev_of(w);
     const int total = m.top * m.ff + m.shared_ff;
     const size_t smem = (size_t)w.width * sizeof(float);
     NT_CHECK(smem <= 200 * 1024, "moe: the activation row does not fit in shared memory");
     const int grid = std::min((total + TK_WARPS - 1) / TK_WARPS, 148 * 8);
 #define NT_CALL(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(moe_up_token_kernel<TY>, 200 * 1024, done); \
-                      launch_k(moe_up_token_kernel<TY>, dim3(grid), dim3(TK_WARPS * 32), smem, s, act, h, sel, m); }
+                      launch_k(moe_up_token_kernel<TY>, dim3(grid), dim3(TK_WARPS * 32), smem, s, act, h, sel, m, logits, sel_out, wt_out); }
     NT_MOE_DT(NT_CALL)
 #undef NT_CALL
     count_launch();
@@ -485,11 +530,11 @@ void moe_expert_down_rows(float* y_rows, const float* act_rows, const int* work,
     count_launch();
 }
 void moe_combine(float* y, const float* y_rows, const int* work, const float* wt, const float* sgate, const float* shared_y, int tokens,
-                 int experts, int top, int width, cudaStream_t s) {
+                 int experts, int top, int width, cudaStream_t s, bool add) {
     const size_t n = (size_t)tokens * width;
     if (!n) return;
     launch_k(moe_combine_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, y, y_rows, work + experts + 1 + (size_t)tokens * top, wt, sgate,
-             shared_y, n, top, width);
+             shared_y, n, top, width, add ? 1 : 0);
     count_launch();
 }
 void moe_gather_rows(float* out, const float* h, const int* work, int tokens, int experts, int top, int width, cudaStream_t s) {

@@ -1,0 +1,418 @@
+// wkv.cu — the WKV time mixer around its projections (engine/layer_spec.h WkvSpec).  Per head with a matrix state S [D, D] in F32
+// (key channel d, value channel j), reading the rows r_t, k_t, v_t and the per-channel decay w_t in (0, 1):
+//       o_t[j] = sum_d r_t[d] S[d, j] + (sum_d r_t[d] u[d] k_t[d]) v_t[j];      S[d, j] <- w_t[d] S[d, j] + k_t[d] v_t[j]
+//   shift_mix_rows   the mixer's inputs m_s[t] = h[t] + (h[t-1] - h[t]) mu_s for several s from one read of h, as F32 rows or as the BF16
+//                    split a tensor-core GEMM reads; h[-1] is the carried row (zeros when the step starts at position 0), which then
+//                    becomes the step's last row
+//   tanh_rows        in place
+//   wkv_prep         a <- exp(-exp(a + w0)) in place [T, H * D];  ruk [T, H] = sum_d r u k
+//   wkv_rows         the recurrence over the rows of a step.  Every column j of S evolves on its own; LN lanes share a column (dim / LN
+//                    state numbers each, in registers).  The carried chain of a row is one multiply-add; the dot products of a tile of
+//                    16 rows stay in registers and are reduced together (a halving exchange between the lanes: 15 shuffles for 16 rows
+//                    instead of 64).  Rows are staged in tiles of 16 by cp.async into two buffers.
+//   wkv_out_norm     o / rms(head) * norm * silu(gate), as F32 rows or as the split of the output projection's input
+//   wkv_token        one decoded token in one launch: decay (second low-rank matrix, exponentials), recurrence, head norm and gate; a CTA
+//                    per head
+// The state [H, D (value), D (key)] is read at the start (zeros when the step starts at position 0) and written back at the end, so a
+// prompt cut anywhere continues exactly.  A step's base position is *pos_dev when given (the captured decode step), else p0.
+// Everything is F32; compiled WITHOUT --use_fast_math (expf / tanhf / division at full precision).
+#include "kernels_internal.h"
+#include "bf16_split.cuh"
+#include "ring.cuh"
+#include <cuda_fp16.h>
+#include <algorithm>
+
+namespace nt { namespace b200 {
+
+namespace {
+
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float decay_of(float z) { return expf(-expf(z)); }
+
+// ---- shift blends ----
+template <bool VEC>
+__global__ void __launch_bounds__(256) shift_mix_kernel(ShiftMix p, const float* __restrict__ h, const float* __restrict__ carried, int width, const int* __restrict__ pos_dev, int p0) {
+    pdl_launch_dependents();
+    pdl_wait();
+    constexpr int V = VEC ? 4 : 1;
+    const int i = (blockIdx.x * 256 + threadIdx.x) * V, t = blockIdx.y;
+    if (i >= width) return;
+    const size_t at = (size_t)t * width + i;
+    float c[V], d[V];
+    if constexpr (VEC) { const float4 f = *reinterpret_cast<const float4*>(h + at); c[0] = f.x; c[1] = f.y; c[2] = f.z; c[3] = f.w; } else c[0] = h[at];
+    const bool none = t == 0 && (pos_dev ? *pos_dev : p0) == 0;
+    const float* pr = t > 0 ? h + at - width : carried + i;
+#pragma unroll
+    for (int e = 0; e < V; e++) d[e] = (none ? 0.f : pr[e]) - c[e];
+    for (int s = 0; s < p.n; s++) {
+        float m[V];
+#pragma unroll
+        for (int e = 0; e < V; e++) m[e] = fmaf(d[e], p.mu[s][i + e], c[e]);
+        if (p.out[s]) {
+            if constexpr (VEC) *reinterpret_cast<float4*>(p.out[s] + at) = make_float4(m[0], m[1], m[2], m[3]);
+            else p.out[s][at] = m[0];
+        }
+        if (p.split[s]) {
+            __nv_bfloat16* hi = static_cast<__nv_bfloat16*>(p.split[s]);
+            if constexpr (VEC) split_store4(hi, hi + p.split_lo, at, m);
+            else split_store1(hi, hi + p.split_lo, at, m[0]);
+        }
+    }
+}
+
+__global__ void tanh_kernel(float* __restrict__ x, size_t n) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = tanhf(x[i]);
+}
+
+// grid (T), 256 threads: a warp per head for the bonus term, all threads for the decays
+__global__ void __launch_bounds__(256) wkv_prep_kernel(float* __restrict__ a, float* __restrict__ ruk, const float* __restrict__ r, const float* __restrict__ k,
+                                                       const float* __restrict__ w0, const float* __restrict__ u, int heads, int dim) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = heads * dim;
+    for (int h = warp; h < heads; h += 8) {
+        float s = 0.f;
+        for (int d = lane; d < dim; d += 32) { const int i = h * dim + d; s = fmaf(r[t * n + i] * u[i], k[t * n + i], s); }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xFFFFFFFFu, s, o);
+        if (lane == 0) ruk[t * heads + h] = s;
+    }
+    for (int i = threadIdx.x; i < n; i += 256) a[t * n + i] = decay_of(a[t * n + i] + w0[i]);
+}
+
+// ---- recurrence over rows ----
+constexpr int WR_TILE = 16;
+
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+// part[0..15] (one number per row and lane) -> sums over the LN lanes of a column: afterwards lane l holds, in part[0..N-1], the rows
+// first_row .. first_row + N - 1.  Every step halves the rows a lane is responsible for and sends the other half to its partner.
+template <int LN>
+__device__ __forceinline__ int reduce_rows(float (&part)[WR_TILE], int l) {
+    int base = 0;
+    constexpr int STEPS = LN == 1 ? 0 : LN == 2 ? 1 : LN == 4 ? 2 : LN == 8 ? 3 : LN == 16 ? 4 : 5;
+#pragma unroll
+    for (int s = 0; s < STEPS; s++) {
+        const int m = LN >> (s + 1);
+        const bool hi = (l & m) != 0;
+        if (s < 4) {
+            const int half = WR_TILE >> (s + 1);
+#pragma unroll
+            for (int j = 0; j < WR_TILE / 2; j++) {
+                if (j < half) {
+                    const float send = hi ? part[j] : part[j + half], keep = hi ? part[j + half] : part[j];
+                    part[j] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, m);
+                }
+            }
+            base += hi ? half : 0;
+        } else part[0] += __shfl_xor_sync(0xFFFFFFFFu, part[0], m);
+    }
+    return base;
+}
+
+// grid (ceil(dim / COLS), heads), 128 threads.  Lane l of a column holds state elements W * (c LN + l) + j, c < CH, j < W.
+template <int LN, int CH, int W>
+__global__ void __launch_bounds__(128) wkv_rows_kernel(float* __restrict__ out, const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v,
+                                                       const float* __restrict__ w, const float* __restrict__ ruk, float* __restrict__ state, int T, int heads, int dim,
+                                                       const int* __restrict__ pos_dev, int p0) {
+    constexpr int THREADS = 128, COLS = THREADS / LN, ROWS_LEFT = LN >= WR_TILE ? 1 : WR_TILE / LN;
+    extern __shared__ __align__(16) float sm[];
+    const int tile_floats = 3 * WR_TILE * dim + WR_TILE * COLS + WR_TILE;      // r | k | w [WR_TILE][dim], v [WR_TILE][COLS], ruk [WR_TILE]
+    const int buf_floats = (tile_floats + 3) & ~3;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.y, n = heads * dim;
+    const int col_l = threadIdx.x / LN, l = threadIdx.x % LN;
+    const int col = blockIdx.x * COLS + col_l;
+    const bool live = col < dim;
+    const bool fresh = (pos_dev ? *pos_dev : p0) == 0;
+    float* st = state + ((size_t)h * dim + (live ? col : 0)) * dim;
+    int d0[CH];
+    bool on[CH];
+    float S[CH][W];
+#pragma unroll
+    for (int c = 0; c < CH; c++) {
+        d0[c] = W * (c * LN + l);
+        on[c] = d0[c] < dim;
+#pragma unroll
+        for (int j = 0; j < W; j++) S[c][j] = 0.f;
+        if (on[c] && live && !fresh) {
+#pragma unroll
+            for (int j = 0; j < W; j++) S[c][j] = st[d0[c] + j];
+        }
+        if (!on[c]) d0[c] = 0;
+    }
+    auto load_tile = [&](int t0, int buf) {
+        float* sr = sm + (size_t)buf * buf_floats;
+        float* sk = sr + WR_TILE * dim;
+        float* sw = sk + WR_TILE * dim;
+        float* sv = sw + WR_TILE * dim;
+        float* sb = sv + WR_TILE * COLS;
+        const int nt = min(WR_TILE, T - t0), dv = dim / W;
+        for (int i = threadIdx.x; i < nt * dv; i += THREADS) {
+            const int tt = i / dv, d = (i - tt * dv) * W;
+            const size_t at = (size_t)(t0 + tt) * n + (size_t)h * dim + d;
+            if constexpr (W == 4) { cp_async16(sr + tt * dim + d, r + at); cp_async16(sk + tt * dim + d, k + at); cp_async16(sw + tt * dim + d, w + at); }
+            else { cp_async4(sr + tt * dim + d, r + at); cp_async4(sk + tt * dim + d, k + at); cp_async4(sw + tt * dim + d, w + at); }
+        }
+        for (int i = threadIdx.x; i < nt * COLS; i += THREADS) {
+            const int tt = i / COLS, c = blockIdx.x * COLS + i % COLS;
+            if (c < dim) cp_async4(sv + i, v + (size_t)(t0 + tt) * n + (size_t)h * dim + c);
+            else sv[i] = 0.f;
+        }
+        for (int i = threadIdx.x; i < nt; i += THREADS) cp_async4(sb + i, ruk + (size_t)(t0 + i) * heads + h);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    const int n_tiles = (T + WR_TILE - 1) / WR_TILE;
+    load_tile(0, 0);
+    for (int q = 0; q < n_tiles; q++) {
+        const int t0 = q * WR_TILE, nt = min(WR_TILE, T - t0), buf = q & 1;
+        if (q + 1 < n_tiles) {
+            load_tile(t0 + WR_TILE, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const float* sr = sm + (size_t)buf * buf_floats;
+        const float* sk = sr + WR_TILE * dim;
+        const float* sw = sk + WR_TILE * dim;
+        const float* sv = sw + WR_TILE * dim;
+        const float* sb = sv + WR_TILE * COLS;
+        float part[WR_TILE];
+        auto step = [&](int tt) {
+            const float vj = sv[tt * COLS + col_l];
+            float p = 0.f;
+#pragma unroll
+            for (int c = 0; c < CH; c++) {
+                float rr[W], kk[W], ww[W];
+                if constexpr (W == 4) {
+                    const float4 a = *reinterpret_cast<const float4*>(sr + tt * dim + d0[c]), b = *reinterpret_cast<const float4*>(sk + tt * dim + d0[c]),
+                                 e = *reinterpret_cast<const float4*>(sw + tt * dim + d0[c]);
+                    rr[0] = a.x; rr[1] = a.y; rr[2] = a.z; rr[3] = a.w; kk[0] = b.x; kk[1] = b.y; kk[2] = b.z; kk[3] = b.w; ww[0] = e.x; ww[1] = e.y; ww[2] = e.z; ww[3] = e.w;
+                } else { rr[0] = sr[tt * dim + d0[c]]; kk[0] = sk[tt * dim + d0[c]]; ww[0] = sw[tt * dim + d0[c]]; }
+                if (CH == 1 || on[c]) {
+#pragma unroll
+                    for (int j = 0; j < W; j++) { p = fmaf(rr[j], S[c][j], p); S[c][j] = fmaf(ww[j], S[c][j], kk[j] * vj); }
+                }
+            }
+            return (CH == 1 && !on[0]) ? 0.f : p;
+        };
+        if (nt == WR_TILE) {
+#pragma unroll
+            for (int tt = 0; tt < WR_TILE; tt++) part[tt] = step(tt);
+        } else {
+#pragma unroll
+            for (int tt = 0; tt < WR_TILE; tt++) part[tt] = tt < nt ? step(tt) : 0.f;
+        }
+        const int row0 = reduce_rows<LN>(part, l);
+#pragma unroll
+        for (int j = 0; j < ROWS_LEFT; j++) {
+            const int tt = row0 + j;
+            if (live && tt < nt && (LN <= WR_TILE || (l & 1) == 0))
+                out[(size_t)(t0 + tt) * n + (size_t)h * dim + col] = fmaf(sb[tt], sv[tt * COLS + col_l], part[j]);
+        }
+        __syncthreads();                       // the buffer is refilled by the load of tile q + 2
+    }
+    if (live) {
+#pragma unroll
+        for (int c = 0; c < CH; c++) {
+            if (on[c]) {
+#pragma unroll
+                for (int j = 0; j < W; j++) st[d0[c] + j] = S[c][j];
+            }
+        }
+    }
+}
+
+// grid (T), 256 threads, a warp per head
+__global__ void __launch_bounds__(256) wkv_out_norm_kernel(float* __restrict__ out, __nv_bfloat16* __restrict__ hi, size_t lo_off, const float* __restrict__ o,
+                                                           const float* __restrict__ gate, const float* __restrict__ norm, float eps, int heads, int dim) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const size_t row = (size_t)blockIdx.x * heads * dim;
+    for (int h = warp; h < heads; h += 8) {
+        const float* oh = o + row + (size_t)h * dim;
+        float ss = 0.f;
+        for (int d = lane; d < dim; d += 32) ss = fmaf(oh[d], oh[d], ss);
+#pragma unroll
+        for (int q = 16; q > 0; q >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, q);
+        const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+        for (int d = lane; d < dim; d += 32) {
+            const int c = h * dim + d;
+            const float y = oh[d] * inv * norm[c] * silu_f(gate[row + c]);
+            if (out) out[row + c] = y;
+            if (hi) split_store1(hi, hi + lo_off, row + c, y);
+        }
+    }
+}
+
+__device__ __forceinline__ float wld(const float* p, size_t i) { return __ldg(p + i); }
+__device__ __forceinline__ float wld(const __half* p, size_t i) { return __half2float(__ushort_as_half(__ldg(reinterpret_cast<const unsigned short*>(p) + i))); }
+__device__ __forceinline__ float wld(const __nv_bfloat16* p, size_t i) { return __uint_as_float((unsigned)__ldg(reinterpret_cast<const unsigned short*>(p) + i) << 16); }
+
+// grid (heads), 256 threads.  a1 [rank]: tanh(W_w1 m) of the token; W2 [heads * dim, rank].  8 lanes per value channel.
+constexpr int WT_LN = 8;
+template <typename T>
+__global__ void __launch_bounds__(256) wkv_token_kernel(float* __restrict__ out, const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v,
+                                                        const float* __restrict__ gate, const float* __restrict__ a1, const T* __restrict__ W2, const float* __restrict__ w0,
+                                                        const float* __restrict__ u, const float* __restrict__ norm, float* __restrict__ state, float eps, int rank,
+                                                        int dim, const int* __restrict__ pos_dev, int p0) {
+    extern __shared__ __align__(16) float sm[];
+    float *rs = sm, *ks = rs + dim, *ws = ks + dim, *os = ws + dim, *as = os + dim;      // [dim] x 4, [rank]
+    __shared__ float red[8];
+    __shared__ float bonus;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const size_t hb = (size_t)h * dim;
+    const bool fresh = (pos_dev ? *pos_dev : p0) == 0;
+    for (int i = threadIdx.x; i < rank; i += 256) as[i] = a1[i];
+    for (int d = threadIdx.x; d < dim; d += 256) { rs[d] = r[hb + d]; ks[d] = k[hb + d]; }
+    __syncthreads();
+    for (int d = warp; d < dim; d += 8) {
+        float z = 0.f;
+        for (int i = lane; i < rank; i += 32) z = fmaf(wld(W2, (hb + d) * rank + i), as[i], z);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) z += __shfl_xor_sync(0xFFFFFFFFu, z, o);
+        if (lane == 0) ws[d] = decay_of(z + w0[hb + d]);
+    }
+    if (warp == 0) {
+        float s = 0.f;
+        for (int d = lane; d < dim; d += 32) s = fmaf(rs[d] * u[hb + d], ks[d], s);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xFFFFFFFFu, s, o);
+        if (lane == 0) bonus = s;
+    }
+    __syncthreads();
+    const int l = threadIdx.x % WT_LN;
+    for (int j0 = 0; j0 < dim; j0 += 256 / WT_LN) {
+        const int j = j0 + threadIdx.x / WT_LN;
+        const bool live = j < dim;
+        float* st = state + (hb + (live ? j : 0)) * dim;
+        const float vj = live ? v[hb + j] : 0.f;
+        float p = 0.f;
+        if (dim % 4 == 0) {
+            for (int d = 4 * l; live && d < dim; d += 4 * WT_LN) {
+                float4 S = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st + d);
+                p = fmaf(rs[d], S.x, p); p = fmaf(rs[d + 1], S.y, p); p = fmaf(rs[d + 2], S.z, p); p = fmaf(rs[d + 3], S.w, p);
+                S.x = fmaf(ws[d], S.x, ks[d] * vj); S.y = fmaf(ws[d + 1], S.y, ks[d + 1] * vj);
+                S.z = fmaf(ws[d + 2], S.z, ks[d + 2] * vj); S.w = fmaf(ws[d + 3], S.w, ks[d + 3] * vj);
+                *reinterpret_cast<float4*>(st + d) = S;
+            }
+        } else {
+            for (int d = l; live && d < dim; d += WT_LN) {
+                const float S = fresh ? 0.f : st[d];
+                p = fmaf(rs[d], S, p);
+                st[d] = fmaf(ws[d], S, ks[d] * vj);
+            }
+        }
+#pragma unroll
+        for (int o = WT_LN / 2; o > 0; o >>= 1) p += __shfl_xor_sync(0xFFFFFFFFu, p, o);
+        if (l == 0 && live) os[j] = fmaf(bonus, vj, p);
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < dim; d += 256) ss = fmaf(os[d], os[d], ss);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    float tot = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) tot += red[w];
+    const float inv = 1.0f / sqrtf(tot / (float)dim + eps);
+    for (int d = threadIdx.x; d < dim; d += 256) out[hb + d] = os[d] * inv * norm[hb + d] * silu_f(gate[hb + d]);
+}
+
+template <int LN, int CH, int W>
+void launch_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int T, int heads, int dim, const int* pos_dev,
+                 int p0, cudaStream_t s) {
+    constexpr int COLS = 128 / LN;
+    const size_t tile = ((size_t)3 * WR_TILE * dim + (size_t)WR_TILE * COLS + WR_TILE + 3) & ~(size_t)3;
+    const size_t smem = sizeof(float) * 2 * tile;
+    static unsigned long long done = 0;
+    if (smem > 48 * 1024) opt_in_dynamic_smem(wkv_rows_kernel<LN, CH, W>, 200 * 1024, done);
+    launch_k(wkv_rows_kernel<LN, CH, W>, dim3((dim + COLS - 1) / COLS, heads), dim3(128), smem, s, out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0);
+}
+
+}  // namespace
+
+void shift_mix_rows(const ShiftMix& p, const float* h, float* carried, int T, int width, const int* pos_dev, int p0, cudaStream_t s) {
+    if (T <= 0) return;
+    NT_CHECK(p.n >= 1 && p.n <= ShiftMix::MAX, "shift_mix_rows: 1..5 blends");
+    bool vec = width % 4 == 0;
+    auto al = [&](const void* q) { if (reinterpret_cast<uintptr_t>(q) & 15) vec = false; };
+    al(h); al(carried);
+    for (int i = 0; i < p.n; i++) { al(p.mu[i]); al(p.out[i]); al(p.split[i]); }
+    const int per = vec ? 1024 : 256;
+    const dim3 grid((width + per - 1) / per, T);
+    if (vec) launch_k(shift_mix_kernel<true>, grid, dim3(256), 0, s, p, h, (const float*)carried, width, pos_dev, p0);
+    else launch_k(shift_mix_kernel<false>, grid, dim3(256), 0, s, p, h, (const float*)carried, width, pos_dev, p0);
+    count_launch();
+    copy(carried, h + (size_t)(T - 1) * width, width, s);
+}
+
+void tanh_rows(float* x, size_t n, cudaStream_t s) {
+    if (!n) return;
+    launch_k(tanh_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, x, n);
+    count_launch();
+}
+
+void wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int T, int heads, int dim, cudaStream_t s) {
+    if (T <= 0) return;
+    launch_k(wkv_prep_kernel, dim3(T), dim3(256), 0, s, a, ruk, r, k, w0, u, heads, dim);
+    count_launch();
+}
+
+void wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int T, int heads, int dim, const int* pos_dev, int p0,
+              cudaStream_t s) {
+    NT_CHECK(dim >= 1 && dim <= WKV_MAX_DIM, "wkv_rows: heads wider than 256 are not covered");
+    if (T <= 0) return;
+    const bool vec = dim % 4 == 0 && ((reinterpret_cast<uintptr_t>(r) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(w)) & 15) == 0;
+#define NT_WR(LN, CH, W) launch_rows<LN, CH, W>(out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0, s)
+    if (vec) {
+        if (dim <= 16) NT_WR(4, 1, 4);
+        else if (dim <= 32) NT_WR(8, 1, 4);
+        else if (dim <= 64) NT_WR(16, 1, 4);
+        else if (dim <= 128) NT_WR(16, 2, 4);
+        else NT_WR(32, 2, 4);
+    } else {
+        if (dim <= 8) NT_WR(8, 1, 1);
+        else if (dim <= 32) NT_WR(16, 2, 1);
+        else if (dim <= 128) NT_WR(16, 8, 1);
+        else NT_WR(16, 16, 1);
+    }
+#undef NT_WR
+    count_launch();
+}
+
+void wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int T, int heads, int dim, cudaStream_t s) {
+    if (T <= 0) return;
+    launch_k(wkv_out_norm_kernel, dim3(T), dim3(256), 0, s, out, static_cast<__nv_bfloat16*>(split), split_lo_offset(T, heads * dim), o, gate, norm, eps, heads, dim);
+    count_launch();
+}
+
+void wkv_token(float* out, const float* r, const float* k, const float* v, const float* gate, const float* a1, const void* W2, DType dt, const float* w0, const float* u,
+               const float* norm, float* state, float eps, int rank, int heads, int dim, const int* pos_dev, int p0, cudaStream_t s) {
+    NT_CHECK(dim >= 1 && dim <= WKV_MAX_DIM && rank >= 1, "wkv_token: heads wider than 256 are not covered");
+    const size_t smem = sizeof(float) * (4 * (size_t)dim + (size_t)rank);
+    NT_CHECK(smem <= 48 * 1024, "wkv_token: decay ranks above 11000 are not covered");
+#define NT_WT(TY) launch_k(wkv_token_kernel<TY>, dim3(heads), dim3(256), smem, s, out, r, k, v, gate, a1, static_cast<const TY*>(W2), w0, u, norm, state, eps, rank, dim, pos_dev, p0)
+    if (dt == DType::F32) NT_WT(float); else if (dt == DType::F16) NT_WT(__half); else if (dt == DType::BF16) NT_WT(__nv_bfloat16);
+    else NT_CHECK(false, "wkv_token: dense dtypes only");
+#undef NT_WT
+    count_launch();
+}
+
+}}  // namespace nt::b200
