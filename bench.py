@@ -964,6 +964,89 @@ def run_family_compare_savidra(args):
                       "dtype": "bf16 weights, f32 activations", "data": "synthetic", "rows": rows}))
 
 
+# width -> latent attention (shared by both models), recurrence (WKV heads x width against scan heads x width x state), experts
+FUVOZEN_SIZES = {
+    "w2048": dict(width=2048, latent=dict(heads=16, dim=64, rot_dim=64, vdim=128, kv_rank=256), q_rank=768, w_heads=32, w_dim=64, decay_rank=64, state=64, experts=16, eff=1408),
+    "w4096": dict(width=4096, latent=dict(heads=32, dim=64, rot_dim=64, vdim=128, kv_rank=512), q_rank=1536, w_heads=64, w_dim=64, decay_rank=128, state=64, experts=16, eff=1536),
+}
+
+
+def time_family_model(model, args, prompt_len, vocab, hbm):
+    """Prompt-pass and decode throughput of one model: CUDA events on the model's stream behind args.warmup steps; prompts differ between steps."""
+    import torch
+    from ntransformer_b200 import kernels as K
+
+    stream = torch.cuda.ExternalStream(model.stream)
+    prompts = [[token_at(i + 97 * j, vocab) for i in range(prompt_len)] for j in range(4)]
+    for i in range(args.warmup):
+        model.forward_async(prompts[i % 4], 0)
+    model.sync()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    n0 = K.launch_count()
+    psteps = max(3, min(args.steps, 8))
+    a.record(stream)
+    for i in range(psteps):
+        model.forward_async(prompts[i % 4], 0)
+    b.record(stream)
+    model.sync()
+    prefill = psteps * prompt_len / (a.elapsed_time(b) / 1e3)
+    dsteps = max(8, min(args.steps, 256))
+    for i in range(args.warmup):
+        model.forward_async([token_at(i, vocab)], prompt_len + i)
+    model.sync()
+    a.record(stream)
+    for i in range(dsteps):
+        model.forward_async([token_at(i + 5, vocab)], prompt_len + args.warmup + i)
+    b.record(stream)
+    model.sync()
+    ms = a.elapsed_time(b) / dsteps
+    bpt = model.bytes_per_token(prompt_len + args.warmup + dsteps // 2)
+    return {"prefill_tok_s": round(prefill, 1), "decode_tok_s": round(1e3 / ms, 1), "decode_ms": round(ms, 4), "decode_bytes_per_token": bpt,
+            "decode_frac_of_hbm_peak": round(bpt / (ms * 1e-3) / (hbm * 1e9), 3), "launches": int(K.launch_count() - n0)}
+
+
+def fuvozen_pair(z, vocab):
+    """(Fuvozen, Tanolorn) configurations of one size: recurrence + dense feed-forward, latent attention + experts, twice.  Equal feed-forward
+    weights: an ungated unit of 3 x width against a gated one of 2 x width; three routed experts and a shared one against four routed ones."""
+    from ntransformer_b200.model_spec import fuvozen_config, tanolorn_config
+
+    w, A = z["width"], z["latent"]
+    fc = fuvozen_config(vocab=vocab, width=w, w_heads=z["w_heads"], w_dim=z["w_dim"], decay_rank=z["decay_rank"], ff=3 * w, experts=z["experts"], top=3, eff=z["eff"],
+                        shared=z["eff"], window=1024, **A)
+    tc = tanolorn_config(vocab=vocab, width=w, pattern=("mamba2", "latent_attention", "mamba2", "latent_attention"), mlp=("dense", "moe", "dense", "moe"),
+                         q_rank=z["q_rank"], s_heads=z["w_heads"], s_vdim=z["w_dim"], state=z["state"], groups=8, norm_groups=8, ff=2 * w, experts=z["experts"], top=4,
+                         eff=z["eff"], route_groups=None, side=0, **A)
+    return fc, tc
+
+
+def run_family_compare_fuvozen(args):
+    """--family-compare --family fuvozen: prompt-pass and decode throughput of the Fuvozen family (BF16 weights; WKV time mixers alternating
+    with windowed latent attention, mixer and feed-forward in parallel, average over depth, grouped norms, experts with a shared one)
+    beside the closest existing family (Tanolorn: state-space scans alternating with latent attention, gated experts) at equal width, layer
+    count, heads, latent rank, recurrent state and active feed-forward weights."""
+    import torch
+    from ntransformer_b200.engine import Model
+    from ntransformer_b200.model_spec import fuvozen_random_tensors, tanolorn_random_tensors
+
+    torch.cuda.set_device(0)
+    vocab, prompt_len, max_seq = 32000, 2048, 4096
+    hbm, hbm_src = measured_peak_hbm()
+    rows = []
+    for name, z in FUVOZEN_SIZES.items():
+        fc, tc = fuvozen_pair(z, vocab)
+        row = {"size": name, "layers": 4, "prompt_tokens": prompt_len, "decode_context": prompt_len}
+        for label, make in (("fuvozen_bf16", lambda: Model.from_config_json(fc, fuvozen_random_tensors(fc), max_context=max_seq)),
+                            ("tanolorn_bf16", lambda: Model.from_config_json(tc, tanolorn_random_tensors(tc), max_context=max_seq))):
+            model = make()
+            row[label] = time_family_model(model, args, prompt_len, vocab, hbm)
+            model.close()
+            del model
+            torch.cuda.empty_cache()
+        rows.append(row)
+    print(json.dumps({"metric": "family_compare", "family": "fuvozen", "unit": "tok/s", "hbm_peak_gbs": hbm, "hbm_peak_source": hbm_src,
+                      "dtype": "bf16 weights, f32 activations", "data": "synthetic", "rows": rows}))
+
+
 def run_family_compare(args):
     """--family-compare: prompt-pass and decode throughput of the Zelunex family (BF16 weights, windowed attention) beside the
     closest GGUF family member (Llama block, F16 weights, full causal attention) at equal layer sizes.  Device-timed with CUDA
@@ -1040,8 +1123,8 @@ def main():
     ap.add_argument("--all-errs", action="store_true", help="--check only: list the error of every step, not the first 8")
     ap.add_argument("--family-compare", action="store_true",
                     help="instead of the workload: Zelunex beside the Llama block at equal layer sizes, prompt pass and decode (1 GPU)")
-    ap.add_argument("--family", default="zelunex", choices=["zelunex", "vebotar", "tanolorn", "savidra"],
-                    help="--family-compare only: zelunex beside the Llama block (default), vebotar beside zelunex, tanolorn beside vebotar, or savidra beside tanolorn")
+    ap.add_argument("--family", default="zelunex", choices=["zelunex", "vebotar", "tanolorn", "savidra", "fuvozen"],
+                    help="--family-compare only: zelunex beside the Llama block (default), vebotar beside zelunex, tanolorn beside vebotar, or savidra / fuvozen beside tanolorn")
     ap.add_argument("--per-token-prompt", action="store_true", help="--check only: our engine replays the prompt token by token like the reference")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
@@ -1051,7 +1134,8 @@ def main():
         sys.exit("bench.py --gpus N > 1 must be launched with torch.distributed.run (one rank per GPU)")
     if args.family_compare:
         if rank == 0:
-            {"vebotar": run_family_compare_vebotar, "tanolorn": run_family_compare_tanolorn, "savidra": run_family_compare_savidra}.get(args.family, run_family_compare)(args)
+            {"vebotar": run_family_compare_vebotar, "tanolorn": run_family_compare_tanolorn, "savidra": run_family_compare_savidra,
+             "fuvozen": run_family_compare_fuvozen}.get(args.family, run_family_compare)(args)
     elif args.check:
         run_check(args, rank, world)
     elif args.impl == "reference":

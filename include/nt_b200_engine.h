@@ -123,6 +123,40 @@ void nt_b200_moe_route_scored(int* sel, float* wt, const float* h, const float* 
                               int width, int tokens, void* stream);
 void nt_b200_moe_glu_experts(float* y, const float* h, const int* sel, const float* wt, const void* const* gate_tab, const void* const* up_tab,
                              const void* const* down_tab, int dtype, int experts, int top, int ff, int width, int tokens, int mode, void* scratch, void* stream);
+/* ---- kernels of the Fuvozen family (rows of a depth-averaged parallel block, WKV time mixer, ...); F32 unless a dtype is given ---- */
+/* prev_dev: one int, the token before the step's first row.  bigram null: the plain embedding.  x1 may be null. */
+void nt_b200_embed_pair_rows(float* x0, float* x1, const void* embed, const void* bigram, int dtype, const int* tokens_dev, const int* prev_dev, int tokens, int width,
+                             long long buckets, long long mul_prev, long long mul_cur, int p0, void* stream);
+/* X: n slots of [rows, width] F32, `slot` floats apart; coef null: the last slot.  split (may be null): BF16 hi / lo workspace of a tensor-core GEMM.
+ * n_mix > 0 (one row): mu / mix_out hold that many pointers. */
+void nt_b200_depth_norm_rows(const float* X, long long slot, int n, const float* coef, float* x_out, float* h_out, void* split, const float* gain, float eps, int rows,
+                             int width, int groups, int n_mix, const void* const* mu, void* const* mix_out, float* carried, int p0, void* stream);
+void nt_b200_shift_mix_rows(int n, const void* const* mu, void* const* out, void* const* split, const float* h, float* carried, int rows, int width, int p0, void* stream);
+void nt_b200_wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int tokens, int heads, int dim, void* stream);
+void nt_b200_wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int tokens, int heads, int dim, int p0,
+                      void* stream);
+void nt_b200_wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int tokens, int heads, int dim, void* stream);
+void nt_b200_wkv_token(float* out, const float* r, const float* k, const float* v, const float* gate, const float* a1, const void* w2, int dtype, const float* w0,
+                       const float* u, const float* norm, float* state, float eps, int rank, int heads, int dim, int p0, void* stream);
+void nt_b200_xielu_rows(float* out, void* split, const float* in, const float* act, int rows, int cols, void* stream);
+/* n matrices with an input each; act[i]: 0 none, 1 tanh, 2 xIELU (act_p[i]: its two numbers) */
+void nt_b200_gemv_multi(int n, const void* const* W, const int* dtype, const void* const* x, void* const* y, const int* out, const int* K, const int* act,
+                        const void* const* act_p, void* stream);
+/* y (+)= W1 x1 + sum_k wt[k] table[sel[k]] x_k (top 0: none) + W2 x2 (W2 null: none) */
+void nt_b200_gemv_sum(float* y, int out, int dtype, int add, const void* W1, const float* x1, int K1, const void* const* table, const int* sel, const float* wt, int top,
+                      const float* xe, int Ke, const void* W2, const float* x2, int K2, void* stream);
+/* Router whose weights are the softmax over all experts times scale */
+void nt_b200_moe_route_all(int* sel, float* wt, const float* h, const float* router, int experts, int top, float scale, int width, int tokens, void* stream);
+/* One token: the choice from the router's logits, then silu(gate) * up of the chosen experts and of the gated shared expert -> act [top * ff + shared_ff] */
+void nt_b200_moe_choose_up(float* act, int* sel, float* wt, const float* h, const float* logits, const void* const* gate_tab, const void* const* up_tab,
+                           const void* shared_gate, const void* shared_up, int dtype, int experts, int top, float scale, int ff, int shared_ff, int width, void* stream);
+/* Windowed attention over one key / value head stored as rows (keys: the first dim numbers, values: the first vdim).  form 0: all heads from one
+ * copy of the rows (returns -1 when the shape is not covered), form 1: one CTA per (query, head).  window 0: full causal. */
+int nt_b200_attention_rows_window(float* out, const float* Q, const void* cache, int cache_dtype, int tokens, int p0, int max_seq, int heads, int dim, int vdim, int row,
+                                  float scale, int window, int form, void* stream);
+/* Tiled windowed attention over BF16 per-head keys [rows, heads, kw] and values [rows, heads, vw] */
+void nt_b200_attention_heads_window(float* out, const float* Q, const void* k, const void* v, int tokens, int p0, int rows, int heads, int kw, int vw, float scale,
+                                    int window, void* stream);
 
 /* forward(tokens[seq_len], start_pos): logits of the last token. logits_host may be NULL.  Returns 0. */
 int  nt_model_forward(nt_model_t m, const int* tokens_host, int seq_len, int start_pos, float* logits_host);

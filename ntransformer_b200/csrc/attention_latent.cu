@@ -102,6 +102,7 @@ __global__ void __launch_bounds__(256) latent_q_absorb_kernel(float* __restrict_
                                                               int dim, int rot_dim, int kv_rank, int dims, int interleaved, double log2_base,
                                                               const int* __restrict__ pos_dev, int p0) {
     extern __shared__ __align__(16) float qs[];           // [LT][dim + rot_dim] | partial sums [4][64][LT]
+    if (T == 1) for (int d = threadIdx.x; d < dim; d += 256) l2_prefetch(W_uk + ((size_t)blockIdx.y * dim + d) * kv_rank + blockIdx.z * 64, min(64, kv_rank - (int)blockIdx.z * 64) * sizeof(WT), 0, 1);
     pdl_launch_dependents();
     pdl_wait();
     const int t0 = blockIdx.x * LT, h = blockIdx.y, qd = dim + rot_dim, od = kv_rank + rot_dim;
@@ -147,6 +148,7 @@ template <typename WT>
 __global__ void __launch_bounds__(256) latent_v_up_kernel(float* __restrict__ out, const float* __restrict__ ol, const WT* __restrict__ W_uv, int T, int heads,
                                                           int vdim, int kv_rank) {
     extern __shared__ __align__(16) float os[];           // [LT][kv_rank]
+    if (T == 1) l2_prefetch(W_uv + ((size_t)blockIdx.y * vdim + blockIdx.z * 32) * kv_rank, (size_t)min(32, vdim - (int)blockIdx.z * 32) * kv_rank * sizeof(WT), threadIdx.x, 256);
     pdl_launch_dependents();
     pdl_wait();
     const int t0 = blockIdx.x * LT, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;

@@ -199,6 +199,54 @@ __global__ void __launch_bounds__(DV_WARPS * 32) gemv_dense_kernel(DenseMats m, 
     }
 }
 
+// n floats into shared memory by the whole CTA, 16 bytes at a time when the source is aligned.  planar (n % 8 == 0): the even and the odd
+// 16-byte pieces go to the first and the second half of dst, so that lanes holding consecutive 8-number pieces of a 16-bit weight row read
+// consecutive 16-byte words of either half (no bank conflicts).
+__device__ __forceinline__ void stage_floats(float* dst, const float* src, int n, bool planar) {
+    const bool al = (reinterpret_cast<uintptr_t>(src) & 15) == 0;
+    if (planar) {
+        const int half = n >> 1, q = n >> 2;
+        if (al) {
+#pragma unroll 4
+            for (int i = threadIdx.x; i < q; i += blockDim.x) *reinterpret_cast<float4*>(dst + ((i & 1) ? half : 0) + (i >> 1) * 4) = *reinterpret_cast<const float4*>(src + 4 * i);
+        } else {
+            for (int i = threadIdx.x; i < n; i += blockDim.x) dst[((i & 4) ? half : 0) + (i >> 3) * 4 + (i & 3)] = src[i];
+        }
+        return;
+    }
+    int done = 0;
+    if (al) {
+        done = n & ~3;
+#pragma unroll 4
+        for (int i = threadIdx.x * 4; i < done; i += blockDim.x * 4) *reinterpret_cast<float4*>(dst + i) = *reinterpret_cast<const float4*>(src + i);
+    }
+    for (int i = done + threadIdx.x; i < n; i += blockDim.x) dst[i] = src[i];
+}
+// acc += <the 16-byte weight piece w, its numbers of the staged vector>; v: the piece's index in the row of K numbers
+template <typename T>
+__device__ __forceinline__ float piece_dot(const uint4& w, const float* xs, int K, int v, float acc) {
+    constexpr int P = Elem<T>::PER16;
+    float f[P];
+    Elem<T>::unpack(w, f);
+    const float4 a = *reinterpret_cast<const float4*>(xs + 4 * v);
+    acc = fmaf(f[0], a.x, acc); acc = fmaf(f[1], a.y, acc); acc = fmaf(f[2], a.z, acc); acc = fmaf(f[3], a.w, acc);
+    if constexpr (P == 8) {
+        const float4 b = *reinterpret_cast<const float4*>(xs + (K >> 1) + 4 * v);
+        acc = fmaf(f[4], b.x, acc); acc = fmaf(f[5], b.y, acc); acc = fmaf(f[6], b.z, acc); acc = fmaf(f[7], b.w, acc);
+    }
+    return acc;
+}
+// batch of up to 128 pieces from v0 on, four 16-byte loads in flight per lane
+template <typename T>
+__device__ __forceinline__ float batch_dot(const unsigned char* row, const float* xs, int K, int nv, int v0, int lane, float acc) {
+    uint4 w[4];
+#pragma unroll
+    for (int u = 0; u < 4; u++) { const int v = v0 + lane + 32 * u; w[u] = v < nv ? ld_stream16(row + (size_t)v * 16) : make_uint4(0u, 0u, 0u, 0u); }
+#pragma unroll
+    for (int u = 0; u < 4; u++) acc = piece_dot<T>(w[u], xs, K, min(v0 + lane + 32 * u, nv - 1), acc);       // past the end the weights are zeros: any valid input will do
+    return acc;
+}
+
 // ---- several matrices, each with its own input vector ----
 struct MultiDev {
     struct One { const unsigned char* W; size_t pitch; const float* x; float* y; const float* act_p; int out, K, act, f32, vec, cta_end; };
@@ -214,53 +262,101 @@ __global__ void __launch_bounds__(DV_WARPS * 32) gemv_multi_kernel(const __grid_
     while (mi + 1 < md.n && (int)blockIdx.x >= md.m[mi].cta_end) { first = md.m[mi].cta_end; mi++; }
     const MultiDev::One& m = md.m[mi];
     const int ctas = m.cta_end - first, r0 = ((int)blockIdx.x - first) * DV_WARPS + warp;
-    pdl_launch_dependents();
+    const size_t row_bytes = (size_t)m.K * (m.f32 ? sizeof(float) : sizeof(T));
+    for (int r = r0; r < m.out; r += ctas * DV_WARPS) l2_prefetch(m.W + (size_t)r * m.pitch, row_bytes, lane, 32);
     pdl_wait();
-    for (int i = threadIdx.x; i < m.K; i += DV_WARPS * 32) xs[i] = m.x[i];
+    const bool wide = !m.f32 && m.vec;                    // 16-bit rows in whole pieces: planar staging
+    stage_floats(xs, m.x, m.K, wide && Elem<T>::PER16 == 8);
     __syncthreads();
     float a = 0.f, b = 0.f;
     if (m.act == GEMV_ACT_XIELU) { a = softplus_f(m.act_p[0]); b = softplus_f(m.act_p[1]); }
     for (int r = r0; r < m.out; r += ctas * DV_WARPS) {
         const unsigned char* row = m.W + (size_t)r * m.pitch;
-        float v = m.f32 ? dense_row_dot<float>(row, xs, m.K, lane, m.vec) : dense_row_dot<T>(row, xs, m.K, lane, m.vec);
+        float v = 0.f;
+        if (wide) {
+            const int nv = m.K / Elem<T>::PER16;
+            for (int v0 = 0; v0 < nv; v0 += 128) v = batch_dot<T>(row, xs, m.K, nv, v0, lane, v);
+            v = warp_sum(v);
+        } else v = m.f32 ? dense_row_dot<float>(row, xs, m.K, lane, m.vec) : dense_row_dot<T>(row, xs, m.K, lane, m.vec);
         if (lane == 0) {
             if (m.act == GEMV_ACT_TANH) v = tanhf(v);
             else if (m.act == GEMV_ACT_XIELU) v = xielu_f(v, a, b);
             m.y[r] = v;
         }
     }
+    pdl_launch_dependents();       // late: CTAs of a small dependent grid placed while this one fills the SMs would crowd onto the few that free up first
 }
 
 // ---- y[r] (+)= sum over terms of <W[r], x> (routed term: sum_k wt[k] <table[sel[k]][r], x_k>) ----
 struct SumDev {
     struct One { const unsigned char* W; const void* const* table; const int* sel; const float* wt; const float* x; int K, top, vec, at; };
     One t[GEMV_SUM_MAX_TERMS];
-    int n, out, add;
+    int n, out, add, nw;
     float* y;
 };
+// A CTA of SV_WARPS warps owns SV_WARPS / nw rows at a time, nw warps per row: the batches of 128 16-byte pieces of a row's terms (of all terms,
+// one count) go round the row's warps; their sums meet in shared memory in a fixed order.
+constexpr int SV_WARPS = 16;
 template <typename T>
-__global__ void __launch_bounds__(DV_WARPS * 32) gemv_sum_kernel(const __grid_constant__ SumDev sd) {
-    extern __shared__ __align__(16) float xs[];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    pdl_launch_dependents();
-    pdl_wait();
-    for (int q = 0; q < sd.n; q++) {
-        const int total = sd.t[q].K * max(1, sd.t[q].top);
-        for (int i = threadIdx.x; i < total; i += DV_WARPS * 32) xs[sd.t[q].at + i] = sd.t[q].x[i];
+__device__ __forceinline__ float row_batches(const unsigned char* row, const float* xs, int K, int lane, bool vec, int& count, int j, int nw) {
+    constexpr int P = Elem<T>::PER16;
+    float acc = 0.f;
+    if (vec) {
+        const int nv = K / P;
+        for (int v0 = 0; v0 < nv; v0 += 128) {
+            if (count++ % nw != j) continue;
+            acc = batch_dot<T>(row, xs, K, nv, v0, lane, acc);
+        }
+    } else {
+        for (int i0 = 0; i0 < K; i0 += 1024) {
+            if (count++ % nw != j) continue;
+            for (int i = i0 + lane; i < min(K, i0 + 1024); i += 32) acc = fmaf(Elem<T>::one(row, i), xs[i], acc);
+        }
     }
+    return acc;
+}
+template <typename T>
+__global__ void __launch_bounds__(SV_WARPS * 32) gemv_sum_kernel(const __grid_constant__ SumDev sd) {
+    extern __shared__ __align__(16) float xs[];
+    __shared__ float part[SV_WARPS];
+    __shared__ const unsigned char* routed[256];       // the chosen experts' matrices and weights of a routed term
+    __shared__ float routed_w[256];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = sd.nw, rows = SV_WARPS / nw, j = warp % nw, rl = warp / nw;
+    for (int r = blockIdx.x * rows + rl; r < sd.out; r += gridDim.x * rows)
+        for (int q = 0; q < sd.n; q++)
+            if (!sd.t[q].table) l2_prefetch(sd.t[q].W + (size_t)r * sd.t[q].K * sizeof(T), (size_t)sd.t[q].K * sizeof(T), lane + 32 * j, 32 * nw);
+    pdl_wait();
+    for (int q = 0; q < sd.n; q++)
+        if (sd.t[q].table)
+            for (int k = threadIdx.x; k < sd.t[q].top; k += SV_WARPS * 32) { routed[k] = static_cast<const unsigned char*>(sd.t[q].table[sd.t[q].sel[k]]); routed_w[k] = sd.t[q].wt[k]; }
+    for (int q = 0; q < sd.n; q++)
+        for (int k = 0; k < sd.t[q].top; k++) stage_floats(xs + sd.t[q].at + k * sd.t[q].K, sd.t[q].x + (size_t)k * sd.t[q].K, sd.t[q].K, sd.t[q].vec && Elem<T>::PER16 == 8);
     __syncthreads();
-    for (int r = blockIdx.x * DV_WARPS + warp; r < sd.out; r += gridDim.x * DV_WARPS) {
+    for (int base = blockIdx.x * rows; base < sd.out; base += gridDim.x * rows) {
+        const int r = base + rl;
         float acc = 0.f;
-        for (int q = 0; q < sd.n; q++) {
-            const SumDev::One& t = sd.t[q];
-            const size_t off = (size_t)r * t.K * sizeof(T);
-            if (!t.table) acc += dense_row_part<T>(t.W + off, xs + t.at, t.K, lane, t.vec);
-            else for (int k = 0; k < t.top; k++)
-                acc = fmaf(t.wt[k], dense_row_part<T>(static_cast<const unsigned char*>(t.table[t.sel[k]]) + off, xs + t.at + k * t.K, t.K, lane, t.vec), acc);
+        if (r < sd.out) {
+            int count = 0;
+            for (int q = 0; q < sd.n; q++) {
+                const SumDev::One& t = sd.t[q];
+                const size_t off = (size_t)r * t.K * sizeof(T);
+                if (!t.table) acc += row_batches<T>(t.W + off, xs + t.at, t.K, lane, t.vec, count, j, nw);
+                else for (int k = 0; k < t.top; k++)
+                    acc = fmaf(routed_w[k], row_batches<T>(routed[k] + off, xs + t.at + k * t.K, t.K, lane, t.vec, count, j, nw), acc);
+            }
         }
         acc = warp_sum(acc);
-        if (lane == 0) sd.y[r] = sd.add ? sd.y[r] + acc : acc;
+        if (lane == 0) part[warp] = acc;
+        __syncthreads();
+        if (threadIdx.x < rows && base + (int)threadIdx.x < sd.out) {
+            float v = 0.f;
+            for (int w = 0; w < nw; w++) v += part[threadIdx.x * nw + w];
+            float* y = sd.y + base + threadIdx.x;
+            *y = sd.add ? *y + v : v;
+        }
+        __syncthreads();
     }
+    pdl_launch_dependents();
 }
 
 template <bool VEC>
@@ -428,8 +524,11 @@ void gemv_sum(float* y, const SumTerm* terms, int n, int out, DType dt, bool add
     SumDev sd{};
     sd.n = n; sd.out = out; sd.add = add ? 1 : 0; sd.y = y;
     int at = 0;
+    int n_routed = 0;
     for (int i = 0; i < n; i++) {
         const SumTerm& t = terms[i];
+        if (t.table) n_routed++;
+        NT_CHECK(!t.table || (n_routed == 1 && t.top >= 1 && t.top <= 256), "gemv_sum: one routed term of at most 256 chosen matrices");
         SumDev::One& o = sd.t[i];
         o.W = static_cast<const unsigned char*>(t.W); o.table = t.table; o.sel = t.sel; o.wt = t.wt; o.x = t.x; o.K = t.K; o.top = t.table ? t.top : 1; o.at = at;
         o.vec = t.K % (dt == DType::F32 ? 4 : 8) == 0 && (t.table ? t.table_aligned : (reinterpret_cast<uintptr_t>(t.W) & 15) == 0);
@@ -437,10 +536,13 @@ void gemv_sum(float* y, const SumTerm* terms, int n, int out, DType dt, bool add
     }
     const size_t smem = (size_t)at * sizeof(float);
     NT_CHECK(smem <= 200 * 1024, "gemv_sum: the input vectors do not fit in shared memory");
-    const int resident = (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)(220 * 1024) / (smem + 1024))) * 148;
-    const int grid = std::min((out + DV_WARPS - 1) / DV_WARPS, resident);
+    // warps per row: as many as keep the grid within what is resident at once (64 warps per SM)
+    const int per_sm = (int)std::max<size_t>(1, std::min<size_t>(4, (size_t)(220 * 1024) / (smem + 1024)));
+    sd.nw = 1;
+    while (sd.nw < 4 && (long)out * sd.nw * 2 <= (long)148 * per_sm * SV_WARPS) sd.nw *= 2;
+    const int rows = SV_WARPS / sd.nw, grid = std::min((out + rows - 1) / rows, 148 * per_sm);
 #define NT_SV(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(gemv_sum_kernel<TY>, 200 * 1024, done); \
-                    launch_k(gemv_sum_kernel<TY>, dim3(grid), dim3(DV_WARPS * 32), smem, s, sd); }
+                    launch_k(gemv_sum_kernel<TY>, dim3(grid), dim3(SV_WARPS * 32), smem, s, sd); }
     if (dt == DType::F32) NT_SV(float) else if (dt == DType::F16) NT_SV(__half) else NT_SV(__nv_bfloat16)
 #undef NT_SV
     count_launch();

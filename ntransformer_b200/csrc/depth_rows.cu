@@ -59,9 +59,13 @@ constexpr int DN_KEEP = 4;       // packs of a thread that stay in registers bet
 template <int VEC>
 __global__ void __launch_bounds__(256) depth_norm_kernel(DepthNorm p) {
     __shared__ float red[8];
+    const int per = p.width / p.groups, c0 = blockIdx.y * per, n = per / VEC, nt = blockDim.x;
+    if (p.n_mix > 0) {
+        l2_prefetch(p.gain + c0, (size_t)per * sizeof(float), threadIdx.x, nt);
+        for (int s = 0; s < p.n_mix; s++) l2_prefetch(p.mu[s] + c0, (size_t)per * sizeof(float), threadIdx.x, nt);
+    }
     pdl_launch_dependents();
     pdl_wait();
-    const int per = p.width / p.groups, c0 = blockIdx.y * per, n = per / VEC, nt = blockDim.x;
     const size_t row = (size_t)blockIdx.x * p.width + c0;
     auto blend = [&](int i) {
         Pack<VEC> a;

@@ -121,6 +121,14 @@ int nt_model_dir_describe(const char* dir, char* out, size_t cap) {
             text += std::string(" ff_kind=") + (L.ff == 0 ? "none" : L.ff_kind == FfKind::GLU ? "dense" : "moe") + " experts=" + std::to_string(L.experts) + " top=" +
                     std::to_string(L.top) + " route_groups=" + std::to_string(L.route.groups) + "/" + std::to_string(L.route.keep) + " side=" + std::to_string(cfg.side_dim);
         }
+        if (L.form == BlockForm::PARALLEL && L.mixer != MixerKind::ATTN_WINDOW) {
+            text += std::string(" mixer=") + (L.mixer == MixerKind::ATTN_LATENT ? "latent" : "wkv");
+            if (L.mixer == MixerKind::ATTN_LATENT) text += " kv_rank=" + std::to_string(L.latent.kv_rank) + " rot_dim=" + std::to_string(L.latent.rot_dim) + " rot=" + std::to_string(L.rot.dims);
+            else text += " decay_rank=" + std::to_string(L.wkv.decay_rank);
+            text += std::string(" ff_kind=") + (L.ff == 0 ? "none" : L.ff_kind == FfKind::MLP ? "dense" : "moe") + " experts=" + std::to_string(L.experts) + " top=" + std::to_string(L.top) +
+                    " route_scale=" + std::to_string(L.route.scale) + " shared_ff=" + std::to_string(L.shared_ff) + " norm_groups=" + std::to_string(cfg.norm_groups) +
+                    " buckets=" + std::to_string(cfg.bigram_buckets);
+        }
         if (L.form == BlockForm::SUM_NORM) {
             auto mixer_text = [](const LayerSpec& M) {
                 if (M.mixer == MixerKind::DELTA_RULE)
@@ -421,6 +429,108 @@ void nt_b200_moe_glu_experts(float* y, const float* h, const int* sel, const flo
     glu_bias_mul(act_rows, gate_rows, act_rows, nullptr, nullptr, tokens * top, ff, false, s);
     moe_expert_down_rows(y_rows, act_rows, work, w, tokens, s);
     moe_combine(y, y_rows, work, wt, nullptr, nullptr, tokens, experts, top, width, s);
+}
+// prev_dev: one int, the token before the step's first row.  bigram null: the plain embedding.  x1 may be null.
+void nt_b200_embed_pair_rows(float* x0, float* x1, const void* embed, const void* bigram, int dtype, const int* tokens_dev, const int* prev_dev, int tokens, int width,
+                             long long buckets, long long mul_prev, long long mul_cur, int p0, void* stream) {
+    embed_bigram_rows(x0, x1, embed, (nt::DType)dtype, bigram, (nt::DType)dtype, tokens_dev, prev_dev, tokens, width, buckets, mul_prev, mul_cur, nullptr, p0,
+                      static_cast<cudaStream_t>(stream));
+}
+// X: n slots of [rows, width] F32, `slot` floats apart; coef null: the last slot.  split (may be null): BF16 hi / lo workspace of a tensor-core GEMM.
+// n_mix > 0 (one row): mu / mix_out hold that many pointers.
+void nt_b200_depth_norm_rows(const float* X, long long slot, int n, const float* coef, float* x_out, float* h_out, void* split, const float* gain, float eps, int rows,
+                             int width, int groups, int n_mix, const void* const* mu, void* const* mix_out, float* carried, int p0, void* stream) {
+    DepthNorm p;
+    p.X = X; p.slot = (size_t)slot; p.n = n; p.coef = coef; p.x_out = x_out; p.h_out = h_out; p.split = split; p.split_lo = ((size_t)rows + 127) / 128 * 128 * (size_t)width;
+    p.gain = gain; p.eps = eps; p.width = width; p.groups = groups; p.carried = carried; p.p0 = p0;
+    NT_CHECK(n_mix >= 0 && n_mix <= DepthNorm::MAX_MIX, "nt_b200_depth_norm_rows: up to five shift blends");
+    p.n_mix = n_mix;
+    for (int i = 0; i < n_mix; i++) { p.mu[i] = static_cast<const float*>(mu[i]); p.mix_out[i] = static_cast<float*>(mix_out[i]); }
+    depth_norm_rows(p, rows, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_shift_mix_rows(int n, const void* const* mu, void* const* out, void* const* split, const float* h, float* carried, int rows, int width, int p0, void* stream) {
+    ShiftMix p;
+    NT_CHECK(n >= 1 && n <= ShiftMix::MAX, "nt_b200_shift_mix_rows: 1..5 blends");
+    p.n = n; p.split_lo = ((size_t)rows + 127) / 128 * 128 * (size_t)width;
+    for (int i = 0; i < n; i++) { p.mu[i] = static_cast<const float*>(mu[i]); p.out[i] = static_cast<float*>(out[i]); p.split[i] = split[i]; }
+    shift_mix_rows(p, h, carried, rows, width, nullptr, p0, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int tokens, int heads, int dim, void* stream) {
+    wkv_prep(a, ruk, r, k, w0, u, tokens, heads, dim, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int tokens, int heads, int dim, int p0,
+                      void* stream) {
+    wkv_rows(out, r, k, v, w, ruk, state, tokens, heads, dim, nullptr, p0, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int tokens, int heads, int dim, void* stream) {
+    wkv_out_norm(out, split, o, gate, norm, eps, tokens, heads, dim, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_wkv_token(float* out, const float* r, const float* k, const float* v, const float* gate, const float* a1, const void* w2, int dtype, const float* w0,
+                       const float* u, const float* norm, float* state, float eps, int rank, int heads, int dim, int p0, void* stream) {
+    wkv_token(out, r, k, v, gate, a1, w2, (nt::DType)dtype, w0, u, norm, state, eps, rank, heads, dim, nullptr, p0, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_xielu_rows(float* out, void* split, const float* in, const float* act, int rows, int cols, void* stream) {
+    xielu_rows(out, split, in, act, rows, cols, static_cast<cudaStream_t>(stream));
+}
+// n matrices with an input each; act[i]: 0 none, 1 tanh, 2 xIELU (act_p[i]: its two numbers)
+void nt_b200_gemv_multi(int n, const void* const* W, const int* dtype, const void* const* x, void* const* y, const int* out, const int* K, const int* act,
+                        const void* const* act_p, void* stream) {
+    MultiMat m[DENSE_MAX_MATS];
+    NT_CHECK(n >= 1 && n <= DENSE_MAX_MATS, "nt_b200_gemv_multi: too many matrices");
+    for (int i = 0; i < n; i++) {
+        m[i].W = W[i]; m[i].dtype = (nt::DType)dtype[i]; m[i].x = static_cast<const float*>(x[i]); m[i].y = static_cast<float*>(y[i]); m[i].out = out[i]; m[i].K = K[i];
+        m[i].act = (GemvAct)act[i]; m[i].act_p = static_cast<const float*>(act_p[i]);
+    }
+    gemv_multi(m, n, static_cast<cudaStream_t>(stream));
+}
+// y (+)= W1 x1 + sum_k wt[k] table[sel[k]] x_k (top 0: none) + W2 x2 (W2 null: none)
+void nt_b200_gemv_sum(float* y, int out, int dtype, int add, const void* W1, const float* x1, int K1, const void* const* table, const int* sel, const float* wt, int top,
+                      const float* xe, int Ke, const void* W2, const float* x2, int K2, void* stream) {
+    SumTerm t[3];
+    int n = 0;
+    t[n].W = W1; t[n].x = x1; t[n++].K = K1;
+    if (top > 0) { t[n].table = table; t[n].sel = sel; t[n].wt = wt; t[n].top = top; t[n].x = xe; t[n++].K = Ke; }
+    if (W2) { t[n].W = W2; t[n].x = x2; t[n++].K = K2; }
+    gemv_sum(y, t, n, out, (nt::DType)dtype, add != 0, static_cast<cudaStream_t>(stream));
+}
+// Router whose weights are the softmax over all experts times scale
+void nt_b200_moe_route_all(int* sel, float* wt, const float* h, const float* router, int experts, int top, float scale, int width, int tokens, void* stream) {
+    MoeWeights w;
+    w.router = router; w.experts = experts; w.top = top; w.width = width; w.all = true; w.scale = scale;
+    moe_route(sel, wt, nullptr, h, w, tokens, static_cast<cudaStream_t>(stream));
+}
+// One token: the choice from the router's logits, then silu(gate) * up of the chosen experts and of the gated shared expert -> act [top * ff + shared_ff]
+void nt_b200_moe_choose_up(float* act, int* sel, float* wt, const float* h, const float* logits, const void* const* gate_tab, const void* const* up_tab,
+                           const void* shared_gate, const void* shared_up, int dtype, int experts, int top, float scale, int ff, int shared_ff, int width, void* stream) {
+    MoeWeights w;
+    w.gate = gate_tab; w.up = up_tab; w.dtype = (nt::DType)dtype; w.experts = experts; w.top = top; w.ff = ff; w.width = width; w.all = true; w.scale = scale;
+    if (shared_ff > 0) { w.shared_up = shared_up; w.shared_gatew = shared_gate; w.shared_ff = shared_ff; }
+    moe_expert_up_token(act, h, nullptr, w, static_cast<cudaStream_t>(stream), logits, sel, wt);
+}
+// Windowed attention over one key / value head stored as rows (keys: the first dim numbers, values: the first vdim).  form 0: all heads from one
+// copy of the rows (returns -1 when the shape is not covered), form 1: one CTA per (query, head).  window 0: full causal.
+int nt_b200_attention_rows_window(float* out, const float* Q, const void* cache, int cache_dtype, int tokens, int p0, int max_seq, int heads, int dim, int vdim, int row,
+                                  float scale, int window, int form, void* stream) {
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const nt::DType dt = (nt::DType)cache_dtype;
+    if (form == 1) {
+        WindowAttn a;
+        a.heads = heads; a.kv_heads = 1; a.dim = dim; a.vdim = vdim; a.scale = scale; a.k_stride = row; a.v_stride = row; a.window = window;
+        attention_window(out, Q, cache, cache, dt, tokens, nullptr, p0, max_seq, a, s);
+        return 0;
+    }
+    if (!attention_shared_rows_supported(heads, dim, vdim, row, dt, cache)) return -1;
+    float* scratch = nullptr;
+    NT_CUDA_CHECK(cudaMalloc(&scratch, sizeof(float) * attention_shared_rows_scratch_floats(heads, vdim)));
+    attention_shared_rows(out, Q, cache, dt, tokens, nullptr, p0, max_seq, heads, dim, vdim, row, scale, scratch, s, window);
+    NT_CUDA_CHECK(cudaStreamSynchronize(s));
+    NT_CUDA_CHECK(cudaFree(scratch));
+    return 0;
+}
+// Tiled windowed attention over BF16 per-head keys [rows, heads, kw] and values [rows, heads, vw]
+void nt_b200_attention_heads_window(float* out, const float* Q, const void* k, const void* v, int tokens, int p0, int rows, int heads, int kw, int vw, float scale,
+                                    int window, void* stream) {
+    attention_heads_mma(out, Q, k, v, tokens, p0, rows, heads, kw, vw, scale, static_cast<cudaStream_t>(stream), window);
 }
 void nt_b200_glu_mul(float* out, const float* gate, const float* up, long long n, int gelu, void* stream) {
     glu_mul(out, gate, up, (size_t)n, gelu != 0, static_cast<cudaStream_t>(stream));

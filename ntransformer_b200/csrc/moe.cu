@@ -239,6 +239,12 @@ __global__ void __launch_bounds__(TK_WARPS * 32) moe_up_token_kernel(float* __re
     __shared__ int sel_s[MAX_EXPERTS];
     __shared__ float wt_s[MAX_EXPERTS];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int r = blockIdx.x * TK_WARPS + warp; r < m.top * m.ff + m.shared_ff; r += gridDim.x * TK_WARPS) {       // the shared expert's rows are known ahead of the choice
+        if (r < m.top * m.ff) continue;
+        const size_t off = (size_t)(r - m.top * m.ff) * m.width * sizeof(T), n = (size_t)m.width * sizeof(T);
+        l2_prefetch(static_cast<const unsigned char*>(m.shared_up) + off, n, lane, 32);
+        if (m.shared_gatew) l2_prefetch(static_cast<const unsigned char*>(m.shared_gatew) + off, n, lane, 32);
+    }
     pdl_launch_dependents();
     pdl_wait();
     for (int i = threadIdx.x; i < m.width; i += TK_WARPS * 32) hs[i] = h[i];

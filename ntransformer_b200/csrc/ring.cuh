@@ -49,6 +49,12 @@ __device__ __forceinline__ int dp4a_ss(int a_s8x4, int b_s8x4, int c) {
 }
 // Programmatic dependent launch: wait for the producer grid / let dependents start.
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+// Hint: bring the 128-byte lines of [p, p + bytes) into L2, the lines shared out over `n` threads (this one is `i`).  Used in front of pdl_wait()
+// on data no kernel of the running step writes (weights, older state): the fetch from HBM overlaps the producer grid's tail.
+__device__ __forceinline__ void l2_prefetch(const void* p, size_t bytes, int i, int n) {
+    const char* c = static_cast<const char*>(p);
+    for (size_t o = (size_t)i * 128; o < bytes; o += (size_t)n * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(c + o));
+}
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
 }}  // namespace nt::b200

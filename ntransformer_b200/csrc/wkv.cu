@@ -261,31 +261,85 @@ __device__ __forceinline__ float wld(const float* p, size_t i) { return __ldg(p 
 __device__ __forceinline__ float wld(const __half* p, size_t i) { return __half2float(__ushort_as_half(__ldg(reinterpret_cast<const unsigned short*>(p) + i))); }
 __device__ __forceinline__ float wld(const __nv_bfloat16* p, size_t i) { return __uint_as_float((unsigned)__ldg(reinterpret_cast<const unsigned short*>(p) + i) << 16); }
 
-// grid (heads), 256 threads.  a1 [rank]: tanh(W_w1 m) of the token; W2 [heads * dim, rank].  8 lanes per value channel.
+template <typename T> struct Chunk;           // 16 bytes of a weight row
+template <> struct Chunk<float> {
+    static constexpr int P = 4;
+    static __device__ __forceinline__ void unpack(const uint4& w, float* f) { f[0] = __uint_as_float(w.x); f[1] = __uint_as_float(w.y); f[2] = __uint_as_float(w.z); f[3] = __uint_as_float(w.w); }
+};
+template <> struct Chunk<__half> {
+    static constexpr int P = 8;
+    static __device__ __forceinline__ void unpack(const uint4& w, float* f) {
+        const unsigned u[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int k = 0; k < 4; k++) { const float2 p = __half22float2(*reinterpret_cast<const __half2*>(&u[k])); f[2 * k] = p.x; f[2 * k + 1] = p.y; }
+    }
+};
+template <> struct Chunk<__nv_bfloat16> {
+    static constexpr int P = 8;
+    static __device__ __forceinline__ void unpack(const uint4& w, float* f) {
+        const unsigned u[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int k = 0; k < 4; k++) { f[2 * k] = __uint_as_float(u[k] << 16); f[2 * k + 1] = __uint_as_float(u[k] & 0xFFFF0000u); }
+    }
+};
+
+// grid (heads), 256 threads.  a1 [rank]: tanh(W_w1 m) of the token; W2 [heads * dim, rank].  8 lanes per value channel; DV > 0: dim is a
+// multiple of 4 and at most 32 DV, a lane's share of a column is DV 16-byte pieces loaded together; DV == 0: any dim.  vec: W2's rows are whole
+// 16-byte pieces, 8 lanes per row.
 constexpr int WT_LN = 8;
-template <typename T>
+template <typename T, int DV>
 __global__ void __launch_bounds__(256) wkv_token_kernel(float* __restrict__ out, const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v,
                                                         const float* __restrict__ gate, const float* __restrict__ a1, const T* __restrict__ W2, const float* __restrict__ w0,
                                                         const float* __restrict__ u, const float* __restrict__ norm, float* __restrict__ state, float eps, int rank,
-                                                        int dim, const int* __restrict__ pos_dev, int p0) {
+                                                        int dim, int vec, const int* __restrict__ pos_dev, int p0) {
     extern __shared__ __align__(16) float sm[];
-    float *rs = sm, *ks = rs + dim, *ws = ks + dim, *os = ws + dim, *as = os + dim;      // [dim] x 4, [rank]
+    const int dp = (dim + 3) & ~3;
+    float *rs = sm, *ks = rs + dp, *ws = ks + dp, *os = ws + dp, *as = os + dp;      // [dim] x 4, [rank]
     __shared__ float red[8];
     __shared__ float bonus;
-    pdl_launch_dependents();
-    pdl_wait();
     const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const size_t hb = (size_t)h * dim;
+    // the state and the constants are older than this step: their way from HBM overlaps the projections
+    l2_prefetch(state + hb * dim, (size_t)dim * dim * sizeof(float), threadIdx.x, 256);
+    l2_prefetch(W2 + hb * rank, (size_t)dim * rank * sizeof(T), threadIdx.x, 256);
+    l2_prefetch(w0 + hb, (size_t)dim * sizeof(float), threadIdx.x, 256);
+    l2_prefetch(u + hb, (size_t)dim * sizeof(float), threadIdx.x, 256);
+    l2_prefetch(norm + hb, (size_t)dim * sizeof(float), threadIdx.x, 256);
+    pdl_launch_dependents();
+    pdl_wait();
     const bool fresh = (pos_dev ? *pos_dev : p0) == 0;
     for (int i = threadIdx.x; i < rank; i += 256) as[i] = a1[i];
     for (int d = threadIdx.x; d < dim; d += 256) { rs[d] = r[hb + d]; ks[d] = k[hb + d]; }
     __syncthreads();
-    for (int d = warp; d < dim; d += 8) {
-        float z = 0.f;
-        for (int i = lane; i < rank; i += 32) z = fmaf(wld(W2, (hb + d) * rank + i), as[i], z);
+    const int l = threadIdx.x % WT_LN;
+    if (vec) {
+        constexpr int P = Chunk<T>::P;
+        const int nc = rank / P;
+#pragma unroll 2
+        for (int d0 = 0; d0 < dim; d0 += 256 / WT_LN) {
+            const int d = d0 + threadIdx.x / WT_LN;
+            float z = 0.f;
+            if (d < dim) {
+                const uint4* row = reinterpret_cast<const uint4*>(W2 + (hb + d) * rank);
+                for (int c = l; c < nc; c += WT_LN) {
+                    float f[P];
+                    Chunk<T>::unpack(__ldg(row + c), f);
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) z += __shfl_xor_sync(0xFFFFFFFFu, z, o);
-        if (lane == 0) ws[d] = decay_of(z + w0[hb + d]);
+                    for (int e = 0; e < P; e++) z = fmaf(f[e], as[c * P + e], z);
+                }
+            }
+#pragma unroll
+            for (int o = WT_LN / 2; o > 0; o >>= 1) z += __shfl_xor_sync(0xFFFFFFFFu, z, o);
+            if (l == 0 && d < dim) ws[d] = decay_of(z + w0[hb + d]);
+        }
+    } else {
+        for (int d = warp; d < dim; d += 8) {
+            float z = 0.f;
+            for (int i = lane; i < rank; i += 32) z = fmaf(wld(W2, (hb + d) * rank + i), as[i], z);
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) z += __shfl_xor_sync(0xFFFFFFFFu, z, o);
+            if (lane == 0) ws[d] = decay_of(z + w0[hb + d]);
+        }
     }
     if (warp == 0) {
         float s = 0.f;
@@ -295,20 +349,29 @@ __global__ void __launch_bounds__(256) wkv_token_kernel(float* __restrict__ out,
         if (lane == 0) bonus = s;
     }
     __syncthreads();
-    const int l = threadIdx.x % WT_LN;
+#pragma unroll 2
     for (int j0 = 0; j0 < dim; j0 += 256 / WT_LN) {
         const int j = j0 + threadIdx.x / WT_LN;
         const bool live = j < dim;
         float* st = state + (hb + (live ? j : 0)) * dim;
         const float vj = live ? v[hb + j] : 0.f;
         float p = 0.f;
-        if (dim % 4 == 0) {
-            for (int d = 4 * l; live && d < dim; d += 4 * WT_LN) {
-                float4 S = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st + d);
-                p = fmaf(rs[d], S.x, p); p = fmaf(rs[d + 1], S.y, p); p = fmaf(rs[d + 2], S.z, p); p = fmaf(rs[d + 3], S.w, p);
-                S.x = fmaf(ws[d], S.x, ks[d] * vj); S.y = fmaf(ws[d + 1], S.y, ks[d + 1] * vj);
-                S.z = fmaf(ws[d + 2], S.z, ks[d + 2] * vj); S.w = fmaf(ws[d + 3], S.w, ks[d + 3] * vj);
-                *reinterpret_cast<float4*>(st + d) = S;
+        if constexpr (DV > 0) {
+            float4 S[DV];
+#pragma unroll
+            for (int c = 0; c < DV; c++) {
+                const int d = 4 * (c * WT_LN + l);
+                S[c] = (live && !fresh && d < dim) ? *reinterpret_cast<const float4*>(st + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int c = 0; c < DV; c++) {
+                const int d = 4 * (c * WT_LN + l);
+                if (live && d < dim) {
+                    const float4 R = *reinterpret_cast<const float4*>(rs + d), K = *reinterpret_cast<const float4*>(ks + d), D = *reinterpret_cast<const float4*>(ws + d);
+                    p = fmaf(R.x, S[c].x, p); p = fmaf(R.y, S[c].y, p); p = fmaf(R.z, S[c].z, p); p = fmaf(R.w, S[c].w, p);
+                    S[c].x = fmaf(D.x, S[c].x, K.x * vj); S[c].y = fmaf(D.y, S[c].y, K.y * vj); S[c].z = fmaf(D.z, S[c].z, K.z * vj); S[c].w = fmaf(D.w, S[c].w, K.w * vj);
+                    *reinterpret_cast<float4*>(st + d) = S[c];
+                }
             }
         } else {
             for (int d = l; live && d < dim; d += WT_LN) {
@@ -406,11 +469,15 @@ void wkv_out_norm(float* out, void* split, const float* o, const float* gate, co
 void wkv_token(float* out, const float* r, const float* k, const float* v, const float* gate, const float* a1, const void* W2, DType dt, const float* w0, const float* u,
                const float* norm, float* state, float eps, int rank, int heads, int dim, const int* pos_dev, int p0, cudaStream_t s) {
     NT_CHECK(dim >= 1 && dim <= WKV_MAX_DIM && rank >= 1, "wkv_token: heads wider than 256 are not covered");
-    const size_t smem = sizeof(float) * (4 * (size_t)dim + (size_t)rank);
+    const size_t smem = sizeof(float) * (4 * (size_t)((dim + 3) & ~3) + (size_t)rank);
     NT_CHECK(smem <= 48 * 1024, "wkv_token: decay ranks above 11000 are not covered");
-#define NT_WT(TY) launch_k(wkv_token_kernel<TY>, dim3(heads), dim3(256), smem, s, out, r, k, v, gate, a1, static_cast<const TY*>(W2), w0, u, norm, state, eps, rank, dim, pos_dev, p0)
-    if (dt == DType::F32) NT_WT(float); else if (dt == DType::F16) NT_WT(__half); else if (dt == DType::BF16) NT_WT(__nv_bfloat16);
-    else NT_CHECK(false, "wkv_token: dense dtypes only");
+    NT_CHECK(dense_dtype(dt), "wkv_token: dense dtypes only");
+    const int vec = rank % (dt == DType::F32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(W2) & 15) == 0;
+    const int dv = dim % 4 || (reinterpret_cast<uintptr_t>(state) & 15) ? 0 : dim <= 32 ? 1 : dim <= 64 ? 2 : dim <= 128 ? 4 : 8;
+#define NT_WD(TY, DV) launch_k(wkv_token_kernel<TY, DV>, dim3(heads), dim3(256), smem, s, out, r, k, v, gate, a1, static_cast<const TY*>(W2), w0, u, norm, state, eps, rank, dim, vec, pos_dev, p0)
+#define NT_WT(TY) { if (dv == 1) NT_WD(TY, 1); else if (dv == 2) NT_WD(TY, 2); else if (dv == 4) NT_WD(TY, 4); else if (dv == 8) NT_WD(TY, 8); else NT_WD(TY, 0); }
+    if (dt == DType::F32) NT_WT(float) else if (dt == DType::F16) NT_WT(__half) else NT_WT(__nv_bfloat16)
+#undef NT_WD
 #undef NT_WT
     count_launch();
 }

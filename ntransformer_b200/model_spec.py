@@ -418,3 +418,89 @@ def savidra_random_tensors(config: dict, seed: int = 1234, device="cuda", dtype=
             t[p + "mlp.up"] = mat(f["ff"], W)
             t[p + "mlp.down"] = mat(W, f["ff"])
     return t
+
+
+# ---- Fuvozen (layer-spec family, model folders): synthetic configurations and random device weights for benchmarks ----
+def fuvozen_config(vocab=32000, width=2048, pattern=("wkv", "latent_attention", "wkv", "latent_attention"), mlp=("dense", "moe", "dense", "moe"), groups=8, eps=1e-5,
+                   buckets=65521, mul_prev=7919, mul_cur=104729, heads=16, dim=64, rot_dim=64, vdim=128, kv_rank=256, window=1024, rot_base=10000.0,
+                   w_heads=32, w_dim=64, decay_rank=64, ff=6144, experts=16, top=3, eff=1408, shared=1408, router_scale=1.0):
+    """The family's config.json as a dict.  pattern: mixer type per layer; mlp: feed-forward kind per layer ("dense", "moe" or None); window: visible
+    positions of the attention layers (0: all); shared: width of the shared expert (0: none).  decay_rank is stated for models made from device
+    tensors; a folder may leave it out (the rows of the decay's first matrix)."""
+    layers = []
+    for i, typ in enumerate(pattern):
+        if typ == "wkv":
+            m = {"heads": w_heads, "dim": w_dim, "decay_rank": decay_rank}
+        else:
+            m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": (dim + rot_dim) ** -0.5, "rot": {"base": rot_base, "dims": rot_dim}}
+            if window:
+                m["mask"] = {"size": window}
+        k = mlp[i % len(mlp)]
+        if k == "dense":
+            f = {"kind": "dense", "ff": ff}
+        elif k == "moe":
+            f = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": experts, "top": top, "scale": router_scale}}
+            if shared:
+                f["shared"] = {"ff": shared}
+        else:
+            f = None
+        layers.append({"type": typ, "mixer": m, "mlp": f})
+    return {"architecture": "Fuvozen", "vocab": vocab, "width": width, "norm": {"eps": eps, "groups": groups},
+            "embedding": {"bigram": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}}, "layers": layers}
+
+
+def fuvozen_random_tensors(config: dict, seed: int = 1234, device="cuda", dtype=None):
+    """Checkpoint name -> random CUDA tensor (matrices and embeddings `dtype`, default bfloat16; gains, blends, decay offsets, router rows and the
+    depth weights float32)."""
+    import torch
+
+    dtype = dtype or torch.bfloat16
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W = config["width"]
+
+    def mat(rows, cols, dt=dtype):
+        return (torch.randn(rows, cols, generator=g, device=device, dtype=torch.float32) * cols ** -0.5).to(dt)
+
+    def vec(n, mean=1.0, std=0.1):
+        return mean + std * torch.randn(n, generator=g, device=device, dtype=torch.float32)
+
+    def uni(n, lo, hi):
+        return lo + (hi - lo) * torch.rand(n, generator=g, device=device, dtype=torch.float32)
+
+    t = {"embed": mat(config["vocab"], W) * W ** 0.5, "bigram": mat(config["embedding"]["bigram"]["buckets"] + 1, W) * W ** 0.5, "final.norm": vec(W)}
+    for i, e in enumerate(config["layers"]):
+        m, p = e["mixer"], "l%d." % i
+        q = p + "mix."
+        t[p + "norm1"] = vec(W)
+        if e["type"] == "wkv":
+            n = m["heads"] * m["dim"]
+            for s in "rkvgw":
+                t[q + "mu." + s] = uni(W, 0.0, 1.0)
+            for s in "rkvg":
+                t[q + s] = mat(n, W)
+            t[q + "w1"] = mat(m["decay_rank"], W)
+            t[q + "w2"] = mat(n, m["decay_rank"])
+            t[q + "w0"] = uni(n, -6.0, 0.0)
+            t[q + "u"] = vec(n, 0.0, 0.5).reshape(m["heads"], m["dim"])
+            t[q + "norm"] = vec(n)
+            t[q + "o"] = mat(W, n)
+        else:
+            t[q + "q"] = mat(m["heads"] * (m["dim"] + m["rot_dim"]), W)
+            t[q + "dkv"] = mat(m["kv_rank"] + m["rot_dim"], W)
+            t[q + "dkv.norm"] = vec(m["kv_rank"])
+            t[q + "uk"] = mat(m["heads"] * m["dim"], m["kv_rank"])
+            t[q + "uv"] = mat(m["heads"] * m["vdim"], m["kv_rank"])
+            t[q + "o"] = mat(W, m["heads"] * m["vdim"])
+        f = e.get("mlp")
+        if f and f["kind"] == "dense":
+            t[p + "mlp.up"], t[p + "mlp.down"] = mat(f["ff"], W), mat(W, f["ff"])
+            t[p + "mlp.act"] = uni(2, -1.0, 0.5)
+        elif f:
+            t[p + "mlp.router"] = mat(f["router"]["experts"], W, torch.float32)
+            names = ["e%d" % x for x in range(f["router"]["experts"])] + (["shared"] if f.get("shared") else [])
+            for x in names:
+                w = f["shared"]["ff"] if x == "shared" else f["expert"]["ff"]
+                t[p + "mlp." + x + ".gate"], t[p + "mlp." + x + ".up"], t[p + "mlp." + x + ".down"] = mat(w, W), mat(w, W), mat(W, w)
+        t[p + "dwa"] = torch.cat([uni(i + 1, -0.1, 0.2), uni(1, 0.9, 1.1)])
+    return t

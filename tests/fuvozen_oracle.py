@@ -207,7 +207,7 @@ def random_model(rng, pattern=("wkv", "latent_attention", "wkv", "latent_attenti
     lay = []
     for i, typ in enumerate(pattern):
         if typ == "wkv":
-            m = {"heads": w_heads, "dim": w_dim}
+            m = {"heads": w_heads, "dim": w_dim, "decay_rank": rank}
         else:
             m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": scale if scale else (dim + rot_dim) ** -0.5,
                  "rot": {"base": rot_base, "dims": rot_dim}}
