@@ -83,7 +83,7 @@ Model::~Model() {
     if (moe_offsets_host_) cudaFreeHost(moe_offsets_host_);
     auto free_layer = [](LayerWeights& L) {
         for (void* p : {(void*)L.e_up_tab, (void*)L.e_down_tab, (void*)L.rot_freq, (void*)L.e_gate_tab, (void*)L.conv_state, (void*)L.ssm_state, (void*)L.shift_state,
-                        (void*)L.q_conv_state, (void*)L.k_conv_state, (void*)L.v_conv_state, (void*)L.delta_state, (void*)L.wkv_state}) if (p) cudaFree(p);
+                        (void*)L.q_conv_state, (void*)L.k_conv_state, (void*)L.v_conv_state, (void*)L.delta_state, (void*)L.wkv_state, L.e_maps}) if (p) cudaFree(p);
     };
     for (LayerWeights& L : layers_) {
         free_layer(L);

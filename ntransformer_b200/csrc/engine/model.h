@@ -69,6 +69,7 @@ struct LayerWeights {
     const float *gate_b = nullptr, *up_b = nullptr, *down_b = nullptr, *route_corr = nullptr;
     std::vector<Weight> e_gate;
     const void** e_gate_tab = nullptr;
+    void* e_maps = nullptr;                // device: tensor maps of the gated experts' gate, up and down matrices [3][experts] (owned; null: CUDA-core form)
     // per-layer token input: gate [side_dim, width], projection [width, side_dim], gain [width]
     Weight side_gate, side_proj;
     const float* side_norm = nullptr;
@@ -243,7 +244,9 @@ private:
     bool latent_expand_ok(const LayerSpec& S, int T) const;
     void ensure_latent_scratch(const LayerSpec& S, size_t rows, size_t tokens);
     void latent_attention_rows(int i, int T, int p0, const float* q, float* out, cudaStream_t s);   // out [T, heads * vdim]
-    bool moe_glu_rows_tc(int i, int T, const float* x, cudaStream_t s);    // routed gated experts of a prompt portion on the tensor cores -> pf_.y_rows
+    void make_expert_maps(const LayerSpec& S, LayerWeights& L);            // LayerWeights::e_maps, when every expert matrix takes the tensor cores
+    // routed gated experts of T prompt rows x, chosen and weighted (pf_.sel, pf_.wt): y (+)= the weighted sum
+    void moe_glu_rows(int i, int T, const float* x, const MoeWeights& w, float* y, bool add, cudaStream_t s);
     RowBufs dec_;                         // POST_NORM decode step: x is hidden_, the rest one scratch row each (stable addresses for the graph)
     std::vector<int> want_;               // places (indices into the current forward's tokens) whose logits are collected
     float* want_out_ = nullptr;           // device [want_cap_, vocab]

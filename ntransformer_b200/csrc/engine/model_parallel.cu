@@ -103,6 +103,7 @@ bool Model::finalize_parallel_layer(int i) {
             NT_CUDA_CHECK(cudaMemcpy(dst, v.data(), sizeof(void*) * v.size(), cudaMemcpyHostToDevice));
         };
         table(M.e_up_tab, up); table(M.e_down_tab, down); table(M.e_gate_tab, gate);
+        make_expert_maps(S, M);
     }
     return true;
 }
@@ -329,22 +330,23 @@ void Model::layer_parallel_rows(int i, int T, int p0, cudaStream_t s) {
         add_product(o, L.wo);
     }
     if (S.ff > 0 && S.ff_kind == FfKind::MLP) {
+        const bool tc = parallel_split_ok(L.down);
+        if (tc && pf_.ws2 && spec_tc_ok(L.up) && S.ff % 8 == 0) {
+            // the activation and the split for the down product in the up GEMM's epilogue: the [T, ff] numbers never reach HBM in FP32
+            TcOpts o; o.bf16 = true;
+            NT_CHECK(gemm_f16_tc_xielu_ws(pf_.ws2, B.hs, L.up.ptr, L.ff_act, T, S.ff, W, s, o), "prefill GEMM (up) rejected");
+            parallel_gemm(x, nullptr, pf_.ws2, L.down, T, true, s);
+            NT_CHECK(cur <= parallel_scratch_width() * (size_t)T, "layer_parallel_rows: scratch rows overrun");
+            return;
+        }
         float* u = take((size_t)S.ff);
         parallel_gemm(u, B.h, hs_of(L.up), L.up, T, false, s);
-        const bool tc = parallel_split_ok(L.down);
         xielu_rows(tc ? nullptr : u, tc ? pf_.ws : nullptr, u, L.ff_act, T, S.ff, s);
         parallel_gemm(x, u, tc ? pf_.ws : nullptr, L.down, T, true, s);
     } else if (S.ff > 0) {
         const MoeWeights w = parallel_moe(i);
         moe_route(pf_.sel, pf_.wt, nullptr, B.h, w, T, s);
-        moe_group(pf_.work, pf_.sel, T, S.experts, S.top, s);
-        if (!moe_glu_rows_tc(i, T, B.h, s)) {
-            moe_expert_gate_rows(pf_.gate_rows, B.h, pf_.work, w, T, s);
-            moe_expert_up_rows(pf_.act_rows, B.h, pf_.work, w, T, s);
-            glu_bias_mul(pf_.act_rows, pf_.gate_rows, pf_.act_rows, nullptr, nullptr, T * S.top, S.ff, false, s);
-            moe_expert_down_rows(pf_.y_rows, pf_.act_rows, pf_.work, w, T, s);
-        }
-        moe_combine(x, pf_.y_rows, pf_.work, pf_.wt, nullptr, nullptr, T, S.experts, S.top, W, s, true);
+        moe_glu_rows(i, T, B.h, w, x, true, s);
         if (S.shared_ff > 0 && pf_.ws && pf_.ws2 && spec_tc_ok(L.sh_glu) && spec_tc_ok(L.sh_up) && spec_tc_ok(L.sh_down) && S.shared_ff % 128 == 0) {
             TcOpts o; o.bf16 = true;
             NT_CHECK(gemm_f16_tc_swiglu_ws(pf_.ws2, B.hs, L.sh_glu.ptr, L.sh_up.ptr, T, S.shared_ff, W, s, o), "prefill GEMM (shared gate / up) rejected");

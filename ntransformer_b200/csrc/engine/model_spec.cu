@@ -283,6 +283,7 @@ bool Model::finalize_spec() {
                 NT_CUDA_CHECK(cudaMemcpy(M.e_up_tab, up.data(), sizeof(void*) * up.size(), cudaMemcpyHostToDevice));
                 NT_CUDA_CHECK(cudaMemcpy(M.e_down_tab, down.data(), sizeof(void*) * down.size(), cudaMemcpyHostToDevice));
                 NT_CUDA_CHECK(cudaMemcpy(M.e_gate_tab, gate.data(), sizeof(void*) * gate.size(), cudaMemcpyHostToDevice));
+                make_expert_maps(S, M);
                 moe_act = std::max(moe_act, S.top * S.ff);
                 topmax = std::max(topmax, S.top);
             }
@@ -517,8 +518,8 @@ void Model::ensure_prefill_buffers_spec(int tokens) {
         if (!post_form) { pf_.xs = dmalloc<float>(T * n_streams() * hidden); pf_.maps = dmalloc<float>(T * mapmax); }
         if (topmax > 0) {
             pf_.sel = dmalloc<int>(T * topmax); pf_.wt = dmalloc<float>(T * topmax); pf_.sgate = dmalloc<float>(T);
-            pf_.work = dmalloc<int>(moe_work_ints((int)T, (int)emax, (int)topmax));
-            pf_.act_rows = dmalloc<float>(T * topmax * effmax); pf_.y_rows = dmalloc<float>(T * topmax * hidden);
+            pf_.work = dmalloc<int>(moe_work_ints((int)T, (int)emax, (int)topmax, 128));
+            pf_.act_rows = dmalloc<float>(T * topmax * effmax); pf_.y_rows = dmalloc<float>(moe_rows_cap((int)T, (int)emax, (int)topmax, 128) * hidden);
             if (!exact32_) {       // the tensor-core path of the routed experts: gathered rows, and a split workspace with every expert's rows padded to a tile
                 pf_.g2 = dmalloc<float>(T * topmax * hidden);
                 pf_.moe_ws = dmalloc<uint8_t>(gemm_f16_tc_workspace_bytes((int)(T * topmax + emax * 128), (int)std::max(hidden, effmax)));
@@ -914,32 +915,49 @@ void Model::latent_attention_rows(int i, int T, int p0, const float* q, float* o
     if (o != out) latent_unpad(out, lat_.o, T, S.heads, S.vdim, vw, s);
 }
 
-// The routed gated experts of T prompt rows on the tensor cores: the per-expert row counts come to the host (one small copy and a wait),
-// then every expert with rows runs, over exactly its rows, the gate / up GEMM pair whose epilogue applies silu(gate) * up and writes the
-// down GEMM's split input, and the down GEMM.  pf_.y_rows [T * top, width] in the grouped order.  false: some matrix does not qualify.
-bool Model::moe_glu_rows_tc(int i, int T, const float* x, cudaStream_t s) {
+// Tensor maps of the gated experts' matrices, kept on the device so that one launch can serve every expert.
+void Model::make_expert_maps(const LayerSpec& S, LayerWeights& L) {
+    const size_t n = (size_t)S.experts, mb = gemm_tc_map_bytes();
+    if (exact32_ || S.act != GluAct::SILU || S.ff % 128 != 0 || cfg_.hidden_size % 4 != 0 || S.experts > 256) return;
+    std::vector<uint8_t> raw(3 * n * mb + 64);
+    uint8_t* host = raw.data() + (64 - reinterpret_cast<uintptr_t>(raw.data()) % 64) % 64;      // maps are encoded on 64-byte boundaries
+    for (size_t e = 0; e < n; e++) {
+        const Weight *g = &L.e_gate[e], *u = &L.e_up[e], *d = &L.e_down[e];
+        if (!spec_tc_ok(*g) || !spec_tc_ok(*u) || !spec_tc_ok(*d)) return;
+        if (!gemm_tc_weight_map(host + e * mb, g->ptr, S.ff, cfg_.hidden_size, true, true) || !gemm_tc_weight_map(host + (n + e) * mb, u->ptr, S.ff, cfg_.hidden_size, true, true) ||
+            !gemm_tc_weight_map(host + (2 * n + e) * mb, d->ptr, cfg_.hidden_size, S.ff, false, true)) return;
+    }
+    L.e_maps = dmalloc<uint8_t>(3 * n * mb);
+    NT_CUDA_CHECK(cudaMemcpy(L.e_maps, host, 3 * n * mb, cudaMemcpyHostToDevice));
+}
+
+// Tensor cores: the rows grouped by expert, every expert's run on a tile boundary, split in place of the gather; one launch runs the gate / up
+// pairs of all experts (the epilogue applies silu(gate) * up and writes the down products' split input), one the down products.  Row counts
+// stay on the device.  Otherwise gathered FP32 GEMMs on CUDA cores.
+void Model::moe_glu_rows(int i, int T, const float* x, const MoeWeights& w, float* y, bool add, cudaStream_t s) {
     const LayerSpec& S = cfg_.layers[(size_t)i];
     const LayerWeights& L = layer_weights(i);
     const int hidden = cfg_.hidden_size;
-    if (!pf_.moe_ws || !pf_.moe_ws2 || !pf_.g2 || !moe_offsets_host_ || S.ff % 128 != 0 || S.experts > 256) return false;
-    for (int e = 0; e < S.experts; e++)
-        if (!spec_tc_ok(L.e_gate[(size_t)e]) || !spec_tc_ok(L.e_up[(size_t)e]) || !spec_tc_ok(L.e_down[(size_t)e])) return false;
-    NT_CUDA_CHECK(cudaMemcpyAsync(moe_offsets_host_, pf_.work, sizeof(int) * (size_t)(S.experts + 1), cudaMemcpyDeviceToHost, s));
-    NT_CUDA_CHECK(cudaStreamSynchronize(s));
-    moe_gather_rows(pf_.g2, x, pf_.work, T, S.experts, S.top, hidden, s);
-    TcOpts o; o.bf16 = true;
-    size_t padded = 0;
-    for (int e = 0; e < S.experts; e++) {
-        const int r0 = moe_offsets_host_[e], cnt = moe_offsets_host_[e + 1] - r0;
-        if (cnt <= 0) continue;
-        void* wi = static_cast<uint8_t*>(pf_.moe_ws) + gemm_f16_tc_workspace_bytes((int)padded, hidden);
-        void* wo = static_cast<uint8_t*>(pf_.moe_ws2) + gemm_f16_tc_workspace_bytes((int)padded, S.ff);
-        split_activations(wi, pf_.g2 + (size_t)r0 * hidden, cnt, hidden, s, true);
-        NT_CHECK(gemm_f16_tc_swiglu_ws(wo, wi, L.e_gate[(size_t)e].ptr, L.e_up[(size_t)e].ptr, cnt, S.ff, hidden, s, o), "expert GEMM (gate / up) rejected");
-        NT_CHECK(gemm_f16_tc_ws(pf_.y_rows + (size_t)r0 * hidden, wo, L.e_down[(size_t)e].ptr, cnt, hidden, S.ff, false, s, o), "expert GEMM (down) rejected");
-        padded += ((size_t)cnt + 127) / 128 * 128;
+    if (L.e_maps && pf_.moe_ws && pf_.moe_ws2 && (reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+        constexpr int PAD = 128;
+        const int cap = (int)moe_rows_cap(T, S.experts, S.top, PAD);
+        const size_t mb = gemm_tc_map_bytes() * (size_t)S.experts;
+        const uint8_t* maps = static_cast<const uint8_t*>(L.e_maps);
+        moe_group(pf_.work, pf_.sel, T, S.experts, S.top, s, PAD);
+        moe_gather_split(pf_.moe_ws, x, pf_.work, T, S.experts, S.top, PAD, hidden, s);
+        const int* counts = moe_counts_of(pf_.work, T, S.experts, S.top, PAD);
+        TcOpts o; o.bf16 = true;
+        NT_CHECK(gemm_f16_tc_grouped_swiglu(pf_.moe_ws2, pf_.moe_ws, maps, maps + mb, pf_.work, counts, S.experts, cap, S.ff, hidden, s, o), "expert GEMM (gate / up) rejected");
+        NT_CHECK(gemm_f16_tc_grouped(pf_.y_rows, pf_.moe_ws2, maps + 2 * mb, pf_.work, counts, S.experts, cap, hidden, S.ff, s, o), "expert GEMM (down) rejected");
+        moe_combine(y, pf_.y_rows, pf_.work, pf_.wt, nullptr, nullptr, T, S.experts, S.top, hidden, s, add, PAD);
+        return;
     }
-    return true;
+    moe_group(pf_.work, pf_.sel, T, S.experts, S.top, s);
+    moe_expert_gate_rows(pf_.gate_rows, x, pf_.work, w, T, s);
+    moe_expert_up_rows(pf_.act_rows, x, pf_.work, w, T, s);
+    glu_bias_mul(pf_.act_rows, pf_.gate_rows, pf_.act_rows, nullptr, nullptr, T * S.top, S.ff, S.act == GluAct::GELU_TANH, s);
+    moe_expert_down_rows(pf_.y_rows, pf_.act_rows, pf_.work, w, T, s);
+    moe_combine(y, pf_.y_rows, pf_.work, pf_.wt, nullptr, nullptr, T, S.experts, S.top, hidden, s, add);
 }
 
 // Scores and values of T rows behind the query projection and the cache write: expanded per-head form for prompt portions, absorbed form on
@@ -1017,14 +1035,7 @@ void Model::layer_postnorm(int i, int T, const int* tok_dev, const int* pos_dev,
             moe_expert_down_token(B.y, moe_act_, moe_sel_, moe_wt_, nullptr, nullptr, w, s);
         } else {
             moe_route(pf_.sel, pf_.wt, nullptr, B.x, w, T, s);
-            moe_group(pf_.work, pf_.sel, T, S.experts, S.top, s);
-            if (S.act != GluAct::SILU || !moe_glu_rows_tc(i, T, B.x, s)) {
-                moe_expert_gate_rows(pf_.gate_rows, B.x, pf_.work, w, T, s);
-                moe_expert_up_rows(pf_.act_rows, B.x, pf_.work, w, T, s);
-                glu_bias_mul(pf_.act_rows, pf_.gate_rows, pf_.act_rows, nullptr, nullptr, T * S.top, S.ff, false, s);
-                moe_expert_down_rows(pf_.y_rows, pf_.act_rows, pf_.work, w, T, s);
-            }
-            moe_combine(B.y, pf_.y_rows, pf_.work, pf_.wt, nullptr, nullptr, T, S.experts, S.top, hidden, s);
+            moe_glu_rows(i, T, B.x, w, B.y, false, s);
         }
         add_rmsnorm_rows(B.x, B.y, L.ffn_norm, nullptr, T, hidden, eps, s);
     }

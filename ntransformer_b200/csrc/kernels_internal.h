@@ -260,15 +260,20 @@ void moe_expert_down_token(float* y, const float* act, const int* sel, const flo
                            const MoeWeights& w, cudaStream_t s, const StreamsIO* sio = nullptr);
 // Prompt rows: assignments grouped per expert (order inside an expert = token order), gathered GEMMs on CUDA cores in F32.
 //   work: ints [experts + 1 (offsets) + tokens*top (row -> token) + tokens*top (assignment -> row)]
-size_t moe_work_ints(int tokens, int experts, int top);
-void moe_group(int* work, const int* sel, int tokens, int experts, int top, cudaStream_t s);
+//   pad > 1: every expert's rows start on a multiple of pad (row runs of the tensor-core GEMM); row numbers count the gaps.
+size_t moe_work_ints(int tokens, int experts, int top, int pad = 1);
+size_t moe_rows_cap(int tokens, int experts, int top, int pad);        // rows the grouped order can take up
+const int* moe_counts_of(const int* work, int tokens, int experts, int top, int pad);     // rows per expert (device); work itself starts with the run starts
+void moe_group(int* work, const int* sel, int tokens, int experts, int top, cudaStream_t s, int pad = 1);
+// h rows in the grouped order as the BF16 split of moe_rows_cap rows (rows between the runs are left alone)
+void moe_gather_split(void* ws, const float* h, const int* work, int tokens, int experts, int top, int pad, int width, cudaStream_t s);
 // [tokens*top, ff]: relu(W_up h)^2, or for gated experts the plain W_up h; moe_expert_gate_rows: W_gate h (combine with glu_bias_mul)
 void moe_expert_up_rows(float* act_rows, const float* h, const int* work, const MoeWeights& w, int tokens, cudaStream_t s);
 void moe_expert_gate_rows(float* gate_rows, const float* h, const int* work, const MoeWeights& w, int tokens, cudaStream_t s);
 void moe_expert_down_rows(float* y_rows, const float* act_rows, const int* work, const MoeWeights& w, int tokens, cudaStream_t s); // [tokens*top, width]
 // y [tokens, width] = sum_k wt[t, k] * y_rows[row(t, k)] (+ sgate[t] * shared_y[t]; sgate null: + shared_y[t]); add: y += that
 void moe_combine(float* y, const float* y_rows, const int* work, const float* wt, const float* sgate, const float* shared_y, int tokens,
-                 int experts, int top, int width, cudaStream_t s, bool add = false);
+                 int experts, int top, int width, cudaStream_t s, bool add = false, int pad = 1);
 // h rows in the grouped order (the tensor-core path splits them per expert): out [tokens*top, width]
 void moe_gather_rows(float* out, const float* h, const int* work, int tokens, int experts, int top, int width, cudaStream_t s);
 void relu2(float* x, size_t n, cudaStream_t s);
@@ -428,12 +433,24 @@ bool gemm_f16_tc_ragged_supported(const void* W_f16, int N, int K, size_t row_pi
 // Variants of the tensor-core GEMM: bf16 — weights and the activation split are BF16 (safetensors families; the same 16-bit
 // layouts, only the MMA's operand format changes); gelu — the gated epilogue uses tanh-GELU instead of SiLU; col_scale / alpha —
 // the store / add epilogue writes C (+)= alpha * col_scale[n] * (A.W^T) (per-channel layer scale and residual multiplier).
-struct TcOpts { bool bf16 = false; bool gelu = false; const float* col_scale = nullptr; float alpha = 1.0f; bool relu = false; /* gated epilogue: ReLU gate */ };
+struct TcOpts { bool bf16 = false; bool gelu = false; const float* col_scale = nullptr; float alpha = 1.0f; bool relu = false; /* gated epilogue: ReLU gate */
+                const float* act_p = nullptr; /* set by gemm_f16_tc_xielu_ws */ };
 void split_activations(void* workspace, const float* A, int M, int K, cudaStream_t s, bool bf16 = false);
 bool gemm_f16_tc_ws(float* C, const void* workspace, const void* W_f16, int M, int N, int K, bool add, cudaStream_t s, const TcOpts& o = TcOpts());
 // workspace_out <- split(silu(A.Wgate^T) * (A.Wup^T)): the FFN's gate/up GEMMs with the SwiGLU + split fused in the epilogue
 bool gemm_f16_tc_swiglu_ws(void* workspace_out, const void* workspace_in, const void* Wgate_f16, const void* Wup_f16, int M, int N, int K,
                            cudaStream_t s, const TcOpts& o = TcOpts());
+// workspace_out <- split(xIELU(A.W^T)), (p, q) = act_p on the device: the up product of an ungated feed-forward; N % 8 == 0
+bool gemm_f16_tc_xielu_ws(void* workspace_out, const void* workspace_in, const void* W_f16, const float* act_p, int M, int N, int K, cudaStream_t s, const TcOpts& o = TcOpts());
+// Routed experts in one launch per product.  Row runs of the split workspace (rows_padded rows in all): run e has count[e] rows from start[e] (a
+// multiple of 128) on; start / count live on the device, so do the experts' tensor maps (gemm_tc_weight_map on the host, then copied;
+// 64-byte aligned).  swiglu: workspace_out <- split(silu(A.Wgate_e^T) * (A.Wup_e^T)), else C rows = A.W_e^T; rows between the runs are not written.
+size_t gemm_tc_map_bytes();
+bool gemm_tc_weight_map(void* map_host, const void* W, int N, int K, bool gated, bool bf16);
+bool gemm_f16_tc_grouped_swiglu(void* workspace_out, const void* workspace_in, const void* maps_gate, const void* maps_up, const int* start, const int* count, int experts,
+                                int rows_padded, int N, int K, cudaStream_t s, const TcOpts& o = TcOpts());
+bool gemm_f16_tc_grouped(float* C, const void* workspace, const void* maps, const int* start, const int* count, int experts, int rows_padded, int N, int K, cudaStream_t s,
+                         const TcOpts& o = TcOpts());
 void rmsnorm_split(void* workspace, const float* x, const float* w, int rows, int hidden, float eps, cudaStream_t s, bool bf16 = false);
 // prefill_dequant.cu: any GGUF weight matrix -> dense F16 pair with W = w_hi + w_lo (operands of two tensor-core GEMMs)
 bool dequant_split_supported(DType dt);

@@ -13,9 +13,11 @@
 // by the plain scores; a router that weights by the softmax over all experts; a gated shared expert.
 // Expert matrices: F32, F16 or BF16 rows.  Compiled WITHOUT --use_fast_math.
 #include "kernels_internal.h"
+#include "bf16_split.cuh"
 #include "ring.cuh"
 #include <cuda_bf16.h>
 #include <cuda_fp16.h>
+#include <algorithm>
 #include <cfloat>
 
 namespace nt { namespace b200 {
@@ -317,8 +319,10 @@ __global__ void __launch_bounds__(TK_WARPS * 32) moe_down_token_kernel(float* __
 }
 
 // ---- prompt rows ----
-// work = [offsets: experts + 1][row_token: n][assign_row: n], n = tokens * top.  One warp per expert; two launches (count, place).
-__global__ void moe_count_kernel(int* __restrict__ work, const int* __restrict__ sel, int n, int experts) {
+// work = [offsets: experts + 1][row_token: cap][assign_row: n][counts: experts], n = tokens * top.  pad == 1: cap = n, an expert's rows follow the
+// last one's; pad > 1: every expert's rows start on a multiple of pad, cap = n rounded up + experts * pad.  One warp per expert; two launches
+// (count, place).
+__global__ void moe_count_kernel(int* __restrict__ counts, const int* __restrict__ sel, int n) {
     pdl_launch_dependents();
     pdl_wait();
     const int e = blockIdx.x, lane = threadIdx.x;
@@ -326,22 +330,21 @@ __global__ void moe_count_kernel(int* __restrict__ work, const int* __restrict__
     for (int a = lane; a < n; a += 32) c += sel[a] == e ? 1 : 0;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) c += __shfl_xor_sync(0xFFFFFFFFu, c, o);
-    if (lane == 0) work[experts + 1 + 2 * (size_t)n + e] = c;      // counts live behind the two tables
+    if (lane == 0) counts[e] = c;
 }
 constexpr int PL_WARPS = 8;
 // One CTA per expert; its warps take consecutive slices of the assignments: count per slice, prefix over the slices, then an
 // ordered placement inside each slice (ballot + popc), so rows of an expert stay in assignment (= token) order.
-__global__ void __launch_bounds__(PL_WARPS * 32) moe_place_kernel(int* __restrict__ work, const int* __restrict__ sel, int n, int experts, int top) {
+__global__ void __launch_bounds__(PL_WARPS * 32) moe_place_kernel(int* __restrict__ work, int* __restrict__ row_token, int* __restrict__ assign_row, const int* __restrict__ counts,
+                                                                  const int* __restrict__ sel, int n, int experts, int top, int pad) {
     __shared__ int slice_count[PL_WARPS];
     pdl_launch_dependents();
     pdl_wait();
     const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int* counts = work + experts + 1 + 2 * (size_t)n;
     int off = 0;
-    for (int x = 0; x < e; x++) off += counts[x];
-    int* row_token = work + experts + 1;
-    int* assign_row = row_token + n;
+    for (int x = 0; x < e; x++) off += (counts[x] + pad - 1) / pad * pad;
     if (threadIdx.x == 0) { work[e] = off; if (e == experts - 1) work[experts] = off + counts[e]; }
+    if (pad > 1) for (int r = off + counts[e] + threadIdx.x; r < off + (counts[e] + pad - 1) / pad * pad; r += PL_WARPS * 32) row_token[r] = -1;      // rows between the runs
     const int per = ((n + PL_WARPS - 1) / PL_WARPS + 31) / 32 * 32;
     const int a_begin = min(n, warp * per), a_end = min(n, a_begin + per);
     int c = 0;
@@ -429,6 +432,47 @@ __global__ void moe_gather_rows_kernel(float* __restrict__ out, const float* __r
     const size_t r = i / width, c = i % width;
     out[i] = h[(size_t)row_token[r] * width + c];
 }
+// The same as the BF16 split of a tensor-core GEMM's input, one CTA per (padded) row; rows between the runs are skipped.  total: one past the last live row
+__global__ void __launch_bounds__(256) moe_gather_split_kernel(__nv_bfloat16* __restrict__ hi, size_t lo, const float* __restrict__ h, const int* __restrict__ row_token,
+                                                               const int* __restrict__ total, int width) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = blockIdx.x;
+    if (r >= *total) return;
+    const int t = row_token[r];
+    if (t < 0) return;
+    const float4* src = reinterpret_cast<const float4*>(h + (size_t)t * width);
+    for (int i = threadIdx.x; i < width / 4; i += blockDim.x) {
+        const float4 f = src[i];
+        const float v[4] = {f.x, f.y, f.z, f.w};
+        split_store4(hi, hi + lo, (size_t)r * width + 4 * (size_t)i, v);
+    }
+}
+// four channels per thread
+__global__ void __launch_bounds__(256) moe_combine4_kernel(float* __restrict__ y, const float* __restrict__ y_rows, const int* __restrict__ assign_row, const float* __restrict__ wt,
+                                                           const float* __restrict__ sgate, const float* __restrict__ shared_y, size_t n4, int top, int width4, int add) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x;
+    if (i >= n4) return;
+    const size_t t = i / width4, c = i % width4;
+    const float4* rows = reinterpret_cast<const float4*>(y_rows);
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int k = 0; k < top; k++) {
+        const float w = wt[t * top + k];
+        const float4 v = rows[(size_t)assign_row[t * top + k] * width4 + c];
+        a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+    }
+    if (shared_y) {
+        const float w = sgate ? sgate[t] : 1.f;
+        const float4 v = reinterpret_cast<const float4*>(shared_y)[i];
+        a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+    }
+    float4* out = reinterpret_cast<float4*>(y) + i;
+    if (add) { const float4 o = *out; a.x += o.x; a.y += o.y; a.z += o.z; a.w += o.w; }
+    *out = a;
+}
 __global__ void moe_combine_kernel(float* __restrict__ y, const float* __restrict__ y_rows, const int* __restrict__ assign_row, const float* __restrict__ wt,
                                    const float* __restrict__ sgate, const float* __restrict__ shared_y, size_t n, int top, int width, int add) {
     pdl_launch_dependents();
@@ -500,13 +544,34 @@ void moe_expert_down_token(float* y, const float* act, const int* sel, const flo
     count_launch();
 }
 
-size_t moe_work_ints(int tokens, int experts, int top) { return (size_t)experts + 1 + 2 * (size_t)tokens * top + (size_t)experts; }
+size_t moe_rows_cap(int tokens, int experts, int top, int pad) {
+    const size_t n = (size_t)tokens * top;
+    return pad > 1 ? (n + pad - 1) / pad * pad + (size_t)experts * pad : n;
+}
+size_t moe_work_ints(int tokens, int experts, int top, int pad) {
+    return (size_t)experts + 1 + moe_rows_cap(tokens, experts, top, pad) + (size_t)tokens * top + (size_t)experts;
+}
+static int* moe_assign_of(int* work, int tokens, int experts, int top, int pad) { return work + experts + 1 + moe_rows_cap(tokens, experts, top, pad); }
+const int* moe_counts_of(const int* work, int tokens, int experts, int top, int pad) {
+    return moe_assign_of(const_cast<int*>(work), tokens, experts, top, pad) + (size_t)tokens * top;
+}
 
-void moe_group(int* work, const int* sel, int tokens, int experts, int top, cudaStream_t s) {
+void moe_group(int* work, const int* sel, int tokens, int experts, int top, cudaStream_t s, int pad) {
     if (tokens <= 0) return;
-    launch_k(moe_count_kernel, dim3(experts), dim3(32), 0, s, work, sel, tokens * top, experts);
-    launch_k(moe_place_kernel, dim3(experts), dim3(PL_WARPS * 32), 0, s, work, sel, tokens * top, experts, top);
+    int* counts = const_cast<int*>(moe_counts_of(work, tokens, experts, top, pad));
+    launch_k(moe_count_kernel, dim3(experts), dim3(32), 0, s, counts, sel, tokens * top);
+    launch_k(moe_place_kernel, dim3(experts), dim3(PL_WARPS * 32), 0, s, work, work + experts + 1, moe_assign_of(work, tokens, experts, top, pad), (const int*)counts, sel,
+             tokens * top, experts, top, pad);
     count_launch(2);
+}
+
+void moe_gather_split(void* ws, const float* h, const int* work, int tokens, int experts, int top, int pad, int width, cudaStream_t s) {
+    if (tokens <= 0) return;
+    NT_CHECK(width % 4 == 0 && pad > 1, "moe_gather_split: padded runs of rows whose width is a multiple of 4");
+    const int cap = (int)moe_rows_cap(tokens, experts, top, pad);
+    launch_k(moe_gather_split_kernel, dim3(cap), dim3(std::min(256, (width / 4 + 31) / 32 * 32)), 0, s, static_cast<__nv_bfloat16*>(ws), (size_t)cap * width, h, work + experts + 1,
+             work + experts, width);
+    count_launch();
 }
 
 void moe_expert_up_rows(float* act_rows, const float* h, const int* work, const MoeWeights& w, int tokens, cudaStream_t s) {
@@ -536,10 +601,16 @@ void moe_expert_down_rows(float* y_rows, const float* act_rows, const int* work,
     count_launch();
 }
 void moe_combine(float* y, const float* y_rows, const int* work, const float* wt, const float* sgate, const float* shared_y, int tokens,
-                 int experts, int top, int width, cudaStream_t s, bool add) {
+                 int experts, int top, int width, cudaStream_t s, bool add, int pad) {
     const size_t n = (size_t)tokens * width;
     if (!n) return;
-    launch_k(moe_combine_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, y, y_rows, work + experts + 1 + (size_t)tokens * top, wt, sgate,
+    const int* assign = moe_assign_of(const_cast<int*>(work), tokens, experts, top, pad);
+    if (width % 4 == 0 && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(y_rows) | reinterpret_cast<uintptr_t>(shared_y)) & 15) == 0) {
+        launch_k(moe_combine4_kernel, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), 0, s, y, y_rows, assign, wt, sgate, shared_y, n / 4, top, width / 4, add ? 1 : 0);
+        count_launch();
+        return;
+    }
+    launch_k(moe_combine_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, s, y, y_rows, assign, wt, sgate,
              shared_y, n, top, width, add ? 1 : 0);
     count_launch();
 }

@@ -15,6 +15,7 @@
 #include <cuda.h>
 #include <cuda_fp16.h>
 #include <cuda_bf16.h>
+#include <algorithm>
 #include <mutex>
 
 namespace nt { namespace b200 {
@@ -44,6 +45,9 @@ __device__ __forceinline__ float gate_act(float g, int gelu) {
     const float u = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return 0.5f * g * (2.0f - 2.0f / (expf(2.0f * u) + 1.0f));
 }
+// xIELU with a = softplus(p), b = softplus(q) of the layer's two numbers
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float xielu_act(float z, float a, float b) { return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(0.5f + b, expm1f(z) - z, 0.5f * z); }
 // a = hi + lo with hi = f16(a), lo = f16(a - hi): 4 floats per thread
 // The same split into two BF16 values (operands of the BF16 tensor-core form, ~16 mantissa bits together): packed pair of 16-bit words
 __device__ __forceinline__ void split_pair(float a, float b, int bf16, uint32_t& hi, uint32_t& lo) {
@@ -94,6 +98,9 @@ __device__ __forceinline__ void tma_load_2d(void* dst, const CUtensorMap* map, i
     asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
                  ::"r"(smem_u32(dst)), "l"(map), "r"(c0), "r"(c1), "r"(smem_u32(bar)) : "memory");
 }
+__device__ __forceinline__ void tensormap_acquire(const CUtensorMap* map) {
+    asm volatile("fence.proxy.tensormap::generic.acquire.sys [%0], 128;" ::"l"(map) : "memory");
+}
 // K-major, SWIZZLE_128B shared-memory matrix descriptor (cute::UMMA::SmemDescriptor bit layout): start address >> 4 in
 // [0,14), leading byte offset [16,30) (unused for swizzled K-major, canonical value 1), stride byte offset [32,46) =
 // 8 rows x 128 B = 1024 B, version 1 at [46,48), layout type SWIZZLE_128B = 2 at [61,64).
@@ -127,7 +134,12 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&v)[32]) {
         : "r"(taddr));
 }
 
-enum : int { MODE_STORE = 0, MODE_ADD = 1, MODE_SWIGLU = 2 };
+enum : int { MODE_STORE = 0, MODE_ADD = 1, MODE_SWIGLU = 2, MODE_XIELU = 3 };
+
+// Grouped form: the rows of A are `experts` runs, run e with count[e] rows from row start[e] (a multiple of BM) on and a weight matrix of its own
+// (maps_b[e], gate / up pairs: maps_b2[e]; encoded on the host, resident in device memory).  The tile list is made on the device from the counts.
+constexpr int MAX_GROUPS = 256;
+struct Grouped { const CUtensorMap* maps_b; const CUtensorMap* maps_b2; const int* start; const int* count; int experts; };
 
 // Persistent, warp-specialised GEMM: CTA b handles output tiles b, b + grid, ...; the shared-memory ring and the two TMEM
 // accumulators run across tile boundaries, so the epilogue of tile i overlaps the MMAs of tile i + 1.
@@ -140,13 +152,16 @@ enum : int { MODE_STORE = 0, MODE_ADD = 1, MODE_SWIGLU = 2 };
 //   MODE_SWIGLU (BN = 256 as 128 gate + 128 up columns, W = gate via map_b, up via map_b2):
 //               split_out = F16 hi/lo split of silu(A.Wg^T) * (A.Wu^T), i.e. the down projection's GEMM input, so the
 //               F32 gate/up activations never touch HBM (ffn.cpp:96-133 computes them as three launches).
-template <int BN, int MODE>
+//   MODE_XIELU  split_out = hi/lo split of xIELU(A.W^T), (p, q) = act_p: the ungated feed-forward's input of the down projection
+template <int BN, int MODE, bool GROUPED>
 __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                                                              const __grid_constant__ CUtensorMap map_b,
                                                              const __grid_constant__ CUtensorMap map_b2,
                                                              float* __restrict__ C, __half* __restrict__ split_out,
                                                              int M, int Mp, int N, int K, int tiles_m, int tiles_n, int n_tiles, int n_outer,
-                                                             int kc_blocks, int bf16, int gelu, const float* __restrict__ col_scale, float alpha) {
+                                                             int kc_blocks, int bf16, int gelu, const float* __restrict__ col_scale, float alpha,
+                                                             const float* __restrict__ act_p, const Grouped grp) {
+    constexpr bool ONE_CHUNK = MODE == MODE_SWIGLU || MODE == MODE_XIELU;       // the epilogue needs the whole sum
     constexpr int STAGES = Cfg<BN>::STAGES, STAGE_BYTES = Cfg<BN>::STAGE_BYTES, TMEM_COLS = 2 * BN;
     constexpr int TN = MODE == MODE_SWIGLU ? 128 : BN;          // output columns per tile
     // BF16 operands: A format at [7,10) and B format at [10,13) become 1 (F16 = 0); layouts, strides and the F32 accumulator are the same
@@ -156,9 +171,24 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ uint64_t full_bar[STAGES], empty_bar[STAGES], tmem_full_bar[2], tmem_empty_bar[2];
     __shared__ uint32_t tmem_base_smem;
+    __shared__ int tile_end[GROUPED ? MAX_GROUPS : 1];          // grouped: tiles of the runs up to and including run e
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (GROUPED) {
+        for (int e = threadIdx.x; e < grp.experts; e += 192) tile_end[e] = (grp.count[e] + BM - 1) / BM * tiles_n;
+        __syncthreads();
+        if (threadIdx.x == 0) for (int e = 1; e < grp.experts; e++) tile_end[e] += tile_end[e - 1];
+        __syncthreads();
+        n_tiles = tile_end[grp.experts - 1];
+    }
+    // tile -> its run (tiles ascend: the run is followed from the last one), first row, first column, one past the last live row
+    auto place = [&](int tile, int& e, int& m0, int& n0, int& m_end) {
+        if (!GROUPED) { m0 = (n_outer ? tile % tiles_m : tile / tiles_n) * BM; n0 = (n_outer ? tile / tiles_m : tile % tiles_n) * TN; m_end = M; return; }
+        while (tile >= tile_end[e]) e++;
+        const int local = tile - (e ? tile_end[e - 1] : 0), cnt = grp.count[e], tm = (cnt + BM - 1) / BM;
+        m0 = grp.start[e] + local % tm * BM; n0 = local / tm * TN; m_end = grp.start[e] + cnt;
+    };
     const int num_kb = K / BK;
-    const int n_kc = (MODE == MODE_SWIGLU) ? 1 : (num_kb + kc_blocks - 1) / kc_blocks;      // accumulation chunks per tile
+    const int n_kc = ONE_CHUNK ? 1 : (num_kb + kc_blocks - 1) / kc_blocks;      // accumulation chunks per tile
 
     if (warp == 0 && lane == 0) {
         for (int s = 0; s < STAGES; s++) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
@@ -177,8 +207,16 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
     if (warp == 0) {
         if (lane == 0) {                               // ---- TMA producer ----
             uint32_t it = 0;                           // k-block counter across all of this CTA's tiles
+            int run = 0, m0 = 0, n0 = 0, m_end = 0, fenced = -1;
             for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
-                const int m0 = (n_outer ? tile % tiles_m : tile / tiles_n) * BM, n0 = (n_outer ? tile / tiles_m : tile % tiles_n) * TN;
+                place(tile, run, m0, n0, m_end);
+                if (GROUPED && run != fenced) {        // maps in global memory: acquire them before this CTA's first use
+                    tensormap_acquire(grp.maps_b + run);
+                    if (MODE == MODE_SWIGLU) tensormap_acquire(grp.maps_b2 + run);
+                    fenced = run;
+                }
+                const CUtensorMap* mb = GROUPED ? grp.maps_b + run : &map_b;
+                const CUtensorMap* mb2 = GROUPED ? grp.maps_b2 + run : &map_b2;
                 for (int kb = 0; kb < num_kb; kb++, it++) {         // chunk boundaries do not matter to the producer
                     const uint32_t s = it % STAGES;
                     wait_or_trap(&empty_bar[s], ((it / STAGES) & 1) ^ 1);
@@ -186,8 +224,8 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                     mbar_expect_tx(&full_bar[s], STAGE_BYTES);
                     tma_load_2d(st, &map_a, kb * BK, m0, &full_bar[s]);                 // A_hi rows [m0, m0+128)
                     tma_load_2d(st + TILE_A, &map_a, kb * BK, Mp + m0, &full_bar[s]);   // A_lo lives below A_hi
-                    tma_load_2d(st + 2 * TILE_A, &map_b, kb * BK, n0, &full_bar[s]);
-                    if (MODE == MODE_SWIGLU) tma_load_2d(st + 2 * TILE_A + 128 * BK * 2, &map_b2, kb * BK, n0, &full_bar[s]);
+                    tma_load_2d(st + 2 * TILE_A, mb, kb * BK, n0, &full_bar[s]);
+                    if (MODE == MODE_SWIGLU) tma_load_2d(st + 2 * TILE_A + 128 * BK * 2, mb2, kb * BK, n0, &full_bar[s]);
                 }
             }
         }
@@ -200,7 +238,7 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                 wait_or_trap(&tmem_empty_bar[acc], acc_phase ^ 1);         // epilogue drained this accumulator
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const uint32_t d = tmem_base + acc * BN;
-                const int kb0 = (MODE == MODE_SWIGLU) ? 0 : kc * kc_blocks, kb1 = (MODE == MODE_SWIGLU) ? num_kb : min(num_kb, kb0 + kc_blocks);
+                const int kb0 = ONE_CHUNK ? 0 : kc * kc_blocks, kb1 = ONE_CHUNK ? num_kb : min(num_kb, kb0 + kc_blocks);
                 for (int kb = kb0; kb < kb1; kb++, it++) {
                     const uint32_t s = it % STAGES;
                     wait_or_trap(&full_bar[s], (it / STAGES) & 1);
@@ -227,11 +265,14 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
         // ---- epilogue: TMEM -> registers -> global (warp w may only touch TMEM lanes [32 * (w % 4), +32)) ----
         const int quarter = warp & 3;
         uint32_t lt = 0;
+        int run = 0, m0 = 0, n0 = 0, m_end = 0;
+        float act_a = 0.f, act_b = 0.f;
+        if (MODE == MODE_XIELU) { act_a = softplus_f(act_p[0]); act_b = softplus_f(act_p[1]); }
         for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x)
         for (int kc = 0; kc < n_kc; kc++, lt++) {
             const uint32_t acc = lt & 1, acc_phase = (lt >> 1) & 1;
             const bool add_c = MODE == MODE_ADD || kc > 0;           // later chunks add their partial sums to what is in C
-            const int m0 = (n_outer ? tile % tiles_m : tile / tiles_n) * BM, n0 = (n_outer ? tile / tiles_m : tile % tiles_n) * TN;
+            if (kc == 0) place(tile, run, m0, n0, m_end);
             const int row = m0 + quarter * 32 + lane;
             wait_or_trap(&tmem_full_bar[acc], acc_phase);
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -244,7 +285,7 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                     uint32_t u[32];
                     tmem_ld32(tacc + 128u + (uint32_t)(c * 32), u);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    if (row < M) {
+                    if (row < m_end) {
                         __half* hi = split_out + (size_t)row * N + n0 + c * 32;
                         __half* lo = hi + (size_t)Mp * N;
 #pragma unroll
@@ -261,9 +302,25 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                             *reinterpret_cast<uint4*>(lo + j) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
                         }
                     }
+                } else if (MODE == MODE_XIELU) {
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (row < m_end) {
+                        __half* hi = split_out + (size_t)row * N + n0 + c * 32;
+                        __half* lo = hi + (size_t)Mp * N;
+#pragma unroll
+                        for (int j = 0; j < 32; j += 8) {
+                            if (n0 + c * 32 + j >= N) break;             // a ragged last tile (N % 8 == 0)
+                            uint32_t ph[4], pl[4];
+#pragma unroll
+                            for (int e = 0; e < 4; e++)
+                                split_pair(xielu_act(__uint_as_float(v[j + 2 * e]), act_a, act_b), xielu_act(__uint_as_float(v[j + 2 * e + 1]), act_a, act_b), bf16, ph[e], pl[e]);
+                            *reinterpret_cast<uint4*>(hi + j) = make_uint4(ph[0], ph[1], ph[2], ph[3]);
+                            *reinterpret_cast<uint4*>(lo + j) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
+                        }
+                    }
                 } else {
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    if (row < M) {
+                    if (row < m_end) {
                         float* crow = C + (size_t)row * N + n0 + c * 32;
 #pragma unroll
                         for (int j = 0; j < 32; j += 4) {
@@ -397,7 +454,7 @@ bool launch_gemm(float* C, __half* split_out, const void* workspace, const void*
         !make_map(&map_b2, W2 ? W2 : W, (uint64_t)N, (uint64_t)K, TN, o.bf16))
         return false;
     static unsigned long long configured = 0;      // bit per device id
-    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE>, (int)(Cfg<BN>::SMEM), configured);
+    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE, false>, (int)(Cfg<BN>::SMEM), configured);
     const int tiles_m = (int)(Mp / BM), tiles_n = (N + TN - 1) / TN, n_tiles = tiles_n * tiles_m;
     const int grid = n_tiles < sm_count() ? n_tiles : sm_count();
     // Tile order: concurrently running CTAs share the operand that is walked in the inner loop, the other one should stay
@@ -412,8 +469,27 @@ bool launch_gemm(float* C, __half* split_out, const void* workspace, const void*
     // 13.5k vs 17.6k on Q4_K_M: the read-modify-write of C per chunk is not free); NT_B200_GEMM_KC=<k-blocks> overrides (0: whole K)
     static const int kc_env = [] { const char* e = getenv("NT_B200_GEMM_KC"); return e ? atoi(e) : 64; }();
     const int kc_blocks = kc_env > 0 ? kc_env : K / BK;
-    gemm_f16_tc_kernel<BN, MODE><<<grid, 192, Cfg<BN>::SMEM, s>>>(map_a, map_b, map_b2, C, split_out, M, (int)Mp, N, K, tiles_m, tiles_n,
-                                                                 n_tiles, n_outer, kc_blocks, o.bf16 ? 1 : 0, o.relu ? 2 : (o.gelu ? 1 : 0), o.col_scale, o.alpha);
+    gemm_f16_tc_kernel<BN, MODE, false><<<grid, 192, Cfg<BN>::SMEM, s>>>(map_a, map_b, map_b2, C, split_out, M, (int)Mp, N, K, tiles_m, tiles_n,
+                                                                        n_tiles, n_outer, kc_blocks, o.bf16 ? 1 : 0, o.relu ? 2 : (o.gelu ? 1 : 0), o.col_scale, o.alpha, o.act_p,
+                                                                        Grouped{});
+    count_launch();
+    return true;
+}
+
+// One launch for every run of the grouped rows; Mp: rows the workspace holds (a multiple of 128, all runs padded).  Tiles never outnumber
+// Mp / 128 per column tile, which bounds the grid.
+template <int BN, int MODE>
+bool launch_grouped(float* C, __half* split_out, const void* workspace, const Grouped& grp, size_t Mp, int N, int K, cudaStream_t s, const TcOpts& o) {
+    constexpr int TN = MODE == MODE_SWIGLU ? 128 : BN;
+    CUtensorMap map_a;
+    if (!make_map(&map_a, workspace, 2 * Mp, (uint64_t)K, BM, o.bf16)) return false;
+    static unsigned long long configured = 0;
+    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE, true>, (int)(Cfg<BN>::SMEM), configured);
+    const int tiles_n = (N + TN - 1) / TN;
+    const int grid = (int)std::min<size_t>((size_t)sm_count(), Mp / BM * tiles_n);
+    gemm_f16_tc_kernel<BN, MODE, true><<<grid, 192, Cfg<BN>::SMEM, s>>>(map_a, map_a, map_a, C, split_out, 0, (int)Mp, N, K, 0, tiles_n, 0, 0, 64, o.bf16 ? 1 : 0,
+                                                                       o.relu ? 2 : (o.gelu ? 1 : 0), nullptr, 1.0f, nullptr, grp);
+    NT_LAUNCH_CHECK();
     count_launch();
     return true;
 }
@@ -438,6 +514,36 @@ bool gemm_f16_tc_swiglu_ws(void* workspace_out, const void* workspace_in, const 
     if (M <= 0 || !gemm_f16_tc_supported(Wgate_f16, N, K, 0) || !gemm_f16_tc_supported(Wup_f16, N, K, 0)) return false;
     const size_t Mp = ((size_t)M + BM - 1) / BM * BM;
     return launch_gemm<256, MODE_SWIGLU>(nullptr, static_cast<__half*>(workspace_out), workspace_in, Wgate_f16, Wup_f16, M, Mp, N, K, s, o);
+}
+
+// workspace_out <- split(xIELU(A.W^T)); N % 8 == 0
+bool gemm_f16_tc_xielu_ws(void* workspace_out, const void* workspace_in, const void* W_f16, const float* act_p, int M, int N, int K, cudaStream_t s, const TcOpts& o_in) {
+    if (M <= 0 || N % 8 != 0 || !gemm_f16_tc_ragged_supported(W_f16, N, K, 0)) return false;
+    const size_t Mp = ((size_t)M + BM - 1) / BM * BM;
+    TcOpts o = o_in;
+    o.act_p = act_p;
+    __half* out = static_cast<__half*>(workspace_out);
+    return N % 256 == 0 ? launch_gemm<256, MODE_XIELU>(nullptr, out, workspace_in, W_f16, nullptr, M, Mp, N, K, s, o)
+                        : launch_gemm<128, MODE_XIELU>(nullptr, out, workspace_in, W_f16, nullptr, M, Mp, N, K, s, o);
+}
+
+// ---- grouped rows (routed experts) ----
+size_t gemm_tc_map_bytes() { return sizeof(CUtensorMap); }
+bool gemm_tc_weight_map(void* map_host, const void* W, int N, int K, bool gated, bool bf16) {
+    return make_map(static_cast<CUtensorMap*>(map_host), W, (uint64_t)N, (uint64_t)K, gated || N % 256 != 0 ? 128 : 256, bf16);
+}
+bool gemm_f16_tc_grouped_swiglu(void* workspace_out, const void* workspace_in, const void* maps_gate, const void* maps_up, const int* start, const int* count, int experts,
+                                int rows_padded, int N, int K, cudaStream_t s, const TcOpts& o) {
+    if (experts < 1 || experts > MAX_GROUPS || N % 128 != 0 || K % BK != 0 || rows_padded % BM != 0) return false;
+    const Grouped g{static_cast<const CUtensorMap*>(maps_gate), static_cast<const CUtensorMap*>(maps_up), start, count, experts};
+    return launch_grouped<256, MODE_SWIGLU>(nullptr, static_cast<__half*>(workspace_out), workspace_in, g, (size_t)rows_padded, N, K, s, o);
+}
+bool gemm_f16_tc_grouped(float* C, const void* workspace, const void* maps, const int* start, const int* count, int experts, int rows_padded, int N, int K, cudaStream_t s,
+                         const TcOpts& o) {
+    if (experts < 1 || experts > MAX_GROUPS || N < 128 || N % 4 != 0 || K % BK != 0 || rows_padded % BM != 0) return false;
+    const Grouped g{static_cast<const CUtensorMap*>(maps), static_cast<const CUtensorMap*>(maps), start, count, experts};
+    return N % 256 == 0 ? launch_grouped<256, MODE_STORE>(C, nullptr, workspace, g, (size_t)rows_padded, N, K, s, o)
+                        : launch_grouped<128, MODE_STORE>(C, nullptr, workspace, g, (size_t)rows_padded, N, K, s, o);
 }
 
 // C[M,N] = A[M,K] . W[N,K]^T ; N % 128 == 0, K % 64 == 0; workspace >= gemm_f16_tc_workspace_bytes(M, K)
