@@ -191,37 +191,64 @@ __global__ void __launch_bounds__(256) latent_rows_f32_kernel(float* __restrict_
     out[e] = wld(cache, ((size_t)r0 + r) * row + i);
 }
 
-// kfull [r, h, kw] = [ku[r - r0, h, :dim] | rotated key part of row r | 0 ...]; vfull [r, h, vw] = [vu[r - r0, h, :vdim] | 0 ...]
+// kfull [r, h, kw] = [ku[r - r0, h, :dim] | rotated key part of row r | 0 ...]; vfull [r, h, vw] = [vu[r - r0, h, :vdim] | 0 ...].  A CTA per row,
+// two channels per thread and store (kw, vw are even).
 __global__ void __launch_bounds__(256) latent_expand_pack_kernel(__nv_bfloat16* __restrict__ kfull, __nv_bfloat16* __restrict__ vfull, const float* __restrict__ ku,
                                                                  const float* __restrict__ vu, const __nv_bfloat16* __restrict__ cache, int row, int kv_rank,
                                                                  int r0, int heads, int dim, int rot_dim, int vdim, int kw, int vw) {
     pdl_launch_dependents();
     pdl_wait();
-    const int r = blockIdx.x, h = blockIdx.y;
+    const int r = blockIdx.x;
     const size_t ar = (size_t)r0 + r;
-    for (int i = threadIdx.x; i < kw; i += 256) {
-        __nv_bfloat16 v = __float2bfloat16_rn(0.f);
-        if (i < dim) v = __float2bfloat16_rn(ku[((size_t)r * heads + h) * dim + i]);
-        else if (i < dim + rot_dim) v = cache[ar * row + kv_rank + (i - dim)];
-        kfull[(ar * heads + h) * kw + i] = v;
+    const __nv_bfloat16* kr = cache + ar * row + kv_rank;
+    const float* kp = ku + (size_t)r * heads * dim;
+    const float* vp = vu + (size_t)r * heads * vdim;
+    for (int e = threadIdx.x * 2; e < heads * kw; e += 512) {
+        const int h = e / kw, i = e - h * kw;
+        float v[2];
+#pragma unroll
+        for (int q = 0; q < 2; q++) {
+            const int c = i + q;
+            v[q] = c < dim ? kp[h * dim + c] : c < dim + rot_dim ? wld(kr, (size_t)(c - dim)) : 0.f;      // 16-bit values survive the round trip
+        }
+        *reinterpret_cast<__nv_bfloat162*>(kfull + ar * heads * kw + e) = __floats2bfloat162_rn(v[0], v[1]);
     }
-    for (int i = threadIdx.x; i < vw; i += 256)
-        vfull[(ar * heads + h) * vw + i] = __float2bfloat16_rn(i < vdim ? vu[((size_t)r * heads + h) * vdim + i] : 0.f);
+    for (int e = threadIdx.x * 2; e < heads * vw; e += 512) {
+        const int h = e / vw, i = e - h * vw;
+        *reinterpret_cast<__nv_bfloat162*>(vfull + ar * heads * vw + e) =
+            __floats2bfloat162_rn(i < vdim ? vp[h * vdim + i] : 0.f, i + 1 < vdim ? vp[h * vdim + i + 1] : 0.f);
+    }
 }
 
-// qp [t, h, kw] = [q[t, h, :dim] | rot(q[t, h, dim:]) | 0 ...]
+// qp [t, h, kw] = [q[t, h, :dim] | rot(q[t, h, dim:]) | 0 ...].  A CTA per token: the position's cosines and sines are computed once for all heads.
 __global__ void __launch_bounds__(256) latent_q_rot_pad_kernel(float* __restrict__ qp, const float* __restrict__ q, int heads, int dim, int rot_dim, int kw, int dims,
                                                                int interleaved, double log2_base, int p0) {
+    extern __shared__ __align__(16) float cs[];           // cos, sin of dims / 2 pairs
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x, h = blockIdx.y, qd = dim + rot_dim;
-    const float* src = q + ((size_t)t * heads + h) * qd;
-    float* dst = qp + ((size_t)t * heads + h) * kw;
-    for (int i = threadIdx.x; i < kw; i += 256) {
-        float v = 0.f;
-        if (i < dim) v = src[i];
-        else if (i < qd) v = rotated(src + dim, i - dim, dims, interleaved, log2_base, p0 + t);
-        dst[i] = v;
+    const int t = blockIdx.x, qd = dim + rot_dim, half = dims >> 1;
+    for (int i = threadIdx.x; i < half; i += 256) {
+        double sn, co;
+        sincos((double)(p0 + t) * exp2(-2.0 * (double)i / (double)dims * log2_base), &sn, &co);
+        cs[2 * i] = (float)co; cs[2 * i + 1] = (float)sn;
+    }
+    __syncthreads();
+    const float* src = q + (size_t)t * heads * qd;
+    float* dst = qp + (size_t)t * heads * kw;
+    for (int e = threadIdx.x; e < heads * kw; e += 256) {
+        const int h = e / kw, i = e - h * kw;
+        const float* qh = src + h * qd;
+        float v = i < qd ? qh[i] : 0.f;
+        const int c = i - dim;
+        if (c >= 0 && c < dims) {
+            int pair, mate;
+            bool first;
+            if (interleaved) { pair = c >> 1; first = (c & 1) == 0; mate = first ? c + 1 : c - 1; }
+            else { first = c < half; pair = first ? c : c - half; mate = first ? c + half : c - half; }
+            const float co = cs[2 * pair], sn = cs[2 * pair + 1], m = qh[dim + mate];
+            v = first ? v * co - m * sn : v * co + m * sn;
+        }
+        dst[e] = v;
     }
 }
 
@@ -455,8 +482,8 @@ void latent_expand_pack(void* kfull, void* vfull, const float* ku, const float* 
                         int dim, int rot_dim, int vdim, int kw, int vw, cudaStream_t s) {
     if (n <= 0) return;
     NT_CHECK(cache_dt == DType::BF16, "latent_expand_pack: BF16 cache rows");
-    NT_CHECK(kw >= dim + rot_dim && vw >= vdim, "latent_expand_pack: padded widths below the head's");
-    launch_k(latent_expand_pack_kernel, dim3(n, heads), dim3(256), 0, s, static_cast<__nv_bfloat16*>(kfull), static_cast<__nv_bfloat16*>(vfull), ku, vu,
+    NT_CHECK(kw >= dim + rot_dim && vw >= vdim && kw % 2 == 0 && vw % 2 == 0, "latent_expand_pack: padded widths below the head's");
+    launch_k(latent_expand_pack_kernel, dim3(n), dim3(256), 0, s, static_cast<__nv_bfloat16*>(kfull), static_cast<__nv_bfloat16*>(vfull), ku, vu,
              static_cast<const __nv_bfloat16*>(cache), kv_rank + rot_dim, kv_rank, r0, heads, dim, rot_dim, vdim, kw, vw);
     count_launch();
 }
@@ -464,7 +491,7 @@ void latent_expand_pack(void* kfull, void* vfull, const float* ku, const float* 
 void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, int rot_dims, bool interleaved, double rot_base, int p0,
                       cudaStream_t s) {
     if (T <= 0) return;
-    launch_k(latent_q_rot_pad_kernel, dim3(T, heads), dim3(256), 0, s, qp, q, heads, dim, rot_dim, kw, rot_dims, interleaved ? 1 : 0, std::log2(rot_base), p0);
+    launch_k(latent_q_rot_pad_kernel, dim3(T), dim3(256), sizeof(float) * (size_t)std::max(2, rot_dims), s, qp, q, heads, dim, rot_dim, kw, rot_dims, interleaved ? 1 : 0, std::log2(rot_base), p0);
     count_launch();
 }
 

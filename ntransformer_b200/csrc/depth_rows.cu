@@ -142,6 +142,90 @@ __global__ void __launch_bounds__(256) depth_norm_kernel(DepthNorm p) {
     for (int i = threadIdx.x + DN_KEEP * nt; i < n; i += nt) emit(i, blend(i));
 }
 
+// The same over prompt rows for groups of at most 32 * DN_KEEP 16-byte pieces: a warp per (row, group), no barrier.
+__global__ void __launch_bounds__(256) depth_norm_warp_kernel(DepthNorm p, int n_items) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int item = (int)blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= n_items) return;
+    const int per = p.width / p.groups, n = per / 4, t = item / p.groups, c0 = (item - t * p.groups) * per;
+    const size_t row = (size_t)t * p.width + c0;
+    Pack<4> keep[DN_KEEP];
+#pragma unroll
+    for (int k = 0; k < DN_KEEP; k++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) keep[k].v[e] = 0.f;
+    for (int j = p.coef ? 0 : p.n - 1; j < p.n; j++) {
+        const float c = p.coef ? __ldg(p.coef + j) : 1.f;
+        const float* x = p.X + (size_t)j * p.slot + row;
+#pragma unroll
+        for (int k = 0; k < DN_KEEP; k++) {
+            const int i = lane + 32 * k;
+            if (i < n) {
+                const Pack<4> v = ldp<4>(x + 4 * i);
+#pragma unroll
+                for (int e = 0; e < 4; e++) keep[k].v[e] = fmaf(c, v.v[e], keep[k].v[e]);
+            }
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < DN_KEEP; k++) {
+        const int i = lane + 32 * k;
+        if (i < n) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) ss = fmaf(keep[k].v[e], keep[k].v[e], ss);
+            if (p.x_out) stp(p.x_out + row + 4 * (size_t)i, keep[k]);
+        }
+    }
+    if (!p.gain) return;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o);
+    const float inv = 1.0f / sqrtf(ss / (float)per + p.eps);
+#pragma unroll
+    for (int k = 0; k < DN_KEEP; k++) {
+        const int i = lane + 32 * k;
+        if (i < n) {
+            const Pack<4> g = ldp<4>(p.gain + c0 + 4 * i);
+            Pack<4> h;
+#pragma unroll
+            for (int e = 0; e < 4; e++) h.v[e] = keep[k].v[e] * inv * g.v[e];
+            if (p.h_out) stp(p.h_out + row + 4 * (size_t)i, h);
+            if (p.split) { __nv_bfloat16* hi = static_cast<__nv_bfloat16*>(p.split); split_store4(hi, hi + p.split_lo, row + 4 * (size_t)i, h.v); }
+        }
+    }
+}
+
+// four channels per thread, BF16 tables
+__global__ void __launch_bounds__(256) embed_bigram4_kernel(float* __restrict__ x0, float* __restrict__ x1, const __nv_bfloat16* __restrict__ E, const __nv_bfloat16* __restrict__ B,
+                                                            const int* __restrict__ tokens, const int* __restrict__ prev, int width, long long buckets, long long mul_prev,
+                                                            long long mul_cur, const int* __restrict__ pos_dev, int p0) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.y, i = (blockIdx.x * 256 + threadIdx.x) * 4;
+    if (i >= width) return;
+    const long long tok = tokens[t];
+    auto load = [&](const __nv_bfloat16* p, float (&f)[4]) {
+        const uint2 w = *reinterpret_cast<const uint2*>(p);
+        f[0] = __uint_as_float(w.x << 16); f[1] = __uint_as_float(w.x & 0xFFFF0000u); f[2] = __uint_as_float(w.y << 16); f[3] = __uint_as_float(w.y & 0xFFFF0000u);
+    };
+    float a[4], b[4] = {0.f, 0.f, 0.f, 0.f};
+    load(E + (size_t)tok * width + i, a);
+    if (B) {
+        const bool first = t == 0 && (pos_dev ? *pos_dev : p0) == 0;
+        long long row = buckets;
+        if (!first) {
+            const long long before = t > 0 ? tokens[t - 1] : *prev;
+            row = (before * mul_prev + tok * mul_cur) % buckets;
+            if (row < 0) row += buckets;
+        }
+        load(B + (size_t)row * width + i, b);
+    }
+    const float4 v = make_float4(a[0] + b[0], a[1] + b[1], a[2] + b[2], a[3] + b[3]);
+    *reinterpret_cast<float4*>(x0 + (size_t)t * width + i) = v;
+    if (x1) *reinterpret_cast<float4*>(x1 + (size_t)t * width + i) = v;
+}
+
 }  // namespace
 
 void embed_bigram_rows(float* x0, float* x1, const void* E, DType edt, const void* B, DType bdt, const int* tokens_dev, const int* prev_dev, int T, int width,
@@ -149,6 +233,13 @@ void embed_bigram_rows(float* x0, float* x1, const void* E, DType edt, const voi
     if (T <= 0) return;
     NT_CHECK(dense_dtype(edt) && (!B || dense_dtype(bdt)), "embed_bigram_rows: dense tables only");
     NT_CHECK(!B || buckets > 0, "embed_bigram_rows: at least one bucket");
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(x0) | reinterpret_cast<uintptr_t>(x1) | reinterpret_cast<uintptr_t>(E) | reinterpret_cast<uintptr_t>(B);
+    if (edt == DType::BF16 && (!B || bdt == DType::BF16) && width % 4 == 0 && (bits & 15) == 0) {
+        launch_k(embed_bigram4_kernel, dim3((width + 1023) / 1024, T), dim3(256), 0, s, x0, x1, static_cast<const __nv_bfloat16*>(E), static_cast<const __nv_bfloat16*>(B), tokens_dev,
+                 prev_dev, width, buckets, mul_prev, mul_cur, pos_dev, p0);
+        count_launch();
+        return;
+    }
     launch_k(embed_bigram_kernel, dim3((width + 255) / 256, T), dim3(256), 0, s, x0, x1, E, (int)edt, B, (int)bdt, tokens_dev, prev_dev, width, buckets, mul_prev, mul_cur,
              pos_dev, p0);
     count_launch();
@@ -164,6 +255,11 @@ void depth_norm_rows(const DepthNorm& p, int T, cudaStream_t s) {
     al(p.X); al(p.x_out); al(p.h_out); al(p.gain); al(p.split); al(p.carried);
     for (int i = 0; i < p.n_mix; i++) { al(p.mu[i]); al(p.mix_out[i]); }
     const int packs = vec ? per / 4 : per;
+    if (vec && T > 1 && packs <= 32 * DN_KEEP) {
+        launch_k(depth_norm_warp_kernel, dim3((unsigned)(((size_t)T * p.groups + 7) / 8)), dim3(256), 0, s, p, T * p.groups);
+        count_launch();
+        return;
+    }
     const int threads = std::min(256, (packs + 31) / 32 * 32);
     if (vec) launch_k(depth_norm_kernel<4>, dim3(T, p.groups), dim3(threads), 0, s, p);
     else launch_k(depth_norm_kernel<1>, dim3(T, p.groups), dim3(threads), 0, s, p);

@@ -21,6 +21,7 @@
 #include "ring.cuh"
 #include <cuda_fp16.h>
 #include <algorithm>
+#include <initializer_list>
 
 namespace nt { namespace b200 {
 
@@ -82,6 +83,34 @@ __global__ void __launch_bounds__(256) wkv_prep_kernel(float* __restrict__ a, fl
         if (lane == 0) ruk[t * heads + h] = s;
     }
     for (int i = threadIdx.x; i < n; i += 256) a[t * n + i] = decay_of(a[t * n + i] + w0[i]);
+}
+
+// The same for heads of whole 16-byte pieces: LN lanes per (row, head), NV pieces each.
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <int LN, int NV>
+__global__ void __launch_bounds__(256) wkv_prep4_kernel(float* __restrict__ a, float* __restrict__ ruk, const float* __restrict__ r, const float* __restrict__ k,
+                                                        const float* __restrict__ w0, const float* __restrict__ u, int rows, int heads, int dim) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int th = (int)(((size_t)blockIdx.x * 256 + threadIdx.x) / LN), l = threadIdx.x % LN;
+    const bool live = th < rows * heads;
+    const int h = live ? th % heads : 0;
+    const size_t base = (size_t)(live ? th : 0) * dim;
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int d = 4 * (l + LN * i);
+        if (live && d < dim) {
+            const float4 R = ld4(r + base + d), K = ld4(k + base + d), U = ld4(u + h * dim + d), O = ld4(w0 + h * dim + d);
+            float4 A = ld4(a + base + d);
+            s = fmaf(R.x * U.x, K.x, s); s = fmaf(R.y * U.y, K.y, s); s = fmaf(R.z * U.z, K.z, s); s = fmaf(R.w * U.w, K.w, s);
+            A.x = decay_of(A.x + O.x); A.y = decay_of(A.y + O.y); A.z = decay_of(A.z + O.z); A.w = decay_of(A.w + O.w);
+            *reinterpret_cast<float4*>(a + base + d) = A;
+        }
+    }
+#pragma unroll
+    for (int o = LN / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xFFFFFFFFu, s, o);
+    if (l == 0 && live) ruk[th] = s;
 }
 
 // ---- recurrence over rows ----
@@ -253,6 +282,39 @@ __global__ void __launch_bounds__(256) wkv_out_norm_kernel(float* __restrict__ o
             const float y = oh[d] * inv * norm[c] * silu_f(gate[row + c]);
             if (out) out[row + c] = y;
             if (hi) split_store1(hi, hi + lo_off, row + c, y);
+        }
+    }
+}
+
+// The same for heads of whole 16-byte pieces: LN lanes per (row, head), NV pieces each.
+template <int LN, int NV>
+__global__ void __launch_bounds__(256) wkv_out_norm4_kernel(float* __restrict__ out, __nv_bfloat16* __restrict__ hi, size_t lo_off, const float* __restrict__ o,
+                                                            const float* __restrict__ gate, const float* __restrict__ norm, float eps, int rows, int heads, int dim) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int th = (int)(((size_t)blockIdx.x * 256 + threadIdx.x) / LN), l = threadIdx.x % LN;
+    const bool live = th < rows * heads;
+    const int h = live ? th % heads : 0;
+    const size_t base = (size_t)(live ? th : 0) * dim;
+    float4 v[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int d = 4 * (l + LN * i);
+        v[i] = (live && d < dim) ? ld4(o + base + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
+    }
+#pragma unroll
+    for (int q = LN / 2; q > 0; q >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, q);
+    const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int d = 4 * (l + LN * i);
+        if (live && d < dim) {
+            const float4 N = ld4(norm + h * dim + d), G = ld4(gate + base + d);
+            const float y[4] = {v[i].x * inv * N.x * silu_f(G.x), v[i].y * inv * N.y * silu_f(G.y), v[i].z * inv * N.z * silu_f(G.z), v[i].w * inv * N.w * silu_f(G.w)};
+            if (out) *reinterpret_cast<float4*>(out + base + d) = make_float4(y[0], y[1], y[2], y[3]);
+            if (hi) split_store4(hi, hi + lo_off, base + d, y);
         }
     }
 }
@@ -434,6 +496,14 @@ void tanh_rows(float* x, size_t n, cudaStream_t s) {
 
 void wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int T, int heads, int dim, cudaStream_t s) {
     if (T <= 0) return;
+    const auto al = [](std::initializer_list<const void*> ps) { uintptr_t b = 0; for (const void* p : ps) b |= reinterpret_cast<uintptr_t>(p); return (b & 15) == 0; };
+    if (dim % 4 == 0 && dim <= 256 && al({a, r, k, w0, u})) {
+#define NT_WP(LN, NV) launch_k(wkv_prep4_kernel<LN, NV>, dim3((unsigned)(((size_t)T * heads * LN + 255) / 256)), dim3(256), 0, s, a, ruk, r, k, w0, u, T, heads, dim)
+        if (dim <= 16) NT_WP(4, 1); else if (dim <= 32) NT_WP(8, 1); else if (dim <= 64) NT_WP(16, 1); else if (dim <= 128) NT_WP(32, 1); else NT_WP(32, 2);
+#undef NT_WP
+        count_launch();
+        return;
+    }
     launch_k(wkv_prep_kernel, dim3(T), dim3(256), 0, s, a, ruk, r, k, w0, u, heads, dim);
     count_launch();
 }
@@ -462,6 +532,15 @@ void wkv_rows(float* out, const float* r, const float* k, const float* v, const 
 
 void wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int T, int heads, int dim, cudaStream_t s) {
     if (T <= 0) return;
+    const auto al = [](std::initializer_list<const void*> ps) { uintptr_t b = 0; for (const void* p : ps) b |= reinterpret_cast<uintptr_t>(p); return (b & 15) == 0; };
+    if (dim % 4 == 0 && dim <= 256 && al({out, split, o, gate, norm})) {
+#define NT_WN(LN, NV) launch_k(wkv_out_norm4_kernel<LN, NV>, dim3((unsigned)(((size_t)T * heads * LN + 255) / 256)), dim3(256), 0, s, out, static_cast<__nv_bfloat16*>(split), \
+                               split_lo_offset(T, heads * dim), o, gate, norm, eps, T, heads, dim)
+        if (dim <= 16) NT_WN(4, 1); else if (dim <= 32) NT_WN(8, 1); else if (dim <= 64) NT_WN(16, 1); else if (dim <= 128) NT_WN(32, 1); else NT_WN(32, 2);
+#undef NT_WN
+        count_launch();
+        return;
+    }
     launch_k(wkv_out_norm_kernel, dim3(T), dim3(256), 0, s, out, static_cast<__nv_bfloat16*>(split), split_lo_offset(T, heads * dim), o, gate, norm, eps, heads, dim);
     count_launch();
 }
