@@ -133,8 +133,10 @@ void nt_b200_depth_norm_rows(const float* X, long long slot, int n, const float*
                              int width, int groups, int n_mix, const void* const* mu, void* const* mix_out, float* carried, int p0, void* stream);
 void nt_b200_shift_mix_rows(int n, const void* const* mu, void* const* out, void* const* split, const float* h, float* carried, int rows, int width, int p0, void* stream);
 void nt_b200_wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int tokens, int heads, int dim, void* stream);
+/* scratch (may be null): nt_b200_wkv_scratch_floats numbers, with which long steps run as segments side by side */
 void nt_b200_wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int tokens, int heads, int dim, int p0,
-                      void* stream);
+                      float* scratch, void* stream);
+long long nt_b200_wkv_scratch_floats(int heads, int dim);
 void nt_b200_wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int tokens, int heads, int dim, void* stream);
 void nt_b200_wkv_token(float* out, const float* r, const float* k, const float* v, const float* gate, const float* a1, const void* w2, int dtype, const float* w0,
                        const float* u, const float* norm, float* state, float eps, int rank, int heads, int dim, int p0, void* stream);

@@ -458,9 +458,13 @@ void nt_b200_shift_mix_rows(int n, const void* const* mu, void* const* out, void
 void nt_b200_wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int tokens, int heads, int dim, void* stream) {
     wkv_prep(a, ruk, r, k, w0, u, tokens, heads, dim, static_cast<cudaStream_t>(stream));
 }
+// scratch (may be null): nt_b200_wkv_scratch_floats numbers, with which long steps run as segments side by side
 void nt_b200_wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int tokens, int heads, int dim, int p0,
-                      void* stream) {
-    wkv_rows(out, r, k, v, w, ruk, state, tokens, heads, dim, nullptr, p0, static_cast<cudaStream_t>(stream));
+                      float* scratch, void* stream) {
+    wkv_rows(out, r, k, v, w, ruk, state, tokens, heads, dim, nullptr, p0, static_cast<cudaStream_t>(stream), scratch);
+}
+long long nt_b200_wkv_scratch_floats(int heads, int dim) {
+    return (long long)wkv_rows_scratch_floats(heads, dim);
 }
 void nt_b200_wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int tokens, int heads, int dim, void* stream) {
     wkv_out_norm(out, split, o, gate, norm, eps, tokens, heads, dim, static_cast<cudaStream_t>(stream));

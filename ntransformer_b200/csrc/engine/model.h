@@ -202,6 +202,7 @@ private:
     struct ParDec { float *slots = nullptr, *h = nullptr, *mix[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}, *wide = nullptr; size_t slot = 0; } par_dec_;   // decode: stable addresses
     struct ParRows { float *slots = nullptr, *h = nullptr, *wide = nullptr; void *hs = nullptr, *mix_s[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}; size_t slot = 0; } par_;
     void latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s);
+    float* wkv_scratch_ = nullptr;            // segment states of the WKV recurrence over prompt rows (owned_)
     Weight bigram_;                           // second embedding over token pairs [buckets + 1, width]
     const LayerSpec& slot_spec(int slot) const { return *slot_spec_[(size_t)slot]; }
     std::vector<const LayerSpec*> slot_spec_;   // the mixer behind every entry of kcs_ / vcs_: the layers first, then the branches that keep rows

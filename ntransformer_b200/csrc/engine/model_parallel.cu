@@ -121,6 +121,9 @@ void Model::finalize_parallel_decode() {
     par_dec_.h = dmalloc0<float>(W);
     for (float*& m : par_dec_.mix) m = dmalloc0<float>(W);
     par_dec_.wide = dmalloc0<float>(parallel_scratch_width());
+    size_t seg = 0;
+    for (const LayerSpec& S : cfg_.layers) if (S.mixer == MixerKind::WKV) seg = std::max(seg, wkv_rows_scratch_floats(S.heads, S.dim));
+    if (seg) { wkv_scratch_ = dmalloc0<float>(seg); owned_.push_back(wkv_scratch_); }
 }
 
 void Model::ensure_parallel_buffers(size_t T) {
@@ -314,7 +317,7 @@ void Model::layer_parallel_rows(int i, int T, int p0, cudaStream_t s) {
         if (w2_tc) split_activations(pf_.ws, a1, T, S.wkv.decay_rank, s, true);
         parallel_gemm(a, a1, w2_tc ? pf_.ws : nullptr, L.wkv_w2, T, false, s);
         wkv_prep(a, ruk, r, k, L.wkv_w0, L.wkv_u, T, S.heads, S.dim, s);
-        wkv_rows(o, r, k, v, a, ruk, L.wkv_state, T, S.heads, S.dim, nullptr, p0, s);
+        wkv_rows(o, r, k, v, a, ruk, L.wkv_state, T, S.heads, S.dim, nullptr, p0, s, wkv_scratch_);
         const bool o_tc = parallel_split_ok(L.wo);
         wkv_out_norm(o_tc ? nullptr : o, o_tc ? pf_.ws : nullptr, o, g, L.wkv_norm, eps, T, S.heads, S.dim, s);
         parallel_gemm(x, o, o_tc ? pf_.ws : nullptr, L.wo, T, true, s);

@@ -399,9 +399,11 @@ void shift_mix_rows(const ShiftMix& p, const float* h, float* carried, int T, in
 void tanh_rows(float* x, size_t n, cudaStream_t s);
 // a [T, heads * dim] <- exp(-exp(a + w0));  ruk [T, heads] = sum_d r u k
 void wkv_prep(float* a, float* ruk, const float* r, const float* k, const float* w0, const float* u, int T, int heads, int dim, cudaStream_t s);
-// out [T, heads * dim] from the recurrence over the step's rows; state [heads, dim (value), dim (key)] read unless the step starts at position 0, written back
+// out [T, heads * dim] from the recurrence over the step's rows; state [heads, dim (value), dim (key)] read unless the step starts at position 0, written back.
+// scratch (wkv_rows_scratch_floats): long steps may run as segments side by side
 void wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int T, int heads, int dim, const int* pos_dev, int p0,
-              cudaStream_t s);
+              cudaStream_t s, float* scratch = nullptr);
+size_t wkv_rows_scratch_floats(int heads, int dim);
 // o / rms(head) * norm * silu(gate), as F32 rows and / or a BF16 split
 void wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int T, int heads, int dim, cudaStream_t s);
 // One token: decay from a1 [rank] (behind the tanh) and W2 [heads * dim, rank], recurrence, head norm and gate -> out [heads * dim]

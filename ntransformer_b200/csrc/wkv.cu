@@ -9,7 +9,8 @@
 //   wkv_rows         the recurrence over the rows of a step.  Every column j of S evolves on its own; LN lanes share a column (dim / LN
 //                    state numbers each, in registers).  The carried chain of a row is one multiply-add; the dot products of a tile of
 //                    16 rows stay in registers and are reduced together (a halving exchange between the lanes: 15 shuffles for 16 rows
-//                    instead of 64).  Rows are staged in tiles of 16 by cp.async into two buffers.
+//                    instead of 64).  Rows are staged in tiles of 16 by cp.async into two buffers.  Long steps are cut into segments that run
+//                    side by side (two launches: the segments' states, then the rows).
 //   wkv_out_norm     o / rms(head) * norm * silu(gate), as F32 rows or as the split of the output projection's input
 //   wkv_token        one decoded token in one launch: decay (second low-rank matrix, exponentials), recurrence, head norm and gate; a CTA
 //                    per head
@@ -148,35 +149,68 @@ __device__ __forceinline__ int reduce_rows(float (&part)[WR_TILE], int l) {
     return base;
 }
 
-// grid (ceil(dim / COLS), heads), 128 threads.  Lane l of a column holds state elements W * (c LN + l) + j, c < CH, j < W.
-template <int LN, int CH, int W>
+// grid (ceil(dim / COLS), heads, segments), 128 threads.  LN lanes share CB neighbouring columns: one read of r, k, w from shared memory (what
+// bounds the kernel) serves CB columns.  Lane l holds state elements W * (c LN + l) + j, c < CH, j < W, of each.
+// PASS 0: the whole step, one segment.  A long step with few columns is cut into segments of seg_len rows that run side by side: the recurrence is
+// linear, so the state behind a segment is (product of its decays) * (state in front) + (state from zero).
+// PASS 1: segments 0 .. segments - 2, state only: seg[z] <- the state from zero (segment 0: from the real one), decay[z] <- the product of the
+//         decays; segment 0 also keeps the step's first state in seg[last].
+// PASS 2: every segment joins the states in front of it, then produces its rows; the last one writes the state back.
+template <int LN, int CH, int W, int CB, int PASS>
 __global__ void __launch_bounds__(128) wkv_rows_kernel(float* __restrict__ out, const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v,
                                                        const float* __restrict__ w, const float* __restrict__ ruk, float* __restrict__ state, int T, int heads, int dim,
-                                                       const int* __restrict__ pos_dev, int p0) {
-    constexpr int THREADS = 128, COLS = THREADS / LN, ROWS_LEFT = LN >= WR_TILE ? 1 : WR_TILE / LN;
+                                                       const int* __restrict__ pos_dev, int p0, float* __restrict__ seg, float* __restrict__ decay, int seg_len, int segments) {
+    constexpr int THREADS = 128, COLS = THREADS / LN * CB, ROWS_LEFT = LN >= WR_TILE ? 1 : WR_TILE / LN;
     extern __shared__ __align__(16) float sm[];
     const int tile_floats = 3 * WR_TILE * dim + WR_TILE * COLS + WR_TILE;      // r | k | w [WR_TILE][dim], v [WR_TILE][COLS], ruk [WR_TILE]
     const int buf_floats = (tile_floats + 3) & ~3;
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.y, n = heads * dim;
-    const int col_l = threadIdx.x / LN, l = threadIdx.x % LN;
+    const int col_l = threadIdx.x / LN * CB, l = threadIdx.x % LN;
     const int col = blockIdx.x * COLS + col_l;
-    const bool live = col < dim;
     const bool fresh = (pos_dev ? *pos_dev : p0) == 0;
-    float* st = state + ((size_t)h * dim + (live ? col : 0)) * dim;
+    const size_t all = (size_t)heads * dim * dim;
+    auto st_off = [&](int b) { return ((size_t)h * dim + col + b) * dim; };       // only for live columns, col + b < dim
+    const int z = PASS == 0 ? 0 : blockIdx.z;
+    if (PASS != 0) {                            // this segment's rows
+        const size_t first = (size_t)z * seg_len;
+        r += first * n; k += first * n; v += first * n; w += first * n; ruk += first * heads; out += first * n;
+        T = min(seg_len, T - z * seg_len);
+    }
     int d0[CH];
     bool on[CH];
-    float S[CH][W];
+    float S[CB][CH][W], prod[PASS == 1 ? CH : 1][W];
 #pragma unroll
     for (int c = 0; c < CH; c++) {
         d0[c] = W * (c * LN + l);
         on[c] = d0[c] < dim;
+        if (PASS == 1) {
 #pragma unroll
-        for (int j = 0; j < W; j++) S[c][j] = 0.f;
-        if (on[c] && live && !fresh) {
+            for (int j = 0; j < W; j++) prod[c][j] = 1.f;
+        }
 #pragma unroll
-            for (int j = 0; j < W; j++) S[c][j] = st[d0[c] + j];
+        for (int b = 0; b < CB; b++) {
+#pragma unroll
+            for (int j = 0; j < W; j++) S[b][c][j] = 0.f;
+            if (!on[c] || col + b >= dim) continue;
+            const size_t at = st_off(b) + d0[c];
+            if (PASS != 2 && z == 0) {
+#pragma unroll
+                for (int j = 0; j < W; j++) {
+                    if (!fresh) S[b][c][j] = state[at + j];
+                    if (PASS == 1) seg[(size_t)(segments - 1) * all + at + j] = S[b][c][j];
+                }
+            }
+            if (PASS == 2) {
+                const float* from = seg + (z == 0 ? (size_t)(segments - 1) * all : 0) + at;
+#pragma unroll
+                for (int j = 0; j < W; j++) S[b][c][j] = from[j];
+                for (int y = 1; y < z; y++) {
+#pragma unroll
+                    for (int j = 0; j < W; j++) S[b][c][j] = fmaf(decay[((size_t)y * heads + h) * dim + d0[c] + j], S[b][c][j], seg[(size_t)y * all + at + j]);
+                }
+            }
         }
         if (!on[c]) d0[c] = 0;
     }
@@ -190,15 +224,15 @@ __global__ void __launch_bounds__(128) wkv_rows_kernel(float* __restrict__ out, 
         for (int i = threadIdx.x; i < nt * dv; i += THREADS) {
             const int tt = i / dv, d = (i - tt * dv) * W;
             const size_t at = (size_t)(t0 + tt) * n + (size_t)h * dim + d;
-            if constexpr (W == 4) { cp_async16(sr + tt * dim + d, r + at); cp_async16(sk + tt * dim + d, k + at); cp_async16(sw + tt * dim + d, w + at); }
-            else { cp_async4(sr + tt * dim + d, r + at); cp_async4(sk + tt * dim + d, k + at); cp_async4(sw + tt * dim + d, w + at); }
+            if constexpr (W == 4) { if (PASS != 1) cp_async16(sr + tt * dim + d, r + at); cp_async16(sk + tt * dim + d, k + at); cp_async16(sw + tt * dim + d, w + at); }
+            else { if (PASS != 1) cp_async4(sr + tt * dim + d, r + at); cp_async4(sk + tt * dim + d, k + at); cp_async4(sw + tt * dim + d, w + at); }
         }
         for (int i = threadIdx.x; i < nt * COLS; i += THREADS) {
             const int tt = i / COLS, c = blockIdx.x * COLS + i % COLS;
             if (c < dim) cp_async4(sv + i, v + (size_t)(t0 + tt) * n + (size_t)h * dim + c);
             else sv[i] = 0.f;
         }
-        for (int i = threadIdx.x; i < nt; i += THREADS) cp_async4(sb + i, ruk + (size_t)(t0 + i) * heads + h);
+        if (PASS != 1) for (int i = threadIdx.x; i < nt; i += THREADS) cp_async4(sb + i, ruk + (size_t)(t0 + i) * heads + h);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     const int n_tiles = (T + WR_TILE - 1) / WR_TILE;
@@ -217,48 +251,76 @@ __global__ void __launch_bounds__(128) wkv_rows_kernel(float* __restrict__ out, 
         const float* sw = sk + WR_TILE * dim;
         const float* sv = sw + WR_TILE * dim;
         const float* sb = sv + WR_TILE * COLS;
-        float part[WR_TILE];
+        float part[CB][WR_TILE];
         auto step = [&](int tt) {
-            const float vj = sv[tt * COLS + col_l];
-            float p = 0.f;
+            float vj[CB], p[CB];
+#pragma unroll
+            for (int b = 0; b < CB; b++) { vj[b] = sv[tt * COLS + col_l + b]; p[b] = 0.f; }
 #pragma unroll
             for (int c = 0; c < CH; c++) {
                 float rr[W], kk[W], ww[W];
                 if constexpr (W == 4) {
-                    const float4 a = *reinterpret_cast<const float4*>(sr + tt * dim + d0[c]), b = *reinterpret_cast<const float4*>(sk + tt * dim + d0[c]),
-                                 e = *reinterpret_cast<const float4*>(sw + tt * dim + d0[c]);
+                    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (PASS != 1) a = *reinterpret_cast<const float4*>(sr + tt * dim + d0[c]);
+                    const float4 b = *reinterpret_cast<const float4*>(sk + tt * dim + d0[c]), e = *reinterpret_cast<const float4*>(sw + tt * dim + d0[c]);
                     rr[0] = a.x; rr[1] = a.y; rr[2] = a.z; rr[3] = a.w; kk[0] = b.x; kk[1] = b.y; kk[2] = b.z; kk[3] = b.w; ww[0] = e.x; ww[1] = e.y; ww[2] = e.z; ww[3] = e.w;
-                } else { rr[0] = sr[tt * dim + d0[c]]; kk[0] = sk[tt * dim + d0[c]]; ww[0] = sw[tt * dim + d0[c]]; }
+                } else { rr[0] = PASS != 1 ? sr[tt * dim + d0[c]] : 0.f; kk[0] = sk[tt * dim + d0[c]]; ww[0] = sw[tt * dim + d0[c]]; }
                 if (CH == 1 || on[c]) {
 #pragma unroll
-                    for (int j = 0; j < W; j++) { p = fmaf(rr[j], S[c][j], p); S[c][j] = fmaf(ww[j], S[c][j], kk[j] * vj); }
+                    for (int j = 0; j < W; j++) {
+#pragma unroll
+                        for (int b = 0; b < CB; b++) {
+                            if (PASS != 1) p[b] = fmaf(rr[j], S[b][c][j], p[b]);
+                            S[b][c][j] = fmaf(ww[j], S[b][c][j], kk[j] * vj[b]);
+                        }
+                        if (PASS == 1) prod[c][j] *= ww[j];
+                    }
                 }
             }
-            return (CH == 1 && !on[0]) ? 0.f : p;
+#pragma unroll
+            for (int b = 0; b < CB; b++) part[b][tt] = (CH == 1 && !on[0]) ? 0.f : p[b];
         };
         if (nt == WR_TILE) {
 #pragma unroll
-            for (int tt = 0; tt < WR_TILE; tt++) part[tt] = step(tt);
+            for (int tt = 0; tt < WR_TILE; tt++) step(tt);
         } else {
 #pragma unroll
-            for (int tt = 0; tt < WR_TILE; tt++) part[tt] = tt < nt ? step(tt) : 0.f;
-        }
-        const int row0 = reduce_rows<LN>(part, l);
+            for (int tt = 0; tt < WR_TILE; tt++) {
+                if (tt < nt) step(tt);
+                else {
 #pragma unroll
-        for (int j = 0; j < ROWS_LEFT; j++) {
-            const int tt = row0 + j;
-            if (live && tt < nt && (LN <= WR_TILE || (l & 1) == 0))
-                out[(size_t)(t0 + tt) * n + (size_t)h * dim + col] = fmaf(sb[tt], sv[tt * COLS + col_l], part[j]);
+                    for (int b = 0; b < CB; b++) part[b][tt] = 0.f;
+                }
+            }
+        }
+        if (PASS != 1) {
+#pragma unroll
+            for (int b = 0; b < CB; b++) {
+                const int row0 = reduce_rows<LN>(part[b], l);
+#pragma unroll
+                for (int j = 0; j < ROWS_LEFT; j++) {
+                    const int tt = row0 + j;
+                    if (col + b < dim && tt < nt && (LN <= WR_TILE || (l & 1) == 0))
+                        out[(size_t)(t0 + tt) * n + (size_t)h * dim + col + b] = fmaf(sb[tt], sv[tt * COLS + col_l + b], part[b][j]);
+                }
+            }
         }
         __syncthreads();                       // the buffer is refilled by the load of tile q + 2
     }
-    if (live) {
+    if (PASS == 2 && z != segments - 1) return;
+    float* to = PASS == 1 ? seg + (size_t)z * all : state;
 #pragma unroll
-        for (int c = 0; c < CH; c++) {
-            if (on[c]) {
+    for (int c = 0; c < CH; c++) {
+        if (!on[c]) continue;
 #pragma unroll
-                for (int j = 0; j < W; j++) st[d0[c] + j] = S[c][j];
-            }
+        for (int b = 0; b < CB; b++) {
+            if (col + b >= dim) continue;
+#pragma unroll
+            for (int j = 0; j < W; j++) to[st_off(b) + d0[c] + j] = S[b][c][j];
+        }
+        if (PASS == 1 && col == 0) {
+#pragma unroll
+            for (int j = 0; j < W; j++) decay[((size_t)z * heads + h) * dim + d0[c] + j] = prod[c][j];
         }
     }
 }
@@ -460,15 +522,33 @@ __global__ void __launch_bounds__(256) wkv_token_kernel(float* __restrict__ out,
     for (int d = threadIdx.x; d < dim; d += 256) out[hb + d] = os[d] * inv * norm[hb + d] * silu_f(gate[hb + d]);
 }
 
-template <int LN, int CH, int W>
+constexpr int WR_MAX_SEGMENTS = 8;
+template <int LN, int CH, int W, int CB>
 void launch_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int T, int heads, int dim, const int* pos_dev,
-                 int p0, cudaStream_t s) {
-    constexpr int COLS = 128 / LN;
+                 int p0, float* scratch, cudaStream_t s) {
+    constexpr int COLS = 128 / LN * CB;
     const size_t tile = ((size_t)3 * WR_TILE * dim + (size_t)WR_TILE * COLS + WR_TILE + 3) & ~(size_t)3;
     const size_t smem = sizeof(float) * 2 * tile;
-    static unsigned long long done = 0;
-    if (smem > 48 * 1024) opt_in_dynamic_smem(wkv_rows_kernel<LN, CH, W>, 200 * 1024, done);
-    launch_k(wkv_rows_kernel<LN, CH, W>, dim3((dim + COLS - 1) / COLS, heads), dim3(128), smem, s, out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0);
+    const int cols = (dim + COLS - 1) / COLS;
+    // segments where the columns leave half of the SMs without a CTA: until about six CTAs stand on every SM, none shorter than eight tiles.  The
+    // state pass costs about half of a full one, so a grid that fills the SMs on its own, or two segments, gain nothing.
+    int segments = 1;
+    if (scratch && 2 * cols * heads <= 148) segments = std::max(1, std::min({WR_MAX_SEGMENTS, (6 * 148 + cols * heads - 1) / (cols * heads), T / (8 * WR_TILE)}));
+    if (segments < 3) segments = 1;
+    const int seg_len = ((T + segments - 1) / segments + WR_TILE - 1) / WR_TILE * WR_TILE;
+    segments = (T + seg_len - 1) / seg_len;
+    static unsigned long long done0 = 0, done1 = 0, done2 = 0;
+    if (segments == 1) {
+        if (smem > 48 * 1024) opt_in_dynamic_smem(wkv_rows_kernel<LN, CH, W, CB, 0>, 200 * 1024, done0);
+        launch_k(wkv_rows_kernel<LN, CH, W, CB, 0>, dim3(cols, heads), dim3(128), smem, s, out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0, (float*)nullptr, (float*)nullptr, T, 1);
+        count_launch();
+        return;
+    }
+    float* decay = scratch + (size_t)WR_MAX_SEGMENTS * heads * dim * dim;
+    if (smem > 48 * 1024) { opt_in_dynamic_smem(wkv_rows_kernel<LN, CH, W, CB, 1>, 200 * 1024, done1); opt_in_dynamic_smem(wkv_rows_kernel<LN, CH, W, CB, 2>, 200 * 1024, done2); }
+    launch_k(wkv_rows_kernel<LN, CH, W, CB, 1>, dim3(cols, heads, segments - 1), dim3(128), smem, s, out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0, scratch, decay, seg_len, segments);
+    launch_k(wkv_rows_kernel<LN, CH, W, CB, 2>, dim3(cols, heads, segments), dim3(128), smem, s, out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0, scratch, decay, seg_len, segments);
+    count_launch(2);
 }
 
 }  // namespace
@@ -508,26 +588,27 @@ void wkv_prep(float* a, float* ruk, const float* r, const float* k, const float*
     count_launch();
 }
 
+size_t wkv_rows_scratch_floats(int heads, int dim) { return (size_t)WR_MAX_SEGMENTS * heads * dim * ((size_t)dim + 1); }
+
 void wkv_rows(float* out, const float* r, const float* k, const float* v, const float* w, const float* ruk, float* state, int T, int heads, int dim, const int* pos_dev, int p0,
-              cudaStream_t s) {
+              cudaStream_t s, float* scratch) {
     NT_CHECK(dim >= 1 && dim <= WKV_MAX_DIM, "wkv_rows: heads wider than 256 are not covered");
     if (T <= 0) return;
     const bool vec = dim % 4 == 0 && ((reinterpret_cast<uintptr_t>(r) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(w)) & 15) == 0;
-#define NT_WR(LN, CH, W) launch_rows<LN, CH, W>(out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0, s)
+#define NT_WR(LN, CH, W, CB) launch_rows<LN, CH, W, CB>(out, r, k, v, w, ruk, state, T, heads, dim, pos_dev, p0, scratch, s)
     if (vec) {
-        if (dim <= 16) NT_WR(4, 1, 4);
-        else if (dim <= 32) NT_WR(8, 1, 4);
-        else if (dim <= 64) NT_WR(16, 1, 4);
-        else if (dim <= 128) NT_WR(16, 2, 4);
-        else NT_WR(32, 2, 4);
+        if (dim <= 16) NT_WR(4, 1, 4, 1);
+        else if (dim <= 32) NT_WR(8, 1, 4, 2);
+        else if (dim <= 64) NT_WR(16, 1, 4, 4);
+        else if (dim <= 128) NT_WR(16, 2, 4, 2);
+        else NT_WR(32, 2, 4, 2);
     } else {
-        if (dim <= 8) NT_WR(8, 1, 1);
-        else if (dim <= 32) NT_WR(16, 2, 1);
-        else if (dim <= 128) NT_WR(16, 8, 1);
-        else NT_WR(16, 16, 1);
+        if (dim <= 8) NT_WR(8, 1, 1, 1);
+        else if (dim <= 32) NT_WR(16, 2, 1, 1);
+        else if (dim <= 128) NT_WR(16, 8, 1, 1);
+        else NT_WR(16, 16, 1, 1);
     }
 #undef NT_WR
-    count_launch();
 }
 
 void wkv_out_norm(float* out, void* split, const float* o, const float* gate, const float* norm, float eps, int T, int heads, int dim, cudaStream_t s) {

@@ -153,15 +153,17 @@ def wkv_inputs(rng, T, H, D, rank=None):
     return r, k, v, raw, w0, u
 
 
-def run_wkv_rows(r, k, v, raw, w0, u, sizes, rng):
+def run_wkv_rows(r, k, v, raw, w0, u, sizes, rng, segments=False):
     T, H, D = r.shape
+    scratch = torch.full((lib().nt_b200_wkv_scratch_floats(H, D),), float("nan"), device="cuda") if segments else None
     state = dev(rng.standard_normal((H, D, D)))                               # stale: a step at position 0 starts from zeros
     got, pos = [], 0
     for n in sizes:
         sl = slice(pos, pos + n)
         dr, dk, a, ruk, out = dev(r[sl]), dev(k[sl]), dev(raw[sl]), torch.empty(n, H, device="cuda"), torch.empty(n, H, D, device="cuda")
         lib().nt_b200_wkv_prep(a.data_ptr(), ruk.data_ptr(), dr.data_ptr(), dk.data_ptr(), dp(w0), dp(u), n, H, D, stream())
-        lib().nt_b200_wkv_rows(out.data_ptr(), dr.data_ptr(), dk.data_ptr(), dp(v[sl]), a.data_ptr(), ruk.data_ptr(), state.data_ptr(), n, H, D, pos, stream())
+        lib().nt_b200_wkv_rows(out.data_ptr(), dr.data_ptr(), dk.data_ptr(), dp(v[sl]), a.data_ptr(), ruk.data_ptr(), state.data_ptr(), n, H, D, pos,
+                               scratch.data_ptr() if segments else None, stream())
         got.append(host(out)); pos += n
     return np.concatenate(got)
 
@@ -174,6 +176,18 @@ def test_wkv_recurrence_and_state_hand_over(H, D):
     ref = O.wkv_recurrence(r, k, v, np.exp(-np.exp(raw + w0)), u)
     for sizes in ([T], [1] * T, [2, 16, 1, 15, 3]):
         np.testing.assert_allclose(run_wkv_rows(r, k, v, raw, w0, u, sizes, rng), ref, rtol=2e-4, atol=2e-5 * np.abs(ref).max())
+
+
+@pytest.mark.parametrize("H,D", [(2, 5), (1, 16), (3, 64), (2, 33), (1, 128), (1, 256), (2, 20)])
+def test_wkv_segments_side_by_side(H, D):
+    """Long steps run as segments whose states are joined; steps that start later, that end inside a tile or a segment, and short ones between."""
+    rng = np.random.default_rng(D)
+    T = 1100
+    r, k, v, raw, w0, u = wkv_inputs(rng, T, H, D)
+    w0 -= 3.0                                                                 # slow decays: states cross many segments
+    ref = O.wkv_recurrence(r, k, v, np.exp(-np.exp(raw + w0)), u)
+    for sizes in ([T], [5, 1000, 95], [517, 583], [1024, 1, 75]):
+        np.testing.assert_allclose(run_wkv_rows(r, k, v, raw, w0, u, sizes, rng, segments=True), ref, rtol=5e-4, atol=1e-4 * np.abs(ref).max())
 
 
 def test_wkv_keeps_a_far_write_under_slow_decay_and_loses_it_under_fast():
