@@ -7,7 +7,7 @@
 // One decoded token, 4 launches for a WKV layer with a dense feed-forward:
 //   [depth average + grouped norm + the five shift blends]  [r, k, v, gate, tanh(W_w1 .) and xielu(W_up .): one launch, an input per matrix]
 //   [decay, recurrence, head norm, gate]  [slot += W_o o + W_down a]
-// and 8 for a latent-attention layer with routed experts:
+// and 9 for a latent-attention layer with routed experts:
 //   [depth average + grouped norm]  [q, key / value latent, router logits]  [latent norm, rotation, cache write]  [absorbed queries]
 //   [attention over the window's rows] [merge]  [values]  [choice + experts and shared expert up]  [slot += W_o o + experts + shared expert].
 // Prompt rows take the tensor-core GEMMs (residual added in the epilogue), the tiled window attention over expanded rows and the tiled
