@@ -12,6 +12,7 @@
 #include <cuda_bf16.h>
 #include <algorithm>
 #include <cmath>
+#include <vector>
 
 namespace nt { namespace b200 {
 
@@ -165,22 +166,28 @@ __global__ void scale_rows_kernel(float* __restrict__ x, float scale, size_t n) 
 
 }  // namespace
 
-float rotary_table(float* freq, int dims, float base, float factor, float original, float fast, float slow) {
+float rotary_table(double* freq, int dims, double base, double factor, double original, double fast, double slow) {
     const int half = dims / 2;
-    const double lnb = std::log((double)base), two_pi = 6.283185307179586476925;
+    const double lnb = std::log(base), two_pi = 6.283185307179586476925;
     // the (fractional) pair index whose wavelength fits `t` times into `original` positions
-    auto turn = [&](double t) { return dims * std::log((double)original / (two_pi * t)) / (2.0 * lnb); };
+    auto turn = [&](double t) { return dims * std::log(original / (two_pi * t)) / (2.0 * lnb); };
     double lo = 0.0, hi = 0.0;
-    if (factor > 0.f) { lo = std::max(std::floor(turn(fast)), 0.0); hi = std::min(std::ceil(turn(slow)), (double)(dims - 1)); }
+    if (factor > 0.0) { lo = std::max(std::floor(turn(fast)), 0.0); hi = std::min(std::ceil(turn(slow)), (double)(dims - 1)); }
     for (int i = 0; i < half; i++) {
         double f = std::exp(-2.0 * i / dims * lnb);
-        if (factor > 0.f) {
+        if (factor > 0.0) {
             const double ramp = std::min(1.0, std::max(0.0, (i - lo) / std::max(hi - lo, 0.001)));
             f = f / factor * ramp + f * (1.0 - ramp);
         }
-        freq[i] = (float)f;
+        freq[i] = f;
     }
-    return factor > 0.f ? (float)(0.1 * std::log((double)factor) + 1.0) : 1.f;
+    return factor > 0.0 ? (float)(0.1 * std::log(factor) + 1.0) : 1.f;
+}
+float rotary_table(float* freq, int dims, float base, float factor, float original, float fast, float slow) {
+    std::vector<double> f((size_t)std::max(1, dims / 2));
+    const float mag = rotary_table(f.data(), dims, (double)base, (double)factor, (double)original, (double)fast, (double)slow);
+    for (int i = 0; i < dims / 2; i++) freq[i] = (float)f[(size_t)i];
+    return mag;
 }
 
 void rope_partial_kv_write(float* Q, const float* K, const float* V, const float* freq, float mag, int dims, bool interleaved, int dim,

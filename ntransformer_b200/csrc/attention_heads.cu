@@ -1,10 +1,11 @@
 // attention_heads.cu — what sits between the projections (and their short convolutions) and attention_window for attention with
 // per-head query / key norm, and the mixing of softmax weights across heads behind it:
 //   head_prep   per token: every dim-wide head of the query and key rows is RMS-normed on its own (x / sqrt(mean x^2 + eps) * gain, one
-//               gain vector of the head's width shared by all heads; null: no norm); the first `dims` channels of every head are rotated
+//               gain vector of the head's width shared by all heads; null: no norm; unit_norm: no gain); the first `dims` channels of every head are rotated
 //               (channel i with i + dims/2 — or 2i with 2i+1 when interleaved — by angle = position * freq[i], F32, the table made on the
 //               host with any frequency scaling folded in); query head h is then multiplied by temp[h] (a per-head score multiplier,
-//               null: none); queries in place, keys into cache row base + t.  Values: v <- (1 - lambda) v + lambda v_first[t] when a
+//               null: none) and by 1 + temp_coef ln(floor((position + 1) / temp_every) + 1) where that is on; queries in place, keys (K null: the
+//               layer reads another layer's rows) into cache row base + t.  Values: v <- (1 - lambda) v + lambda v_first[t] when a
 //               blend is given (v_first: the values another layer computed for the same tokens, F32, [T, vdim]); the values as the layer
 //               computed them are published to v_publish when given; then into the cache row.
 //   talk_mix    out[t, h, :] = sum_g M[h, g] A[t, g, kv(h), :] where A[t, g, c, :] = sum_j w_g(t, j) v_c(j) is what attention_window
@@ -25,15 +26,15 @@ __device__ __forceinline__ void cst(float* p, size_t i, float v) { p[i] = v; }
 __device__ __forceinline__ void cst(__nv_bfloat16* p, size_t i, float v) { p[i] = __float2bfloat16_rn(v); }
 
 // One head in shared memory: norm, rotate; `row` [dim] is overwritten with the result.  Called by one warp.
-__device__ __forceinline__ void norm_rotate_head(float* row, int dim, const float* __restrict__ gain, float eps, int dims, bool interleaved,
+__device__ __forceinline__ void norm_rotate_head(float* row, int dim, const float* __restrict__ gain, bool unit, float eps, int dims, bool interleaved,
                                                  const float* cs, const float* sn, int lane) {
-    if (gain) {
+    if (gain || unit) {
         float ss = 0.f;
         for (int i = lane; i < dim; i += 32) ss = fmaf(row[i], row[i], ss);
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o);
         const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
-        for (int i = lane; i < dim; i += 32) row[i] = row[i] * inv * gain[i];
+        for (int i = lane; i < dim; i += 32) row[i] = gain ? row[i] * inv * gain[i] : row[i] * inv;
         __syncwarp();
     }
     const int half = dims >> 1;
@@ -63,16 +64,18 @@ __global__ void __launch_bounds__(256) head_prep_kernel(float* __restrict__ Q, c
     for (int i = threadIdx.x; i < half; i += 256) sincosf((float)pos * p.freq[i], &sn[i], &cs[i]);
     __syncthreads();
     float* row = rows + (size_t)warp * p.dim;
-    const int n_heads = p.heads + p.kv_heads;
+    const int n_heads = p.heads + (K ? p.kv_heads : 0);
+    float pos_temp = 1.f;
+    if (p.temp_every > 0.0) pos_temp = 1.0f + p.temp_coef * logf((float)floor((double)(pos + 1) / p.temp_every) + 1.0f);
     for (int hh = blockIdx.y * 8 + warp; hh < n_heads; hh += 8 * gridDim.y) {
         const bool is_q = hh < p.heads;
         const int h = is_q ? hh : hh - p.heads;
         const float* src = is_q ? Q + ((size_t)t * p.heads + h) * p.dim : K + ((size_t)t * p.kv_heads + h) * p.dim;
         for (int i = lane; i < p.dim; i += 32) row[i] = src[i];
         __syncwarp();
-        norm_rotate_head(row, p.dim, is_q ? p.q_gain : p.k_gain, p.eps, p.rot_dims, p.interleaved != 0, cs, sn, lane);
+        norm_rotate_head(row, p.dim, is_q ? p.q_gain : p.k_gain, p.unit_norm != 0, p.eps, p.rot_dims, p.interleaved != 0, cs, sn, lane);
         if (is_q) {
-            const float m = p.temp ? p.temp[h] : 1.f;
+            const float m = (p.temp ? p.temp[h] : 1.f) * pos_temp;
             float* dst = Q + ((size_t)t * p.heads + h) * p.dim;
             for (int i = lane; i < p.dim; i += 32) dst[i] = row[i] * m;
         } else {
@@ -81,6 +84,7 @@ __global__ void __launch_bounds__(256) head_prep_kernel(float* __restrict__ Q, c
         }
         __syncwarp();
     }
+    if (!K) return;
     const int vw = p.kv_heads * p.vdim;
     const float lam = p.v_lambda ? *p.v_lambda : 0.f;
     for (int i = blockIdx.y * 256 + threadIdx.x; i < vw; i += 256 * gridDim.y) {

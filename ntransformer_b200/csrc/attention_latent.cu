@@ -14,7 +14,7 @@
 // [row, head, width] operands) and runs the tiled tensor-core attention kernel over them (attention_heads_mma): heads * (dim + rot_dim +
 // vdim) multiply-adds per (query, key) instead of heads * (2 kv_rank + rot_dim).  latent_q_rot_pad rotates and pads the queries.
 // Rotation: channel i of the rotated part pairs with channel i + dims/2 (or 2i with 2i+1), angle pos * base^(-2i/dims), computed
-// in double and applied in F32; channels past `dims` pass unchanged.  Norms, angles and sums are F32 or better.
+// in double (or position * a table entry: LatentRot::freq) and applied in F32 times LatentRot::mag; channels past `dims` pass unchanged.  Norms, angles and sums are F32 or better.
 // Compiled WITHOUT --use_fast_math.
 #include "kernels_internal.h"
 #include "ring.cuh"
@@ -36,18 +36,31 @@ __device__ __forceinline__ float wld(const __nv_bfloat16* p, size_t i) { return 
 __device__ __forceinline__ void cst(float* p, size_t i, float v) { p[i] = v; }
 __device__ __forceinline__ void cst(__nv_bfloat16* p, size_t i, float v) { p[i] = __float2bfloat16_rn(v); }
 
+// LatentRot as the kernels see it
+struct RotDev {
+    int dims, interleaved;
+    double log2_base;
+    const double* freq;
+    float mag;
+    __device__ __forceinline__ void cos_sin(int pair, int pos, float& c, float& s) const {
+        double sn, cs;
+        sincos((double)pos * (freq ? freq[pair] : exp2(-2.0 * (double)pair / (double)dims * log2_base)), &sn, &cs);
+        c = (float)cs * mag; s = (float)sn * mag;
+    }
+};
+RotDev dev_of(const LatentRot& r) { return RotDev{r.dims, r.interleaved ? 1 : 0, std::log2(r.base), r.freq, r.mag}; }
+
 // out[i] for channel i of a rot_dim-wide vector `src` at position pos
-__device__ __forceinline__ float rotated(const float* src, int i, int dims, int interleaved, double log2_base, int pos) {
+__device__ __forceinline__ float rotated(const float* src, int i, const RotDev& rot, int pos) {
+    const int dims = rot.dims, interleaved = rot.interleaved;
     if (i >= dims) return src[i];
     const int half = dims >> 1;
     int pair, mate;
     bool first;
     if (interleaved) { pair = i >> 1; first = (i & 1) == 0; mate = first ? i + 1 : i - 1; }
     else { first = i < half; pair = first ? i : i - half; mate = first ? i + half : i - half; }
-    const double ang = (double)pos * exp2(-2.0 * (double)pair / (double)dims * log2_base);
-    double sn, cs;
-    sincos(ang, &sn, &cs);
-    const float c = (float)cs, sv = (float)sn;
+    float c, sv;
+    rot.cos_sin(pair, pos, c, sv);
     // (u, v) -> (u cos - v sin, v cos + u sin)
     return first ? src[i] * c - src[mate] * sv : src[i] * c + src[mate] * sv;
 }
@@ -68,7 +81,7 @@ __device__ __forceinline__ float block_sum_256(float v, float* red) {
 template <typename KT>
 __global__ void __launch_bounds__(256) latent_prep_kernel(float* __restrict__ cq, int q_rank, const float* __restrict__ q_gain, const float* __restrict__ dkv,
                                                           int kv_rank, int rot_dim, const float* __restrict__ kv_gain, float eps, KT* __restrict__ cache,
-                                                          int dims, int interleaved, double log2_base, const int* __restrict__ pos_dev, int p0) {
+                                                          const RotDev rot, const int* __restrict__ pos_dev, int p0) {
     __shared__ float red[8];
     pdl_launch_dependents();
     pdl_wait();
@@ -89,7 +102,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(float* __restrict__ cq
     for (int i = threadIdx.x; i < kv_rank; i += 256) ss = fmaf(r[i], r[i], ss);
     const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)kv_rank + eps);
     for (int i = threadIdx.x; i < kv_rank; i += 256) cst(cache, (size_t)pos * row + i, r[i] * inv * kv_gain[i]);
-    for (int i = threadIdx.x; i < rot_dim; i += 256) cst(cache, (size_t)pos * row + kv_rank + i, rotated(r + kv_rank, i, dims, interleaved, log2_base, pos));
+    for (int i = threadIdx.x; i < rot_dim; i += 256) cst(cache, (size_t)pos * row + kv_rank + i, rotated(r + kv_rank, i, rot, pos));
 }
 
 constexpr int LT = 8;      // tokens per CTA in the two per-head products
@@ -99,7 +112,7 @@ constexpr int LT = 8;      // tokens per CTA in the two per-head products
 // shared memory.  One decoded token then has heads * kv_rank / 64 CTAs with short chains instead of `heads` CTAs with long ones.
 template <typename WT>
 __global__ void __launch_bounds__(256) latent_q_absorb_kernel(float* __restrict__ qa, const float* __restrict__ q, const WT* __restrict__ W_uk, int T, int heads,
-                                                              int dim, int rot_dim, int kv_rank, int dims, int interleaved, double log2_base,
+                                                              int dim, int rot_dim, int kv_rank, const RotDev rot,
                                                               const int* __restrict__ pos_dev, int p0) {
     extern __shared__ __align__(16) float qs[];           // [LT][dim + rot_dim] | partial sums [4][64][LT]
     if (T == 1) for (int d = threadIdx.x; d < dim; d += 256) l2_prefetch(W_uk + ((size_t)blockIdx.y * dim + d) * kv_rank + blockIdx.z * 64, min(64, kv_rank - (int)blockIdx.z * 64) * sizeof(WT), 0, 1);
@@ -138,7 +151,7 @@ __global__ void __launch_bounds__(256) latent_q_absorb_kernel(float* __restrict_
     const int base = pos_dev ? *pos_dev : p0;
     for (int e = threadIdx.x; e < nt * rot_dim; e += 256) {
         const int tt = e / rot_dim, i = e % rot_dim;
-        qa[((size_t)(t0 + tt) * heads + h) * od + kv_rank + i] = rotated(qs + tt * qd + dim, i, dims, interleaved, log2_base, base + t0 + tt);
+        qa[((size_t)(t0 + tt) * heads + h) * od + kv_rank + i] = rotated(qs + tt * qd + dim, i, rot, base + t0 + tt);
     }
 }
 
@@ -146,7 +159,7 @@ __global__ void __launch_bounds__(256) latent_q_absorb_kernel(float* __restrict_
 // channel, 32 channels per CTA.
 template <typename WT>
 __global__ void __launch_bounds__(256) latent_v_up_kernel(float* __restrict__ out, const float* __restrict__ ol, const WT* __restrict__ W_uv, int T, int heads,
-                                                          int vdim, int kv_rank) {
+                                                          int vdim, int kv_rank, const float* __restrict__ gate) {
     extern __shared__ __align__(16) float os[];           // [LT][kv_rank]
     if (T == 1) l2_prefetch(W_uv + ((size_t)blockIdx.y * vdim + blockIdx.z * 32) * kv_rank, (size_t)min(32, vdim - (int)blockIdx.z * 32) * kv_rank * sizeof(WT), threadIdx.x, 256);
     pdl_launch_dependents();
@@ -174,7 +187,10 @@ __global__ void __launch_bounds__(256) latent_v_up_kernel(float* __restrict__ ou
             for (int o = 16; o > 0; o >>= 1) acc[tt] += __shfl_xor_sync(0xFFFFFFFFu, acc[tt], o);
         }
         if (lane == 0)
-            for (int tt = 0; tt < nt; tt++) out[(size_t)(t0 + tt) * heads * vdim + (size_t)h * vdim + v] = acc[tt];
+            for (int tt = 0; tt < nt; tt++) {
+                const size_t at = (size_t)(t0 + tt) * heads * vdim + (size_t)h * vdim + v;
+                out[at] = gate ? acc[tt] / (1.0f + expf(-gate[at])) : acc[tt];
+            }
     }
 }
 
@@ -221,17 +237,14 @@ __global__ void __launch_bounds__(256) latent_expand_pack_kernel(__nv_bfloat16* 
 }
 
 // qp [t, h, kw] = [q[t, h, :dim] | rot(q[t, h, dim:]) | 0 ...].  A CTA per token: the position's cosines and sines are computed once for all heads.
-__global__ void __launch_bounds__(256) latent_q_rot_pad_kernel(float* __restrict__ qp, const float* __restrict__ q, int heads, int dim, int rot_dim, int kw, int dims,
-                                                               int interleaved, double log2_base, int p0) {
+__global__ void __launch_bounds__(256) latent_q_rot_pad_kernel(float* __restrict__ qp, const float* __restrict__ q, int heads, int dim, int rot_dim, int kw, const RotDev rot,
+                                                               int p0) {
     extern __shared__ __align__(16) float cs[];           // cos, sin of dims / 2 pairs
     pdl_launch_dependents();
     pdl_wait();
+    const int dims = rot.dims, interleaved = rot.interleaved;
     const int t = blockIdx.x, qd = dim + rot_dim, half = dims >> 1;
-    for (int i = threadIdx.x; i < half; i += 256) {
-        double sn, co;
-        sincos((double)(p0 + t) * exp2(-2.0 * (double)i / (double)dims * log2_base), &sn, &co);
-        cs[2 * i] = (float)co; cs[2 * i + 1] = (float)sn;
-    }
+    for (int i = threadIdx.x; i < half; i += 256) rot.cos_sin(i, p0 + t, cs[2 * i], cs[2 * i + 1]);
     __syncthreads();
     const float* src = q + (size_t)t * heads * qd;
     float* dst = qp + (size_t)t * heads * kw;
@@ -430,40 +443,40 @@ __global__ void __launch_bounds__(256) latent_shared_merge_kernel(float* __restr
 }  // namespace
 
 void latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache,
-                 DType cache_dt, int rot_dims, bool interleaved, double rot_base, int T, const int* pos_dev, int p0, cudaStream_t s) {
+                 DType cache_dt, const LatentRot& rot, int T, const int* pos_dev, int p0, cudaStream_t s) {
     if (T <= 0) return;
     NT_CHECK(cache_dt == DType::F32 || cache_dt == DType::BF16, "latent_prep: F32 or BF16 cache");
-    const double l2b = std::log2(rot_base);
+    const RotDev rd = dev_of(rot);
     if (cache_dt == DType::F32)
         launch_k(latent_prep_kernel<float>, dim3(T, cq ? 2 : 1), dim3(256), 0, s, cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps, static_cast<float*>(cache),
-                 rot_dims, interleaved ? 1 : 0, l2b, pos_dev, p0);
+                 rd, pos_dev, p0);
     else
         launch_k(latent_prep_kernel<__nv_bfloat16>, dim3(T, cq ? 2 : 1), dim3(256), 0, s, cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps,
-                 static_cast<__nv_bfloat16*>(cache), rot_dims, interleaved ? 1 : 0, l2b, pos_dev, p0);
+                 static_cast<__nv_bfloat16*>(cache), rd, pos_dev, p0);
     count_launch();
 }
 
-void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, int rot_dims,
-                     bool interleaved, double rot_base, const int* pos_dev, int p0, cudaStream_t s) {
+void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, const LatentRot& rot,
+                     const int* pos_dev, int p0, cudaStream_t s) {
     if (T <= 0) return;
     const size_t smem = sizeof(float) * (LT * (size_t)(dim + rot_dim) + 4 * 64 * LT);
     NT_CHECK(smem <= 48 * 1024, "latent_q_absorb: query heads wider than 1280 are not covered");
-    const double l2b = std::log2(rot_base);
+    const RotDev rd = dev_of(rot);
     const dim3 grid((T + LT - 1) / LT, heads, (kv_rank + 63) / 64);
-#define NT_QA(TY) launch_k(latent_q_absorb_kernel<TY>, grid, dim3(256), smem, s, qa, q, static_cast<const TY*>(W_uk), T, heads, dim, rot_dim, kv_rank, rot_dims, \
-                           interleaved ? 1 : 0, l2b, pos_dev, p0)
+#define NT_QA(TY) launch_k(latent_q_absorb_kernel<TY>, grid, dim3(256), smem, s, qa, q, static_cast<const TY*>(W_uk), T, heads, dim, rot_dim, kv_rank, rd, \
+                           pos_dev, p0)
     if (dt == DType::F32) NT_QA(float); else if (dt == DType::F16) NT_QA(__half); else if (dt == DType::BF16) NT_QA(__nv_bfloat16);
     else NT_CHECK(false, "latent_q_absorb: dense dtypes only");
 #undef NT_QA
     count_launch();
 }
 
-void latent_v_up(float* out, const float* ol, const void* W_uv, DType dt, int T, int heads, int vdim, int kv_rank, cudaStream_t s) {
+void latent_v_up(float* out, const float* ol, const void* W_uv, DType dt, int T, int heads, int vdim, int kv_rank, cudaStream_t s, const float* gate) {
     if (T <= 0) return;
     const size_t smem = sizeof(float) * LT * (size_t)kv_rank;
     NT_CHECK(smem <= 48 * 1024, "latent_v_up: latents wider than 1536 are not covered");
     const dim3 grid((T + LT - 1) / LT, heads, (vdim + 31) / 32);
-#define NT_VU(TY) launch_k(latent_v_up_kernel<TY>, grid, dim3(256), smem, s, out, ol, static_cast<const TY*>(W_uv), T, heads, vdim, kv_rank)
+#define NT_VU(TY) launch_k(latent_v_up_kernel<TY>, grid, dim3(256), smem, s, out, ol, static_cast<const TY*>(W_uv), T, heads, vdim, kv_rank, gate)
     if (dt == DType::F32) NT_VU(float); else if (dt == DType::F16) NT_VU(__half); else if (dt == DType::BF16) NT_VU(__nv_bfloat16);
     else NT_CHECK(false, "latent_v_up: dense dtypes only");
 #undef NT_VU
@@ -488,10 +501,10 @@ void latent_expand_pack(void* kfull, void* vfull, const float* ku, const float* 
     count_launch();
 }
 
-void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, int rot_dims, bool interleaved, double rot_base, int p0,
+void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, const LatentRot& rot, int p0,
                       cudaStream_t s) {
     if (T <= 0) return;
-    launch_k(latent_q_rot_pad_kernel, dim3(T), dim3(256), sizeof(float) * (size_t)std::max(2, rot_dims), s, qp, q, heads, dim, rot_dim, kw, rot_dims, interleaved ? 1 : 0, std::log2(rot_base), p0);
+    launch_k(latent_q_rot_pad_kernel, dim3(T), dim3(256), sizeof(float) * (size_t)std::max(2, rot.dims), s, qp, q, heads, dim, rot_dim, kw, dev_of(rot), p0);
     count_launch();
 }
 

@@ -61,7 +61,7 @@ __global__ void __launch_bounds__(128, 2) prefill_mma_kernel(float* __restrict__
                                                              const __half* __restrict__ kc, const __half* __restrict__ vc,
                                                              int seq_len, int start_pos, int n_heads, int n_kv, int max_seq,
                                                              float scale, int window, int keep, float softcap, int maps, int chunk,
-                                                             const float* __restrict__ sink, int joint_v) {
+                                                             const float* __restrict__ sink, int joint_v, const float* __restrict__ slopes) {
     constexpr int LD = HD + PAD, LDV = HDV + PAD, KS = HD / 16, NT = HDV / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __half* sK = reinterpret_cast<__half*>(smem_raw);                 // [2][BKV][LD]
@@ -70,6 +70,7 @@ __global__ void __launch_bounds__(128, 2) prefill_mma_kernel(float* __restrict__
     const int head = blockIdx.y, vh = (head / maps) / ((n_heads / maps) / n_kv), kvh = vh * maps + head % maps, n_k = n_kv * maps;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int r0 = qb * BQ + warp * 16 + g, r1 = r0 + 8;              // this thread's two query rows (chunk-relative)
+    const float slope = slopes ? slopes[head / maps] : 0.f;           // slope * (p - key) is taken off the score
     const int p0 = start_pos + r0, p1 = start_pos + r1;               // their absolute positions == last visible key
 
     // ---- Q fragments (A operand, 16 x HD per warp), split into F16 hi + lo ----
@@ -151,6 +152,7 @@ __global__ void __launch_bounds__(128, 2) prefill_mma_kernel(float* __restrict__
                 const bool seen = key <= p && (chunk > 0 ? key >= p / chunk * chunk : (window <= 0 || p - key < window || key < keep));
                 float v = s[n][i] * scale;
                 if (softcap > 0.f) v = softcap * (1.0f - 2.0f / (__expf(2.0f * v / softcap) + 1.0f));     // cap * tanh(v / cap)
+                v -= slope * (float)(p - key);
                 v = seen ? v : -INFINITY;
                 s[n][i] = v;
                 if (i & 2) mx1 = fmaxf(mx1, v); else mx0 = fmaxf(mx0, v);
@@ -220,12 +222,12 @@ __global__ void __launch_bounds__(128, 2) prefill_mma_kernel(float* __restrict__
 template <int HD, int HDV, bool BF>
 void launch(float* out, const float* Q, const __half* kc, const __half* vc, int seq_len, int start_pos, int n_heads, int n_kv,
             int max_seq, float scale, int window, int keep, float softcap, cudaStream_t s, int maps = 1, int chunk = 0, const float* sink = nullptr,
-            int joint_v = 0) {
+            int joint_v = 0, const float* slopes = nullptr) {
     const int smem = 2 * BKV * (HD + PAD + HDV + PAD) * (int)sizeof(__half);
     static unsigned long long configured = 0;      // bit per device id
     opt_in_dynamic_smem(prefill_mma_kernel<HD, HDV, BF>, (int)(smem), configured);
     prefill_mma_kernel<HD, HDV, BF><<<dim3((seq_len + BQ - 1) / BQ, n_heads * maps), 128, smem, s>>>(out, Q, kc, vc, seq_len, start_pos, n_heads * maps, n_kv,
-                                                                                                    max_seq, scale, window, keep, softcap, maps, chunk, sink, joint_v);
+                                                                                                    max_seq, scale, window, keep, softcap, maps, chunk, sink, joint_v, slopes);
     NT_LAUNCH_CHECK();
     count_launch();
 }
@@ -244,20 +246,21 @@ void attention_prefill_mma(float* out, const float* Q, const void* kc, const voi
     else launch<64, 64, false>(out, Q, k, v, seq_len, start_pos, n_heads, n_kv, max_seq, scale, 0, 0, 0.f, s);
 }
 
-// Windowed / block-masked / soft-capped form over a BF16 cache: (dim, vdim) in {(64, 64), (128, 128), (32, 64), (64, 128)}, one or
+// Windowed / block-masked / soft-capped / distance-biased form over a BF16 cache: (dim, vdim) in {(64, 64), (96, 96), (128, 128), (32, 64), (64, 128)}, one or
 // two score maps per head, at least 16 queries.
 bool attention_window_mma_supported(int tokens, const WindowAttn& a, DType cache_dt) {
-    const bool shape = (a.dim == a.vdim && (a.dim == 64 || a.dim == 128)) || (a.vdim == 2 * a.dim && (a.dim == 32 || a.dim == 64));
+    const bool shape = (a.dim == a.vdim && (a.dim == 64 || a.dim == 96 || a.dim == 128)) || (a.vdim == 2 * a.dim && (a.dim == 32 || a.dim == 64));
     // joint values: one value row of width vdim per key, packed (the stride equals the width)
     const bool strides = a.k_stride == 0 && (a.joint_v ? (a.v_stride == a.vdim && a.maps == 1) : a.v_stride == 0);
-    return cache_dt == DType::BF16 && shape && strides && a.maps >= 1 && a.maps <= 2 && tokens >= 16 && a.kv_heads > 0 && a.heads % a.kv_heads == 0;
+    return cache_dt == DType::BF16 && shape && strides && !a.head_gate && a.maps >= 1 && a.maps <= 2 && tokens >= 16 && a.kv_heads > 0 && a.heads % a.kv_heads == 0;
 }
 void attention_window_mma(float* out, const float* Q, const void* kc, const void* vc, int tokens, int p0, int max_seq, const WindowAttn& a,
                           cudaStream_t s) {
     const __half* k = static_cast<const __half*>(kc);       // 16-bit words either way; the BF instantiation reads them as BF16
     const __half* v = static_cast<const __half*>(vc);
-#define NT_AW(D, V) launch<D, V, true>(out, Q, k, v, tokens, p0, a.heads, a.kv_heads, max_seq, a.scale, a.window, a.keep, a.softcap, s, a.maps, a.chunk, a.sink, a.joint_v)
+#define NT_AW(D, V) launch<D, V, true>(out, Q, k, v, tokens, p0, a.heads, a.kv_heads, max_seq, a.scale, a.window, a.keep, a.softcap, s, a.maps, a.chunk, a.sink, a.joint_v, a.slope)
     if (a.dim == 128) NT_AW(128, 128);
+    else if (a.dim == 96) NT_AW(96, 96);
     else if (a.dim == 64 && a.vdim == 64) NT_AW(64, 64);
     else if (a.dim == 64) NT_AW(64, 128);
     else NT_AW(32, 64);

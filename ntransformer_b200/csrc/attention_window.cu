@@ -12,6 +12,7 @@
 //   value width go to the tiled tensor-core form in attention_prefill_mma.cu instead.
 // WindowAttn::sink adds exp(sink_h) to head h's denominator (a learned term without key or value); WindowAttn::joint_v makes every query
 // head sum one value row per key that spans all value heads, which attention_heads.cu's talk_mix turns into head-mixed softmax weights.
+// WindowAttn::slope takes slope_h * (i - j) off the scaled (and capped) score; WindowAttn::head_gate multiplies head h's result by sigmoid(gate).
 // Compiled WITHOUT --use_fast_math (tanhf / expf at full precision).
 #include "kernels_internal.h"
 #include "ring.cuh"
@@ -101,6 +102,8 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(float* 
     const size_t vstride = a.v_stride > 0 ? (size_t)a.v_stride : (size_t)a.kv_heads * a.vdim;
     constexpr int PER16 = 16 / (int)sizeof(KT);
     const bool vec = a.dim % PER16 == 0 && kstride % PER16 == 0 && (reinterpret_cast<uintptr_t>(kc) & 15) == 0;      // every key row then starts on 16 bytes
+    const float slope = a.slope ? a.slope[h] : 0.f;
+    const float gate = a.head_gate ? 1.0f / (1.0f + expf(-a.head_gate[(size_t)t * a.gate_stride + h])) : 1.f;
     float m = -FLT_MAX, l = 0.f, acc[AW_MAXV];
 #pragma unroll
     for (int e = 0; e < AW_MAXV; e++) acc[e] = 0.f;
@@ -112,6 +115,7 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(float* 
         if (valid) {
             sc = dot_row(kc + (size_t)j * kstride + (size_t)gk * a.dim, qs, a.dim, vec) * a.scale;
             if (a.softcap > 0.f) sc = a.softcap * tanhf(sc / a.softcap);
+            sc -= slope * (float)(pos - j);
         }
         float gmax = sc;
 #pragma unroll
@@ -154,7 +158,7 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(float* 
         for (int i = threadIdx.x; i < a.vdim; i += AW_WARPS * 32) {
             float v = 0.f;
             for (int w = 0; w < AW_WARPS; w++) v += accs[w * a.vdim + i] * expf(ms[w] - M);
-            o[i] = v * fix / L;
+            o[i] = v * fix / L * gate;
         }
         return;
     }
@@ -177,7 +181,7 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(float* 
     for (int i = threadIdx.x; i < a.vdim; i += AW_WARPS * 32) {
         float v = 0.f;
         for (int r = 0; r < splits; r++) v += part[(size_t)r * (a.vdim + 2) + 2 + i] * expf(part[(size_t)r * (a.vdim + 2)] - MM);
-        o[i] = v / LL;
+        o[i] = v / LL * gate;
     }
 }
 

@@ -281,6 +281,7 @@ __global__ void __launch_bounds__(DV_WARPS * 32) gemv_multi_kernel(const __grid_
         if (lane == 0) {
             if (m.act == GEMV_ACT_TANH) v = tanhf(v);
             else if (m.act == GEMV_ACT_XIELU) v = xielu_f(v, a, b);
+            else if (m.act == GEMV_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
             m.y[r] = v;
         }
     }

@@ -259,12 +259,12 @@ void nt_b200_moe_experts(float* y, const float* h, const int* sel, const float* 
 // ---- kernel entries of the mechanisms added with the Tanolorn family (numerics tests) ----
 void nt_b200_latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache,
                          int cache_dtype, int rot_dims, int interleaved, float rot_base, int tokens, int p0, void* stream) {
-    latent_prep(cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps, cache, (nt::DType)cache_dtype, rot_dims, interleaved != 0, rot_base, tokens, nullptr, p0,
+    latent_prep(cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps, cache, (nt::DType)cache_dtype, LatentRot{rot_dims, interleaved != 0, rot_base}, tokens, nullptr, p0,
                 static_cast<cudaStream_t>(stream));
 }
 void nt_b200_latent_q_absorb(float* qa, const float* q, const void* W_uk, int dtype, int tokens, int heads, int dim, int rot_dim, int kv_rank, int rot_dims,
                              int interleaved, float rot_base, int p0, void* stream) {
-    latent_q_absorb(qa, q, W_uk, (nt::DType)dtype, tokens, heads, dim, rot_dim, kv_rank, rot_dims, interleaved != 0, rot_base, nullptr, p0, static_cast<cudaStream_t>(stream));
+    latent_q_absorb(qa, q, W_uk, (nt::DType)dtype, tokens, heads, dim, rot_dim, kv_rank, LatentRot{rot_dims, interleaved != 0, rot_base}, nullptr, p0, static_cast<cudaStream_t>(stream));
 }
 void nt_b200_latent_v_up(float* out, const float* ol, const void* W_uv, int dtype, int tokens, int heads, int vdim, int kv_rank, void* stream) {
     latent_v_up(out, ol, W_uv, (nt::DType)dtype, tokens, heads, vdim, kv_rank, static_cast<cudaStream_t>(stream));
@@ -287,7 +287,7 @@ int nt_b200_latent_attention_expanded(float* out, const float* q, const void* ca
     gemm_dense(ku, c32, W_uk, (nt::DType)dtype, 0, (int)P, heads * dim, kv_rank, DENSE_STORE, nullptr, 1.f, s);
     gemm_dense(vu, c32, W_uv, (nt::DType)dtype, 0, (int)P, heads * vdim, kv_rank, DENSE_STORE, nullptr, 1.f, s);
     latent_expand_pack(kf, vf, ku, vu, cache, nt::DType::BF16, kv_rank, 0, (int)P, heads, dim, rot_dim, vdim, kw, vw, s);
-    latent_q_rot_pad(qp, q, tokens, heads, dim, rot_dim, kw, rot_dims, interleaved != 0, rot_base, p0, s);
+    latent_q_rot_pad(qp, q, tokens, heads, dim, rot_dim, kw, LatentRot{rot_dims, interleaved != 0, rot_base}, p0, s);
     attention_heads_mma(op, qp, kf, vf, tokens, p0, (int)P, heads, kw, vw, scale, s);
     latent_unpad(out, op, tokens, heads, vdim, vw, s);
     NT_CUDA_CHECK(cudaStreamSynchronize(s));

@@ -17,11 +17,14 @@ enum class MixerKind { ATTN_ROPE_CAUSAL = 0,     // rotary positions, full causa
                                                  // corrected towards the new value along the new key and read with the query; no cache rows
                        BRANCHES = 5,           // several mixers side by side reading the same input; their outputs are summed with fixed weights
                                                  // (LayerSpec::branches / branch_scale); each branch keeps its own cache rows or state
-                       WKV = 6 };                // token-shifted linear recurrence with a data-dependent decay per key channel (WkvSpec): a matrix state
+                       WKV = 6,                  // token-shifted linear recurrence with a data-dependent decay per key channel (WkvSpec): a matrix state
                                                  // per head; no cache rows
+                       MLSTM = 7 };              // matrix memory with exponential input gate, normalizer and stabilizer (MlstmSpec); no cache rows
 enum class QKNorm { NONE = 0, WHOLE = 1,         // WHOLE: one RMS norm across ALL heads of the projection (gain vector of that length)
-                    PER_HEAD = 2 };              // every head is RMS-normed on its own with one gain vector of the head's width shared by all heads
+                    PER_HEAD = 2,                // every head is RMS-normed on its own with one gain vector of the head's width shared by all heads
+                    UNIT = 3 };                  // the same without a gain
 enum class GluAct { SILU = 0, GELU_TANH = 1, RELU = 2,
+                    RELU2 = 4,               // relu(z)^2
                     XIELU = 3 };             // two learned numbers (p, q) per layer: z > 0: softplus(p) z^2 + z / 2; z <= 0: (1/2 + softplus(q))(e^z - 1 - z) + z / 2
 enum class BlockForm { SEQUENTIAL = 0,           // x += mixer(norm1 x) ; x += ff(norm2 x)
                        PARALLEL = 1,             // h = norm1 x ; x += m * (ls1 * mixer(h) + ls2 * ff(h)); with ModelConfig::depth_average the next layer reads
@@ -29,8 +32,11 @@ enum class BlockForm { SEQUENTIAL = 0,           // x += mixer(norm1 x) ; x += f
                        STREAMS = 2,              // SEQUENTIAL over several residual streams: a sublayer reads a learned blend of the streams and
                                                  // its output enters every stream through a learned stream-mixing matrix (ModelConfig::streams)
                        POST_NORM = 3,            // x += norm1(mixer(x)) ; x += norm2(ff(x)): the sublayers read x itself, the norm sits on their output
-                       SUM_NORM = 4 };           // x <- norm1(a x + mixer(x)) ; x <- norm2(a x + ff(x)): the norm sits on the residual sum itself, the
+                       SUM_NORM = 4,             // x <- norm1(a x + mixer(x)) ; x <- norm2(a x + ff(x)): the norm sits on the residual sum itself, the
                                                  // skip path is multiplied by a = ModelConfig::skip_scale
+                       SANDWICH = 5 };           // x += norm1b(mixer(norm1 x)) ; x += norm2b(ff(norm2 x)): a norm in front of and behind each sublayer
+enum class OutGate { NONE = 0, PER_HEAD = 1,     // what the mixer's joined heads are multiplied by before the output projection: sigmoid(W_g h), one number
+                     PER_CHANNEL = 2 };          // per head or one per channel; h is the input the projections read
 enum class FfKind { GLU = 0,                     // W_down (act(W_gate h) * W_up h)
                     MOE_RELU2 = 1,               // routed experts W_down relu(W_up h)^2, top-k softmax over the chosen logits, optional gated shared expert
                     MOE_GLU = 2,               // routed gated experts W_down (act(W_gate h) * W_up h); how they are chosen and weighted: RouteSpec
@@ -45,7 +51,7 @@ struct RotarySpec {
     int dims = 0;
     double base = 10000.0;
     bool interleaved = true;     // pairs (2i, 2i+1); false: (i, i + dims/2)
-    float factor = 0.f, original = 0.f, fast = 0.f, slow = 0.f;
+    double factor = 0.0, original = 0.0, fast = 0.0, slow = 0.0;
     float divide = 1.f;          // linear position scaling: every angular frequency is divided by this
 };
 
@@ -65,11 +71,12 @@ struct ScanSpec {
 // How a mixture of experts chooses and weights.  sigmoid: scores are sigmoid(logit) (else softmax over the chosen logits);
 // correction: a per-expert vector added to the scores for the CHOICE only; groups > 0: experts form `groups` equal runs of
 // neighbours, a run scores the sum of its two largest choice scores and only the best `keep` runs can be chosen from.
-// all: scores are the softmax over ALL experts; the chosen experts' scores times `scale` are the weights, not renormalized.
+// all: scores are the softmax over ALL experts; the chosen experts' scores times `scale` are the weights, not renormalized — or, with
+// renorm, divided by their sum.  With `all` a run of neighbours scores its largest score instead.
 struct RouteSpec {
     bool sigmoid = false, correction = false;
     int groups = 0, keep = 0;
-    bool all = false;
+    bool all = false, renorm = false;
     float scale = 1.f;
 };
 
@@ -89,6 +96,19 @@ struct DeltaSpec {
 // divided by its root mean square per head, times a gain over all heads, times the gate, then W_o.  The sequence's state is S and h'.
 struct WkvSpec {
     int decay_rank = 0;
+};
+
+// Matrix memory with exponential gating.  q (times dim^-1/2), k [heads, dim], v [heads, vdim] from projections; per head a log input gate
+// i = c(W_i h + b_i) and a log forget gate f = logsigmoid(c(W_f h + b_f)), c(z) = gate_cap tanh(z / gate_cap).  With S [dim, vdim], n [dim] and the
+// stabilizer m from zero, all F32:  m' = max(f + m, i);  S <- e^(f+m-m') S + e^(i-m') k v^T, n likewise with k alone;
+// o = S^T q / (max(|<n, q>|, e^-m') + 1e-6), over its root mean square per head, times a gain over all heads, times sigmoid(W_g h).
+struct MlstmSpec {
+    float gate_cap = 0.f;
+};
+// Queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  every == 0: off.
+struct QueryTempSpec {
+    float coef = 0.f;
+    double every = 0.0;
 };
 
 struct LayerSpec {
@@ -138,6 +158,12 @@ struct LayerSpec {
     // ---- mechanisms added with the Fuvozen family ----
     WkvSpec wkv;                 // WKV (heads and dim above apply too; vdim == dim)
     bool shared_glu = false;     // MOE_GLU: the shared expert (shared_ff) is a gated unit added as it is, without a sigmoid weight
+    // ---- mechanisms added with the Tibelix family ----
+    MlstmSpec mlstm;             // MLSTM (heads, dim and vdim above apply too)
+    QueryTempSpec q_temp;        // attention: position-dependent multiplier of the queries
+    bool distance_bias = false;  // attention: slope_h (i - j) is taken off the scaled score, slope_h = 2^(-8 (h + 1) / heads)
+    bool unit_sink = false;      // attention: the softmax denominator also holds 1 (a sink of score 0 without key or value)
+    OutGate out_gate = OutGate::NONE;
     int cache_slot = -1;         // set when the model is finalized: which entry of the model's per-mixer cache table holds this mixer's rows
 };
 

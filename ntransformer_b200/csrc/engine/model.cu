@@ -83,7 +83,7 @@ Model::~Model() {
     if (moe_offsets_host_) cudaFreeHost(moe_offsets_host_);
     auto free_layer = [](LayerWeights& L) {
         for (void* p : {(void*)L.e_up_tab, (void*)L.e_down_tab, (void*)L.rot_freq, (void*)L.e_gate_tab, (void*)L.conv_state, (void*)L.ssm_state, (void*)L.shift_state,
-                        (void*)L.q_conv_state, (void*)L.k_conv_state, (void*)L.v_conv_state, (void*)L.delta_state, (void*)L.wkv_state, L.e_maps}) if (p) cudaFree(p);
+                        (void*)L.q_conv_state, (void*)L.k_conv_state, (void*)L.v_conv_state, (void*)L.delta_state, (void*)L.wkv_state, L.e_maps, (void*)L.ml_state, (void*)L.ml_m, (void*)L.rot_freq64}) if (p) cudaFree(p);
     };
     for (LayerWeights& L : layers_) {
         free_layer(L);
@@ -441,6 +441,7 @@ size_t Model::weight_bytes() const {
             const LayerWeights& L = layer_weights(i);
             b += L.wq.bytes() + L.wk.bytes() + L.wv.bytes() + L.wo.bytes() + L.gate.bytes() + L.up.bytes() + L.down.bytes();
             b += L.w_dq.bytes() + L.w_uq.bytes() + L.w_dkv.bytes() + L.w_uk.bytes() + L.w_uv.bytes() + L.ssm_in.bytes() + L.side_gate.bytes() + L.side_proj.bytes();
+            b += L.out_gate.bytes() + L.ml_i.bytes() + L.ml_f.bytes();
             b += L.wkv_g.bytes() + L.wkv_w1.bytes() + L.wkv_w2.bytes();
             for (const LayerWeights& m : L.branch)
                 b += m.wq.bytes() + m.wk.bytes() + m.wv.bytes() + m.wo.bytes() + m.d_beta.bytes() + m.d_a1.bytes() + m.d_a2.bytes() + m.d_g1.bytes() + m.d_g2.bytes();
@@ -467,6 +468,7 @@ size_t Model::bytes_per_token(int ctx) const {
             size_t kw = 0, vw = 0;
             cache_row_widths(L.kv_from >= 0 ? L.kv_from : i, kw, vw);
             b += (size_t)std::min(ctx, L.chunk > 0 ? L.chunk : (L.window > 0 ? L.window + L.keep_first : ctx)) * (kw + vw) * dtype_size(cache_dt_);
+            if (L.mixer == MixerKind::MLSTM) b += (size_t)2 * L.heads * (L.vdim + 1) * L.dim * 4;
             if (L.mixer == MixerKind::WKV) b += (size_t)2 * L.heads * L.dim * L.dim * 4;
             if (L.mixer == MixerKind::SSM_SCAN) b += (size_t)2 * L.heads * L.vdim * L.scan.state * 4;      // the state is read and written
             for (const LayerSpec& m : L.branches) {

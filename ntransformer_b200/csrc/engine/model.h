@@ -96,6 +96,16 @@ struct LayerWeights {
     // weights of the average over depth [layer + 2], the activation's two numbers, gate matrix of a gated shared expert
     const float *depth_w = nullptr, *ff_act = nullptr;
     Weight sh_glu;
+    // norms behind the sublayers (SANDWICH), output gate of the mixer; matrix memory: input / forget gate rows and biases [heads], output gain
+    // [heads * vdim], the short gate rows stacked and zero-padded for the tensor cores (owned), the sequence's state [heads, vdim + 1, dim] and
+    // stabilizer [heads] in F32 (owned)
+    const float *norm1b = nullptr, *norm2b = nullptr;
+    Weight out_gate, ml_i, ml_f, ml_if;
+    const float *ml_ib = nullptr, *ml_fb = nullptr, *ml_norm = nullptr;
+    float *ml_state = nullptr, *ml_m = nullptr;
+    double* rot_freq64 = nullptr;          // device, rot.dims / 2: the latent attention's frequencies where a long-context blend is configured (owned)
+    const float* slopes = nullptr;         // device [heads]: distance bias; device [heads] of zeros: unit sink (model-owned)
+    const float* zero_sink = nullptr;
     // MixerKind::BRANCHES: each branch's tensors and state
     std::vector<LayerWeights> branch;
 };
@@ -197,11 +207,25 @@ private:
     void layer_parallel_token(int i, cudaStream_t s);
     void prefill_parallel(int T, int p0, cudaStream_t s);   // T prompt rows: embedding, all layers -> pf_.x
     void layer_parallel_rows(int i, int T, int p0, cudaStream_t s);
-    MoeWeights parallel_moe(int i) const;
+    MoeWeights gated_moe(int i) const;
     void ensure_parallel_buffers(size_t T);
     struct ParDec { float *slots = nullptr, *h = nullptr, *mix[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}, *wide = nullptr; size_t slot = 0; } par_dec_;   // decode: stable addresses
     struct ParRows { float *slots = nullptr, *h = nullptr, *wide = nullptr; void *hs = nullptr, *mix_s[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}; size_t slot = 0; } par_;
-    void latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s);
+    // gate [T, heads * vdim] (absorbed form only): the values are multiplied by sigmoid(gate)
+    void latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s, const float* gate = nullptr);
+    LatentRot latent_rot(int i) const;
+    // SANDWICH block form (attention with distance bias, latent attention, matrix memory): engine/model_sandwich.cu
+    bool finalize_sandwich_layer(int i);
+    void finalize_sandwich_decode();
+    size_t sandwich_scratch_width() const;    // floats per row of the layers' intermediates
+    void step_sandwich(cudaStream_t s);       // one decoded token: embedding, all layers -> hidden_
+    void prefill_sandwich(int T, int p0, cudaStream_t s);      // T prompt rows: embedding, all layers -> pf_.x
+    void sandwich_mixer_token(int i, float* y, cudaStream_t s);
+    void sandwich_ff_token(int i, float* y, cudaStream_t s);
+    void sandwich_mixer_rows(int i, int T, int p0, float* y, cudaStream_t s);
+    void sandwich_ff_rows(int i, int T, float* y, cudaStream_t s);
+    bool rows_take_tc(const Weight& w) const { return pf_.ws && (w.tc_ptr || spec_tc_ok(w)); }
+    float* ml_scratch_ = nullptr;             // segment states of the matrix memory over prompt rows (owned_)
     float* wkv_scratch_ = nullptr;            // segment states of the WKV recurrence over prompt rows (owned_)
     Weight bigram_;                           // second embedding over token pairs [buckets + 1, width]
     const LayerSpec& slot_spec(int slot) const { return *slot_spec_[(size_t)slot]; }

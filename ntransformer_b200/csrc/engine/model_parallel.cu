@@ -224,12 +224,12 @@ void Model::layer_parallel_token(int i, cudaStream_t s) {
         mats[n++] = multi(L.wq, B.h, q); mats[n++] = multi(L.w_dkv, B.h, dkv);
         ff_mats();
         gemv_multi(mats, n, s);
-        latent_prep(nullptr, 0, nullptr, dkv, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, S.rot.dims, S.rot.interleaved, S.rot.base, 1, pos_dev, 0, s);
+        latent_prep(nullptr, 0, nullptr, dkv, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, latent_rot(i), 1, pos_dev, 0, s);
         latent_mixer_core(i, 1, pos_dev, 0, q, qa, ol, o, s);
     }
     NT_CHECK(cur <= parallel_scratch_width(), "layer_parallel_token: scratch overrun");
     if (moe) {
-        const MoeWeights w = parallel_moe(i);
+        const MoeWeights w = gated_moe(i);
         moe_expert_up_token(act, B.h, nullptr, w, s, logits, moe_sel_, moe_wt_);
     }
     SumTerm t[GEMV_SUM_MAX_TERMS];
@@ -245,13 +245,13 @@ void Model::layer_parallel_token(int i, cudaStream_t s) {
     gemv_sum(x, t, nt, cfg_.hidden_size, L.wo.dtype, true, s);
 }
 
-MoeWeights Model::parallel_moe(int i) const {
+MoeWeights Model::gated_moe(int i) const {
     const LayerSpec& S = cfg_.layers[(size_t)i];
     const LayerWeights& L = layers_[(size_t)i];
     MoeWeights w;
     w.router = L.router; w.up = L.e_up_tab; w.down = L.e_down_tab; w.gate = L.e_gate_tab; w.dtype = L.e_up[0].dtype;
     w.experts = S.experts; w.top = S.top; w.ff = S.ff; w.width = cfg_.hidden_size;
-    w.all = true; w.scale = S.route.scale;
+    w.all = true; w.scale = S.route.scale; w.renorm = S.route.renorm; w.groups = S.route.groups; w.keep = S.route.keep;
     if (S.shared_ff > 0) { w.shared_up = L.sh_up.ptr; w.shared_down = L.sh_down.ptr; w.shared_gatew = L.sh_glu.ptr; w.shared_ff = S.shared_ff; }
     return w;
 }
@@ -328,7 +328,7 @@ void Model::layer_parallel_rows(int i, int T, int p0, cudaStream_t s) {
               *o = take(H * (size_t)S.vdim);
         parallel_gemm(q, B.h, hs_of(L.wq), L.wq, T, false, s);
         parallel_gemm(dkv, B.h, hs_of(L.w_dkv), L.w_dkv, T, false, s);
-        latent_prep(nullptr, 0, nullptr, dkv, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, S.rot.dims, S.rot.interleaved, S.rot.base, T, nullptr, p0, s);
+        latent_prep(nullptr, 0, nullptr, dkv, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, latent_rot(i), T, nullptr, p0, s);
         latent_mixer_core(i, T, nullptr, p0, q, qa, ol, o, s);
         add_product(o, L.wo);
     }
@@ -347,7 +347,7 @@ void Model::layer_parallel_rows(int i, int T, int p0, cudaStream_t s) {
         xielu_rows(tc ? nullptr : u, tc ? pf_.ws : nullptr, u, L.ff_act, T, S.ff, s);
         parallel_gemm(x, u, tc ? pf_.ws : nullptr, L.down, T, true, s);
     } else if (S.ff > 0) {
-        const MoeWeights w = parallel_moe(i);
+        const MoeWeights w = gated_moe(i);
         moe_route(pf_.sel, pf_.wt, nullptr, B.h, w, T, s);
         moe_glu_rows(i, T, B.h, w, x, true, s);
         if (S.shared_ff > 0 && pf_.ws && pf_.ws2 && spec_tc_ok(L.sh_glu) && spec_tc_ok(L.sh_up) && spec_tc_ok(L.sh_down) && S.shared_ff % 128 == 0) {

@@ -7,7 +7,7 @@
 namespace nt { namespace b200 {
 
 const std::vector<const ModelFamily*>& model_families() {
-    static const std::vector<const ModelFamily*> all = {zelunex_family(), vebotar_family(), tanolorn_family(), savidra_family(), fuvozen_family()};
+    static const std::vector<const ModelFamily*> all = {zelunex_family(), vebotar_family(), tanolorn_family(), savidra_family(), fuvozen_family(), tibelix_family()};
     return all;
 }
 
@@ -19,7 +19,8 @@ bool slot_is_f32_table(TensorSlot s) {
         case TensorSlot::W_DQ: case TensorSlot::W_UQ: case TensorSlot::W_DKV: case TensorSlot::W_UK: case TensorSlot::W_UV:
         case TensorSlot::SSM_IN: case TensorSlot::SIDE_EMBED: case TensorSlot::SIDE_GATE: case TensorSlot::SIDE_PROJ:
         case TensorSlot::DELTA_BETA: case TensorSlot::DELTA_A1: case TensorSlot::DELTA_A2: case TensorSlot::DELTA_G1: case TensorSlot::DELTA_G2:
-        case TensorSlot::BIGRAM: case TensorSlot::WKV_G: case TensorSlot::WKV_W1: case TensorSlot::WKV_W2: case TensorSlot::SHARED_GLU: return false;
+        case TensorSlot::BIGRAM: case TensorSlot::WKV_G: case TensorSlot::WKV_W1: case TensorSlot::WKV_W2: case TensorSlot::SHARED_GLU:
+        case TensorSlot::OUT_GATE: case TensorSlot::MLSTM_I: case TensorSlot::MLSTM_F: return false;
         default: return true;
     }
 }

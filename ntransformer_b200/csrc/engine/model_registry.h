@@ -25,6 +25,8 @@ enum class TensorSlot { EMBED, HEAD, OUT_NORM, NORM1, NORM2, WQ, WK, WV, WO, Q_N
                         DELTA_BETA, DELTA_A1, DELTA_A2, DELTA_DT_BIAS, DELTA_A_LOG, DELTA_NORM, DELTA_G1, DELTA_G2,   // gated delta rule
                         BIGRAM, DEPTH_AVG,                                                // second embedding over token pairs; weights of the average over depth
                         WKV_MU, WKV_G, WKV_W1, WKV_W2, WKV_W0, WKV_U, WKV_NORM,           // WKV mixer (WKV_MU: index r, k, v, g, w; r, k, v are WQ, WK, WV)
+                        NORM1B, NORM2B, OUT_GATE,                                         // norms behind the sublayers; output gate of a mixer
+                        MLSTM_I, MLSTM_F, MLSTM_IB, MLSTM_FB, MLSTM_NORM,                 // matrix memory: input / forget gate rows and biases, output gain
                         FF_ACT, SHARED_GLU };                                             // the activation's numbers; gate matrix of a gated shared expert
 
 struct TensorBinding {
@@ -60,5 +62,6 @@ const ModelFamily* vebotar_family();      // engine/vebotar.cpp
 const ModelFamily* tanolorn_family();     // engine/tanolorn.cpp
 const ModelFamily* savidra_family();      // engine/savidra.cpp
 const ModelFamily* fuvozen_family();      // engine/fuvozen.cpp
+const ModelFamily* tibelix_family();      // engine/tibelix.cpp
 
 }}  // namespace nt::b200

@@ -3,7 +3,8 @@
 // mechanisms (windowed / soft-capped attention, whole-projection q/k norm, parallel block with layer scale, GELU-gated unit,
 // layers sharing tensors) combine freely.  Same buffers, stream, CUDA-graph replay, logits and sampler as the GGUF families
 // (engine/model.cu); the KV cache is per layer because layers may differ in width.  Layers of BlockForm::SUM_NORM live in
-// engine/model_sumnorm.cu, layers of the PARALLEL form with latent-attention or WKV mixers in engine/model_parallel.cu.
+// engine/model_sumnorm.cu, layers of the PARALLEL form with latent-attention or WKV mixers in engine/model_parallel.cu, layers of the
+// SANDWICH form in engine/model_sandwich.cu.
 //
 // Arithmetic: the residual stream, norms, softmax and every accumulation are F32.  Weights stay in their stored dtype (BF16)
 // and are widened in registers, or — exact 32-bit mode — are widened once at load.  The cache stores BF16 (F32 in exact mode).
@@ -65,6 +66,14 @@ bool Model::bind_slot(TensorSlot slot, int layer, const void* ptr, DType dt, int
     LayerWeights& L = *Lp;
     switch (slot) {
         case TensorSlot::SHIFT_MU: return V(L.shift_mu);
+        case TensorSlot::NORM1B: return V(L.norm1b);
+        case TensorSlot::NORM2B: return V(L.norm2b);
+        case TensorSlot::OUT_GATE: return W(L.out_gate);
+        case TensorSlot::MLSTM_I: return W(L.ml_i);
+        case TensorSlot::MLSTM_F: return W(L.ml_f);
+        case TensorSlot::MLSTM_IB: return V(L.ml_ib);
+        case TensorSlot::MLSTM_FB: return V(L.ml_fb);
+        case TensorSlot::MLSTM_NORM: return V(L.ml_norm);
         case TensorSlot::WKV_MU: return index >= 0 && index < 5 && V(L.wkv_mu[index]);
         case TensorSlot::WKV_G: return W(L.wkv_g);
         case TensorSlot::WKV_W1: return W(L.wkv_w1);
@@ -240,6 +249,11 @@ bool Model::finalize_spec() {
             if (S.ff > 0 && S.ff_kind == FfKind::MOE_GLU) topmax = std::max(topmax, S.top);
             continue;
         }
+        if (S.form == BlockForm::SANDWICH) {
+            if (!finalize_sandwich_layer(i)) return false;
+            if (S.ff > 0 && S.ff_kind == FfKind::MOE_GLU) topmax = std::max(topmax, S.top);
+            continue;
+        }
         if (S.form == BlockForm::SUM_NORM) {
             if (!finalize_sumnorm_layer(i)) return false;
             ffmax = std::max(ffmax, S.ff);
@@ -350,10 +364,14 @@ bool Model::finalize_spec() {
             g = d;
         };
         fold(out_norm_);
-        for (LayerWeights& L : layers_) { fold(L.attn_norm); fold(L.ffn_norm); }
+        for (LayerWeights& L : layers_) { fold(L.attn_norm); fold(L.ffn_norm); fold(L.norm1b); fold(L.norm2b); }
     }
     if (parallel_rows()) {
         finalize_parallel_decode();
+        moe_sel_ = dmalloc<int>(topmax); moe_wt_ = dmalloc<float>(topmax);
+    }
+    if (cfg_.layers[0].form == BlockForm::SANDWICH) {
+        finalize_sandwich_decode();
         moe_sel_ = dmalloc<int>(topmax); moe_wt_ = dmalloc<float>(topmax);
     }
     if (cfg_.layers[0].form == BlockForm::SUM_NORM) {
@@ -438,6 +456,7 @@ void Model::step_body_spec(cudaStream_t s) {
     const int* pos_dev = step_dev_ + 1;
     const float m = cfg_.residual_mult;
     if (parallel_rows()) { step_parallel(s); return; }
+    if (cfg_.layers[0].form == BlockForm::SANDWICH) { step_sandwich(s); return; }
     embed_rows(hidden_, embd_.ptr, embd_.dtype, step_dev_, 1, hidden, s);
     if (cfg_.layers[0].form == BlockForm::POST_NORM) {
         RowBufs B = dec_;
@@ -499,11 +518,13 @@ void Model::ensure_prefill_buffers_spec(int tokens) {
     size_t qmax = 1, kmax = 1, vmax = 1, omax = 1, ffmax = 1, mapmax = 1, topmax = 0, emax = 1, effmax = 1;
     const bool par_form = parallel_rows();
     const bool sum_form = cfg_.layers[0].form == BlockForm::SUM_NORM;
-    const bool post_form = cfg_.layers[0].form == BlockForm::POST_NORM || sum_form || par_form;       // the first two keep five scratch rows of the widest intermediate
+    const bool sand_form = cfg_.layers[0].form == BlockForm::SANDWICH;
+    const bool post_form = cfg_.layers[0].form == BlockForm::POST_NORM || sum_form || par_form || sand_form;       // the first two keep five scratch rows of the widest intermediate
     if (sum_form) pf_.wide = dmalloc<float>(T * sumnorm_scratch_width());
+    if (sand_form) pf_.wide = dmalloc<float>(T * sandwich_scratch_width());
     for (const LayerSpec& S : cfg_.layers) {
         if (post_form) {                  // five scratch rows of the widest intermediate; routed experts as below
-            if (!par_form) qmax = kmax = vmax = omax = ffmax = row_scratch_width();
+            if (!par_form && !sand_form) qmax = kmax = vmax = omax = ffmax = row_scratch_width();
             if (S.ff_kind == FfKind::MOE_GLU && S.ff > 0) { topmax = std::max(topmax, (size_t)S.top); emax = std::max(emax, (size_t)S.experts); effmax = std::max(effmax, (size_t)S.ff); }
             continue;
         }
@@ -538,7 +559,7 @@ void Model::ensure_prefill_buffers_spec(int tokens) {
     for (int i = 0; i < cfg_.n_layers; i++) {
         const LayerWeights& L = layer_weights(i);
         for (const Weight* w : {&L.wq, &L.wk, &L.wv, &L.wo, &L.gate, &L.up, &L.down, &L.sh_up, &L.sh_down, &L.w_dq, &L.w_uq, &L.w_dkv, &L.ssm_in, &L.side_gate, &L.side_proj, &L.wkv_g, &L.wkv_w1,
-                                &L.wkv_w2, &L.sh_glu})
+                                &L.wkv_w2, &L.sh_glu, &L.w_uk, &L.w_uv, &L.out_gate, &L.ml_if})
             any_tc = any_tc || (w->ptr && (spec_tc_ok(*w) || w->tc_ptr));
         for (const LayerWeights& b : L.branch)
             for (const Weight* w : {&b.wq, &b.wk, &b.wv, &b.wo, &b.d_beta, &b.d_a1, &b.d_a2, &b.d_g1, &b.d_g2}) {
@@ -551,7 +572,11 @@ void Model::ensure_prefill_buffers_spec(int tokens) {
         ensure_parallel_buffers(T);
         if (any_tc) for (const LayerSpec& S : cfg_.layers) ffmax = std::max({ffmax, (size_t)S.shared_ff, (size_t)S.wkv.decay_rank});
     }
-    if ((sum_form || par_form) && any_tc) {             // the gated feed-forward's fused gate / up GEMM writes the down GEMM's split input here
+    if (sand_form && any_tc) {
+        for (const LayerSpec& S : cfg_.layers) ffmax = std::max({ffmax, (size_t)S.ff, (size_t)S.shared_ff, (size_t)S.latent.q_rank});
+        pf_.hws = dmalloc<uint8_t>(gemm_f16_tc_workspace_bytes((int)T, (int)hidden));
+    }
+    if ((sum_form || par_form || sand_form) && any_tc) {             // the gated feed-forward's fused gate / up GEMM writes the down GEMM's split input here
         size_t ffw = 1;
         for (const LayerSpec& S : cfg_.layers) ffw = std::max({ffw, (size_t)S.ff, (size_t)S.shared_ff});
         pf_.ws2 = dmalloc<uint8_t>(gemm_f16_tc_workspace_bytes((int)T, (int)ffw));
@@ -603,6 +628,11 @@ void Model::prefill_spec(const int* tokens, int seq_len, int start_pos) {
         NT_CUDA_CHECK(cudaMemcpyAsync(pf_.tok, tokens + c0, sizeof(int) * (size_t)T, cudaMemcpyHostToDevice, s));
         if (parallel_rows()) {
             prefill_parallel(T, p0, s);
+            if (!want_.empty()) emit_wanted(pf_.x, c0, T, s);
+            continue;
+        }
+        if (cfg_.layers[0].form == BlockForm::SANDWICH) {
+            prefill_sandwich(T, p0, s);
             if (!want_.empty()) emit_wanted(pf_.x, c0, T, s);
             continue;
         }
@@ -794,7 +824,7 @@ void Model::layer_streams_rows(int i, int T, int p0, cudaStream_t s) {
 
 void Model::cache_row_widths(int i, size_t& k, size_t& v) const {
     const LayerSpec& S = slot_spec(i);
-    if (S.mixer == MixerKind::SSM_SCAN || S.mixer == MixerKind::DELTA_RULE || S.mixer == MixerKind::BRANCHES || S.mixer == MixerKind::WKV) { k = v = 0; return; }      // a state, no rows (branches own theirs)
+    if (S.mixer == MixerKind::SSM_SCAN || S.mixer == MixerKind::DELTA_RULE || S.mixer == MixerKind::BRANCHES || S.mixer == MixerKind::WKV || S.mixer == MixerKind::MLSTM) { k = v = 0; return; }      // a state, no rows (branches own theirs)
     if (S.mixer == MixerKind::ATTN_LATENT) { k = (size_t)S.latent.kv_rank + S.latent.rot_dim; v = 0; return; }   // [latent | rotated key part]
     k = (size_t)S.kv_heads * S.maps * S.dim;
     v = (size_t)S.kv_heads * S.vdim;
@@ -909,7 +939,7 @@ void Model::latent_attention_rows(int i, int T, int p0, const float* q, float* o
         spec_gemm(lat_.vu, lat_.c32, tv ? lat_.ws : nullptr, L.w_uv, n, DENSE_STORE, nullptr, 1.f, s);
         latent_expand_pack(lat_.k, lat_.v, lat_.ku, lat_.vu, rows, cache_dt_, A.kv_rank, r0, n, S.heads, S.dim, A.rot_dim, S.vdim, kw, vw, s);
     }
-    latent_q_rot_pad(lat_.q, q, T, S.heads, S.dim, A.rot_dim, kw, S.rot.dims, S.rot.interleaved, S.rot.base, p0, s);
+    latent_q_rot_pad(lat_.q, q, T, S.heads, S.dim, A.rot_dim, kw, latent_rot(i), p0, s);
     float* o = vw == S.vdim ? out : lat_.o;
     attention_heads_mma(o, lat_.q, lat_.k, lat_.v, T, p0 - lo, P, S.heads, kw, vw, S.scale, s, S.window);
     if (o != out) latent_unpad(out, lat_.o, T, S.heads, S.vdim, vw, s);
@@ -960,15 +990,23 @@ void Model::moe_glu_rows(int i, int T, const float* x, const MoeWeights& w, floa
     moe_combine(y, pf_.y_rows, pf_.work, pf_.wt, nullptr, nullptr, T, S.experts, S.top, hidden, s, add);
 }
 
+LatentRot Model::latent_rot(int i) const {
+    const RotarySpec& R = cfg_.layers[(size_t)i].rot;
+    const LayerWeights& L = layer_weights(i);
+    LatentRot r;
+    r.dims = R.dims; r.interleaved = R.interleaved; r.base = R.base; r.freq = L.rot_freq64; r.mag = L.rot_freq64 ? L.rot_mag : 1.f;
+    return r;
+}
+
 // Scores and values of T rows behind the query projection and the cache write: expanded per-head form for prompt portions, absorbed form on
 // the cached rows otherwise.  q [T, heads, dim + rot_dim]; qa, ol: scratch [T, heads, kv_rank + rot_dim], [T, heads, kv_rank]; o (may be q) [T, heads * vdim].
-void Model::latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s) {
+void Model::latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s, const float* gate) {
     const LayerSpec& S = cfg_.layers[(size_t)i];
     const LayerWeights& L = layer_weights(i);
     const LatentSpec& A = S.latent;
     const int row = A.kv_rank + A.rot_dim;
-    if (!pos_dev && latent_expand_ok(S, T)) { latent_attention_rows(i, T, p0, q, o, s); return; }
-    latent_q_absorb(qa, q, L.w_uk.ptr, L.w_uv.dtype, T, S.heads, S.dim, A.rot_dim, A.kv_rank, S.rot.dims, S.rot.interleaved, S.rot.base, pos_dev, p0, s);
+    if (!pos_dev && !gate && latent_expand_ok(S, T)) { latent_attention_rows(i, T, p0, q, o, s); return; }
+    latent_q_absorb(qa, q, L.w_uk.ptr, L.w_uv.dtype, T, S.heads, S.dim, A.rot_dim, A.kv_rank, latent_rot(i), pos_dev, p0, s);
     if (lat_part_ && attention_shared_rows_supported(S.heads, row, A.kv_rank, row, cache_dt_, kcs_[(size_t)i])) {
         attention_shared_rows(ol, qa, kcs_[(size_t)i], cache_dt_, T, pos_dev, p0, cfg_.max_seq_len, S.heads, row, A.kv_rank, row, S.scale, lat_part_, s, S.window);
     } else {
@@ -976,7 +1014,7 @@ void Model::latent_mixer_core(int i, int T, const int* pos_dev, int p0, const fl
         a.heads = S.heads; a.kv_heads = 1; a.dim = row; a.vdim = A.kv_rank; a.scale = S.scale; a.k_stride = row; a.v_stride = row; a.window = S.window;
         attention_window(ol, qa, kcs_[(size_t)i], kcs_[(size_t)i], cache_dt_, T, pos_dev, p0, cfg_.max_seq_len, a, s);
     }
-    latent_v_up(o, ol, L.w_uv.ptr, L.w_uv.dtype, T, S.heads, S.vdim, A.kv_rank, s);
+    latent_v_up(o, ol, L.w_uv.ptr, L.w_uv.dtype, T, S.heads, S.vdim, A.kv_rank, s, gate);
 }
 
 // One layer over T rows: x += norm1(mixer(x)); x += norm2(ff(x)); x += side(x, token).  The sublayers read x itself.
@@ -996,8 +1034,8 @@ void Model::layer_postnorm(int i, int T, const int* tok_dev, const int* pos_dev,
             rows_matmul(cq, B.x, L.w_dq, T, s);
             if (S.kv_from < 0) rows_matmul(dkv, B.x, L.w_dkv, T, s);
         }
-        latent_prep(cq, A.q_rank, L.dq_norm, S.kv_from < 0 ? dkv : nullptr, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, S.rot.dims,
-                    S.rot.interleaved, S.rot.base, T, pos_dev, p0, s);
+        latent_prep(cq, A.q_rank, L.dq_norm, S.kv_from < 0 ? dkv : nullptr, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, latent_rot(i),
+                    T, pos_dev, p0, s);
         rows_matmul(q, cq, L.w_uq, T, s);
         latent_mixer_core(i, T, pos_dev, p0, q, qa, ol, o, s);
         rows_matmul(B.y, o, L.wo, T, s);

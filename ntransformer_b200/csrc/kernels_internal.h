@@ -149,7 +149,7 @@ void gemv_dense(const GemvMat* mats, int n_mat, int K, const float* x, DenseEpil
 constexpr int DENSE_MAX_NORM_GROUPS = 256;
 // Several matrices with an input vector each, one launch; act is applied to a matrix's own rows.  One 16-bit dtype per launch, F32 matrices
 // (router tables) may stand beside it.
-enum GemvAct { GEMV_ACT_NONE = 0, GEMV_ACT_TANH = 1, GEMV_ACT_XIELU = 2 /* two learned numbers: act_p */ };
+enum GemvAct { GEMV_ACT_NONE = 0, GEMV_ACT_TANH = 1, GEMV_ACT_XIELU = 2 /* two learned numbers: act_p */, GEMV_ACT_RELU2 = 3 };
 struct MultiMat {
     const void* W = nullptr; DType dtype = DType::F32; size_t row_pitch = 0;
     const float* x = nullptr; float* y = nullptr;
@@ -187,6 +187,9 @@ struct WindowAttn {
     int k_stride = 0, v_stride = 0;    // elements between consecutive positions' key / value rows; 0: packed (kv_heads*maps*dim, kv_heads*vdim).
                                        // With strides the two caches may be one buffer (values = a slice of the key rows: latent attention)
     const float* sink = nullptr;       // [heads] (device): exp(sink[h]) joins head h's softmax denominator; it has no key and no value
+    const float* slope = nullptr;      // [heads] (device): slope[h] * (i - j) is taken off head h's scaled score
+    const float* head_gate = nullptr;  // [tokens, heads] (device): head h's result is multiplied by sigmoid(head_gate[t * gate_stride + h])
+    int gate_stride = 0;
     int joint_v = 0;                   // 1: every query head sums ONE value row per key, vdim wide, at the start of the key's value row (whatever its
                                        // key head): with vdim = kv_heads * (a head's width) each head's weights are applied to every value head at once
 };
@@ -210,6 +213,7 @@ void qk_norm_kv_write(float* Q, const float* K, const float* V, const float* q_g
 // Host: the dims/2 angular frequencies base^(-2i/dims) of a rotary layer, blended for long contexts when factor > 0 (see
 // engine/layer_spec.h RotarySpec), computed in double; returns the multiplier of cos and sin.
 float rotary_table(float* freq_host, int dims, float base, float factor, float original, float fast, float slow);
+float rotary_table(double* freq_host, int dims, double base, double factor, double original, double fast, double slow);
 void rope_partial_kv_write(float* Q, const float* K, const float* V, const float* freq, float mag, int dims, bool interleaved, int dim,
                            void* kc, void* vc, DType cache_dt, int tokens, const int* pos_dev, int p0, int qdim, int kdim, int vdim, cudaStream_t s);
 // Differential combination of two attention maps: A [tokens, heads, 2, vdim] -> out [tokens, heads * vdim],
@@ -240,8 +244,9 @@ struct MoeWeights {
     bool sigmoid = false;
     const float* correction = nullptr;
     int groups = 0, keep = 0;
-    // all: scores are the softmax over ALL experts, weight = the chosen experts' scores times scale (not renormalized)
-    bool all = false;
+    // all: scores are the softmax over ALL experts, weight = the chosen experts' scores times scale (not renormalized), or with renorm
+    // divided by their sum (+ 1e-20); a run of neighbours (groups > 0) then scores its largest score
+    bool all = false, renorm = false;
     float scale = 1.f;
     const void* shared_gatew = nullptr;  // [shared_ff, width]: the shared expert is a gated unit too (decode kernels; sgate null: added as it is)
 };
@@ -279,22 +284,25 @@ void moe_gather_rows(float* out, const float* h, const int* work, int tokens, in
 void relu2(float* x, size_t n, cudaStream_t s);
 
 // ---- attention_latent.cu / ssm_scan.cu / postnorm.cu: mechanisms added with the third layer-spec family ----
+// Rotation of the latent attention's rotated part: pairs turn by position * base^(-2i/dims), or by position * freq[i] when a table is given
+// (device, dims / 2 numbers; long-context blends); cos and sin times mag.
+struct LatentRot { int dims = 0; bool interleaved = true; double base = 10000.0; const double* freq = nullptr; float mag = 1.f; };
 // Latent attention (engine/layer_spec.h LatentSpec).  cq [T, q_rank]: RMS-normed in place (gain).  dkv [T, kv_rank + rot_dim] (null: the layer
 // reads another layer's rows; cq null: the queries have no latent): [RMS-normed first part | rotated rest] -> cache row base + t of `cache` ([max_seq, kv_rank + rot_dim]).
 void latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache,
-                 DType cache_dt, int rot_dims, bool interleaved, double rot_base, int T, const int* pos_dev, int p0, cudaStream_t s);
+                 DType cache_dt, const LatentRot& rot, int T, const int* pos_dev, int p0, cudaStream_t s);
 // q [T, heads, dim + rot_dim] -> qa [T, heads, kv_rank + rot_dim] = [W_uk,h^T q_unrotated | rot(q_rotated)];  W_uk [heads * dim, kv_rank]
-void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, int rot_dims,
-                     bool interleaved, double rot_base, const int* pos_dev, int p0, cudaStream_t s);
-// ol [T, heads, kv_rank] -> out [T, heads * vdim] = W_uv,h ol_h;  W_uv [heads * vdim, kv_rank]
-void latent_v_up(float* out, const float* ol, const void* W_uv, DType dt, int T, int heads, int vdim, int kv_rank, cudaStream_t s);
+void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, const LatentRot& rot,
+                     const int* pos_dev, int p0, cudaStream_t s);
+// ol [T, heads, kv_rank] -> out [T, heads * vdim] = W_uv,h ol_h;  W_uv [heads * vdim, kv_rank].  gate [T, heads * vdim] (may be null): times sigmoid(gate)
+void latent_v_up(float* out, const float* ol, const void* W_uv, DType dt, int T, int heads, int vdim, int kv_rank, cudaStream_t s, const float* gate = nullptr);
 // Prompt portions: F32 latents of cache rows r0.. (input of the two up-projection GEMMs); their results packed with the rotated key part
 // into 16-bit per-head operands kfull [row, heads, kw] / vfull [row, heads, vw] (zero padded); queries rotated and padded to kw; the
 // padded outputs [T, heads, vw] back to [T, heads * vdim].
 void latent_rows_f32(float* out, const void* cache, DType cache_dt, int row, int kv_rank, int r0, int n, cudaStream_t s);
 void latent_expand_pack(void* kfull, void* vfull, const float* ku, const float* vu, const void* cache, DType cache_dt, int kv_rank, int r0, int n, int heads,
                         int dim, int rot_dim, int vdim, int kw, int vw, cudaStream_t s);
-void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, int rot_dims, bool interleaved, double rot_base, int p0,
+void latent_q_rot_pad(float* qp, const float* q, int T, int heads, int dim, int rot_dim, int kw, const LatentRot& rot, int p0,
                       cudaStream_t s);
 void latent_unpad(float* out, const float* o, int T, int heads, int vdim, int vw, cudaStream_t s);
 // Attention of a few queries over ONE key / value head stored as rows (keys: the first dim numbers of a row, values: the first vdim),
@@ -320,6 +328,13 @@ void ssm_gate_norm(float* out, const float* y, const float* u, int ld, int z_col
 // Post-norm block form: x[t] += rms(y[t] + bias) * gain;  out = act(gate + b_g) * (up + b_u);  g[t, j] <- gelu_tanh(g[t, j]) * E[token_t, col0 + j]
 void add_rmsnorm_rows(float* x, const float* y, const float* gain, const float* bias, int rows, int width, float eps, cudaStream_t s);
 void glu_bias_mul(float* out, const float* gate, const float* up, const float* gate_bias, const float* up_bias, int rows, int cols, bool gelu, cudaStream_t s);
+// The sandwich form's step between sublayers: x[t] += rms(y[t]) * gain_y (y null: x as it is), then h = rms(x[t]) * gain_h -> F32 rows and / or the
+// BF16 split of a tensor-core GEMM's input (gain_h null: x only).
+void sandwich_norm_rows(float* x, const float* y, const float* gain_y, const float* gain_h, float* h, void* split, int rows, int width, float eps, cudaStream_t s);
+// o [T, cols] * sigmoid(gate[t * ld + c / per]) -> F32 rows (in place is fine) and / or the BF16 split
+void sigmoid_gate_rows(float* out, void* split, const float* o, const float* gate, int ld, int per, int T, int cols, cudaStream_t s);
+// relu(z)^2 of a [T, cols], as F32 rows (in place is fine) and / or the BF16 split
+void relu2_rows(float* out, void* split, const float* in, int T, int cols, cudaStream_t s);
 void side_gate_rows(float* g, const void* E, DType dt, int e_cols, int col0, const int* tokens_dev, int rows, int dim, cudaStream_t s);
 
 // ---- short_conv.cu / delta_rule.cu / sumnorm.cu / attention_heads.cu: mechanisms added with the fourth layer-spec family ----
@@ -357,6 +372,8 @@ void token_shift_rows(float* h, const float* x, const float* mu, float* carried,
 struct HeadPrep {
     int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
     const float* q_gain = nullptr; const float* k_gain = nullptr; float eps = 0.f;      // [dim] each; null: no norm
+    int unit_norm = 0;                      // 1: every query and key head over its root mean square, without a gain
+    float temp_coef = 0.f; double temp_every = 0.0;      // temp_every > 0: queries times 1 + temp_coef ln(floor((position + 1) / temp_every) + 1)
     int rot_dims = 0, interleaved = 0; const float* freq = nullptr;                      // [rot_dims / 2] angular frequencies (device)
     const float* temp = nullptr;            // [heads] or null
     const float* v_lambda = nullptr;        // one number (device); used with v_first
@@ -410,6 +427,24 @@ void wkv_out_norm(float* out, void* split, const float* o, const float* gate, co
 void wkv_token(float* out, const float* r, const float* k, const float* v, const float* gate, const float* a1, const void* W2, DType dt, const float* w0, const float* u,
                const float* norm, float* state, float eps, int rank, int heads, int dim, const int* pos_dev, int p0, cudaStream_t s);
 
+// ---- mlstm.cu: matrix memory with exponential gates (engine/layer_spec.h MlstmSpec), added with the sixth layer-spec family ----
+// State of a sequence: [heads, vdim + 1, dim] (rows 0 .. vdim - 1: S by value channel, row vdim: the normalizer n) and m [heads], F32; both read
+// as zeros when the step starts at position 0.
+// gates: zi, zf: pre-activations without bias, row t at + t * ld -> a = e^(f+m-m'), b = e^(i-m'), em = e^-m' [T, heads] each; m: read and replaced.
+void mlstm_gates(float* a, float* b, float* em, const float* zi, const float* zf, int ld, const float* bi, const float* bf, float cap, float* m, int T, int heads,
+                 const int* pos_dev, int p0, cudaStream_t s);
+// rows: o [T, heads, vdim] = S^T q q_scale, den [T, heads] = <n, q> q_scale.  scratch (mlstm_rows_scratch_floats; may be null): long steps may run as
+// segments side by side.  out_norm: o / (max(|den|, em) + 1e-6), over its root mean square, times norm [heads * vdim] and sigmoid(gate).
+constexpr int MLSTM_MAX_DIM = 512;
+void mlstm_rows(float* o, float* den, const float* q, const float* k, const float* v, const float* a, const float* b, float* state, float q_scale, int T, int heads, int dim,
+                int vdim, const int* pos_dev, int p0, cudaStream_t s, float* scratch = nullptr);
+size_t mlstm_rows_scratch_floats(int heads, int dim, int vdim);
+void mlstm_out_norm(float* out, void* split, const float* o, const float* den, const float* em, const float* gate, const float* norm, float eps, int T, int heads, int vdim,
+                    cudaStream_t s);
+// One token: gates, memory, head norm and output gate in one launch -> out [heads * vdim]
+void mlstm_token(float* out, const float* q, const float* k, const float* v, const float* gate, const float* zi, const float* zf, const float* bi, const float* bf,
+                 const float* norm, float* state, float* m, float cap, float q_scale, float eps, int heads, int dim, int vdim, const int* pos_dev, int p0, cudaStream_t s);
+
 // Programmatic dependent launch (PDL): when enabled, kernels are launched with
 // cudaLaunchAttributeProgrammaticStreamSerialization so that a kernel's prologue (barrier init, TMA weight
 // prefetch) overlaps the tail of its predecessor; every kernel executes griddepcontrol.wait before it touches
@@ -444,6 +479,8 @@ bool gemm_f16_tc_swiglu_ws(void* workspace_out, const void* workspace_in, const 
                            cudaStream_t s, const TcOpts& o = TcOpts());
 // workspace_out <- split(xIELU(A.W^T)), (p, q) = act_p on the device: the up product of an ungated feed-forward; N % 8 == 0
 bool gemm_f16_tc_xielu_ws(void* workspace_out, const void* workspace_in, const void* W_f16, const float* act_p, int M, int N, int K, cudaStream_t s, const TcOpts& o = TcOpts());
+// the same with relu(z)^2
+bool gemm_f16_tc_relu2_ws(void* workspace_out, const void* workspace_in, const void* W_f16, int M, int N, int K, cudaStream_t s, const TcOpts& o = TcOpts());
 // Routed experts in one launch per product.  Row runs of the split workspace (rows_padded rows in all): run e has count[e] rows from start[e] (a
 // multiple of 128) on; start / count live on the device, so do the experts' tensor maps (gemm_tc_weight_map on the host, then copied;
 // 64-byte aligned).  swiglu: workspace_out <- split(silu(A.Wgate_e^T) * (A.Wup_e^T)), else C rows = A.W_e^T; rows between the runs are not written.

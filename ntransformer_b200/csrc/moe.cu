@@ -10,7 +10,8 @@
 //                            result does not depend on which other tokens share its tile.
 // Variants (MoeWeights): gated experts W_down (silu(W_gate h) * W_up h) through a third pointer table; a router that scores by
 // sigmoid, adds a correction vector for the choice only, restricts the choice to the best runs of neighbouring experts and weights
-// by the plain scores; a router that weights by the softmax over all experts; a gated shared expert.
+// by the plain scores; a router that weights by the softmax over all experts (or by the chosen ones' share of it, choosing inside the runs of
+// neighbours with the largest score); a gated shared expert.
 // Expert matrices: F32, F16 or BF16 rows.  Compiled WITHOUT --use_fast_math.
 #include "kernels_internal.h"
 #include "bf16_split.cuh"
@@ -94,8 +95,9 @@ __device__ __forceinline__ float warp_dot(const unsigned char* row, const float*
 constexpr int RT_WARPS = 8;
 constexpr int MAX_EXPERTS = 256;
 
-// One warp: softmax over all experts of z, the `top` largest (lowest index on ties) with their share times `scale`, largest first.
-__device__ __forceinline__ void choose_of_all(const float* z, int experts, int top, float scale, int lane, int* sel, float* wt) {
+// One warp: softmax over all experts of z, the `top` largest (lowest index on ties) with their share times `scale`, largest first.  groups > 0: only
+// experts of the `keep` equal runs of neighbours whose largest score is largest.  renorm: the shares are divided by their sum.
+__device__ __forceinline__ void choose_of_all(const float* z, int experts, int top, float scale, int groups, int keep, int renorm, int lane, int* sel, float* wt) {
     float v[MAX_EXPERTS / 32], mx = -INFINITY, den = 0.f;
 #pragma unroll
     for (int i = 0; i < MAX_EXPERTS / 32; i++) { const int e = lane + 32 * i; v[i] = e < experts ? z[e] : -INFINITY; mx = fmaxf(mx, v[i]); }
@@ -105,7 +107,41 @@ __device__ __forceinline__ void choose_of_all(const float* z, int experts, int t
     for (int i = 0; i < MAX_EXPERTS / 32; i++) den += lane + 32 * i < experts ? expf(v[i] - mx) : 0.f;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xFFFFFFFFu, den, o);
-    unsigned taken = 0;                            // bit i: this lane's expert lane + 32 i is chosen
+    unsigned taken = 0;                            // bit i: this lane's expert lane + 32 i is chosen (or cannot be)
+    if (groups > 0) {
+        const int per = experts / groups;
+        float gs[MAX_EXPERTS / 32];                // this lane's runs lane + 32 j
+        unsigned kept = 0;
+#pragma unroll
+        for (int j = 0; j < MAX_EXPERTS / 32; j++) {
+            const int g = lane + 32 * j;
+            gs[j] = -INFINITY;
+            if (g < groups) for (int e = g * per; e < (g + 1) * per; e++) gs[j] = fmaxf(gs[j], z[e]);
+        }
+        for (int k = 0; k < keep; k++) {
+            float bv = -INFINITY;
+            int bg = MAX_EXPERTS;
+#pragma unroll
+            for (int j = 0; j < MAX_EXPERTS / 32; j++) {
+                const int g = lane + 32 * j;
+                if (g < groups && !(kept >> j & 1u) && (gs[j] > bv || bg == MAX_EXPERTS)) { bv = gs[j]; bg = g; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xFFFFFFFFu, bv, o);
+                const int og = __shfl_xor_sync(0xFFFFFFFFu, bg, o);
+                if (og < MAX_EXPERTS && (bg == MAX_EXPERTS || ov > bv || (ov == bv && og < bg))) { bv = ov; bg = og; }
+            }
+            if ((bg & 31) == lane) kept |= 1u << (bg >> 5);
+        }
+#pragma unroll
+        for (int i = 0; i < MAX_EXPERTS / 32; i++) {
+            const int e = lane + 32 * i, g = e < experts ? e / per : 0;
+            const unsigned k = __shfl_sync(0xFFFFFFFFu, kept, g & 31);
+            if (!(k >> (g >> 5) & 1u)) taken |= 1u << i;
+        }
+    }
+    float sum = 0.f;
     for (int k = 0; k < top; k++) {
         float bv = -INFINITY;
         int be = MAX_EXPERTS;
@@ -121,14 +157,17 @@ __device__ __forceinline__ void choose_of_all(const float* z, int experts, int t
             if (oe < MAX_EXPERTS && (be == MAX_EXPERTS || ov > bv || (ov == bv && oe < be))) { bv = ov; be = oe; }
         }
         if ((be & 31) == lane) taken |= 1u << (be >> 5);
-        if (lane == 0) { sel[k] = be; wt[k] = expf(bv - mx) / den * scale; }
+        const float share = expf(bv - mx) / den;
+        sum += share;
+        if (lane == 0) { sel[k] = be; wt[k] = share * scale; }
     }
+    if (renorm && lane == 0) for (int k = 0; k < top; k++) wt[k] /= sum + 1e-20f;
 }
 
 __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(int* __restrict__ sel, float* __restrict__ wt, float* __restrict__ sgate,
                                                                   const float* __restrict__ h, const float* __restrict__ router,
                                                                   const float* __restrict__ shared_gate, int experts, int top, int width,
-                                                                  int sigmoid, const float* __restrict__ correction, int groups, int keep, int all, float scale, StreamsIO sio, const float* __restrict__ norm_w, float eps, float* __restrict__ h_out) {
+                                                                  int sigmoid, const float* __restrict__ correction, int groups, int keep, int all, int renorm, float scale, StreamsIO sio, const float* __restrict__ norm_w, float eps, float* __restrict__ h_out) {
     extern __shared__ __align__(16) float hs[];
     __shared__ float z[MAX_EXPERTS + 1];
     __shared__ float sc[MAX_EXPERTS];
@@ -169,7 +208,7 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(int* __restric
     __syncthreads();
     if (all) {
         if (threadIdx.x == 0 && shared_gate) sgate[t] = 1.0f / (1.0f + expf(-z[experts]));
-        if (warp == 0) choose_of_all(z, experts, top, scale, lane, sel + (size_t)t * top, wt + (size_t)t * top);
+        if (warp == 0) choose_of_all(z, experts, top, scale, groups, keep, renorm, lane, sel + (size_t)t * top, wt + (size_t)t * top);
         return;
     }
     if (threadIdx.x != 0) return;
@@ -230,6 +269,7 @@ struct MoeDev {
     const void* shared_up; const void* shared_down; const void* shared_gatew;
     int top, ff, width, shared_ff, experts;
     float scale;
+    int groups, keep, renorm;
 };
 
 constexpr int TK_WARPS = 8;
@@ -251,7 +291,7 @@ __global__ void __launch_bounds__(TK_WARPS * 32) moe_up_token_kernel(float* __re
     pdl_wait();
     for (int i = threadIdx.x; i < m.width; i += TK_WARPS * 32) hs[i] = h[i];
     if (logits) {                                  // every CTA makes the same choice from the router's logits; the first one publishes it
-        if (warp == 0) choose_of_all(logits, m.experts, m.top, m.scale, lane, sel_s, wt_s);
+        if (warp == 0) choose_of_all(logits, m.experts, m.top, m.scale, m.groups, m.keep, m.renorm, lane, sel_s, wt_s);
     } else for (int k = threadIdx.x; k < m.top; k += TK_WARPS * 32) sel_s[k] = sel[k];
     __syncthreads();
     if (logits && blockIdx.x == 0) for (int k = threadIdx.x; k < m.top; k += TK_WARPS * 32) { sel_out[k] = sel_s[k]; wt_out[k] = wt_s[k]; }
@@ -492,7 +532,7 @@ __global__ void relu2_kernel(float* __restrict__ x, size_t n) {
     if (i < n) { const float z = fmaxf(x[i], 0.f); x[i] = z * z; }
 }
 
-MoeDev dev_of(const MoeWeights& w) { return MoeDev{w.gate, w.up, w.down, w.shared_up, w.shared_down, w.shared_gatew, w.top, w.ff, w.width, w.shared_up ? w.shared_ff : 0, w.experts, w.scale}; }
+MoeDev dev_of(const MoeWeights& w) { return MoeDev{w.gate, w.up, w.down, w.shared_up, w.shared_down, w.shared_gatew, w.top, w.ff, w.width, w.shared_up ? w.shared_ff : 0, w.experts, w.scale, w.groups, w.keep, w.renorm ? 1 : 0}; }
 
 }  // namespace
 
@@ -500,7 +540,7 @@ void moe_route(int* sel, float* wt, float* sgate, const float* h, const MoeWeigh
                const float* norm_w, float eps, float* h_out) {
     const StreamsIO sio = sio_p ? *sio_p : StreamsIO();
     NT_CHECK(w.experts >= 1 && w.experts <= MAX_EXPERTS && w.top >= 1 && w.top <= w.experts, "moe_route: 1 <= top <= experts <= 256");
-    NT_CHECK(w.groups == 0 || (w.sigmoid && w.experts % w.groups == 0 && w.keep >= 1 && w.keep <= w.groups && w.keep * (w.experts / w.groups) >= w.top),
+    NT_CHECK(w.groups == 0 || ((w.sigmoid || w.all) && w.experts % w.groups == 0 && w.keep >= 1 && w.keep <= w.groups && w.keep * (w.experts / w.groups) >= w.top),
              "moe_route: expert groups must be equal runs whose kept part holds at least top experts");
     if (tokens <= 0) return;
     const size_t smem = (size_t)w.width * sizeof(float);
@@ -508,7 +548,7 @@ void moe_route(int* sel, float* wt, float* sgate, const float* h, const MoeWeigh
     static unsigned long long done = 0;
     if (smem > 40 * 1024) opt_in_dynamic_smem(moe_route_kernel, 160 * 1024, done);
     launch_k(moe_route_kernel, dim3(tokens), dim3(RT_WARPS * 32), smem, s, sel, wt, sgate, h, w.router, w.shared_gate, w.experts, w.top, w.width,
-             w.sigmoid ? 1 : 0, w.correction, w.groups, w.keep, w.all ? 1 : 0, w.scale, sio, norm_w, eps, h_out);
+             w.sigmoid ? 1 : 0, w.correction, w.groups, w.keep, w.all ? 1 : 0, w.renorm ? 1 : 0, w.scale, sio, norm_w, eps, h_out);
     count_launch();
 }
 

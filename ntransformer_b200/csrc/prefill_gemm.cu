@@ -134,7 +134,7 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&v)[32]) {
         : "r"(taddr));
 }
 
-enum : int { MODE_STORE = 0, MODE_ADD = 1, MODE_SWIGLU = 2, MODE_XIELU = 3 };
+enum : int { MODE_STORE = 0, MODE_ADD = 1, MODE_SWIGLU = 2, MODE_XIELU = 3, MODE_RELU2 = 4 };
 
 // Grouped form: the rows of A are `experts` runs, run e with count[e] rows from row start[e] (a multiple of BM) on and a weight matrix of its own
 // (maps_b[e], gate / up pairs: maps_b2[e]; encoded on the host, resident in device memory).  The tile list is made on the device from the counts.
@@ -153,6 +153,7 @@ struct Grouped { const CUtensorMap* maps_b; const CUtensorMap* maps_b2; const in
 //               split_out = F16 hi/lo split of silu(A.Wg^T) * (A.Wu^T), i.e. the down projection's GEMM input, so the
 //               F32 gate/up activations never touch HBM (ffn.cpp:96-133 computes them as three launches).
 //   MODE_XIELU  split_out = hi/lo split of xIELU(A.W^T), (p, q) = act_p: the ungated feed-forward's input of the down projection
+//   MODE_RELU2  the same with relu(z)^2
 template <int BN, int MODE, bool GROUPED>
 __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                                                              const __grid_constant__ CUtensorMap map_b,
@@ -161,7 +162,7 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                                                              int M, int Mp, int N, int K, int tiles_m, int tiles_n, int n_tiles, int n_outer,
                                                              int kc_blocks, int bf16, int gelu, const float* __restrict__ col_scale, float alpha,
                                                              const float* __restrict__ act_p, const Grouped grp) {
-    constexpr bool ONE_CHUNK = MODE == MODE_SWIGLU || MODE == MODE_XIELU;       // the epilogue needs the whole sum
+    constexpr bool ONE_CHUNK = MODE == MODE_SWIGLU || MODE == MODE_XIELU || MODE == MODE_RELU2;       // the epilogue needs the whole sum
     constexpr int STAGES = Cfg<BN>::STAGES, STAGE_BYTES = Cfg<BN>::STAGE_BYTES, TMEM_COLS = 2 * BN;
     constexpr int TN = MODE == MODE_SWIGLU ? 128 : BN;          // output columns per tile
     // BF16 operands: A format at [7,10) and B format at [10,13) become 1 (F16 = 0); layouts, strides and the F32 accumulator are the same
@@ -302,7 +303,7 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                             *reinterpret_cast<uint4*>(lo + j) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
                         }
                     }
-                } else if (MODE == MODE_XIELU) {
+                } else if (MODE == MODE_XIELU || MODE == MODE_RELU2) {
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                     if (row < m_end) {
                         __half* hi = split_out + (size_t)row * N + n0 + c * 32;
@@ -312,8 +313,11 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                             if (n0 + c * 32 + j >= N) break;             // a ragged last tile (N % 8 == 0)
                             uint32_t ph[4], pl[4];
 #pragma unroll
-                            for (int e = 0; e < 4; e++)
-                                split_pair(xielu_act(__uint_as_float(v[j + 2 * e]), act_a, act_b), xielu_act(__uint_as_float(v[j + 2 * e + 1]), act_a, act_b), bf16, ph[e], pl[e]);
+                            for (int e = 0; e < 4; e++) {
+                                const float z0 = __uint_as_float(v[j + 2 * e]), z1 = __uint_as_float(v[j + 2 * e + 1]);
+                                if (MODE == MODE_XIELU) split_pair(xielu_act(z0, act_a, act_b), xielu_act(z1, act_a, act_b), bf16, ph[e], pl[e]);
+                                else { const float r0 = fmaxf(z0, 0.f), r1 = fmaxf(z1, 0.f); split_pair(r0 * r0, r1 * r1, bf16, ph[e], pl[e]); }
+                            }
                             *reinterpret_cast<uint4*>(hi + j) = make_uint4(ph[0], ph[1], ph[2], ph[3]);
                             *reinterpret_cast<uint4*>(lo + j) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
                         }
@@ -525,6 +529,15 @@ bool gemm_f16_tc_xielu_ws(void* workspace_out, const void* workspace_in, const v
     __half* out = static_cast<__half*>(workspace_out);
     return N % 256 == 0 ? launch_gemm<256, MODE_XIELU>(nullptr, out, workspace_in, W_f16, nullptr, M, Mp, N, K, s, o)
                         : launch_gemm<128, MODE_XIELU>(nullptr, out, workspace_in, W_f16, nullptr, M, Mp, N, K, s, o);
+}
+
+// workspace_out <- split(relu(A.W^T)^2); N % 8 == 0
+bool gemm_f16_tc_relu2_ws(void* workspace_out, const void* workspace_in, const void* W_f16, int M, int N, int K, cudaStream_t s, const TcOpts& o) {
+    if (M <= 0 || N % 8 != 0 || !gemm_f16_tc_ragged_supported(W_f16, N, K, 0)) return false;
+    const size_t Mp = ((size_t)M + BM - 1) / BM * BM;
+    __half* out = static_cast<__half*>(workspace_out);
+    return N % 256 == 0 ? launch_gemm<256, MODE_RELU2>(nullptr, out, workspace_in, W_f16, nullptr, M, Mp, N, K, s, o)
+                        : launch_gemm<128, MODE_RELU2>(nullptr, out, workspace_in, W_f16, nullptr, M, Mp, N, K, s, o);
 }
 
 // ---- grouped rows (routed experts) ----
