@@ -1047,6 +1047,59 @@ def run_family_compare_fuvozen(args):
                       "dtype": "bf16 weights, f32 activations", "data": "synthetic", "rows": rows}))
 
 
+# width -> latent attention (shared by both models), matrix memory against WKV of equal state volume, grouped-query attention, experts
+TIBELIX_SIZES = {
+    "w2048": dict(width=2048, latent=dict(dim=64, rot_dim=64, kv_rank=256), l_heads=16, vdim=128, q_rank=768, m_heads=8, m_dim=128, w_heads=32, w_dim=64, decay_rank=64,
+                  heads=16, kv_heads=4, experts=16, eff=1408),
+    "w4096": dict(width=4096, latent=dict(dim=64, rot_dim=64, kv_rank=512), l_heads=32, vdim=128, q_rank=1536, m_heads=16, m_dim=128, w_heads=64, w_dim=64, decay_rank=128,
+                  heads=32, kv_heads=8, experts=16, eff=1536),
+}
+
+
+def tibelix_pair(z, vocab, mixers=("mlstm", "latent_attention")):
+    """(Tibelix, Fuvozen) configurations of one size: recurrence + dense feed-forward, attention + experts, twice.  Equal width, latent heads and
+    ranks, feed-forward widths and experts; the recurrences' states hold equally many numbers (heads x 128 x 128 against 4 heads x 64 x 64)."""
+    from ntransformer_b200.model_spec import fuvozen_config, tibelix_config
+
+    w = z["width"]
+    tc = tibelix_config(vocab=vocab, width=w, pattern=mixers * 2, l_heads=z["l_heads"], l_dim=z["latent"]["dim"], rot_dim=z["latent"]["rot_dim"], l_vdim=z["vdim"],
+                        kv_rank=z["latent"]["kv_rank"], q_rank=z["q_rank"], m_heads=z["m_heads"], m_dim=z["m_dim"], m_vdim=z["m_dim"], heads=z["heads"], kv_heads=z["kv_heads"],
+                        ff=3 * w, experts=z["experts"], top=3, eff=z["eff"], shared=z["eff"])
+    fc = fuvozen_config(vocab=vocab, width=w, heads=z["l_heads"], vdim=z["vdim"], w_heads=z["w_heads"], w_dim=z["w_dim"], decay_rank=z["decay_rank"], ff=3 * w,
+                        experts=z["experts"], top=3, eff=z["eff"], shared=z["eff"], window=0, **z["latent"])
+    return tc, fc
+
+
+def run_family_compare_tibelix(args):
+    """--family-compare --family tibelix: prompt-pass and decode throughput of the Tibelix family (BF16 weights; matrix memories alternating with
+    latent attention or with distance-biased attention, norms in front of and behind each sublayer, experts with a shared one) beside the closest
+    existing family (Fuvozen: WKV time mixers alternating with latent attention, experts with a shared one) at equal width, layer count, heads,
+    latent rank, recurrent state and feed-forward weights."""
+    import torch
+    from ntransformer_b200.engine import Model
+    from ntransformer_b200.model_spec import fuvozen_random_tensors, tibelix_random_tensors
+
+    torch.cuda.set_device(0)
+    vocab, prompt_len, max_seq = 32000, 2048, 4096
+    hbm, hbm_src = measured_peak_hbm()
+    rows = []
+    for name, z in TIBELIX_SIZES.items():
+        tc, fc = tibelix_pair(z, vocab)
+        ac, _ = tibelix_pair(z, vocab, ("mlstm", "attention"))
+        row = {"size": name, "layers": 4, "prompt_tokens": prompt_len, "decode_context": prompt_len}
+        for label, make in (("tibelix_bf16", lambda: Model.from_config_json(tc, tibelix_random_tensors(tc), max_context=max_seq)),
+                            ("tibelix_biased_attention_bf16", lambda: Model.from_config_json(ac, tibelix_random_tensors(ac), max_context=max_seq)),
+                            ("fuvozen_bf16", lambda: Model.from_config_json(fc, fuvozen_random_tensors(fc), max_context=max_seq))):
+            model = make()
+            row[label] = time_family_model(model, args, prompt_len, vocab, hbm)
+            model.close()
+            del model
+            torch.cuda.empty_cache()
+        rows.append(row)
+    print(json.dumps({"metric": "family_compare", "family": "tibelix", "unit": "tok/s", "hbm_peak_gbs": hbm, "hbm_peak_source": hbm_src,
+                      "dtype": "bf16 weights, f32 activations", "data": "synthetic", "rows": rows}))
+
+
 def run_family_compare(args):
     """--family-compare: prompt-pass and decode throughput of the Zelunex family (BF16 weights, windowed attention) beside the
     closest GGUF family member (Llama block, F16 weights, full causal attention) at equal layer sizes.  Device-timed with CUDA
@@ -1123,8 +1176,8 @@ def main():
     ap.add_argument("--all-errs", action="store_true", help="--check only: list the error of every step, not the first 8")
     ap.add_argument("--family-compare", action="store_true",
                     help="instead of the workload: Zelunex beside the Llama block at equal layer sizes, prompt pass and decode (1 GPU)")
-    ap.add_argument("--family", default="zelunex", choices=["zelunex", "vebotar", "tanolorn", "savidra", "fuvozen"],
-                    help="--family-compare only: zelunex beside the Llama block (default), vebotar beside zelunex, tanolorn beside vebotar, or savidra / fuvozen beside tanolorn")
+    ap.add_argument("--family", default="zelunex", choices=["zelunex", "vebotar", "tanolorn", "savidra", "fuvozen", "tibelix"],
+                    help="--family-compare only: zelunex beside the Llama block (default), vebotar beside zelunex, tanolorn beside vebotar, savidra / fuvozen beside tanolorn, or tibelix beside fuvozen")
     ap.add_argument("--per-token-prompt", action="store_true", help="--check only: our engine replays the prompt token by token like the reference")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
@@ -1135,7 +1188,7 @@ def main():
     if args.family_compare:
         if rank == 0:
             {"vebotar": run_family_compare_vebotar, "tanolorn": run_family_compare_tanolorn, "savidra": run_family_compare_savidra,
-             "fuvozen": run_family_compare_fuvozen}.get(args.family, run_family_compare)(args)
+             "fuvozen": run_family_compare_fuvozen, "tibelix": run_family_compare_tibelix}.get(args.family, run_family_compare)(args)
     elif args.check:
         run_check(args, rank, world)
     elif args.impl == "reference":

@@ -160,6 +160,41 @@ int nt_b200_attention_rows_window(float* out, const float* Q, const void* cache,
 void nt_b200_attention_heads_window(float* out, const float* Q, const void* k, const void* v, int tokens, int p0, int rows, int heads, int kw, int vw, float scale,
                                     int window, void* stream);
 
+/* ---- kernels of the Tibelix family (norms around a sublayer, attention with distance bias and unit sink, long-context latent rotation, matrix memory); F32 unless a dtype is given ---- */
+/* x += rms(y) * gain_y (y null: x as it is); h = rms(x) * gain_h -> h and / or the BF16 split (gain_h null: x only) */
+void nt_b200_sandwich_norm_rows(float* x, const float* y, const float* gain_y, const float* gain_h, float* h, void* split, int rows, int width, float eps, void* stream);
+void nt_b200_sigmoid_gate_rows(float* out, void* split, const float* o, const float* gate, int ld, int per, int rows, int cols, void* stream);
+void nt_b200_relu2_rows(float* out, void* split, const float* in, int rows, int cols, void* stream);
+/* Queries and keys over their root mean square per head, queries times 1 + coef ln(floor((p + 1) / every) + 1) (every 0: off); K null: queries only */
+void nt_b200_head_prep_unit(float* Q, const float* K, const float* V, int heads, int kv_heads, int dim, int vdim, float eps, float coef, double every, void* kc, void* vc,
+                            int cache_dtype, int tokens, int p0, void* stream);
+/* Causal grouped-query attention with a distance bias (slopes [heads] or null), a per-head sink (or null) and an output gate (raw [tokens, heads] or null) */
+void nt_b200_attention_biased(float* out, const float* Q, const void* kc, const void* vc, int cache_dtype, int tokens, int p0, int max_seq, int heads, int kv_heads, int dim,
+                              int vdim, float scale, const float* slopes, const float* sink, const float* gate, void* stream);
+/* The latent attention's cache rows and absorbed queries with a frequency table (freq: device, dims / 2 doubles; host side: nt_b200_rotary_table64) */
+double nt_b200_rotary_table64(double* freq_host, int dims, double base, double factor, double original, double fast, double slow);
+void nt_b200_latent_rotated(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache, int cache_dtype,
+                            int dims, int interleaved, const double* freq, float mag, int tokens, int p0, float* qa, const float* q, const void* W_uk, int dtype, int heads, int dim,
+                            float* q_padded, int kw, void* stream);
+void nt_b200_latent_v_up_gated(float* out, const float* ol, const void* W_uv, int dtype, int tokens, int heads, int vdim, int kv_rank, const float* gate, void* stream);
+/* Router whose weights are the chosen experts' share of the softmax; groups > 0: chosen inside the `keep` runs of neighbours with the largest score.
+ * choose_up: one token's choice from its logits, then silu(gate) * up of the chosen experts -> act [top * ff] */
+void nt_b200_moe_route_shares(int* sel, float* wt, const float* h, const float* router, int experts, int top, int groups, int keep, int width, int tokens, void* stream);
+void nt_b200_moe_choose_up_shares(float* act, int* sel, float* wt, const float* h, const float* logits, const void* const* gate_tab, const void* const* up_tab, int dtype, int experts,
+                                  int top, int groups, int keep, int ff, int width, void* stream);
+void nt_b200_mlstm_gates(float* a, float* b, float* em, const float* zi, const float* zf, int ld, const float* bi, const float* bf, float cap, float* m, int tokens, int heads, int p0,
+                         void* stream);
+/* scratch (may be null): nt_b200_mlstm_scratch_floats numbers, with which long steps run as segments side by side */
+void nt_b200_mlstm_rows(float* o, float* den, const float* q, const float* k, const float* v, const float* a, const float* b, float* state, float q_scale, int tokens, int heads, int dim,
+                        int vdim, int p0, float* scratch, void* stream);
+long long nt_b200_mlstm_scratch_floats(int heads, int dim, int vdim);
+void nt_b200_mlstm_out_norm(float* out, void* split, const float* o, const float* den, const float* em, const float* gate, const float* norm, float eps, int tokens, int heads, int vdim,
+                            void* stream);
+void nt_b200_mlstm_token(float* out, const float* q, const float* k, const float* v, const float* gate, const float* zi, const float* zf, const float* bi, const float* bf,
+                         const float* norm, float* state, float* m, float cap, float q_scale, float eps, int heads, int dim, int vdim, int p0, void* stream);
+/* The tensor-core GEMM with relu(z)^2 in its epilogue: split_out <- split(relu(A W^T)^2) from BF16 W and F32 A (workspace: the split of A).  -1: shape not covered */
+int nt_b200_gemm_relu2(void* split_out, const float* A, const void* W, int M, int N, int K, void* workspace, void* stream);
+
 /* forward(tokens[seq_len], start_pos): logits of the last token. logits_host may be NULL.  Returns 0. */
 int  nt_model_forward(nt_model_t m, const int* tokens_host, int seq_len, int start_pos, float* logits_host);
 /* asynchronous launch only (no sync, no copy); nt_model_sync waits for the model's stream */

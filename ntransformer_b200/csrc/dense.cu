@@ -474,7 +474,7 @@ void gemv_dense(const GemvMat* mats, int n_mat, int K, const float* x, DenseEpil
     int grid = (total + DV_WARPS - 1) / DV_WARPS;
     const int resident = (int)std::max<size_t>(1, std::min<size_t>(8, (size_t)(220 * 1024) / (smem + 1024))) * 148;
     grid = std::min(grid, resident);
-#define NT_DV(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(gemv_dense_kernel<TY>, 200 * 1024, done); \
+#define NT_DV(TY) { static unsigned long long done = 0; if (smem > 40 * 1024) opt_in_dynamic_smem(gemv_dense_kernel<TY>, 200 * 1024, done); \
                     launch_k(gemv_dense_kernel<TY>, dim3(grid), dim3(DV_WARPS * 32), smem, s, m, x, K, (int)ep, row_scale, alpha, vec, norm_w, eps, sio, norm_groups); }
     if (dt == DType::F32) NT_DV(float) else if (dt == DType::F16) NT_DV(__half) else NT_DV(__nv_bfloat16)
 #undef NT_DV
@@ -512,7 +512,7 @@ void gemv_multi(const MultiMat* mats, int n_mat, cudaStream_t s) {
         end += std::max(1, std::min(full, share));
         md.m[i].cta_end = end;
     }
-#define NT_MV(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(gemv_multi_kernel<TY>, 200 * 1024, done); \
+#define NT_MV(TY) { static unsigned long long done = 0; if (smem > 40 * 1024) opt_in_dynamic_smem(gemv_multi_kernel<TY>, 200 * 1024, done); \
                     launch_k(gemv_multi_kernel<TY>, dim3(end), dim3(DV_WARPS * 32), smem, s, md); }
     if (dt == DType::F32) NT_MV(float) else if (dt == DType::F16) NT_MV(__half) else NT_MV(__nv_bfloat16)
 #undef NT_MV
@@ -542,7 +542,7 @@ void gemv_sum(float* y, const SumTerm* terms, int n, int out, DType dt, bool add
     sd.nw = 1;
     while (sd.nw < 4 && (long)out * sd.nw * 2 <= (long)148 * per_sm * SV_WARPS) sd.nw *= 2;
     const int rows = SV_WARPS / sd.nw, grid = std::min((out + rows - 1) / rows, 148 * per_sm);
-#define NT_SV(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(gemv_sum_kernel<TY>, 200 * 1024, done); \
+#define NT_SV(TY) { static unsigned long long done = 0; if (smem > 40 * 1024) opt_in_dynamic_smem(gemv_sum_kernel<TY>, 200 * 1024, done); \
                     launch_k(gemv_sum_kernel<TY>, dim3(grid), dim3(SV_WARPS * 32), smem, s, sd); }
     if (dt == DType::F32) NT_SV(float) else if (dt == DType::F16) NT_SV(__half) else NT_SV(__nv_bfloat16)
 #undef NT_SV

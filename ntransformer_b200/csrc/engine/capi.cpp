@@ -129,6 +129,17 @@ int nt_model_dir_describe(const char* dir, char* out, size_t cap) {
                     " route_scale=" + std::to_string(L.route.scale) + " shared_ff=" + std::to_string(L.shared_ff) + " norm_groups=" + std::to_string(cfg.norm_groups) +
                     " buckets=" + std::to_string(cfg.bigram_buckets);
         }
+        if (L.form == BlockForm::SANDWICH) {
+            if (L.mixer == MixerKind::ATTN_LATENT)
+                text += " mixer=latent q_rank=" + std::to_string(L.latent.q_rank) + " kv_rank=" + std::to_string(L.latent.kv_rank) + " rot_dim=" + std::to_string(L.latent.rot_dim) +
+                        " rot=" + std::to_string(L.rot.dims) + " factor=" + std::to_string(L.rot.factor);
+            else if (L.mixer == MixerKind::MLSTM) text += " mixer=mlstm cap=" + std::to_string(L.mlstm.gate_cap);
+            else
+                text += " mixer=attention temp=" + std::to_string(L.q_temp.coef) + "/" + std::to_string(L.q_temp.every) + " kv_from=" + std::to_string(L.kv_from) + " bias=" +
+                        std::to_string(L.distance_bias) + " unit_sink=" + std::to_string(L.unit_sink);
+            text += std::string(" ff_kind=") + (L.ff == 0 ? "none" : L.ff_kind == FfKind::MLP ? "dense" : "moe") + " experts=" + std::to_string(L.experts) + " top=" + std::to_string(L.top) +
+                    " route_groups=" + std::to_string(L.route.groups) + "/" + std::to_string(L.route.keep) + " shared_ff=" + std::to_string(L.shared_ff);
+        }
         if (L.form == BlockForm::SUM_NORM) {
             auto mixer_text = [](const LayerSpec& M) {
                 if (M.mixer == MixerKind::DELTA_RULE)
@@ -535,6 +546,89 @@ int nt_b200_attention_rows_window(float* out, const float* Q, const void* cache,
 void nt_b200_attention_heads_window(float* out, const float* Q, const void* k, const void* v, int tokens, int p0, int rows, int heads, int kw, int vw, float scale,
                                     int window, void* stream) {
     attention_heads_mma(out, Q, k, v, tokens, p0, rows, heads, kw, vw, scale, static_cast<cudaStream_t>(stream), window);
+}
+// ---- kernels of the Tibelix family ----
+// x += rms(y) * gain_y (y null: x as it is); h = rms(x) * gain_h -> h and / or the BF16 split (gain_h null: x only)
+void nt_b200_sandwich_norm_rows(float* x, const float* y, const float* gain_y, const float* gain_h, float* h, void* split, int rows, int width, float eps, void* stream) {
+    sandwich_norm_rows(x, y, gain_y, gain_h, h, split, rows, width, eps, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_sigmoid_gate_rows(float* out, void* split, const float* o, const float* gate, int ld, int per, int rows, int cols, void* stream) {
+    sigmoid_gate_rows(out, split, o, gate, ld, per, rows, cols, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_relu2_rows(float* out, void* split, const float* in, int rows, int cols, void* stream) {
+    relu2_rows(out, split, in, rows, cols, static_cast<cudaStream_t>(stream));
+}
+// Queries and keys over their root mean square per head, queries times 1 + coef ln(floor((p + 1) / every) + 1) (every 0: off); K null: queries only
+void nt_b200_head_prep_unit(float* Q, const float* K, const float* V, int heads, int kv_heads, int dim, int vdim, float eps, float coef, double every, void* kc, void* vc,
+                            int cache_dtype, int tokens, int p0, void* stream) {
+    HeadPrep p;
+    p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.eps = eps; p.unit_norm = 1; p.temp_coef = coef; p.temp_every = every;
+    head_prep(Q, K, V, p, kc, vc, (nt::DType)cache_dtype, tokens, nullptr, p0, static_cast<cudaStream_t>(stream));
+}
+// Causal grouped-query attention with a distance bias (slopes [heads] or null), a per-head sink (or null) and an output gate (raw [tokens, heads] or null)
+void nt_b200_attention_biased(float* out, const float* Q, const void* kc, const void* vc, int cache_dtype, int tokens, int p0, int max_seq, int heads, int kv_heads, int dim,
+                              int vdim, float scale, const float* slopes, const float* sink, const float* gate, void* stream) {
+    WindowAttn a;
+    a.heads = heads; a.kv_heads = kv_heads; a.dim = dim; a.vdim = vdim; a.scale = scale; a.slope = slopes; a.sink = sink; a.head_gate = gate; a.gate_stride = heads;
+    attention_window(out, Q, kc, vc, (nt::DType)cache_dtype, tokens, nullptr, p0, max_seq, a, static_cast<cudaStream_t>(stream));
+}
+// The latent attention's cache rows and absorbed queries with a frequency table (freq: device, dims / 2 doubles; host side: nt_b200_rotary_table64)
+double nt_b200_rotary_table64(double* freq_host, int dims, double base, double factor, double original, double fast, double slow) {
+    return rotary_table(freq_host, dims, base, factor, original, fast, slow);
+}
+void nt_b200_latent_rotated(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache, int cache_dtype,
+                            int dims, int interleaved, const double* freq, float mag, int tokens, int p0, float* qa, const float* q, const void* W_uk, int dtype, int heads, int dim,
+                            float* q_padded, int kw, void* stream) {
+    LatentRot r;
+    r.dims = dims; r.interleaved = interleaved != 0; r.freq = freq; r.mag = mag;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    latent_prep(cq, q_rank, q_gain, dkv, kv_rank, rot_dim, kv_gain, eps, cache, (nt::DType)cache_dtype, r, tokens, nullptr, p0, s);
+    if (qa) latent_q_absorb(qa, q, W_uk, (nt::DType)dtype, tokens, heads, dim, rot_dim, kv_rank, r, nullptr, p0, s);
+    if (q_padded) latent_q_rot_pad(q_padded, q, tokens, heads, dim, rot_dim, kw, r, p0, s);
+}
+void nt_b200_latent_v_up_gated(float* out, const float* ol, const void* W_uv, int dtype, int tokens, int heads, int vdim, int kv_rank, const float* gate, void* stream) {
+    latent_v_up(out, ol, W_uv, (nt::DType)dtype, tokens, heads, vdim, kv_rank, static_cast<cudaStream_t>(stream), gate);
+}
+// Router whose weights are the chosen experts' share of the softmax; groups > 0: chosen inside the `keep` runs of neighbours with the largest score.
+// choose_up: one token's choice from its logits, then silu(gate) * up of the chosen experts -> act [top * ff]
+void nt_b200_moe_route_shares(int* sel, float* wt, const float* h, const float* router, int experts, int top, int groups, int keep, int width, int tokens, void* stream) {
+    MoeWeights w;
+    w.router = router; w.experts = experts; w.top = top; w.width = width; w.all = true; w.renorm = true; w.groups = groups; w.keep = keep;
+    moe_route(sel, wt, nullptr, h, w, tokens, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_moe_choose_up_shares(float* act, int* sel, float* wt, const float* h, const float* logits, const void* const* gate_tab, const void* const* up_tab, int dtype, int experts,
+                                  int top, int groups, int keep, int ff, int width, void* stream) {
+    MoeWeights w;
+    w.gate = gate_tab; w.up = up_tab; w.dtype = (nt::DType)dtype; w.experts = experts; w.top = top; w.ff = ff; w.width = width; w.all = true; w.renorm = true; w.groups = groups; w.keep = keep;
+    moe_expert_up_token(act, h, nullptr, w, static_cast<cudaStream_t>(stream), logits, sel, wt);
+}
+void nt_b200_mlstm_gates(float* a, float* b, float* em, const float* zi, const float* zf, int ld, const float* bi, const float* bf, float cap, float* m, int tokens, int heads, int p0,
+                         void* stream) {
+    mlstm_gates(a, b, em, zi, zf, ld, bi, bf, cap, m, tokens, heads, nullptr, p0, static_cast<cudaStream_t>(stream));
+}
+// scratch (may be null): nt_b200_mlstm_scratch_floats numbers, with which long steps run as segments side by side
+void nt_b200_mlstm_rows(float* o, float* den, const float* q, const float* k, const float* v, const float* a, const float* b, float* state, float q_scale, int tokens, int heads, int dim,
+                        int vdim, int p0, float* scratch, void* stream) {
+    mlstm_rows(o, den, q, k, v, a, b, state, q_scale, tokens, heads, dim, vdim, nullptr, p0, static_cast<cudaStream_t>(stream), scratch);
+}
+long long nt_b200_mlstm_scratch_floats(int heads, int dim, int vdim) {
+    return (long long)mlstm_rows_scratch_floats(heads, dim, vdim);
+}
+void nt_b200_mlstm_out_norm(float* out, void* split, const float* o, const float* den, const float* em, const float* gate, const float* norm, float eps, int tokens, int heads, int vdim,
+                            void* stream) {
+    mlstm_out_norm(out, split, o, den, em, gate, norm, eps, tokens, heads, vdim, static_cast<cudaStream_t>(stream));
+}
+void nt_b200_mlstm_token(float* out, const float* q, const float* k, const float* v, const float* gate, const float* zi, const float* zf, const float* bi, const float* bf,
+                         const float* norm, float* state, float* m, float cap, float q_scale, float eps, int heads, int dim, int vdim, int p0, void* stream) {
+    mlstm_token(out, q, k, v, gate, zi, zf, bi, bf, norm, state, m, cap, q_scale, eps, heads, dim, vdim, nullptr, p0, static_cast<cudaStream_t>(stream));
+}
+// The tensor-core GEMM with relu(z)^2 in its epilogue: split_out <- split(relu(A W^T)^2) from BF16 W and F32 A (workspace: the split of A).  -1: shape not covered
+int nt_b200_gemm_relu2(void* split_out, const float* A, const void* W, int M, int N, int K, void* workspace, void* stream) {
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    TcOpts o;
+    o.bf16 = true;
+    split_activations(workspace, A, M, K, s, true);
+    return gemm_f16_tc_relu2_ws(split_out, workspace, W, M, N, K, s, o) ? 0 : -1;
 }
 void nt_b200_glu_mul(float* out, const float* gate, const float* up, long long n, int gelu, void* stream) {
     glu_mul(out, gate, up, (size_t)n, gelu != 0, static_cast<cudaStream_t>(stream));

@@ -459,7 +459,9 @@ inline void launch_k(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t sme
     at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     at[0].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
     cfg.attrs = at; cfg.numAttrs = 1;
-    NT_CUDA_CHECK(cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...));
+    const cudaError_t rc = cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+    if (rc != cudaSuccess) fprintf(stderr, "launch of grid (%u, %u, %u), block %u, %zu bytes of shared memory:\n", grid.x, grid.y, grid.z, block.x, smem);
+    NT_CUDA_CHECK(rc);
 }
 
 // prefill_gemm.cu: tcgen05/TMEM GEMM, C[M,N] = A[M,K] (F32, split hi+lo F16) . W[N,K]^T (F16)

@@ -497,7 +497,7 @@ void mlstm_token(float* out, const float* q, const float* k, const float* v, con
     while (splits < MT_MAX_SPLITS && splits * heads < 148 && vdim >= 64 * splits) splits *= 2;
     const int per = (vdim + splits - 1) / splits;
     const size_t smem = sizeof(float) * (3 * (size_t)((dim + 3) & ~3) + (size_t)per);
-    NT_CHECK(smem <= 48 * 1024, "mlstm_token: the head does not fit in shared memory");
+    NT_CHECK(smem <= 47 * 1024, "mlstm_token: the head does not fit in shared memory");
     const int dv = dim % 4 || !aligned16({state}) ? 0 : dim <= 32 ? 1 : dim <= 64 ? 2 : dim <= 128 ? 4 : dim <= 256 ? 8 : 16;
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(splits, heads); cfg.blockDim = dim3(256); cfg.dynamicSmemBytes = smem; cfg.stream = s;

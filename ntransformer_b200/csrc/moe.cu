@@ -563,7 +563,7 @@ void moe_expert_up_token(float* act, const float* h, const int* sel, const MoeWe
     const size_t smem = (size_t)w.width * sizeof(float);
     NT_CHECK(smem <= 200 * 1024, "moe: the activation row does not fit in shared memory");
     const int grid = std::min((total + TK_WARPS - 1) / TK_WARPS, 148 * 8);
-#define NT_CALL(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(moe_up_token_kernel<TY>, 200 * 1024, done); \
+#define NT_CALL(TY) { static unsigned long long done = 0; if (smem > 40 * 1024) opt_in_dynamic_smem(moe_up_token_kernel<TY>, 200 * 1024, done); \
                       launch_k(moe_up_token_kernel<TY>, dim3(grid), dim3(TK_WARPS * 32), smem, s, act, h, sel, m, logits, sel_out, wt_out); }
     NT_MOE_DT(NT_CALL)
 #undef NT_CALL
@@ -577,7 +577,7 @@ void moe_expert_down_token(float* y, const float* act, const int* sel, const flo
     const size_t smem = (size_t)(m.top * m.ff + m.shared_ff) * sizeof(float);
     NT_CHECK(smem <= 200 * 1024, "moe: the chosen experts' activations do not fit in shared memory");
     const int grid = std::min((w.width + TK_WARPS - 1) / TK_WARPS, 148 * 8);
-#define NT_CALL(TY) { static unsigned long long done = 0; if (smem > 48 * 1024) opt_in_dynamic_smem(moe_down_token_kernel<TY>, 200 * 1024, done); \
+#define NT_CALL(TY) { static unsigned long long done = 0; if (smem > 40 * 1024) opt_in_dynamic_smem(moe_down_token_kernel<TY>, 200 * 1024, done); \
                       launch_k(moe_down_token_kernel<TY>, dim3(grid), dim3(TK_WARPS * 32), smem, s, y, act, sel, wt, sgate, m, sio); }
     NT_MOE_DT(NT_CALL)
 #undef NT_CALL

@@ -504,3 +504,89 @@ def fuvozen_random_tensors(config: dict, seed: int = 1234, device="cuda", dtype=
                 t[p + "mlp." + x + ".gate"], t[p + "mlp." + x + ".up"], t[p + "mlp." + x + ".down"] = mat(w, W), mat(w, W), mat(W, w)
         t[p + "dwa"] = torch.cat([uni(i + 1, -0.1, 0.2), uni(1, 0.9, 1.1)])
     return t
+
+
+# ---- Tibelix (layer-spec family, model folders): synthetic configurations and random device weights for benchmarks ----
+def tibelix_config(vocab=32000, width=2048, pattern=("mlstm", "latent_attention", "mlstm", "attention"), mlp=("dense", "moe", "dense", "moe"), kv_from=None, eps=1e-6,
+                   heads=16, kv_heads=4, dim=128, vdim=128, temp=(0.1, 4096), l_heads=16, l_dim=64, rot_dim=64, l_vdim=128, q_rank=768, kv_rank=256, rot_base=10000.0,
+                   scaling=(4.0, 4096, 32.0, 1.0), m_heads=8, m_dim=128, m_vdim=128, cap=15.0, ff=6144, experts=16, top=3, groups=(4, 2), eff=1408, shared=1408):
+    """The family's config.json as a dict.  pattern: mixer type per layer; mlp: feed-forward kind per layer ("dense", "moe" or None); kv_from: {layer:
+    earlier attention layer whose cache rows it reads}; temp (coefficient, every), scaling (factor, original, fast, slow) and groups (count, keep) may
+    be None; shared: width of the shared expert (0: none)."""
+    kv_from = kv_from or {}
+    layers = []
+    for i, typ in enumerate(pattern):
+        if typ == "attention":
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5}
+            if temp:
+                m["q_temp"] = {"coef": temp[0], "every": temp[1]}
+            if i in kv_from:
+                m["kv_from"] = kv_from[i]
+        elif typ == "latent_attention":
+            m = {"heads": l_heads, "dim": l_dim, "rot_dim": rot_dim, "vdim": l_vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": (l_dim + rot_dim) ** -0.5,
+                 "rot": {"base": rot_base, "dims": rot_dim}}
+            if scaling:
+                m["rot"]["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+        else:
+            m = {"heads": m_heads, "dim": m_dim, "vdim": m_vdim, "gate_cap": cap}
+        k = mlp[i % len(mlp)]
+        if k == "dense":
+            f = {"kind": "dense", "ff": ff}
+        elif k == "moe":
+            f = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": experts, "top": top}}
+            if groups:
+                f["router"]["groups"] = {"count": groups[0], "keep": groups[1]}
+            if shared:
+                f["shared"] = {"ff": shared}
+        else:
+            f = None
+        layers.append({"type": typ, "mixer": m, "mlp": f})
+    return {"architecture": "Tibelix", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+
+
+def tibelix_random_tensors(config: dict, seed: int = 1234, device="cuda", dtype=None):
+    """Checkpoint name -> random CUDA tensor (matrices and embedding `dtype`, default bfloat16; gains, gate biases and router rows float32)."""
+    import torch
+
+    dtype = dtype or torch.bfloat16
+    g = torch.Generator(device=device)
+    g.manual_seed(seed)
+    W = config["width"]
+
+    def mat(rows, cols, dt=dtype):
+        return (torch.randn(rows, cols, generator=g, device=device, dtype=torch.float32) * cols ** -0.5).to(dt)
+
+    def vec(n, mean=0.0, std=0.1):
+        return mean + std * torch.randn(n, generator=g, device=device, dtype=torch.float32)
+
+    t = {"embed": mat(config["vocab"], W) * W ** 0.5, "final.norm": vec(W)}
+    for i, e in enumerate(config["layers"]):
+        m, p = e["mixer"], "l%d." % i
+        q, H, D, V = p + "mix.", m["heads"], m["dim"], m["vdim"]
+        t[p + "norm1"], t[p + "norm1b"] = vec(W), vec(W)
+        if e["type"] == "latent_attention":
+            R, r = m["rot_dim"], m["kv_rank"]
+            t[q + "dq"], t[q + "dq.norm"], t[q + "uq"] = mat(m["q_rank"], W), vec(m["q_rank"], 1.0), mat(H * (D + R), m["q_rank"])
+            t[q + "dkv"], t[q + "dkv.norm"] = mat(r + R, W), vec(r, 1.0)
+            t[q + "uk"], t[q + "uv"] = mat(H * D, r), mat(H * V, r)
+        else:
+            G = m.get("kv_heads", H)
+            t[q + "q"] = mat(H * D, W)
+            if "kv_from" not in m:
+                t[q + "k"], t[q + "v"] = mat(G * D, W), mat(G * V, W)
+        t[q + "g"] = mat(H if e["type"] == "attention" else H * V, W)
+        if e["type"] == "mlstm":
+            t[q + "i"], t[q + "f"] = mat(H, W), mat(H, W)
+            t[q + "i.b"], t[q + "f.b"], t[q + "norm"] = vec(H, -2.0, 1.0), vec(H, 4.0, 1.0), vec(H * V, 1.0)
+        t[q + "o"] = mat(W, H * V)
+        f = e.get("mlp")
+        if f:
+            t[p + "norm2"], t[p + "norm2b"] = vec(W), vec(W)
+        if f and f["kind"] == "dense":
+            t[p + "mlp.up"], t[p + "mlp.down"] = mat(f["ff"], W), mat(W, f["ff"])
+        elif f:
+            t[p + "mlp.router"] = mat(f["router"]["experts"], W, torch.float32)
+            for x in ["e%d" % n for n in range(f["router"]["experts"])] + (["shared"] if f.get("shared") else []):
+                w = f["shared"]["ff"] if x == "shared" else f["expert"]["ff"]
+                t[p + "mlp." + x + ".gate"], t[p + "mlp." + x + ".up"], t[p + "mlp." + x + ".down"] = mat(w, W), mat(w, W), mat(W, w)
+    return t
