@@ -37,23 +37,26 @@ constexpr float kDenEps = 1e-6f;
 struct MaxPlus { float F, M; };                                     // m -> max(F + m, M)
 __device__ __forceinline__ MaxPlus then(const MaxPlus& a, const MaxPlus& b) { return {a.F + b.F, fmaxf(a.M + b.F, b.M)}; }      // first a, then b
 
-// grid (heads), 256 threads: a thread composes a run of consecutive rows, the runs are scanned over the CTA
-__global__ void __launch_bounds__(256) mlstm_gates_kernel(float* __restrict__ a, float* __restrict__ b, float* __restrict__ em, const float* __restrict__ zi,
+// grid (heads), GT_THREADS threads: the log gates of all rows first (independent loads in flight together), then a thread composes a run of consecutive
+// rows and the runs are scanned over the CTA
+constexpr int GT_THREADS = 512;
+__global__ void __launch_bounds__(GT_THREADS) mlstm_gates_kernel(float* __restrict__ a, float* __restrict__ b, float* __restrict__ em, const float* __restrict__ zi,
                                                           const float* __restrict__ zf, int ld, const float* __restrict__ bi, const float* __restrict__ bf, float cap,
                                                           float* __restrict__ m_state, int T, int heads, const int* __restrict__ pos_dev, int p0) {
-    __shared__ MaxPlus warp_tot[8];
+    __shared__ MaxPlus warp_tot[GT_THREADS / 32];
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int per = (T + 255) / 256, t0 = min(T, (int)threadIdx.x * per), t1 = min(T, t0 + per);
+    const int per = (T + GT_THREADS - 1) / GT_THREADS, t0 = min(T, (int)threadIdx.x * per), t1 = min(T, t0 + per);
     const float m0 = (pos_dev ? *pos_dev : p0) == 0 ? 0.f : m_state[h], bih = bi[h], bfh = bf[h];
     MaxPlus run = {0.f, -INFINITY};                                 // the identity
-    for (int t = t0; t < t1; t++) {
-        const float i = capped(zi[(size_t)t * ld + h] + bih, cap), f = log_sigmoid(capped(zf[(size_t)t * ld + h] + bfh, cap));
-        a[(size_t)t * heads + h] = f;
-        b[(size_t)t * heads + h] = i;
-        run = then(run, {f, i});
+#pragma unroll 4
+    for (int t = threadIdx.x; t < T; t += GT_THREADS) {
+        a[(size_t)t * heads + h] = log_sigmoid(capped(zf[(size_t)t * ld + h] + bfh, cap));
+        b[(size_t)t * heads + h] = capped(zi[(size_t)t * ld + h] + bih, cap);
     }
+    __syncthreads();
+    for (int t = t0; t < t1; t++) run = then(run, {a[(size_t)t * heads + h], b[(size_t)t * heads + h]});
     MaxPlus inc = run;                                              // inclusive scan over the warp, then over the warps
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -68,7 +71,7 @@ __global__ void __launch_bounds__(256) mlstm_gates_kernel(float* __restrict__ a,
     for (int w = 0; w < warp; w++) ahead = then(ahead, warp_tot[w]);
     before = then(ahead, before);
     float m = fmaxf(before.F + m0, before.M);
-    for (int t = t0; t < t1; t++) {                                 // a thread reads back what it wrote itself
+    for (int t = t0; t < t1; t++) {                                 // the run's numbers are this thread's alone by now
         const size_t at = (size_t)t * heads + h;
         const float f = a[at], i = b[at], mn = fmaxf(f + m, i);
         a[at] = expf(f + m - mn);
@@ -449,7 +452,7 @@ void mlstm_gates(float* a, float* b, float* em, const float* zi, const float* zf
                  const int* pos_dev, int p0, cudaStream_t s) {
     if (T <= 0) return;
     NT_CHECK(cap > 0.f, "mlstm_gates: the gates' cap must be positive");
-    launch_k(mlstm_gates_kernel, dim3(heads), dim3(256), 0, s, a, b, em, zi, zf, ld, bi, bf, cap, m, T, heads, pos_dev, p0);
+    launch_k(mlstm_gates_kernel, dim3(heads), dim3(GT_THREADS), 0, s, a, b, em, zi, zf, ld, bi, bf, cap, m, T, heads, pos_dev, p0);
     count_launch();
 }
 

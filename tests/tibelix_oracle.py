@@ -2,7 +2,8 @@
 
 Test infrastructure: nothing under ntransformer_b200/ imports it and it shares no code with the product path.  It keeps no cache and
 no state: every function sees the whole sequence (the matrix memory is a loop over time), so the product's cache, state hand-over and
-schedules are checked against something that cannot have the same fault.
+schedules are checked against something that cannot have the same fault.  `store`, where a function takes it, is applied to whatever the product
+keeps in 16 bits (cache rows, and the per-head keys and values it expands latent rows to): None keeps everything in float64.
 
 Notation.  X is [T, width]; weights are [out, in] and applied as x @ W.T.  `cfg` is the parsed config.json, `P` maps tensor names to
 float64 arrays.
@@ -71,10 +72,14 @@ def softmax_rows(s, mask):
     return e / e.sum(axis=-1, keepdims=True)
 
 
-def attention_kv(h, P, p, m, eps):
+def kept(x, store):
+    return store(x) if store else x
+
+
+def attention_kv(h, P, p, m, eps, store=None):
     """Keys [T, G, dim] (unit root mean square per head) and values [T, G, vdim]."""
     T, G = h.shape[0], m["kv_heads"]
-    return rms((h @ P[p + "k"].T).reshape(T, G, m["dim"]), eps), (h @ P[p + "v"].T).reshape(T, G, m["vdim"])
+    return kept(rms((h @ P[p + "k"].T).reshape(T, G, m["dim"]), eps), store), kept((h @ P[p + "v"].T).reshape(T, G, m["vdim"]), store)
 
 
 def biased_attention(q, k, v, scale, slope):
@@ -131,7 +136,7 @@ def rotate_pairs(v, pos, rot):
     return out
 
 
-def latent_attention(h, P, p, m, eps):
+def latent_attention(h, P, p, m, eps, store=None, expanded=False):
     T = h.shape[0]
     H, D, R, V, r = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
     pos = np.arange(T)
@@ -139,8 +144,10 @@ def latent_attention(h, P, p, m, eps):
     q = (cq @ P[p + "uq"].T).reshape(T, H, D + R)
     qn, qr = q[:, :, :D], rotate_pairs(q[:, :, D:], pos, m.get("rot"))
     d = h @ P[p + "dkv"].T
-    c, kr = norm_plain(d[:, :r], P[p + "dkv.norm"], eps), rotate_pairs(d[:, r:], pos, m.get("rot"))
+    c, kr = kept(norm_plain(d[:, :r], P[p + "dkv.norm"], eps), store), kept(rotate_pairs(d[:, r:], pos, m.get("rot")), store)
     kn, v = (c @ P[p + "uk"].T).reshape(T, H, D), (c @ P[p + "uv"].T).reshape(T, H, V)
+    if expanded:
+        kn, v = kept(kn, store), kept(v, store)
     out = np.zeros((T, H, V))
     for x in range(H):
         s = (qn[:, x] @ kn[:, x].T + qr[:, x] @ kr.T) * m["scale"]
@@ -216,7 +223,7 @@ def moe_ff(h, P, p, mlp):
 
 
 # ---------------------------------------------------------------- model
-def layers(cfg, P, tokens):
+def layers(cfg, P, tokens, store=None, expanded=False):
     """The embedding output, then the residual after every layer."""
     eps = cfg["norm"]["eps"]
     x = P["embed"][np.asarray(tokens)]
@@ -226,10 +233,12 @@ def layers(cfg, P, tokens):
         h = norm_zero(x, P[p + "norm1"], eps)
         if e["type"] == "attention":
             if "kv_from" not in m:
-                kv[i] = attention_kv(h, P, p + "mix.", m, eps)
+                kv[i] = attention_kv(h, P, p + "mix.", m, eps, store)
             y = attention(h, P, p + "mix.", m, eps, kv[m.get("kv_from", i)])
+        elif e["type"] == "latent_attention":
+            y = latent_attention(h, P, p + "mix.", m, eps, store, expanded)
         else:
-            y = (latent_attention if e["type"] == "latent_attention" else mlstm)(h, P, p + "mix.", m, eps)
+            y = mlstm(h, P, p + "mix.", m, eps)
         x = x + norm_zero(y, P[p + "norm1b"], eps)
         f = e.get("mlp")
         if f:
@@ -240,8 +249,8 @@ def layers(cfg, P, tokens):
     return out
 
 
-def forward(cfg, P, tokens):
-    return norm_zero(layers(cfg, P, tokens)[-1], P["final.norm"], cfg["norm"]["eps"]) @ P["embed"].T
+def forward(cfg, P, tokens, store=None, expanded=False):
+    return norm_zero(layers(cfg, P, tokens, store, expanded)[-1], P["final.norm"], cfg["norm"]["eps"]) @ P["embed"].T
 
 
 # ---------------------------------------------------------------- random models
