@@ -192,6 +192,17 @@ void nt_b200_mlstm_out_norm(float* out, void* split, const float* o, const float
                             void* stream);
 void nt_b200_mlstm_token(float* out, const float* q, const float* k, const float* v, const float* gate, const float* zi, const float* zf, const float* bi, const float* bf,
                          const float* norm, float* state, float* m, float cap, float q_scale, float eps, int heads, int dim, int vdim, int p0, void* stream);
+/* One row: x_out = x + rms(y) * gain_y, h = rms(x_out) * gain_h, logits [experts] = router . h.  -1: width not covered */
+int nt_b200_sandwich_norm_router(float* x_out, const float* x, const float* y, const float* gain_y, const float* gain_h, float* h, const float* router, float* logits, int experts,
+                                 int width, float eps, void* stream);
+/* y = W (x / sqrt(mean x^2 + eps) * gain) */
+void nt_b200_gemv_normed(float* y, const void* W, int dtype, const float* x, const float* gain, float eps, int out, int K, void* stream);
+/* One decoded token of the latent attention behind its queries, in three launches: absorbed queries and the cache row, the slices, merge and gated values.
+ * rot: base, no table.  -1: shape not covered.  Scratch is allocated and freed here. */
+int nt_b200_latent_token(float* out, const float* q, const float* dkv, const float* kv_gain, float eps, void* cache, int cache_dtype, const void* W_uk, const void* W_uv, int dtype, int p0,
+                         int max_seq, int heads, int dim, int rot_dim, int vdim, int kv_rank, int rot_dims, float rot_base, float scale, const float* gate, void* stream);
+/* C[i] [M, N[i]] = A W[i]^T for n BF16 matrices in one launch (workspace: the split of A).  -1: shape not covered */
+int nt_b200_gemm_multi(float* const* C, const float* A, const void* const* W, const int* N, int n, int M, int K, void* workspace, void* stream);
 /* The tensor-core GEMM with relu(z)^2 in its epilogue: split_out <- split(relu(A W^T)^2) from BF16 W and F32 A (workspace: the split of A).  -1: shape not covered */
 int nt_b200_gemm_relu2(void* split_out, const float* A, const void* W, int M, int N, int K, void* workspace, void* stream);
 

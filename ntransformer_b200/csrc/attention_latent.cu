@@ -77,6 +77,18 @@ __device__ __forceinline__ float block_sum_256(float v, float* red) {
     return tot;
 }
 
+// One key / value row: the first kv_rank numbers RMS-normed, the rest rotated, into the cache row of its position.  Called by a CTA of 256 threads.
+template <typename KT>
+__device__ __forceinline__ void store_row(const float* __restrict__ r, int kv_rank, int rot_dim, const float* __restrict__ kv_gain, float eps, KT* __restrict__ cache, const RotDev& rot,
+                                          int pos, float* red) {
+    const int row = kv_rank + rot_dim;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < kv_rank; i += 256) ss = fmaf(r[i], r[i], ss);
+    const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)kv_rank + eps);
+    for (int i = threadIdx.x; i < kv_rank; i += 256) cst(cache, (size_t)pos * row + i, r[i] * inv * kv_gain[i]);
+    for (int i = threadIdx.x; i < rot_dim; i += 256) cst(cache, (size_t)pos * row + kv_rank + i, rotated(r + kv_rank, i, rot, pos));
+}
+
 // grid (T, 2): y == 0 the query latent, y == 1 the key / value row; grid (T, 1) without a query latent
 template <typename KT>
 __global__ void __launch_bounds__(256) latent_prep_kernel(float* __restrict__ cq, int q_rank, const float* __restrict__ q_gain, const float* __restrict__ dkv,
@@ -96,25 +108,29 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(float* __restrict__ cq
     }
     if (!dkv) return;
     const int pos = (pos_dev ? *pos_dev : p0) + t;
-    const int row = kv_rank + rot_dim;
-    const float* r = dkv + (size_t)t * row;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < kv_rank; i += 256) ss = fmaf(r[i], r[i], ss);
-    const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)kv_rank + eps);
-    for (int i = threadIdx.x; i < kv_rank; i += 256) cst(cache, (size_t)pos * row + i, r[i] * inv * kv_gain[i]);
-    for (int i = threadIdx.x; i < rot_dim; i += 256) cst(cache, (size_t)pos * row + kv_rank + i, rotated(r + kv_rank, i, rot, pos));
+    store_row(dkv + (size_t)t * (kv_rank + rot_dim), kv_rank, rot_dim, kv_gain, eps, cache, rot, pos, red);
 }
 
 constexpr int LT = 8;      // tokens per CTA in the two per-head products
 
 // grid (ceil(T / LT), heads, ceil(kv_rank / 64)).  q [T, heads, dim + rot_dim]; qa [T, heads, kv_rank + rot_dim]; W_uk [heads * dim, kv_rank].
 // A CTA owns 64 latent channels of a head: thread (r, part) sums every fourth row of W_uk,h for channel r, the four parts meet in
-// shared memory.  One decoded token then has heads * kv_rank / 64 CTAs with short chains instead of `heads` CTAs with long ones.
+// shared memory.  One decoded token then has heads * kv_rank / 64 CTAs with short chains instead of `heads` CTAs with long ones; with a LatentRow one more
+// CTA (y == heads) writes the token's cache row.
 template <typename WT>
 __global__ void __launch_bounds__(256) latent_q_absorb_kernel(float* __restrict__ qa, const float* __restrict__ q, const WT* __restrict__ W_uk, int T, int heads,
                                                               int dim, int rot_dim, int kv_rank, const RotDev rot,
-                                                              const int* __restrict__ pos_dev, int p0) {
+                                                              const int* __restrict__ pos_dev, int p0, const LatentRow lr) {
     extern __shared__ __align__(16) float qs[];           // [LT][dim + rot_dim] | partial sums [4][64][LT]
+    if ((int)blockIdx.y == heads) {
+        pdl_launch_dependents();
+        pdl_wait();
+        if (blockIdx.z != 0) return;
+        const int pos = pos_dev ? *pos_dev : p0;
+        if (lr.cache_dt == DType::F32) store_row(lr.dkv, kv_rank, rot_dim, lr.gain, lr.eps, static_cast<float*>(lr.cache), rot, pos, qs);
+        else store_row(lr.dkv, kv_rank, rot_dim, lr.gain, lr.eps, static_cast<__nv_bfloat16*>(lr.cache), rot, pos, qs);
+        return;
+    }
     if (T == 1) for (int d = threadIdx.x; d < dim; d += 256) l2_prefetch(W_uk + ((size_t)blockIdx.y * dim + d) * kv_rank + blockIdx.z * 64, min(64, kv_rank - (int)blockIdx.z * 64) * sizeof(WT), 0, 1);
     pdl_launch_dependents();
     pdl_wait();
@@ -440,6 +456,56 @@ __global__ void __launch_bounds__(256) latent_shared_merge_kernel(float* __restr
     if (g == 0 && c < vdim) out[((size_t)t * heads + h) * vdim + c] = ((sums[0][cl] + sums[1][cl]) + (sums[2][cl] + sums[3][cl])) / L;
 }
 
+// The merge for one query with the up-projection of the values behind it: grid (1, heads, ceil(v_up / 32)).  Every CTA of a head joins the head's slices
+// itself (they come from L2), then a warp per output channel.
+template <typename WT>
+__global__ void __launch_bounds__(256) latent_merge_up_kernel(float* __restrict__ out, const float* __restrict__ part, int n_slices, int heads, int vdim, const WT* __restrict__ W_uv,
+                                                              int v_up, const float* __restrict__ gate) {
+    extern __shared__ __align__(16) float sm_mu[];         // slice weights [n_slices] | joined vector [vdim]
+    __shared__ float red[8];
+    const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, v0 = blockIdx.z * 32, v1 = min(v_up, v0 + 32);
+    float *wsm = sm_mu, *os = sm_mu + ((n_slices + 3) & ~3);
+    l2_prefetch(W_uv + ((size_t)h * v_up + v0) * vdim, (size_t)(v1 - v0) * vdim * sizeof(WT), threadIdx.x, 256);
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* base = part + (size_t)h * (vdim + 2);
+    const size_t step = (size_t)heads * (vdim + 2);
+    float mx = -FLT_MAX;
+    for (int s = threadIdx.x; s < n_slices; s += 256) mx = fmaxf(mx, base[s * step]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, o));
+    if (lane == 0) red[warp] = mx;
+    __syncthreads();
+    float M = -FLT_MAX;
+#pragma unroll
+    for (int w = 0; w < 8; w++) M = fmaxf(M, red[w]);
+    float ls = 0.f;
+    for (int s = threadIdx.x; s < n_slices; s += 256) { const float w = expf(base[s * step] - M); wsm[s] = w; ls = fmaf(base[s * step + 1], w, ls); }
+    const float inv = 1.0f / block_sum_256(ls, red);       // its barriers also publish wsm
+    for (int c = threadIdx.x; c < vdim; c += 256) {
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        int s = 0;
+#pragma unroll 4
+        for (; s + 4 <= n_slices; s += 4) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) v[e] = fmaf(base[(s + e) * step + 2 + c], wsm[s + e], v[e]);
+        }
+        for (; s < n_slices; s++) v[0] = fmaf(base[s * step + 2 + c], wsm[s], v[0]);
+        os[c] = ((v[0] + v[1]) + (v[2] + v[3])) * inv;
+    }
+    __syncthreads();
+    for (int v = v0 + warp; v < v1; v += 8) {
+        const WT* wr = W_uv + ((size_t)h * v_up + v) * vdim;
+        float acc = 0.f;
+#pragma unroll 8
+        for (int r = lane; r < vdim; r += 32) acc = fmaf(wld(wr, r), os[r], acc);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xFFFFFFFFu, acc, o);
+        const size_t at = (size_t)h * v_up + v;
+        if (lane == 0) out[at] = gate ? acc / (1.0f + expf(-gate[at])) : acc;
+    }
+}
+
 }  // namespace
 
 void latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache,
@@ -457,14 +523,16 @@ void latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, i
 }
 
 void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, const LatentRot& rot,
-                     const int* pos_dev, int p0, cudaStream_t s) {
+                     const int* pos_dev, int p0, cudaStream_t s, const LatentRow* row) {
     if (T <= 0) return;
     const size_t smem = sizeof(float) * (LT * (size_t)(dim + rot_dim) + 4 * 64 * LT);
     NT_CHECK(smem <= 48 * 1024, "latent_q_absorb: query heads wider than 1280 are not covered");
     const RotDev rd = dev_of(rot);
-    const dim3 grid((T + LT - 1) / LT, heads, (kv_rank + 63) / 64);
+    NT_CHECK(!row || (T == 1 && (row->cache_dt == DType::F32 || row->cache_dt == DType::BF16)), "latent_q_absorb: a cache row rides along with one token only");
+    const LatentRow lr = row ? *row : LatentRow();
+    const dim3 grid((T + LT - 1) / LT, heads + (row ? 1 : 0), (kv_rank + 63) / 64);
 #define NT_QA(TY) launch_k(latent_q_absorb_kernel<TY>, grid, dim3(256), smem, s, qa, q, static_cast<const TY*>(W_uk), T, heads, dim, rot_dim, kv_rank, rd, \
-                           pos_dev, p0)
+                           pos_dev, p0, lr)
     if (dt == DType::F32) NT_QA(float); else if (dt == DType::F16) NT_QA(__half); else if (dt == DType::BF16) NT_QA(__nv_bfloat16);
     else NT_CHECK(false, "latent_q_absorb: dense dtypes only");
 #undef NT_QA
@@ -532,32 +600,52 @@ int attention_shared_rows_slices(int tokens, int max_seq, int window) {
 }
 size_t attention_shared_rows_scratch_floats(int heads, int vdim) { return (size_t)LS_MAX_PARTS * heads * ((size_t)vdim + 2); }
 
+namespace {
+// the slices of nt queries -> scratch; returns their number
+int shared_rows_slices(float* scratch, const float* Q, const void* cache, DType cache_dt, int nt, const int* pos_dev, int p0, int max_seq, int heads, int dim, int vdim, int row, float scale,
+                       int window, cudaStream_t s) {
+    const bool f32 = cache_dt == DType::F32;
+    const int vn = f32 ? 4 : 8;
+    const size_t smem = sizeof(float) * ((size_t)heads * dim + (size_t)heads * LS_KEYS) + (size_t)LS_KEYS * (dim + vn) * (f32 ? 4 : 2);
+    const int slices = attention_shared_rows_slices(nt, max_seq, window);
+    static unsigned long long cfg_f = 0, cfg_b = 0;
+    if (f32) {
+        opt_in_dynamic_smem(latent_shared_attn_kernel<float>, 200 * 1024, cfg_f);
+        launch_k(latent_shared_attn_kernel<float>, dim3(nt, slices), dim3(256), smem, s, scratch, Q, static_cast<const float*>(cache), pos_dev, p0, heads, dim, vdim, row, scale, window);
+    } else {
+        opt_in_dynamic_smem(latent_shared_attn_kernel<__nv_bfloat16>, 200 * 1024, cfg_b);
+        launch_k(latent_shared_attn_kernel<__nv_bfloat16>, dim3(nt, slices), dim3(256), smem, s, scratch, Q, static_cast<const __nv_bfloat16*>(cache), pos_dev, p0, heads, dim, vdim, row,
+                 scale, window);
+    }
+    count_launch();
+    return slices;
+}
+}  // namespace
+
 // out [tokens, heads, vdim]; Q [tokens, heads, dim]; scratch >= attention_shared_rows_scratch_floats.  The grid depends on tokens and
 // max_seq only, never on the position: the captured decode step replays it unchanged.
 void attention_shared_rows(float* out, const float* Q, const void* cache, DType cache_dt, int tokens, const int* pos_dev, int p0, int max_seq, int heads, int dim,
                            int vdim, int row, float scale, float* scratch, cudaStream_t s, int window) {
     if (tokens <= 0) return;
     NT_CHECK(attention_shared_rows_supported(heads, dim, vdim, row, cache_dt, cache), "attention_shared_rows: shape not covered");
-    const bool f32 = cache_dt == DType::F32;
-    const int vn = f32 ? 4 : 8;
-    const size_t smem = sizeof(float) * ((size_t)heads * dim + (size_t)heads * LS_KEYS) + (size_t)LS_KEYS * (dim + vn) * (f32 ? 4 : 2);
     for (int t0 = 0; t0 < tokens; t0 += LS_MAX_PARTS) {           // long portions (exact mode): blocks of queries with one slice each
         const int nt = std::min(LS_MAX_PARTS, tokens - t0);
-        const int slices = attention_shared_rows_slices(nt, max_seq, window);
-        static unsigned long long cfg_f = 0, cfg_b = 0;
-        if (f32) {
-            opt_in_dynamic_smem(latent_shared_attn_kernel<float>, 200 * 1024, cfg_f);
-            launch_k(latent_shared_attn_kernel<float>, dim3(nt, slices), dim3(256), smem, s, scratch, Q + (size_t)t0 * heads * dim, static_cast<const float*>(cache), pos_dev,
-                     p0 + t0, heads, dim, vdim, row, scale, window);
-        } else {
-            opt_in_dynamic_smem(latent_shared_attn_kernel<__nv_bfloat16>, 200 * 1024, cfg_b);
-            launch_k(latent_shared_attn_kernel<__nv_bfloat16>, dim3(nt, slices), dim3(256), smem, s, scratch, Q + (size_t)t0 * heads * dim,
-                     static_cast<const __nv_bfloat16*>(cache), pos_dev, p0 + t0, heads, dim, vdim, row, scale, window);
-        }
-        count_launch();
+        const int slices = shared_rows_slices(scratch, Q + (size_t)t0 * heads * dim, cache, cache_dt, nt, pos_dev, p0 + t0, max_seq, heads, dim, vdim, row, scale, window, s);
         launch_k(latent_shared_merge_kernel, dim3(nt, heads, (vdim + 63) / 64), dim3(256), sizeof(float) * slices, s, out + (size_t)t0 * heads * vdim, (const float*)scratch, slices, heads, vdim);
         count_launch();
     }
+}
+
+void attention_shared_rows_up(float* out, const float* Q, const void* cache, DType cache_dt, const int* pos_dev, int p0, int max_seq, int heads, int dim, int vdim, int row, float scale,
+                              float* scratch, const void* W_uv, DType wdt, int v_up, const float* gate, cudaStream_t s, int window) {
+    NT_CHECK(attention_shared_rows_supported(heads, dim, vdim, row, cache_dt, cache) && dense_dtype(wdt), "attention_shared_rows_up: shape not covered");
+    const int slices = shared_rows_slices(scratch, Q, cache, cache_dt, 1, pos_dev, p0, max_seq, heads, dim, vdim, row, scale, window, s);
+    const size_t smem = sizeof(float) * ((size_t)((slices + 3) & ~3) + (size_t)vdim);
+    const dim3 grid(1, heads, (v_up + 31) / 32);
+#define NT_MU(TY) launch_k(latent_merge_up_kernel<TY>, grid, dim3(256), smem, s, out, (const float*)scratch, slices, heads, vdim, static_cast<const TY*>(W_uv), v_up, gate)
+    if (wdt == DType::F32) NT_MU(float); else if (wdt == DType::F16) NT_MU(__half); else NT_MU(__nv_bfloat16);
+#undef NT_MU
+    count_launch();
 }
 
 }}  // namespace nt::b200

@@ -249,7 +249,7 @@ __device__ __forceinline__ float batch_dot(const unsigned char* row, const float
 
 // ---- several matrices, each with its own input vector ----
 struct MultiDev {
-    struct One { const unsigned char* W; size_t pitch; const float* x; float* y; const float* act_p; int out, K, act, f32, vec, cta_end; };
+    struct One { const unsigned char* W; size_t pitch; const float* x; float* y; const float* act_p; const float* norm_w; float eps; int out, K, act, f32, vec, cta_end; };
     One m[DENSE_MAX_MATS];
     int n;
 };
@@ -266,7 +266,25 @@ __global__ void __launch_bounds__(DV_WARPS * 32) gemv_multi_kernel(const __grid_
     for (int r = r0; r < m.out; r += ctas * DV_WARPS) l2_prefetch(m.W + (size_t)r * m.pitch, row_bytes, lane, 32);
     pdl_wait();
     const bool wide = !m.f32 && m.vec;                    // 16-bit rows in whole pieces: planar staging
-    stage_floats(xs, m.x, m.K, wide && Elem<T>::PER16 == 8);
+    float inv = 1.f;
+    if (m.norm_w) {                                       // the gain goes into the staged vector, the root mean square onto the results
+        __shared__ float red[DV_WARPS];
+        const bool planar = wide && Elem<T>::PER16 == 8;
+        const int half = m.K >> 1;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < m.K; i += DV_WARPS * 32) {
+            const float v = m.x[i];
+            ss = fmaf(v, v, ss);
+            xs[planar ? ((i & 4) ? half : 0) + (i >> 3) * 4 + (i & 3) : i] = v * m.norm_w[i];
+        }
+        ss = warp_sum(ss);
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        float tot = 0.f;
+#pragma unroll
+        for (int w = 0; w < DV_WARPS; w++) tot += red[w];
+        inv = 1.0f / sqrtf(tot / (float)m.K + m.eps);
+    } else stage_floats(xs, m.x, m.K, wide && Elem<T>::PER16 == 8);
     __syncthreads();
     float a = 0.f, b = 0.f;
     if (m.act == GEMV_ACT_XIELU) { a = softplus_f(m.act_p[0]); b = softplus_f(m.act_p[1]); }
@@ -279,6 +297,7 @@ __global__ void __launch_bounds__(DV_WARPS * 32) gemv_multi_kernel(const __grid_
             v = warp_sum(v);
         } else v = m.f32 ? dense_row_dot<float>(row, xs, m.K, lane, m.vec) : dense_row_dot<T>(row, xs, m.K, lane, m.vec);
         if (lane == 0) {
+            v *= inv;
             if (m.act == GEMV_ACT_TANH) v = tanhf(v);
             else if (m.act == GEMV_ACT_XIELU) v = xielu_f(v, a, b);
             else if (m.act == GEMV_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
@@ -495,7 +514,7 @@ void gemv_multi(const MultiMat* mats, int n_mat, cudaStream_t s) {
         NT_CHECK(a.act != GEMV_ACT_XIELU || a.act_p, "gemv_multi: the activation's two numbers are missing");
         MultiDev::One& o = md.m[i];
         o.W = static_cast<const unsigned char*>(a.W); o.pitch = a.row_pitch ? a.row_pitch : dtype_row_size(a.dtype, (size_t)a.K);
-        o.x = a.x; o.y = a.y; o.act_p = a.act_p; o.out = a.out; o.K = a.K; o.act = a.act; o.f32 = a.dtype == DType::F32 ? 1 : 0;
+        o.x = a.x; o.y = a.y; o.act_p = a.act_p; o.norm_w = a.norm_w; o.eps = a.eps; o.out = a.out; o.K = a.K; o.act = a.act; o.f32 = a.dtype == DType::F32 ? 1 : 0;
         o.vec = a.K % (o.f32 ? 4 : 8) == 0 && (reinterpret_cast<uintptr_t>(a.W) & 15) == 0 && (o.pitch & 15) == 0;
         bytes[i] = (size_t)a.out * o.pitch; total += bytes[i];
         K = std::max(K, a.K); rows += a.out;

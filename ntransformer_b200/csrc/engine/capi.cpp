@@ -622,6 +622,45 @@ void nt_b200_mlstm_token(float* out, const float* q, const float* k, const float
                          const float* norm, float* state, float* m, float cap, float q_scale, float eps, int heads, int dim, int vdim, int p0, void* stream) {
     mlstm_token(out, q, k, v, gate, zi, zf, bi, bf, norm, state, m, cap, q_scale, eps, heads, dim, vdim, nullptr, p0, static_cast<cudaStream_t>(stream));
 }
+// One row: x_out = x + rms(y) * gain_y, h = rms(x_out) * gain_h, logits [experts] = router . h.  -1: width not covered
+int nt_b200_sandwich_norm_router(float* x_out, const float* x, const float* y, const float* gain_y, const float* gain_h, float* h, const float* router, float* logits, int experts,
+                                 int width, float eps, void* stream) {
+    return sandwich_norm_router(x_out, x, y, gain_y, gain_h, h, router, logits, experts, width, eps, static_cast<cudaStream_t>(stream)) ? 0 : -1;
+}
+// y = W (x / sqrt(mean x^2 + eps) * gain)
+void nt_b200_gemv_normed(float* y, const void* W, int dtype, const float* x, const float* gain, float eps, int out, int K, void* stream) {
+    MultiMat m;
+    m.W = W; m.dtype = (nt::DType)dtype; m.x = x; m.y = y; m.out = out; m.K = K; m.norm_w = gain; m.eps = eps;
+    gemv_multi(&m, 1, static_cast<cudaStream_t>(stream));
+}
+// One decoded token of the latent attention behind its queries, in three launches: absorbed queries and the cache row, the slices, merge and gated values.
+// rot: base, no table.  -1: shape not covered.  Scratch is allocated and freed here.
+int nt_b200_latent_token(float* out, const float* q, const float* dkv, const float* kv_gain, float eps, void* cache, int cache_dtype, const void* W_uk, const void* W_uv, int dtype, int p0,
+                         int max_seq, int heads, int dim, int rot_dim, int vdim, int kv_rank, int rot_dims, float rot_base, float scale, const float* gate, void* stream) {
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const int row = kv_rank + rot_dim;
+    const nt::DType ct = (nt::DType)cache_dtype, wt = (nt::DType)dtype;
+    if (!attention_shared_rows_supported(heads, row, kv_rank, row, ct, cache)) return -1;
+    float *qa = nullptr, *scratch = nullptr;
+    NT_CUDA_CHECK(cudaMalloc(&qa, sizeof(float) * (size_t)heads * row));
+    NT_CUDA_CHECK(cudaMalloc(&scratch, sizeof(float) * attention_shared_rows_scratch_floats(heads, kv_rank)));
+    LatentRow lr;
+    lr.dkv = dkv; lr.gain = kv_gain; lr.eps = eps; lr.cache = cache; lr.cache_dt = ct;
+    latent_q_absorb(qa, q, W_uk, wt, 1, heads, dim, rot_dim, kv_rank, LatentRot{rot_dims, true, rot_base}, nullptr, p0, s, &lr);
+    attention_shared_rows_up(out, qa, cache, ct, nullptr, p0, max_seq, heads, row, kv_rank, row, scale, scratch, W_uv, wt, vdim, gate, s);
+    NT_CUDA_CHECK(cudaStreamSynchronize(s));
+    cudaFree(qa);
+    cudaFree(scratch);
+    return 0;
+}
+// C[i] [M, N[i]] = A W[i]^T for n BF16 matrices in one launch (workspace: the split of A).  -1: shape not covered
+int nt_b200_gemm_multi(float* const* C, const float* A, const void* const* W, const int* N, int n, int M, int K, void* workspace, void* stream) {
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    TcOpts o;
+    o.bf16 = true;
+    split_activations(workspace, A, M, K, s, true);
+    return gemm_f16_tc_multi_ws(C, workspace, W, N, n, M, K, s, o) ? 0 : -1;
+}
 // The tensor-core GEMM with relu(z)^2 in its epilogue: split_out <- split(relu(A W^T)^2) from BF16 W and F32 A (workspace: the split of A).  -1: shape not covered
 int nt_b200_gemm_relu2(void* split_out, const float* A, const void* W, int M, int N, int K, void* workspace, void* stream) {
     cudaStream_t s = static_cast<cudaStream_t>(stream);

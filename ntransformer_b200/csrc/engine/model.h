@@ -211,8 +211,8 @@ private:
     void ensure_parallel_buffers(size_t T);
     struct ParDec { float *slots = nullptr, *h = nullptr, *mix[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}, *wide = nullptr; size_t slot = 0; } par_dec_;   // decode: stable addresses
     struct ParRows { float *slots = nullptr, *h = nullptr, *wide = nullptr; void *hs = nullptr, *mix_s[5] = {nullptr, nullptr, nullptr, nullptr, nullptr}; size_t slot = 0; } par_;
-    // gate [T, heads * vdim] (absorbed form only): the values are multiplied by sigmoid(gate)
-    void latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s, const float* gate = nullptr);
+    // gate [T, heads * vdim] (absorbed form only): the values are multiplied by sigmoid(gate); cache_row (one token): its key / value row, written on the way
+    void latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s, const float* gate = nullptr, const LatentRow* cache_row = nullptr);
     LatentRot latent_rot(int i) const;
     // SANDWICH block form (attention with distance bias, latent attention, matrix memory): engine/model_sandwich.cu
     bool finalize_sandwich_layer(int i);
@@ -221,10 +221,11 @@ private:
     void step_sandwich(cudaStream_t s);       // one decoded token: embedding, all layers -> hidden_
     void prefill_sandwich(int T, int p0, cudaStream_t s);      // T prompt rows: embedding, all layers -> pf_.x
     void sandwich_mixer_token(int i, float* y, cudaStream_t s);
-    void sandwich_ff_token(int i, float* y, cudaStream_t s);
+    void sandwich_ff_token(int i, float* y, bool with_logits, cudaStream_t s);
     void sandwich_mixer_rows(int i, int T, int p0, float* y, cudaStream_t s);
     void sandwich_ff_rows(int i, int T, float* y, cudaStream_t s);
     bool rows_take_tc(const Weight& w) const { return pf_.ws && (w.tc_ptr || spec_tc_ok(w)); }
+    float* moe_logits_ = nullptr;             // decode: the router's logits of one token (owned_)
     float* ml_scratch_ = nullptr;             // segment states of the matrix memory over prompt rows (owned_)
     float* wkv_scratch_ = nullptr;            // segment states of the WKV recurrence over prompt rows (owned_)
     Weight bigram_;                           // second embedding over token pairs [buckets + 1, width]

@@ -7,10 +7,11 @@
 // Everything between two sublayers — norm of the output, residual sum, norm of the next input — is one launch (sandwich_norm_rows), so a decoded
 // token takes
 //   attention layer, 5:  [q, k, v, gate rows]  [head norm, query multiplier, cache write]  [attention, gated]  [W_o]  [between]
-//   latent layer, 9:     [query latent, key / value latent, gate]  [latent norms, rotation, cache write]  [queries]  [absorbed queries]  [attention]  [merge]
-//                        [values, gated]  [W_o]  [between]
+//   latent layer, 7:     [query latent, key / value latent, gate]  [queries from the normed latent]  [absorbed queries + cache row]  [attention]
+//                        [merge + values, gated]  [W_o]  [between]
 //   matrix memory, 4:    [q, k, v, gate, input / forget gate rows]  [gates, memory, head norm, output gate]  [W_o]  [between]
-//   dense feed-forward, 3:  [relu(W_up .)^2]  [W_down]  [between]      experts, 4:  [router logits]  [choice + experts and shared one up]  [down, weighted]  [between]
+//   dense feed-forward, 3:  [relu(W_up .)^2]  [W_down]  [between]      experts, 3:  (router logits come with the launch between mixer and feed-forward)
+//                        [choice + experts and shared one up]  [down, weighted]  [between]
 // Prompt rows take the tensor-core GEMMs, the tiled attention kernels and the tiled recurrence.  What a sequence carries between steps — cache rows, the
 // matrix memory with its normalizer and stabilizer — is written by the step that owns the tokens and read by later steps only from there; the memory
 // reads as zeros when a step starts at position 0, so a new request needs no clearing.
@@ -152,7 +153,11 @@ size_t Model::sandwich_scratch_width() const {
 
 void Model::finalize_sandwich_decode() {
     dec_.y = dmalloc0<float>((size_t)cfg_.hidden_size);
-    dec_.t[0] = dmalloc0<float>((size_t)cfg_.hidden_size);
+    for (int t = 0; t < 2; t++) dec_.t[t] = dmalloc0<float>((size_t)cfg_.hidden_size);
+    int experts = 1;
+    for (const LayerSpec& S : cfg_.layers) if (S.ff_kind == FfKind::MOE_GLU) experts = std::max(experts, S.experts);
+    moe_logits_ = dmalloc0<float>((size_t)experts);
+    owned_.push_back(moe_logits_);
     dec_.wide = dmalloc0<float>(sandwich_scratch_width());
     size_t seg = 0;
     for (const LayerSpec& S : cfg_.layers) if (S.mixer == MixerKind::MLSTM) seg = std::max(seg, mlstm_rows_scratch_floats(S.heads, S.dim, S.vdim));
@@ -176,7 +181,11 @@ static WindowAttn biased_attn_of(const LayerSpec& S, const LayerWeights& L) {
 void Model::step_sandwich(cudaStream_t s) {
     const int W = cfg_.hidden_size;
     const float eps = cfg_.norm_eps;
-    float *x = hidden_, *h = dec_.t[0], *y = dec_.y;
+    // a launch that also routes writes the residual into the other of two rows; start so that the last result lands in hidden_
+    float *x = hidden_, *other = dec_.t[1], *h = dec_.t[0], *y = dec_.y;
+    int routed_layers = 0;
+    for (const LayerSpec& S : cfg_.layers) routed_layers += S.ff > 0 && S.ff_kind == FfKind::MOE_GLU;
+    if (routed_layers & 1) std::swap(x, other);
     embed_rows(x, embd_.ptr, embd_.dtype, step_dev_, 1, W, s);
     sandwich_norm_rows(x, nullptr, nullptr, layers_[0].attn_norm, h, nullptr, 1, W, eps, s);
     for (int i = 0; i < cfg_.n_layers; i++) {
@@ -184,11 +193,15 @@ void Model::step_sandwich(cudaStream_t s) {
         const float* next = i + 1 < cfg_.n_layers ? layers_[(size_t)i + 1].attn_norm : nullptr;       // the head normalises the last result itself
         const bool ff = cfg_.layers[(size_t)i].ff > 0;
         sandwich_mixer_token(i, y, s);
-        sandwich_norm_rows(x, y, L.norm1b, ff ? L.ffn_norm : next, h, nullptr, 1, W, eps, s);
+        const bool routed = ff && cfg_.layers[(size_t)i].ff_kind == FfKind::MOE_GLU;
+        const bool with_logits = routed && sandwich_norm_router(other, x, y, L.norm1b, L.ffn_norm, h, L.router, moe_logits_, cfg_.layers[(size_t)i].experts, W, eps, s);
+        if (with_logits) std::swap(x, other);
+        else sandwich_norm_rows(x, y, L.norm1b, ff ? L.ffn_norm : next, h, nullptr, 1, W, eps, s);
         if (!ff) continue;
-        sandwich_ff_token(i, y, s);
+        sandwich_ff_token(i, y, with_logits, s);
         sandwich_norm_rows(x, y, L.norm2b, next, h, nullptr, 1, W, eps, s);
     }
+    if (x != hidden_) copy(hidden_, x, W, s);
 }
 
 // y = mixer(h), h = dec_.t[0]
@@ -222,10 +235,12 @@ void Model::sandwich_mixer_token(int i, float* y, cudaStream_t s) {
         mats[n++] = multi(L.w_dq, h, cq); mats[n++] = multi(L.w_dkv, h, dkv);
         if (g) mats[n++] = multi(L.out_gate, h, g);
         gemv_multi(mats, n, s);
-        latent_prep(cq, A.q_rank, L.dq_norm, dkv, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, latent_rot(i), 1, pos_dev, 0, s);
         mats[0] = multi(L.w_uq, cq, q);
+        mats[0].norm_w = L.dq_norm; mats[0].eps = eps;
         gemv_multi(mats, 1, s);
-        latent_mixer_core(i, 1, pos_dev, 0, q, qa, ol, o, s, g);
+        LatentRow row;
+        row.dkv = dkv; row.gain = L.dkv_norm; row.eps = eps; row.cache = kcs_[(size_t)i]; row.cache_dt = cache_dt_;
+        latent_mixer_core(i, 1, pos_dev, 0, q, qa, ol, o, s, g, &row);
     } else {
         float *q = take(H * D), *k = take(H * D), *v = take(H * V), *zi = take(H), *zf = take(H);
         mats[n++] = multi(L.wq, h, q); mats[n++] = multi(L.wk, h, k); mats[n++] = multi(L.wv, h, v); mats[n++] = multi(L.out_gate, h, g);
@@ -239,8 +254,8 @@ void Model::sandwich_mixer_token(int i, float* y, cudaStream_t s) {
     gemv_sum(y, &t, 1, cfg_.hidden_size, L.wo.dtype, false, s);
 }
 
-// y = ff(h), h = dec_.t[0]
-void Model::sandwich_ff_token(int i, float* y, cudaStream_t s) {
+// y = ff(h), h = dec_.t[0]; with_logits: the router's logits are already in moe_logits_
+void Model::sandwich_ff_token(int i, float* y, bool with_logits, cudaStream_t s) {
     const LayerSpec& S = cfg_.layers[(size_t)i];
     const LayerWeights& L = layers_[(size_t)i];
     const float* h = dec_.t[0];
@@ -255,12 +270,14 @@ void Model::sandwich_ff_token(int i, float* y, cudaStream_t s) {
         gemv_multi(&m, 1, s);
         t[nt].W = L.down.ptr; t[nt].x = a; t[nt++].K = S.ff;
     } else {
-        float *act = take((size_t)S.top * S.ff + S.shared_ff), *logits = take((size_t)S.experts);
-        MultiMat m;
-        m.W = L.router; m.dtype = DType::F32; m.x = h; m.y = logits; m.out = S.experts; m.K = cfg_.hidden_size;
-        gemv_multi(&m, 1, s);
+        float* act = take((size_t)S.top * S.ff + S.shared_ff);
+        if (!with_logits) {
+            MultiMat m;
+            m.W = L.router; m.dtype = DType::F32; m.x = h; m.y = moe_logits_; m.out = S.experts; m.K = cfg_.hidden_size;
+            gemv_multi(&m, 1, s);
+        }
         const MoeWeights w = gated_moe(i);
-        moe_expert_up_token(act, h, nullptr, w, s, logits, moe_sel_, moe_wt_);
+        moe_expert_up_token(act, h, nullptr, w, s, moe_logits_, moe_sel_, moe_wt_);
         bool aligned = true;
         for (const Weight& d : L.e_down) aligned = aligned && (reinterpret_cast<uintptr_t>(d.ptr) & 15) == 0;
         t[nt].table = L.e_down_tab; t[nt].table_aligned = aligned; t[nt].sel = moe_sel_; t[nt].wt = moe_wt_; t[nt].top = S.top; t[nt].x = act; t[nt++].K = S.ff;
@@ -334,11 +351,32 @@ void Model::sandwich_mixer_rows(int i, int T, int p0, float* y, cudaStream_t s) 
         copy_cols(P, C, T, w.rows, ld, s);
         return P;
     };
-    auto h_split = [&](const Weight& w) { return rows_take_tc(w) ? pf_.hws : nullptr; };
+    // the products that read h: those of 256 rows or more are collected and run as one launch, the others at once
+    float* many_C[TC_MULTI_MAX];
+    const Weight* many[TC_MULTI_MAX];
+    int n_many = 0;
+    auto of_h = [&](const Weight& w, int* ld = nullptr) {
+        if (rows_take_tc(w) && !w.tc_ptr && w.rows >= 256 && n_many < TC_MULTI_MAX) {
+            many[n_many] = &w;
+            if (ld) *ld = w.rows;
+            return many_C[n_many++] = take((size_t)w.rows);
+        }
+        const void* split = rows_take_tc(w) ? pf_.hws : nullptr;
+        return ld ? product(w, pf_.h, split, *ld) : packed(w, pf_.h, split);
+    };
+    auto run_many = [&]() {
+        const void* W[TC_MULTI_MAX];
+        int N[TC_MULTI_MAX];
+        for (int x = 0; x < n_many; x++) { W[x] = many[x]->ptr; N[x] = many[x]->rows; }
+        TcOpts opt; opt.bf16 = true;
+        if (n_many == 1) NT_CHECK(gemm_f16_tc_ws(many_C[0], pf_.hws, W[0], T, N[0], cfg_.hidden_size, false, s, opt), "prefill GEMM rejected");
+        else if (n_many > 1) NT_CHECK(gemm_f16_tc_multi_ws(many_C, pf_.hws, W, N, n_many, T, cfg_.hidden_size, s, opt), "prefill GEMM (several matrices) rejected");
+    };
     const bool o_tc = rows_take_tc(L.wo);
     float* o = take(H * V);
     if (S.mixer == MixerKind::MLSTM) {
-        float *q = packed(L.wq, pf_.h, h_split(L.wq)), *k = packed(L.wk, pf_.h, h_split(L.wk)), *v = packed(L.wv, pf_.h, h_split(L.wv)), *g = packed(L.out_gate, pf_.h, h_split(L.out_gate));
+        float *q = of_h(L.wq), *k = of_h(L.wk), *v = of_h(L.wv), *g = of_h(L.out_gate);
+        run_many();
         int ld = 0;
         const float *zi = nullptr, *zf = nullptr;
         if (L.ml_if.ptr && rows_take_tc(L.ml_if)) { zi = product(L.ml_if, nullptr, pf_.hws, ld); zf = zi + H; }
@@ -350,16 +388,18 @@ void Model::sandwich_mixer_rows(int i, int T, int p0, float* y, cudaStream_t s) 
     } else {
         const float* g = nullptr;
         int g_ld = 0;
-        if (S.out_gate != OutGate::NONE) g = product(L.out_gate, pf_.h, h_split(L.out_gate), g_ld);
+        if (S.out_gate != OutGate::NONE) g = of_h(L.out_gate, &g_ld);
         if (S.mixer == MixerKind::ATTN_WINDOW) {
-            float *q = packed(L.wq, pf_.h, h_split(L.wq)), *k = nullptr, *v = nullptr;
-            if (S.kv_from < 0) { k = packed(L.wk, pf_.h, h_split(L.wk)); v = packed(L.wv, pf_.h, h_split(L.wv)); }
+            float *q = of_h(L.wq), *k = nullptr, *v = nullptr;
+            if (S.kv_from < 0) { k = of_h(L.wk); v = of_h(L.wv); }
+            run_many();
             void *kc = kcs_[(size_t)i], *vc = vcs_[(size_t)i];
             head_prep(q, k, v, head_prep_of(S, eps), kc, vc, cache_dt_, T, nullptr, p0, s);
             attention_window(o, q, kc, vc, cache_dt_, T, nullptr, p0, cfg_.max_seq_len, biased_attn_of(S, L), s);
         } else {
             const LatentSpec& A = S.latent;
-            float *cq = packed(L.w_dq, pf_.h, h_split(L.w_dq)), *dkv = packed(L.w_dkv, pf_.h, h_split(L.w_dkv));
+            float *cq = of_h(L.w_dq), *dkv = of_h(L.w_dkv);
+            run_many();
             latent_prep(cq, A.q_rank, L.dq_norm, dkv, A.kv_rank, A.rot_dim, L.dkv_norm, eps, kcs_[(size_t)i], cache_dt_, latent_rot(i), T, nullptr, p0, s);
             const bool uq_tc = rows_take_tc(L.w_uq);
             if (uq_tc) split_activations(pf_.ws, cq, T, A.q_rank, s, true);

@@ -1000,13 +1000,18 @@ LatentRot Model::latent_rot(int i) const {
 
 // Scores and values of T rows behind the query projection and the cache write: expanded per-head form for prompt portions, absorbed form on
 // the cached rows otherwise.  q [T, heads, dim + rot_dim]; qa, ol: scratch [T, heads, kv_rank + rot_dim], [T, heads, kv_rank]; o (may be q) [T, heads * vdim].
-void Model::latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s, const float* gate) {
+void Model::latent_mixer_core(int i, int T, const int* pos_dev, int p0, const float* q, float* qa, float* ol, float* o, cudaStream_t s, const float* gate, const LatentRow* cache_row) {
     const LayerSpec& S = cfg_.layers[(size_t)i];
     const LayerWeights& L = layer_weights(i);
     const LatentSpec& A = S.latent;
     const int row = A.kv_rank + A.rot_dim;
     if (!pos_dev && !gate && latent_expand_ok(S, T)) { latent_attention_rows(i, T, p0, q, o, s); return; }
-    latent_q_absorb(qa, q, L.w_uk.ptr, L.w_uv.dtype, T, S.heads, S.dim, A.rot_dim, A.kv_rank, latent_rot(i), pos_dev, p0, s);
+    latent_q_absorb(qa, q, L.w_uk.ptr, L.w_uv.dtype, T, S.heads, S.dim, A.rot_dim, A.kv_rank, latent_rot(i), pos_dev, p0, s, cache_row);
+    if (T == 1 && lat_part_ && attention_shared_rows_supported(S.heads, row, A.kv_rank, row, cache_dt_, kcs_[(size_t)i])) {
+        attention_shared_rows_up(o, qa, kcs_[(size_t)i], cache_dt_, pos_dev, p0, cfg_.max_seq_len, S.heads, row, A.kv_rank, row, S.scale, lat_part_, L.w_uv.ptr, L.w_uv.dtype, S.vdim, gate,
+                                 s, S.window);
+        return;
+    }
     if (lat_part_ && attention_shared_rows_supported(S.heads, row, A.kv_rank, row, cache_dt_, kcs_[(size_t)i])) {
         attention_shared_rows(ol, qa, kcs_[(size_t)i], cache_dt_, T, pos_dev, p0, cfg_.max_seq_len, S.heads, row, A.kv_rank, row, S.scale, lat_part_, s, S.window);
     } else {

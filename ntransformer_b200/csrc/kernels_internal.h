@@ -155,6 +155,7 @@ struct MultiMat {
     const float* x = nullptr; float* y = nullptr;
     int out = 0, K = 0;
     GemvAct act = GEMV_ACT_NONE; const float* act_p = nullptr;
+    const float* norm_w = nullptr; float eps = 0.f;      // norm_w given: the input is x / sqrt(mean(x^2) + eps) * norm_w
 };
 void gemv_multi(const MultiMat* mats, int n_mat, cudaStream_t s);
 // y[out] (+)= the sum of up to GEMV_SUM_MAX_TERMS matrix-vector products.  A term is one matrix W [out, K] with x [K], or `top` routed ones:
@@ -291,9 +292,11 @@ struct LatentRot { int dims = 0; bool interleaved = true; double base = 10000.0;
 // reads another layer's rows; cq null: the queries have no latent): [RMS-normed first part | rotated rest] -> cache row base + t of `cache` ([max_seq, kv_rank + rot_dim]).
 void latent_prep(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache,
                  DType cache_dt, const LatentRot& rot, int T, const int* pos_dev, int p0, cudaStream_t s);
+// row (T == 1): the token's key / value row [kv_rank + rot_dim] in front of its norm is prepared and written to the cache by the same launch
+struct LatentRow { const float* dkv = nullptr; const float* gain = nullptr; float eps = 0.f; void* cache = nullptr; DType cache_dt = DType::F32; };
 // q [T, heads, dim + rot_dim] -> qa [T, heads, kv_rank + rot_dim] = [W_uk,h^T q_unrotated | rot(q_rotated)];  W_uk [heads * dim, kv_rank]
 void latent_q_absorb(float* qa, const float* q, const void* W_uk, DType dt, int T, int heads, int dim, int rot_dim, int kv_rank, const LatentRot& rot,
-                     const int* pos_dev, int p0, cudaStream_t s);
+                     const int* pos_dev, int p0, cudaStream_t s, const LatentRow* row = nullptr);
 // ol [T, heads, kv_rank] -> out [T, heads * vdim] = W_uv,h ol_h;  W_uv [heads * vdim, kv_rank].  gate [T, heads * vdim] (may be null): times sigmoid(gate)
 void latent_v_up(float* out, const float* ol, const void* W_uv, DType dt, int T, int heads, int vdim, int kv_rank, cudaStream_t s, const float* gate = nullptr);
 // Prompt portions: F32 latents of cache rows r0.. (input of the two up-projection GEMMs); their results packed with the rotated key part
@@ -312,6 +315,9 @@ bool attention_shared_rows_supported(int heads, int dim, int vdim, int row, DTyp
 size_t attention_shared_rows_scratch_floats(int heads, int vdim);
 void attention_shared_rows(float* out, const float* Q, const void* cache, DType cache_dt, int tokens, const int* pos_dev, int p0, int max_seq, int heads, int dim,
                            int vdim, int row, float scale, float* scratch, cudaStream_t s, int window = 0);
+// One query: the same, the merge of the slices and the up-projection of the values in one launch: out [heads * v_up] = W_uv,h o_h (times sigmoid(gate))
+void attention_shared_rows_up(float* out, const float* Q, const void* cache, DType cache_dt, const int* pos_dev, int p0, int max_seq, int heads, int dim, int vdim, int row, float scale,
+                              float* scratch, const void* W_uv, DType wdt, int v_up, const float* gate, cudaStream_t s, int window = 0);
 // attention_prefill_mma.cu: causal (window > 0: the last `window` positions) attention of `tokens` queries [tokens, heads, kw] at positions p0.. over BF16 per-head keys
 // [rows, heads, kw] and values [rows, heads, vw]; (kw, vw) from attention_heads_mma_widths.  out [tokens, heads, vw].
 bool attention_heads_mma_widths(int key_dim, int value_dim, int* kw, int* vw);
@@ -331,6 +337,10 @@ void glu_bias_mul(float* out, const float* gate, const float* up, const float* g
 // The sandwich form's step between sublayers: x[t] += rms(y[t]) * gain_y (y null: x as it is), then h = rms(x[t]) * gain_h -> F32 rows and / or the
 // BF16 split of a tensor-core GEMM's input (gain_h null: x only).
 void sandwich_norm_rows(float* x, const float* y, const float* gain_y, const float* gain_h, float* h, void* split, int rows, int width, float eps, cudaStream_t s);
+// One row, with the router's logits [experts] = router [experts, width] . h from the same launch; x_out (not x): the new residual.  false: width or alignment
+// not covered, nothing launched.
+bool sandwich_norm_router(float* x_out, const float* x, const float* y, const float* gain_y, const float* gain_h, float* h, const float* router, float* logits, int experts, int width,
+                          float eps, cudaStream_t s);
 // o [T, cols] * sigmoid(gate[t * ld + c / per]) -> F32 rows (in place is fine) and / or the BF16 split
 void sigmoid_gate_rows(float* out, void* split, const float* o, const float* gate, int ld, int per, int T, int cols, cudaStream_t s);
 // relu(z)^2 of a [T, cols], as F32 rows (in place is fine) and / or the BF16 split
@@ -476,6 +486,9 @@ struct TcOpts { bool bf16 = false; bool gelu = false; const float* col_scale = n
                 const float* act_p = nullptr; /* set by gemm_f16_tc_xielu_ws */ };
 void split_activations(void* workspace, const float* A, int M, int K, cudaStream_t s, bool bf16 = false);
 bool gemm_f16_tc_ws(float* C, const void* workspace, const void* W_f16, int M, int N, int K, bool add, cudaStream_t s, const TcOpts& o = TcOpts());
+// Several matrices of at least 256 rows over the same input rows in one launch: C[i] [M, N[i]] = A . W[i]^T
+constexpr int TC_MULTI_MAX = 6;
+bool gemm_f16_tc_multi_ws(float* const* C, const void* workspace, const void* const* W, const int* N, int n, int M, int K, cudaStream_t s, const TcOpts& o = TcOpts());
 // workspace_out <- split(silu(A.Wgate^T) * (A.Wup^T)): the FFN's gate/up GEMMs with the SwiGLU + split fused in the epilogue
 bool gemm_f16_tc_swiglu_ws(void* workspace_out, const void* workspace_in, const void* Wgate_f16, const void* Wup_f16, int M, int N, int K,
                            cudaStream_t s, const TcOpts& o = TcOpts());

@@ -407,7 +407,7 @@ __global__ void __launch_bounds__(256) mlstm_token_kernel(float* __restrict__ ou
     for (int j = j_first + threadIdx.x; j < j_end; j += 256) out[hv + j] = os[j - j_first] * inv * norm[hv + j] * sigmoid_f(gate[hv + j]);
 }
 
-constexpr int MR_MAX_SEGMENTS = 8;
+constexpr int MR_MAX_SEGMENTS = 16;
 template <int LN, int CH, int W, int CB>
 void launch_rows(float* o, float* den, const float* q, const float* k, const float* v, const float* a, const float* b, float* state, float q_scale, int T, int heads, int dim,
                  int vdim, const int* pos_dev, int p0, float* scratch, cudaStream_t s) {
@@ -467,7 +467,7 @@ void mlstm_rows(float* o, float* den, const float* q, const float* k, const floa
         if (dim <= 16) NT_MR(4, 1, 4, 1);
         else if (dim <= 32) NT_MR(8, 1, 4, 2);
         else if (dim <= 64) NT_MR(16, 1, 4, 4);
-        else if (dim <= 128) NT_MR(16, 2, 4, 4);
+        else if (dim <= 128) NT_MR(32, 1, 4, 4);
         else if (dim <= 256) NT_MR(32, 2, 4, 4);
         else NT_MR(32, 4, 4, 2);
     } else {

@@ -4,7 +4,8 @@
 //   glu_bias_mul       out = act(gate + b_g) * (up + b_u)      (biases may be null)
 //   side_gate_rows     g[t, j] <- gelu_tanh(g[t, j]) * E[token_t, col0 + j]     (E: a second embedding table, any dense dtype)
 //   sandwich_norm_rows x[t] += rms(y[t]) * gain_y; h = rms(x[t]) * gain_h as F32 rows and / or the BF16 split of a GEMM's input: what lies between two
-//                      sublayers when a norm sits in front of and behind each; both rows are kept in registers
+//                      sublayers when a norm sits in front of and behind each; both rows are kept in registers.  sandwich_norm_router: one
+//                      decoded token's row, with the router's logits from the same launch
 //   sigmoid_gate_rows  o * sigmoid(gate), one gate per run of `per` channels, as F32 rows and / or the split
 //   relu2_rows         relu(z)^2, likewise
 // One CTA per row; a row is read twice (sum of squares, then the update), both times from L1/L2.
@@ -86,10 +87,12 @@ __device__ __forceinline__ float row_sum(float v, float* red) {        // over t
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float sq4(const float4& v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))); }
 
-// KEEP 16-byte pieces of the row per thread
-template <int KEEP>
-__global__ void __launch_bounds__(1024) sandwich_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ gain_y, const float* __restrict__ gain_h,
-                                                             float* __restrict__ h, __nv_bfloat16* __restrict__ hi, size_t lo, int width, float eps) {
+// KEEP 16-byte pieces of the row per thread.  ROUTER (one row): every CTA works out the whole row, the first one writes it (x_out is not x), and the CTAs
+// share the router's rows out: logits[e] = <router row e, h>.
+template <int KEEP, bool ROUTER>
+__global__ void __launch_bounds__(1024) sandwich_norm_kernel(float* x_out, const float* x, const float* __restrict__ y, const float* __restrict__ gain_y, const float* __restrict__ gain_h,
+                                                             float* __restrict__ h, __nv_bfloat16* __restrict__ hi, size_t lo, int width, float eps, const float* __restrict__ router,
+                                                             float* __restrict__ logits, int experts) {
     __shared__ float red[32];
     const int n = width / 4, nt = blockDim.x;
     float4 gy[KEEP], gh[KEEP];                     // constants: their way from memory overlaps the producer of y
@@ -99,9 +102,11 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(float* __restrict__
         gy[k] = (y && i < n) ? ld4(gain_y + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
         gh[k] = (gain_h && i < n) ? ld4(gain_h + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    if (ROUTER) for (int e = blockIdx.x; e < experts; e += gridDim.x) l2_prefetch(router + (size_t)e * width, (size_t)width * sizeof(float), threadIdx.x, nt);
     pdl_launch_dependents();
     pdl_wait();
-    const size_t row = (size_t)blockIdx.x * width;
+    const size_t row = ROUTER ? 0 : (size_t)blockIdx.x * width;
+    const bool writes = !ROUTER || blockIdx.x == 0;
     float4 xv[KEEP];
 #pragma unroll
     for (int k = 0; k < KEEP; k++) { const int i = threadIdx.x + k * nt; xv[k] = i < n ? ld4(x + row + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f); }
@@ -117,7 +122,7 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(float* __restrict__
             if (i >= n) continue;
             xv[k].x = fmaf(yv[k].x * inv, gy[k].x, xv[k].x); xv[k].y = fmaf(yv[k].y * inv, gy[k].y, xv[k].y);
             xv[k].z = fmaf(yv[k].z * inv, gy[k].z, xv[k].z); xv[k].w = fmaf(yv[k].w * inv, gy[k].w, xv[k].w);
-            *reinterpret_cast<float4*>(x + row + 4 * i) = xv[k];
+            if (writes) *reinterpret_cast<float4*>(x_out + row + 4 * i) = xv[k];
         }
     }
     if (!gain_h) return;
@@ -130,8 +135,21 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(float* __restrict__
         const int i = threadIdx.x + k * nt;
         if (i >= n) continue;
         const float v[4] = {xv[k].x * inv * gh[k].x, xv[k].y * inv * gh[k].y, xv[k].z * inv * gh[k].z, xv[k].w * inv * gh[k].w};
-        if (h) *reinterpret_cast<float4*>(h + row + 4 * i) = make_float4(v[0], v[1], v[2], v[3]);
+        if (h && writes) *reinterpret_cast<float4*>(h + row + 4 * i) = make_float4(v[0], v[1], v[2], v[3]);
         if (hi) split_store4(hi, hi + lo, row + 4 * (size_t)i, v);
+        if (ROUTER) xv[k] = make_float4(v[0], v[1], v[2], v[3]);
+    }
+    if (ROUTER) for (int e = blockIdx.x; e < experts; e += gridDim.x) {
+        float d = 0.f;
+#pragma unroll
+        for (int k = 0; k < KEEP; k++) {
+            const int i = threadIdx.x + k * nt;
+            if (i >= n) continue;
+            const float4 r = ld4(router + (size_t)e * width + 4 * i);
+            d = fmaf(r.x, xv[k].x, d); d = fmaf(r.y, xv[k].y, d); d = fmaf(r.z, xv[k].z, d); d = fmaf(r.w, xv[k].w, d);
+        }
+        d = row_sum(d, red);
+        if (threadIdx.x == 0) logits[e] = d;
     }
 }
 // any width and alignment
@@ -241,11 +259,26 @@ void sandwich_norm_rows(float* x, const float* y, const float* gain_y, const flo
     const int n = width / 4, most = rows == 1 ? 1024 : 256;        // one row: the whole row in flight at once
     const int threads = std::min(most, (n + 31) / 32 * 32), keep = (n + std::max(threads, 1) - 1) / std::max(threads, 1);
     if (width % 4 == 0 && (bits & 15) == 0 && keep <= 4) {
-#define NT_SN(K) launch_k(sandwich_norm_kernel<K>, dim3(rows), dim3(threads), 0, s, x, y, gain_y, gain_h, h, hi, lo, width, eps)
+#define NT_SN(K) launch_k(sandwich_norm_kernel<K, false>, dim3(rows), dim3(threads), 0, s, x, (const float*)x, y, gain_y, gain_h, h, hi, lo, width, eps, (const float*)nullptr, (float*)nullptr, 0)
         if (keep <= 1) NT_SN(1); else if (keep <= 2) NT_SN(2); else NT_SN(4);
 #undef NT_SN
     } else launch_k(sandwich_norm_any_kernel, dim3(rows), dim3(256), 0, s, x, y, gain_y, gain_h, h, hi, lo, width, eps);
     count_launch();
+}
+
+bool sandwich_norm_router(float* x_out, const float* x, const float* y, const float* gain_y, const float* gain_h, float* h, const float* router, float* logits, int experts, int width,
+                          float eps, cudaStream_t s) {
+    uintptr_t bits = 0;
+    for (const void* p : {(const void*)x_out, (const void*)x, (const void*)y, (const void*)gain_y, (const void*)gain_h, (const void*)h, (const void*)router}) bits |= reinterpret_cast<uintptr_t>(p);
+    const int n = width / 4, threads = std::min(1024, (n + 31) / 32 * 32), keep = (n + std::max(threads, 1) - 1) / std::max(threads, 1);
+    if (width % 4 != 0 || (bits & 15) != 0 || keep > 4 || keep < 1) return false;
+    NT_CHECK(x_out != x && y && gain_y && gain_h && h && experts >= 1, "sandwich_norm_router: a row of its own for the new residual, both norms and the router's rows");
+    const int grid = std::min(experts, 64);
+#define NT_SR(K) launch_k(sandwich_norm_kernel<K, true>, dim3(grid), dim3(threads), 0, s, x_out, x, y, gain_y, gain_h, h, (__nv_bfloat16*)nullptr, (size_t)0, width, eps, router, logits, experts)
+    if (keep <= 1) NT_SR(1); else if (keep <= 2) NT_SR(2); else NT_SR(4);
+#undef NT_SR
+    count_launch();
+    return true;
 }
 
 void sigmoid_gate_rows(float* out, void* split, const float* o, const float* gate, int ld, int per, int T, int cols, cudaStream_t s) {

@@ -140,6 +140,14 @@ enum : int { MODE_STORE = 0, MODE_ADD = 1, MODE_SWIGLU = 2, MODE_XIELU = 3, MODE
 // (maps_b[e], gate / up pairs: maps_b2[e]; encoded on the host, resident in device memory).  The tile list is made on the device from the counts.
 constexpr int MAX_GROUPS = 256;
 struct Grouped { const CUtensorMap* maps_b; const CUtensorMap* maps_b2; const int* start; const int* count; int experts; };
+// Several weight matrices over the same rows of A in one launch (MODE_STORE): matrix i's product goes to C[i] [M, N[i]]; its tiles are those up to
+// tile_end[i].  Narrow matrices leave SMs idle one by one and fill them together.
+struct alignas(64) Multi { CUtensorMap map[TC_MULTI_MAX]; float* C[TC_MULTI_MAX]; int N[TC_MULTI_MAX]; int tile_end[TC_MULTI_MAX]; };
+struct Plain {};
+enum : int { KIND_PLAIN = 0, KIND_GROUPED = 1, KIND_MULTI = 2 };
+template <int KIND> struct KindArg { using type = Plain; };
+template <> struct KindArg<KIND_GROUPED> { using type = Grouped; };
+template <> struct KindArg<KIND_MULTI> { using type = Multi; };
 
 // Persistent, warp-specialised GEMM: CTA b handles output tiles b, b + grid, ...; the shared-memory ring and the two TMEM
 // accumulators run across tile boundaries, so the epilogue of tile i overlaps the MMAs of tile i + 1.
@@ -154,14 +162,16 @@ struct Grouped { const CUtensorMap* maps_b; const CUtensorMap* maps_b2; const in
 //               F32 gate/up activations never touch HBM (ffn.cpp:96-133 computes them as three launches).
 //   MODE_XIELU  split_out = hi/lo split of xIELU(A.W^T), (p, q) = act_p: the ungated feed-forward's input of the down projection
 //   MODE_RELU2  the same with relu(z)^2
-template <int BN, int MODE, bool GROUPED>
+template <int BN, int MODE, int KIND>
 __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                                                              const __grid_constant__ CUtensorMap map_b,
                                                              const __grid_constant__ CUtensorMap map_b2,
                                                              float* __restrict__ C, __half* __restrict__ split_out,
                                                              int M, int Mp, int N, int K, int tiles_m, int tiles_n, int n_tiles, int n_outer,
                                                              int kc_blocks, int bf16, int gelu, const float* __restrict__ col_scale, float alpha,
-                                                             const float* __restrict__ act_p, const Grouped grp) {
+                                                             const float* __restrict__ act_p, const __grid_constant__ typename KindArg<KIND>::type grp) {
+    constexpr bool GROUPED = KIND == KIND_GROUPED, MULTI = KIND == KIND_MULTI;
+    static_assert(!MULTI || MODE == MODE_STORE, "several matrices: plain stores");
     constexpr bool ONE_CHUNK = MODE == MODE_SWIGLU || MODE == MODE_XIELU || MODE == MODE_RELU2;       // the epilogue needs the whole sum
     constexpr int STAGES = Cfg<BN>::STAGES, STAGE_BYTES = Cfg<BN>::STAGE_BYTES, TMEM_COLS = 2 * BN;
     constexpr int TN = MODE == MODE_SWIGLU ? 128 : BN;          // output columns per tile
@@ -174,7 +184,7 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
     __shared__ uint32_t tmem_base_smem;
     __shared__ int tile_end[GROUPED ? MAX_GROUPS : 1];          // grouped: tiles of the runs up to and including run e
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    if (GROUPED) {
+    if constexpr (GROUPED) {
         for (int e = threadIdx.x; e < grp.experts; e += 192) tile_end[e] = (grp.count[e] + BM - 1) / BM * tiles_n;
         __syncthreads();
         if (threadIdx.x == 0) for (int e = 1; e < grp.experts; e++) tile_end[e] += tile_end[e - 1];
@@ -183,10 +193,16 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
     }
     // tile -> its run (tiles ascend: the run is followed from the last one), first row, first column, one past the last live row
     auto place = [&](int tile, int& e, int& m0, int& n0, int& m_end) {
-        if (!GROUPED) { m0 = (n_outer ? tile % tiles_m : tile / tiles_n) * BM; n0 = (n_outer ? tile / tiles_m : tile % tiles_n) * TN; m_end = M; return; }
-        while (tile >= tile_end[e]) e++;
-        const int local = tile - (e ? tile_end[e - 1] : 0), cnt = grp.count[e], tm = (cnt + BM - 1) / BM;
-        m0 = grp.start[e] + local % tm * BM; n0 = local / tm * TN; m_end = grp.start[e] + cnt;
+        if constexpr (KIND == KIND_PLAIN) { m0 = (n_outer ? tile % tiles_m : tile / tiles_n) * BM; n0 = (n_outer ? tile / tiles_m : tile % tiles_n) * TN; m_end = M; }
+        else if constexpr (MULTI) {
+            while (tile >= grp.tile_end[e]) e++;
+            const int local = tile - (e ? grp.tile_end[e - 1] : 0);
+            m0 = local % tiles_m * BM; n0 = local / tiles_m * TN; m_end = M;
+        } else {
+            while (tile >= tile_end[e]) e++;
+            const int local = tile - (e ? tile_end[e - 1] : 0), cnt = grp.count[e], tm = (cnt + BM - 1) / BM;
+            m0 = grp.start[e] + local % tm * BM; n0 = local / tm * TN; m_end = grp.start[e] + cnt;
+        }
     };
     const int num_kb = K / BK;
     const int n_kc = ONE_CHUNK ? 1 : (num_kb + kc_blocks - 1) / kc_blocks;      // accumulation chunks per tile
@@ -211,13 +227,16 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
             int run = 0, m0 = 0, n0 = 0, m_end = 0, fenced = -1;
             for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
                 place(tile, run, m0, n0, m_end);
-                if (GROUPED && run != fenced) {        // maps in global memory: acquire them before this CTA's first use
-                    tensormap_acquire(grp.maps_b + run);
-                    if (MODE == MODE_SWIGLU) tensormap_acquire(grp.maps_b2 + run);
-                    fenced = run;
+                const CUtensorMap *mb = &map_b, *mb2 = &map_b2;
+                if constexpr (GROUPED) {
+                    mb = grp.maps_b + run; mb2 = grp.maps_b2 + run;
+                    if (run != fenced) {               // maps in global memory: acquire them before this CTA's first use
+                        tensormap_acquire(mb);
+                        if (MODE == MODE_SWIGLU) tensormap_acquire(mb2);
+                        fenced = run;
+                    }
                 }
-                const CUtensorMap* mb = GROUPED ? grp.maps_b + run : &map_b;
-                const CUtensorMap* mb2 = GROUPED ? grp.maps_b2 + run : &map_b2;
+                if constexpr (MULTI) mb = &grp.map[run];
                 for (int kb = 0; kb < num_kb; kb++, it++) {         // chunk boundaries do not matter to the producer
                     const uint32_t s = it % STAGES;
                     wait_or_trap(&empty_bar[s], ((it / STAGES) & 1) ^ 1);
@@ -324,11 +343,14 @@ __global__ void __launch_bounds__(192, 1) gemm_f16_tc_kernel(const __grid_consta
                     }
                 } else {
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    int Nc = N;
+                    float* Cc = C;
+                    if constexpr (MULTI) { Nc = grp.N[run]; Cc = grp.C[run]; }
                     if (row < m_end) {
-                        float* crow = C + (size_t)row * N + n0 + c * 32;
+                        float* crow = Cc + (size_t)row * Nc + n0 + c * 32;
 #pragma unroll
                         for (int j = 0; j < 32; j += 4) {
-                            if (n0 + c * 32 + j >= N) break;             // a ragged last tile (N % 4 == 0): TMA filled the missing weight rows with zeros
+                            if (n0 + c * 32 + j >= Nc) break;            // a ragged last tile (N % 4 == 0): TMA filled the missing weight rows with zeros
                             float4* dst = reinterpret_cast<float4*>(crow + j);
                             float4 o = make_float4(__uint_as_float(v[j]), __uint_as_float(v[j + 1]), __uint_as_float(v[j + 2]), __uint_as_float(v[j + 3]));
                             if (col_scale || alpha != 1.0f) {           // C (+)= alpha * col_scale[n] * acc: layer scale and residual multiplier
@@ -458,7 +480,7 @@ bool launch_gemm(float* C, __half* split_out, const void* workspace, const void*
         !make_map(&map_b2, W2 ? W2 : W, (uint64_t)N, (uint64_t)K, TN, o.bf16))
         return false;
     static unsigned long long configured = 0;      // bit per device id
-    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE, false>, (int)(Cfg<BN>::SMEM), configured);
+    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE, KIND_PLAIN>, (int)(Cfg<BN>::SMEM), configured);
     const int tiles_m = (int)(Mp / BM), tiles_n = (N + TN - 1) / TN, n_tiles = tiles_n * tiles_m;
     const int grid = n_tiles < sm_count() ? n_tiles : sm_count();
     // Tile order: concurrently running CTAs share the operand that is walked in the inner loop, the other one should stay
@@ -473,9 +495,9 @@ bool launch_gemm(float* C, __half* split_out, const void* workspace, const void*
     // 13.5k vs 17.6k on Q4_K_M: the read-modify-write of C per chunk is not free); NT_B200_GEMM_KC=<k-blocks> overrides (0: whole K)
     static const int kc_env = [] { const char* e = getenv("NT_B200_GEMM_KC"); return e ? atoi(e) : 64; }();
     const int kc_blocks = kc_env > 0 ? kc_env : K / BK;
-    gemm_f16_tc_kernel<BN, MODE, false><<<grid, 192, Cfg<BN>::SMEM, s>>>(map_a, map_b, map_b2, C, split_out, M, (int)Mp, N, K, tiles_m, tiles_n,
+    gemm_f16_tc_kernel<BN, MODE, KIND_PLAIN><<<grid, 192, Cfg<BN>::SMEM, s>>>(map_a, map_b, map_b2, C, split_out, M, (int)Mp, N, K, tiles_m, tiles_n,
                                                                         n_tiles, n_outer, kc_blocks, o.bf16 ? 1 : 0, o.relu ? 2 : (o.gelu ? 1 : 0), o.col_scale, o.alpha, o.act_p,
-                                                                        Grouped{});
+                                                                        Plain{});
     count_launch();
     return true;
 }
@@ -488,10 +510,10 @@ bool launch_grouped(float* C, __half* split_out, const void* workspace, const Gr
     CUtensorMap map_a;
     if (!make_map(&map_a, workspace, 2 * Mp, (uint64_t)K, BM, o.bf16)) return false;
     static unsigned long long configured = 0;
-    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE, true>, (int)(Cfg<BN>::SMEM), configured);
+    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE, KIND_GROUPED>, (int)(Cfg<BN>::SMEM), configured);
     const int tiles_n = (N + TN - 1) / TN;
     const int grid = (int)std::min<size_t>((size_t)sm_count(), Mp / BM * tiles_n);
-    gemm_f16_tc_kernel<BN, MODE, true><<<grid, 192, Cfg<BN>::SMEM, s>>>(map_a, map_a, map_a, C, split_out, 0, (int)Mp, N, K, 0, tiles_n, 0, 0, 64, o.bf16 ? 1 : 0,
+    gemm_f16_tc_kernel<BN, MODE, KIND_GROUPED><<<grid, 192, Cfg<BN>::SMEM, s>>>(map_a, map_a, map_a, C, split_out, 0, (int)Mp, N, K, 0, tiles_n, 0, 0, 64, o.bf16 ? 1 : 0,
                                                                        o.relu ? 2 : (o.gelu ? 1 : 0), nullptr, 1.0f, nullptr, grp);
     NT_LAUNCH_CHECK();
     count_launch();
@@ -510,6 +532,34 @@ bool gemm_f16_tc_ws(float* C, const void* workspace, const void* W_f16, int M, i
                    : launch_gemm<256, MODE_STORE>(C, nullptr, workspace, W_f16, nullptr, M, Mp, N, K, s, o);
     return add ? launch_gemm<128, MODE_ADD>(C, nullptr, workspace, W_f16, nullptr, M, Mp, N, K, s, o)
                : launch_gemm<128, MODE_STORE>(C, nullptr, workspace, W_f16, nullptr, M, Mp, N, K, s, o);
+}
+
+// C[i] [M, N[i]] = split(A)[M, K] . W[i]^T for n matrices with at least 256 rows each
+bool gemm_f16_tc_multi_ws(float* const* C, const void* workspace, const void* const* W, const int* N, int n, int M, int K, cudaStream_t s, const TcOpts& o) {
+    constexpr int BN = 256;
+    if (M <= 0 || n < 1 || n > TC_MULTI_MAX) return false;
+    const size_t Mp = ((size_t)M + BM - 1) / BM * BM;
+    Multi mu{};
+    CUtensorMap map_a;
+    if (!make_map(&map_a, workspace, 2 * Mp, (uint64_t)K, BM, o.bf16)) return false;
+    const int tiles_m = (int)(Mp / BM);
+    int tiles = 0;
+    for (int i = 0; i < TC_MULTI_MAX; i++) {
+        if (i < n) {
+            if (N[i] < BN || !gemm_f16_tc_ragged_supported(W[i], N[i], K, 0) || !make_map(&mu.map[i], W[i], (uint64_t)N[i], (uint64_t)K, BN, o.bf16)) return false;
+            mu.C[i] = C[i]; mu.N[i] = N[i];
+            tiles += (N[i] + BN - 1) / BN * tiles_m;
+        }
+        mu.tile_end[i] = tiles;
+    }
+    static unsigned long long configured = 0;
+    opt_in_dynamic_smem(gemm_f16_tc_kernel<BN, MODE_STORE, KIND_MULTI>, (int)(Cfg<BN>::SMEM), configured);
+    const int kc_blocks = 64;                      // accumulation chunk, as for one matrix
+    gemm_f16_tc_kernel<BN, MODE_STORE, KIND_MULTI><<<std::min(tiles, sm_count()), 192, Cfg<BN>::SMEM, s>>>(map_a, map_a, map_a, nullptr, nullptr, M, (int)Mp, 0, K, tiles_m, 0, tiles, 0,
+                                                                                                          kc_blocks, o.bf16 ? 1 : 0, 0, nullptr, 1.0f, nullptr, mu);
+    NT_LAUNCH_CHECK();
+    count_launch();
+    return true;
 }
 
 // workspace_out <- split(silu(A.Wgate^T) * (A.Wup^T)) for A already split into workspace_in; N = rows of Wgate/Wup

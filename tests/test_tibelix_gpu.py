@@ -108,6 +108,51 @@ def test_squared_relu_in_rows_and_in_the_product(M, N, K):
     np.testing.assert_allclose(joined(sp, M, N), ref, rtol=1e-3, atol=2e-4 * ref.max())
 
 
+def ptrs(ts):
+    return (C.c_void_p * len(ts))(*[t.data_ptr() for t in ts])
+
+
+@pytest.mark.parametrize("M,K,Ns", [(1, 64, [256, 260]), (130, 128, [512, 320, 256]), (300, 192, [256] * 6), (77, 64, [1000])])
+def test_several_products_of_the_same_rows_in_one_launch(M, K, Ns):
+    rng = np.random.default_rng(M)
+    A = rng.standard_normal((M, K))
+    Ws = [O.bf16_grid(rng.standard_normal((n, K)) * K ** -0.5) for n in Ns]
+    Wd, Cd, ws = [dev(W, torch.bfloat16) for W in Ws], [torch.full((M + 1, n), 7.0, device="cuda") for n in Ns], split_buffer(M, K)
+    rc = lib().nt_b200_gemm_multi(ptrs(Cd), dp(A), ptrs(Wd), (C.c_int * len(Ns))(*Ns), len(Ns), M, K, ws.data_ptr(), stream())
+    assert rc == 0
+    for c, W in zip(Cd, Ws):
+        np.testing.assert_allclose(host(c)[:M], A @ W.T, rtol=1e-3, atol=2e-4)
+        assert (host(c)[M] == 7.0).all()                                      # nothing behind the live rows
+    assert lib().nt_b200_gemm_multi(ptrs(Cd[:1]), dp(A), ptrs(Wd[:1]), (C.c_int * 1)(128), 1, M, K, ws.data_ptr(), stream()) == -1      # too narrow
+
+
+@pytest.mark.parametrize("width,experts", [(4, 1), (36, 5), (1024, 3), (2048, 16), (4100, 100), (8192, 256), (16384, 7)])
+def test_norms_around_a_sublayer_with_the_routers_logits(width, experts):
+    rng = np.random.default_rng(width)
+    eps = 1e-3
+    x, y, gy, gh = rng.standard_normal((1, width)), rng.standard_normal((1, width)) * 3, 1 + 0.3 * rng.standard_normal(width), 1 + 0.3 * rng.standard_normal(width)
+    R = rng.standard_normal((experts, width)) * width ** -0.5
+    x_ref = x + O.norm_plain(y, gy, eps)
+    h_ref = O.norm_plain(x_ref, gh, eps)
+    xd, xo, h, z = dev(x), torch.empty(1, width, device="cuda"), torch.empty(1, width, device="cuda"), torch.empty(experts, device="cuda")
+    assert lib().nt_b200_sandwich_norm_router(xo.data_ptr(), xd.data_ptr(), dp(y), dp(gy), dp(gh), h.data_ptr(), dp(R), z.data_ptr(), experts, width, eps, stream()) == 0
+    np.testing.assert_allclose(host(xo), x_ref, rtol=2e-5, atol=2e-5)
+    np.testing.assert_allclose(host(h), h_ref, rtol=3e-5, atol=3e-5)
+    np.testing.assert_allclose(host(z), (R @ h_ref[0]), rtol=1e-4, atol=1e-4)
+    np.testing.assert_array_equal(host(xd), host(dev(x)))
+    assert lib().nt_b200_sandwich_norm_router(xo.data_ptr(), xd.data_ptr(), dp(y), dp(gy), dp(gh), h.data_ptr(), dp(R), z.data_ptr(), experts, 7, eps, stream()) == -1
+
+
+@pytest.mark.parametrize("dt", [DType.F32, DType.BF16])
+@pytest.mark.parametrize("out,K", [(5, 13), (300, 64), (1, 1), (64, 1544), (2000, 768)])
+def test_a_product_of_a_normed_input(dt, out, K):
+    rng = np.random.default_rng(K)
+    W, x, g = O.bf16_grid(rng.standard_normal((out, K)) * K ** -0.5), rng.standard_normal((1, K)) * 5, 1 + 0.3 * rng.standard_normal(K)
+    y = torch.empty(out, device="cuda")
+    lib().nt_b200_gemv_normed(y.data_ptr(), dp(W, TORCH_DT[dt]), int(dt), dp(x), dp(g), 1e-2, out, K, stream())
+    np.testing.assert_allclose(host(y), W @ O.norm_plain(x, g, 1e-2)[0], rtol=3e-5, atol=3e-5)
+
+
 # ---------------------------------------------------------------- attention
 @pytest.mark.parametrize("dt", [DType.F32, DType.BF16])
 @pytest.mark.parametrize("H,G,D,V,every", [(2, 1, 8, 5, 4), (6, 3, 10, 7, 1), (1, 1, 1, 1, 7), (4, 2, 96, 64, 16), (3, 3, 33, 130, 1000), (2, 2, 7, 7, 2.5)])
@@ -231,6 +276,31 @@ def test_latent_values_with_an_output_gate(dt):
         lib().nt_b200_latent_v_up_gated(out.data_ptr(), dp(ol), dp(Wv, TORCH_DT[dt]), int(dt), T, H, V, r, dp(g), stream())
         ref = np.einsum("thr,hvr->thv", ol, Wv.reshape(H, V, r)).reshape(T, H * V) * O.sigmoid(g)
         np.testing.assert_allclose(host(out), ref, rtol=3e-5, atol=3e-5)
+
+
+@pytest.mark.parametrize("dt", [DType.F32, DType.BF16])
+@pytest.mark.parametrize("H,D,R,V,r,p0", [(3, 9, 8, 7, 16, 0), (2, 40, 16, 48, 64, 37), (5, 8, 8, 33, 40, 300), (20, 16, 32, 64, 480, 130), (1, 4, 8, 1, 8, 5)])
+def test_a_decoded_token_of_the_latent_attention(dt, H, D, R, V, r, p0):
+    """Absorbed queries with the cache row on the way, slices, merge with the gated values."""
+    rng = np.random.default_rng(r)
+    eps, rot, S = 1e-5, {"dims": R, "base": 700.0}, p0 + 1
+    c, kr = O.bf16_grid(rng.standard_normal((S, r))), O.bf16_grid(rng.standard_normal((S, R)))
+    dkv, gk, q, g = rng.standard_normal((1, r + R)), 1 + 0.2 * rng.standard_normal(r), rng.standard_normal((1, H, D + R)), rng.standard_normal((1, H * V)) * 2
+    Wk, Wv = O.bf16_grid(rng.standard_normal((H * D, r)) * r ** -0.5), O.bf16_grid(rng.standard_normal((H * V, r)) * r ** -0.5)
+    cache = dev(np.concatenate([c, kr], 1), TORCH_DT[dt])
+    cache[p0] = 99.0                                                          # overwritten by the token's own row
+    out, scale = torch.empty(H * V, device="cuda"), (D + R) ** -0.5
+    rc = lib().nt_b200_latent_token(out.data_ptr(), dp(q), dp(dkv), dp(gk), eps, cache.data_ptr(), int(dt), dp(Wk, TORCH_DT[dt]), dp(Wv, TORCH_DT[dt]), int(dt), p0, 1000, H, D, R, V, r, R,
+                                    700.0, scale, dp(g), stream())
+    assert rc == 0
+    own = np.concatenate([O.norm_plain(dkv[:, :r], gk, eps), O.rotate_pairs(dkv[:, r:], [p0], rot)], 1)
+    np.testing.assert_allclose(host(cache)[p0:], own, **(dict(rtol=3e-5, atol=3e-5) if dt == DType.F32 else dict(rtol=8e-3, atol=8e-3)))
+    rows = host(cache)
+    k, v = np.einsum("sr,hdr->shd", rows[:, :r], Wk.reshape(H, D, r)), np.einsum("sr,hvr->shv", rows[:, :r], Wv.reshape(H, V, r))
+    qr = O.rotate_pairs(q[:, :, D:], [p0], rot)
+    s = (np.einsum("hd,shd->hs", q[0, :, :D], k) + np.einsum("hd,sd->hs", qr[0], rows[:, r:])) * scale
+    ref = np.einsum("hs,shv->hv", O.softmax_rows(s, np.ones_like(s, dtype=bool)), v).reshape(-1) * O.sigmoid(g[0])
+    np.testing.assert_allclose(host(out), ref, rtol=2e-4, atol=1e-4)
 
 
 # ---------------------------------------------------------------- matrix memory
@@ -432,6 +502,8 @@ CONFIGS = {
                               ff=192, experts=4, top=2, groups=(2, 1), eff=128, shared=128),
     "tensor_core_tiles_ragged": dict(width=192, vocab=100, heads=6, kv_heads=2, dim=96, vdim=96, l_heads=3, l_dim=64, rot_dim=32, l_vdim=80, q_rank=192, kv_rank=96, m_heads=3, m_dim=64,
                                      m_vdim=64, ff=320, experts=6, top=3, groups=(3, 2), eff=64, shared=192),
+    "wide_projections_in_one_launch": dict(pattern=(ML, LA, AT, ML), mlp=("moe",), width=128, vocab=90, heads=8, kv_heads=4, dim=64, vdim=128, l_heads=8, l_dim=32, rot_dim=32, l_vdim=64,
+                                           q_rank=256, kv_rank=224, m_heads=4, m_dim=64, m_vdim=96, experts=8, top=3, groups=(4, 2), eff=128, shared=256),
     "sixty_four_gate_rows": dict(pattern=(ML, AT), mlp=("dense",), width=128, m_heads=64, m_dim=4, m_vdim=4, heads=8, kv_heads=2, dim=64, vdim=128, ff=128),
 }
 
