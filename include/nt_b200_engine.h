@@ -171,6 +171,11 @@ void nt_b200_head_prep_unit(float* Q, const float* K, const float* V, int heads,
 /* Causal grouped-query attention with a distance bias (slopes [heads] or null), a per-head sink (or null) and an output gate (raw [tokens, heads] or null) */
 void nt_b200_attention_biased(float* out, const float* Q, const void* kc, const void* vc, int cache_dtype, int tokens, int p0, int max_seq, int heads, int kv_heads, int dim,
                               int vdim, float scale, const float* slopes, const float* sink, const float* gate, void* stream);
+/* One decoded token of the same over BF16 rows, the query heads of a key head served together; window 0: all positions; kc == vc: values are the first vdim
+ * numbers of the key rows.  scratch: nt_b200_attention_rows_decode_scratch_floats numbers.  -1: shape not covered */
+int nt_b200_attention_rows_decode(float* out, const float* Q, const void* kc, const void* vc, int p0, int max_seq, int heads, int kv_heads, int dim, int vdim, int k_stride, int v_stride,
+                                  float scale, int window, const float* slopes, const float* sink, const float* gate, float* scratch, void* stream);
+long long nt_b200_attention_rows_decode_scratch_floats(int heads, int vdim);
 /* The latent attention's cache rows and absorbed queries with a frequency table (freq: device, dims / 2 doubles; host side: nt_b200_rotary_table64) */
 double nt_b200_rotary_table64(double* freq_host, int dims, double base, double factor, double original, double fast, double slow);
 void nt_b200_latent_rotated(float* cq, int q_rank, const float* q_gain, const float* dkv, int kv_rank, int rot_dim, const float* kv_gain, float eps, void* cache, int cache_dtype,

@@ -23,7 +23,7 @@ COMMON = ["-std=c++17", "-O3", "-lineinfo", "--use_fast_math", "-Xcompiler", "-f
           "-ccbin", shutil.which("g++") or "g++"]
 # Kernels whose 32-bit mode must be exact to rounding (tanh / exp / division at full precision): no --use_fast_math.
 PRECISE = {"dense.cu", "attention_window.cu", "attention_diff.cu", "moe.cu", "attention_latent.cu", "ssm_scan.cu", "postnorm.cu",
-           "short_conv.cu", "delta_rule.cu", "sumnorm.cu", "attention_heads.cu", "depth_rows.cu", "wkv.cu", "mlstm.cu"}
+           "short_conv.cu", "delta_rule.cu", "sumnorm.cu", "attention_heads.cu", "depth_rows.cu", "wkv.cu", "mlstm.cu", "attention_rows_decode.cu"}
 
 
 def _nvcc() -> str:

@@ -422,18 +422,26 @@ __global__ void __launch_bounds__(256) latent_shared_attn_kernel(float* __restri
     }
 }
 
+// slices that hold anything at position pos: slice s starts with the s-th tile of the visible positions
+__device__ __forceinline__ int live_slices(int n_slices, int tile, int pos, int window) {
+    const int n_vis = window > 0 ? min(pos + 1, window) : pos + 1;
+    return min(n_slices, (n_vis + tile - 1) / tile);
+}
+
 // grid (tokens, heads, ceil(vdim / 64)): out [t, h, :] = sum_s acc_s exp(m_s - M) / sum_s l_s exp(m_s - M).  Thread (channel, g) sums
 // every fourth slice of its channel; the four partial sums meet in shared memory.
-__global__ void __launch_bounds__(256) latent_shared_merge_kernel(float* __restrict__ out, const float* __restrict__ part, int n_slices, int heads, int vdim) {
+__global__ void __launch_bounds__(256) latent_shared_merge_kernel(float* __restrict__ out, const float* __restrict__ part, int n_slices, int heads, int vdim, int tile,
+                                                                  const int* __restrict__ pos_dev, int p0, int window, const float* __restrict__ sink, const float* __restrict__ gate) {
     extern __shared__ __align__(16) float wsm[];           // [n_slices]
     __shared__ float red[8];
     __shared__ float sums[4][64];
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x, h = blockIdx.y;
-    const float* base = part + ((size_t)t * n_slices * heads + h) * (vdim + 2);
+    const int t = blockIdx.x, h = blockIdx.y, stored = n_slices;
+    n_slices = live_slices(n_slices, tile, (pos_dev ? *pos_dev : p0) + t, window);
+    const float* base = part + ((size_t)t * stored * heads + h) * (vdim + 2);
     const size_t step = (size_t)heads * (vdim + 2);
-    float mx = -FLT_MAX;
+    float mx = sink ? sink[h] : -FLT_MAX;                  // the sink joins the denominator as one more term
     for (int s = threadIdx.x; s < n_slices; s += 256) mx = fmaxf(mx, base[s * step]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, o));
@@ -444,7 +452,9 @@ __global__ void __launch_bounds__(256) latent_shared_merge_kernel(float* __restr
     for (int w = 0; w < 8; w++) M = fmaxf(M, red[w]);
     float ls = 0.f;
     for (int s = threadIdx.x; s < n_slices; s += 256) { const float w = expf(base[s * step] - M); wsm[s] = w; ls = fmaf(base[s * step + 1], w, ls); }
-    const float L = block_sum_256(ls, red);                // its barriers also publish wsm
+    float L = block_sum_256(ls, red);                      // its barriers also publish wsm
+    if (sink) L += expf(sink[h] - M);
+    const float k = gate ? 1.0f / (L * (1.0f + expf(-gate[h]))) : 1.0f / L;
     const int cl = threadIdx.x & 63, g = threadIdx.x >> 6, c = blockIdx.z * 64 + cl;
     float v = 0.f;
     if (c < vdim) {
@@ -453,14 +463,14 @@ __global__ void __launch_bounds__(256) latent_shared_merge_kernel(float* __restr
     }
     sums[g][cl] = v;
     __syncthreads();
-    if (g == 0 && c < vdim) out[((size_t)t * heads + h) * vdim + c] = ((sums[0][cl] + sums[1][cl]) + (sums[2][cl] + sums[3][cl])) / L;
+    if (g == 0 && c < vdim) out[((size_t)t * heads + h) * vdim + c] = ((sums[0][cl] + sums[1][cl]) + (sums[2][cl] + sums[3][cl])) * k;
 }
 
 // The merge for one query with the up-projection of the values behind it: grid (1, heads, ceil(v_up / 32)).  Every CTA of a head joins the head's slices
 // itself (they come from L2), then a warp per output channel.
 template <typename WT>
-__global__ void __launch_bounds__(256) latent_merge_up_kernel(float* __restrict__ out, const float* __restrict__ part, int n_slices, int heads, int vdim, const WT* __restrict__ W_uv,
-                                                              int v_up, const float* __restrict__ gate) {
+__global__ void __launch_bounds__(256) latent_merge_up_kernel(float* __restrict__ out, const float* __restrict__ part, int n_slices, int heads, int vdim, int tile,
+                                                              const int* __restrict__ pos_dev, int p0, int window, const WT* __restrict__ W_uv, int v_up, const float* __restrict__ gate) {
     extern __shared__ __align__(16) float sm_mu[];         // slice weights [n_slices] | joined vector [vdim]
     __shared__ float red[8];
     const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, v0 = blockIdx.z * 32, v1 = min(v_up, v0 + 32);
@@ -468,6 +478,7 @@ __global__ void __launch_bounds__(256) latent_merge_up_kernel(float* __restrict_
     l2_prefetch(W_uv + ((size_t)h * v_up + v0) * vdim, (size_t)(v1 - v0) * vdim * sizeof(WT), threadIdx.x, 256);
     pdl_launch_dependents();
     pdl_wait();
+    n_slices = live_slices(n_slices, tile, pos_dev ? *pos_dev : p0, window);
     const float* base = part + (size_t)h * (vdim + 2);
     const size_t step = (size_t)heads * (vdim + 2);
     float mx = -FLT_MAX;
@@ -631,18 +642,28 @@ void attention_shared_rows(float* out, const float* Q, const void* cache, DType 
     for (int t0 = 0; t0 < tokens; t0 += LS_MAX_PARTS) {           // long portions (exact mode): blocks of queries with one slice each
         const int nt = std::min(LS_MAX_PARTS, tokens - t0);
         const int slices = shared_rows_slices(scratch, Q + (size_t)t0 * heads * dim, cache, cache_dt, nt, pos_dev, p0 + t0, max_seq, heads, dim, vdim, row, scale, window, s);
-        launch_k(latent_shared_merge_kernel, dim3(nt, heads, (vdim + 63) / 64), dim3(256), sizeof(float) * slices, s, out + (size_t)t0 * heads * vdim, (const float*)scratch, slices, heads, vdim);
+        launch_k(latent_shared_merge_kernel, dim3(nt, heads, (vdim + 63) / 64), dim3(256), sizeof(float) * slices, s, out + (size_t)t0 * heads * vdim, (const float*)scratch, slices, heads, vdim,
+                 LS_KEYS, pos_dev, p0 + t0, window, (const float*)nullptr, (const float*)nullptr);
         count_launch();
     }
+}
+
+void attention_slices_merge(float* out, const float* part, int n_slices, int tile, const int* pos_dev, int p0, int window, int heads, int vdim, const float* sink, const float* gate,
+                            cudaStream_t s) {
+    launch_k(latent_shared_merge_kernel, dim3(1, heads, (vdim + 63) / 64), dim3(256), sizeof(float) * n_slices, s, out, part, n_slices, heads, vdim, tile, pos_dev, p0, window, sink, gate);
+    count_launch();
 }
 
 void attention_shared_rows_up(float* out, const float* Q, const void* cache, DType cache_dt, const int* pos_dev, int p0, int max_seq, int heads, int dim, int vdim, int row, float scale,
                               float* scratch, const void* W_uv, DType wdt, int v_up, const float* gate, cudaStream_t s, int window) {
     NT_CHECK(attention_shared_rows_supported(heads, dim, vdim, row, cache_dt, cache) && dense_dtype(wdt), "attention_shared_rows_up: shape not covered");
-    const int slices = shared_rows_slices(scratch, Q, cache, cache_dt, 1, pos_dev, p0, max_seq, heads, dim, vdim, row, scale, window, s);
+    const bool tiles = attention_rows_decode_supported(heads, 1, dim, vdim, row, row, cache_dt, cache, cache);       // the tensor-core form
+    const int slices = tiles ? attention_rows_decode(scratch, Q, cache, cache, pos_dev, p0, max_seq, heads, 1, dim, vdim, row, row, scale, window, nullptr, s)
+                             : shared_rows_slices(scratch, Q, cache, cache_dt, 1, pos_dev, p0, max_seq, heads, dim, vdim, row, scale, window, s);
+    const int tile = tiles ? ROWS_DECODE_TILE : LS_KEYS;
     const size_t smem = sizeof(float) * ((size_t)((slices + 3) & ~3) + (size_t)vdim);
     const dim3 grid(1, heads, (v_up + 31) / 32);
-#define NT_MU(TY) launch_k(latent_merge_up_kernel<TY>, grid, dim3(256), smem, s, out, (const float*)scratch, slices, heads, vdim, static_cast<const TY*>(W_uv), v_up, gate)
+#define NT_MU(TY) launch_k(latent_merge_up_kernel<TY>, grid, dim3(256), smem, s, out, (const float*)scratch, slices, heads, vdim, tile, pos_dev, p0, window, static_cast<const TY*>(W_uv), v_up, gate)
     if (wdt == DType::F32) NT_MU(float); else if (wdt == DType::F16) NT_MU(__half); else NT_MU(__nv_bfloat16);
 #undef NT_MU
     count_launch();

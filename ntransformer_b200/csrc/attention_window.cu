@@ -232,6 +232,14 @@ void attention_window(float* out, const float* Q, const void* kc, const void* vc
                       int max_seq, const WindowAttn& a, cudaStream_t s) {
     static const bool no_mma = getenv("NT_B200_NO_WINDOW_MMA") != nullptr;
     if (!pos_dev && !no_mma && attention_window_mma_supported(tokens, a, cache_dt)) { attention_window_mma(out, Q, kc, vc, tokens, p0, max_seq, a, s); return; }
+    if (tokens == 1 && a.scratch && a.maps == 1 && !a.joint_v && a.keep == 0 && a.chunk == 0 && a.softcap == 0.f) {
+        const int ks = a.k_stride > 0 ? a.k_stride : a.kv_heads * a.dim, vs = a.v_stride > 0 ? a.v_stride : a.kv_heads * a.vdim;
+        if (attention_rows_decode_supported(a.heads, a.kv_heads, a.dim, a.vdim, ks, vs, cache_dt, kc, vc)) {
+            const int n = attention_rows_decode(a.scratch, Q, kc, vc, pos_dev, p0, max_seq, a.heads, a.kv_heads, a.dim, a.vdim, ks, vs, a.scale, a.window, a.slope, s);
+            attention_slices_merge(out, a.scratch, n, ROWS_DECODE_TILE, pos_dev, p0, a.window, a.heads, a.vdim, a.sink, a.head_gate, s);
+            return;
+        }
+    }
     NT_CHECK(a.vdim <= 512, "attention_window: value heads wider than 512 are not covered");
     NT_CHECK(a.heads % a.kv_heads == 0, "attention_window: heads must be a multiple of kv_heads");
     NT_CHECK(cache_dt == DType::F32 || cache_dt == DType::BF16, "attention_window: F32 or BF16 cache");

@@ -572,6 +572,19 @@ void nt_b200_attention_biased(float* out, const float* Q, const void* kc, const 
     a.heads = heads; a.kv_heads = kv_heads; a.dim = dim; a.vdim = vdim; a.scale = scale; a.slope = slopes; a.sink = sink; a.head_gate = gate; a.gate_stride = heads;
     attention_window(out, Q, kc, vc, (nt::DType)cache_dtype, tokens, nullptr, p0, max_seq, a, static_cast<cudaStream_t>(stream));
 }
+// One decoded token of the same over BF16 rows, query heads of a key head served together (attention_rows_decode.cu); window 0: all positions.
+// scratch: nt_b200_attention_rows_decode_scratch_floats numbers.  -1: shape not covered
+int nt_b200_attention_rows_decode(float* out, const float* Q, const void* kc, const void* vc, int p0, int max_seq, int heads, int kv_heads, int dim, int vdim, int k_stride, int v_stride,
+                                  float scale, int window, const float* slopes, const float* sink, const float* gate, float* scratch, void* stream) {
+    if (!attention_rows_decode_supported(heads, kv_heads, dim, vdim, k_stride, v_stride, nt::DType::BF16, kc, vc)) return -1;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const int n = attention_rows_decode(scratch, Q, kc, vc, nullptr, p0, max_seq, heads, kv_heads, dim, vdim, k_stride, v_stride, scale, window, slopes, s);
+    attention_slices_merge(out, scratch, n, ROWS_DECODE_TILE, nullptr, p0, window, heads, vdim, sink, gate, s);
+    return 0;
+}
+long long nt_b200_attention_rows_decode_scratch_floats(int heads, int vdim) {
+    return (long long)attention_rows_decode_scratch_floats(heads, vdim);
+}
 // The latent attention's cache rows and absorbed queries with a frequency table (freq: device, dims / 2 doubles; host side: nt_b200_rotary_table64)
 double nt_b200_rotary_table64(double* freq_host, int dims, double base, double factor, double original, double fast, double slow) {
     return rotary_table(freq_host, dims, base, factor, original, fast, slow);

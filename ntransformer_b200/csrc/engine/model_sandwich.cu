@@ -6,7 +6,7 @@
 //
 // Everything between two sublayers — norm of the output, residual sum, norm of the next input — is one launch (sandwich_norm_rows), so a decoded
 // token takes
-//   attention layer, 5:  [q, k, v, gate rows]  [head norm, query multiplier, cache write]  [attention, gated]  [W_o]  [between]
+//   attention layer, 6:  [q, k, v, gate rows]  [head norm, query multiplier, cache write]  [attention]  [merge, gated]  [W_o]  [between]
 //   latent layer, 7:     [query latent, key / value latent, gate]  [queries from the normed latent]  [absorbed queries + cache row]  [attention]
 //                        [merge + values, gated]  [W_o]  [between]
 //   matrix memory, 4:    [q, k, v, gate, input / forget gate rows]  [gates, memory, head norm, output gate]  [W_o]  [between]
@@ -226,7 +226,7 @@ void Model::sandwich_mixer_token(int i, float* y, cudaStream_t s) {
         void *kc = kcs_[(size_t)i], *vc = vcs_[(size_t)i];
         head_prep(q, k, v, head_prep_of(S, eps), kc, vc, cache_dt_, 1, pos_dev, 0, s);
         WindowAttn a = biased_attn_of(S, L);
-        a.head_gate = g; a.gate_stride = S.heads;
+        a.head_gate = g; a.gate_stride = S.heads; a.scratch = lat_part_;
         attention_window(o, q, kc, vc, cache_dt_, 1, pos_dev, 0, cfg_.max_seq_len, a, s);
     } else if (S.mixer == MixerKind::ATTN_LATENT) {
         const LatentSpec& A = S.latent;

@@ -390,6 +390,7 @@ bool Model::finalize_spec() {
         size_t parts = 0;                          // per-slice partial results of the attention that serves all heads from one copy of the rows
         for (const LayerSpec& S : cfg_.layers)
             if (S.mixer == MixerKind::ATTN_LATENT) parts = std::max(parts, attention_shared_rows_scratch_floats(S.heads, S.latent.kv_rank));
+            else if (S.form == BlockForm::SANDWICH && S.mixer == MixerKind::ATTN_WINDOW) parts = std::max(parts, attention_rows_decode_scratch_floats(S.heads, S.vdim));
         if (parts) { lat_part_ = dmalloc<float>(parts); owned_.push_back(lat_part_); }
     }
     hidden_ = dmalloc<float>(hidden);

@@ -191,6 +191,7 @@ struct WindowAttn {
     const float* slope = nullptr;      // [heads] (device): slope[h] * (i - j) is taken off head h's scaled score
     const float* head_gate = nullptr;  // [tokens, heads] (device): head h's result is multiplied by sigmoid(head_gate[t * gate_stride + h])
     int gate_stride = 0;
+    float* scratch = nullptr;          // attention_rows_decode_scratch_floats (device): lets one decoded token take attention_rows_decode.cu
     int joint_v = 0;                   // 1: every query head sums ONE value row per key, vdim wide, at the start of the key's value row (whatever its
                                        // key head): with vdim = kv_heads * (a head's width) each head's weights are applied to every value head at once
 };
@@ -200,6 +201,17 @@ struct WindowAttn {
 // with dim == vdim in {64, 128} take attention_prefill_mma.cu's tiles, everything else one CTA per (token, head).
 void attention_window(float* out, const float* Q, const void* kc, const void* vc, DType cache_dt, int tokens, const int* pos_dev, int p0,
                       int max_seq, const WindowAttn& a, cudaStream_t s);
+// attention_rows_decode.cu: one query over BF16 rows, the query heads of a key head served together; slices of the positions -> part [slice, heads, vdim + 2]
+// (max, sum, unnormalised vector); returns the number of slices.  k == v: values are the first vdim numbers of the key rows.
+constexpr int ROWS_DECODE_TILE = 64, ROWS_DECODE_MAX_SLICES = 148;
+bool attention_rows_decode_supported(int heads, int kv_heads, int dim, int vdim, int k_stride, int v_stride, DType cache_dt, const void* k, const void* v);
+int attention_rows_decode_slices(int max_seq, int kv_heads, int window);
+size_t attention_rows_decode_scratch_floats(int heads, int vdim);
+int attention_rows_decode(float* part, const float* Q, const void* k, const void* v, const int* pos_dev, int p0, int max_seq, int heads, int kv_heads, int dim, int vdim, int k_stride,
+                          int v_stride, float scale, int window, const float* slopes, cudaStream_t s);
+// Joins the slices: out [heads, vdim] (attention_latent.cu); sink, gate [heads] or null as in WindowAttn
+void attention_slices_merge(float* out, const float* part, int n_slices, int tile, const int* pos_dev, int p0, int window, int heads, int vdim, const float* sink, const float* gate,
+                            cudaStream_t s);
 bool attention_window_mma_supported(int tokens, const WindowAttn& a, DType cache_dt);
 void attention_window_mma(float* out, const float* Q, const void* kc, const void* vc, int tokens, int p0, int max_seq, const WindowAttn& a,
                           cudaStream_t s);

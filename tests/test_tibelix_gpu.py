@@ -235,6 +235,38 @@ def test_a_far_key_outweighs_the_bias_by_exactly_its_distance(at, D):
     assert not np.allclose(run_biased(q, k, v, 1.0, slope, None, DType.F32, [S], unit_sink=False), ref, atol=1e-2)      # the sink shows
 
 
+@pytest.mark.parametrize("H,G,D,V", [(2, 1, 16, 16), (6, 2, 48, 32), (4, 4, 64, 64), (16, 4, 128, 128), (20, 1, 96, 96), (32, 1, 64, 512), (17, 1, 32, 144), (8, 1, 320, 256), (32, 1, 576, 512)])
+@pytest.mark.parametrize("joint", [False, True])
+def test_one_decoded_token_with_the_heads_of_a_key_head_together(H, G, D, V, joint):
+    """Positions at the first token, around tile borders and where slices wrap over several tiles; distance bias, sink and gate on and off; a window;
+    values in rows of their own or at the start of the key rows."""
+    if (joint and (G > 1 or V > D)) or (not joint and D + V > 1000):
+        pytest.skip("values at the start of the key rows: one key head, values no wider than the keys; the widest rows fit shared memory in that form only")
+    rng = np.random.default_rng(H + D)
+    S, max_seq, scale = 700, 1024, D ** -0.5
+    k = O.bf16_grid(rng.standard_normal((S, G, D)))
+    v = k[:, :, :V] if joint else O.bf16_grid(rng.standard_normal((S, G, V)))
+    kc = dev(k, torch.bfloat16)
+    vc = kc if joint else dev(v, torch.bfloat16)
+    scratch = torch.full((lib().nt_b200_attention_rows_decode_scratch_floats(H, V),), float("nan"), device="cuda")
+    slopes, zeros = O.slopes(H), np.zeros(H)
+    for pos in (0, 1, 15, 62, 63, 64, 65, 127, 128, 500, 699):
+        q, gate = rng.standard_normal((1, H, D)), rng.standard_normal(H)
+        for window, seq, full in ((0, max_seq, True), (0, 64, False), (37, max_seq, False), (64, max_seq, True), (300, max_seq, False)):
+            lo = max(0, pos + 1 - window) if window else 0
+            ref = np.zeros((H, V))
+            for h in range(H):
+                g = h // (H // G)
+                s = k[lo:pos + 1, g] @ q[0, h] * scale - full * slopes[h] * (pos - np.arange(lo, pos + 1))
+                ones = np.ones((1, len(s)), dtype=bool)
+                ref[h] = (O.sink_softmax(s[None], ones) if full else O.softmax_rows(s[None], ones))[0] @ v[lo:pos + 1, g] * (O.sigmoid(gate[h]) if full else 1.0)
+            out = torch.empty(H, V, device="cuda")
+            rc = lib().nt_b200_attention_rows_decode(out.data_ptr(), dp(q), kc.data_ptr(), vc.data_ptr(), pos, seq, H, G, D, V, G * D, G * D if joint else G * V, scale, window,
+                                                     dp(slopes) if full else None, dp(zeros) if full else None, dp(gate) if full else None, scratch.data_ptr(), stream())
+            assert rc == 0
+            np.testing.assert_allclose(host(out), ref, rtol=3e-4, atol=3e-4)
+
+
 def table64(rot):
     sc = rot.get("scaling")
     f = np.zeros(max(1, rot["dims"] // 2))
