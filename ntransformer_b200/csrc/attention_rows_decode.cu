@@ -10,6 +10,7 @@
 // The grid depends on the cache's length only, never on the position: the captured decode step replays it unchanged.
 // Compiled WITHOUT --use_fast_math.
 #include "kernels_internal.h"
+#include "bf16_split.cuh"
 #include "ring.cuh"
 #include <cuda_bf16.h>
 #include <algorithm>
@@ -67,26 +68,30 @@ __global__ void __launch_bounds__(256) rows_decode_kernel(float* __restrict__ pa
     const int pos = pos_dev ? *pos_dev : p0, lo = window > 0 ? max(0, pos + 1 - window) : 0, n_vis = pos + 1 - lo;
     auto load_tile = [&](int t0) {
         const int ck = dim / 8, cv = vdim / 8;
-        for (int i = threadIdx.x; i < TK * ck; i += 256) {
-            const int r = i / ck, c = i - r * ck, j = lo + min(t0 + r, n_vis - 1);      // rows past the last visible one are masked below
-            cp16(kt + (size_t)r * ldq + c * 8, kc + (size_t)j * k_stride + (size_t)g0 * dim + c * 8);
-        }
-        if (!same)
-            for (int i = threadIdx.x; i < TK * cv; i += 256) {
-                const int r = i / cv, c = i - r * cv, j = lo + min(t0 + r, n_vis - 1);
-                cp16(vt + (size_t)r * ldv + c * 8, vc + (size_t)j * v_stride + (size_t)g0 * vdim + c * 8);
+        // 8 or 32 lanes per row: no division, whole sectors
+        const int lanes = ck <= 16 ? 8 : 32, l0 = threadIdx.x & (lanes - 1), rows_at_once = 256 / lanes;
+        for (int r = threadIdx.x / lanes; r < TK; r += rows_at_once) {
+            const int j = lo + min(t0 + r, n_vis - 1);                         // rows past the last visible one are masked below
+            const __nv_bfloat16* src = kc + (size_t)j * k_stride + (size_t)g0 * dim;
+            for (int c = l0; c < ck; c += lanes) cp16(kt + (size_t)r * ldq + c * 8, src + c * 8);
+            if (!same) {
+                const __nv_bfloat16* vs = vc + (size_t)j * v_stride + (size_t)g0 * vdim;
+                for (int c = l0; c < cv; c += lanes) cp16(vt + (size_t)r * ldv + c * 8, vs + c * 8);
             }
+        }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     int t0 = slice * TK;
     if (t0 < n_vis) load_tile(t0);
     if (t0 < n_vis)
-        for (int i = threadIdx.x; i < ROWS * dim; i += 256) {
-            const int r = i / dim, c = i - r * dim;
-            const float v = r < group ? Q[((size_t)g0 * group + r) * dim + c] : 0.f;
-            const __nv_bfloat16 hb = __float2bfloat16_rn(v);
-            qh[(size_t)r * ldq + c] = hb;
-            ql[(size_t)r * ldq + c] = __float2bfloat16_rn(v - __bfloat162float(hb));
+        for (int r = warp; r < ROWS; r += 8) {
+            const float* q = Q + ((size_t)g0 * group + r) * dim;
+#pragma unroll 2
+            for (int c = lane * 4; c < dim; c += 128) {
+                float v[4] = {0.f, 0.f, 0.f, 0.f};
+                if (r < group) { const float4 f = *reinterpret_cast<const float4*>(q + c); v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w; }
+                split_store4(qh, ql, (size_t)r * ldq + c, v);
+            }
         }
     const int srow = threadIdx.x / TPR, sl = threadIdx.x % TPR;
     const float slope = slopes && srow < group ? slopes[g0 * group + srow] : 0.f;
@@ -225,6 +230,7 @@ size_t attention_rows_decode_scratch_floats(int heads, int vdim) { return (size_
 int attention_rows_decode(float* part, const float* Q, const void* k, const void* v, const int* pos_dev, int p0, int max_seq, int heads, int kv_heads, int dim, int vdim, int k_stride,
                           int v_stride, float scale, int window, const float* slopes, cudaStream_t s) {
     NT_CHECK(attention_rows_decode_supported(heads, kv_heads, dim, vdim, k_stride, v_stride, DType::BF16, k, v), "attention_rows_decode: shape not covered");
+    NT_CHECK((reinterpret_cast<uintptr_t>(Q) & 15) == 0, "attention_rows_decode: the queries must start on 16 bytes");
     const int mt = heads / kv_heads > 16 ? 2 : 1, slices = attention_rows_decode_slices(max_seq, kv_heads, window);
     const size_t smem = smem_bytes(mt, dim, vdim, k == v);
     const __nv_bfloat16 *kb = static_cast<const __nv_bfloat16*>(k), *vb = static_cast<const __nv_bfloat16*>(v);
