@@ -12,6 +12,7 @@
 //   value width go to the tiled tensor-core form in attention_prefill_mma.cu instead.
 // WindowAttn::sink adds exp(sink_h) to head h's denominator (a learned term without key or value); WindowAttn::joint_v makes every query
 // head sum one value row per key that spans all value heads, which attention_heads.cu's talk_mix turns into head-mixed softmax weights.
+// WindowAttn::scratch lets one decoded token over BF16 rows take attention_rows_decode.cu where the shape fits it.
 // WindowAttn::slope takes slope_h * (i - j) off the scaled (and capped) score; WindowAttn::head_gate multiplies head h's result by sigmoid(gate).
 // Compiled WITHOUT --use_fast_math (tanhf / expf at full precision).
 #include "kernels_internal.h"

@@ -263,7 +263,6 @@ void Model::sandwich_ff_token(int i, float* y, bool with_logits, cudaStream_t s)
     auto take = [&](size_t n) { float* p = dec_.wide + cur; cur += up4(n); return p; };
     SumTerm t[2];
     int nt = 0;
-    DType dt = L.wo.dtype;
     if (S.ff_kind == FfKind::MLP) {
         float* a = take((size_t)S.ff);
         const MultiMat m = multi(L.up, h, a, GEMV_ACT_RELU2);
@@ -284,7 +283,7 @@ void Model::sandwich_ff_token(int i, float* y, bool with_logits, cudaStream_t s)
         if (S.shared_ff > 0) { t[nt].W = L.sh_down.ptr; t[nt].x = act + (size_t)S.top * S.ff; t[nt++].K = S.shared_ff; }
     }
     NT_CHECK(cur <= sandwich_scratch_width(), "sandwich_ff_token: scratch overrun");
-    gemv_sum(y, t, nt, cfg_.hidden_size, dt, false, s);
+    gemv_sum(y, t, nt, cfg_.hidden_size, L.wo.dtype, false, s);
 }
 
 // ---- prompt rows ----
@@ -326,7 +325,7 @@ void Model::sandwich_mixer_rows(int i, int T, int p0, float* y, cudaStream_t s) 
     const LayerSpec& S = cfg_.layers[(size_t)i];
     LayerWeights& L = layers_[(size_t)i];
     const float eps = cfg_.norm_eps;
-    const size_t H = (size_t)S.heads, G = (size_t)S.kv_heads, D = (size_t)S.dim, V = (size_t)S.vdim;
+    const size_t H = (size_t)S.heads, V = (size_t)S.vdim;
     size_t cur = 0;
     auto take = [&](size_t n) { float* p = pf_.wide + cur; cur += up4(n * (size_t)T); return p; };
     // rows . w^T; a short matrix goes through its padded copy, whose product has rows of ld = Weight::tc_rows numbers
@@ -410,7 +409,6 @@ void Model::sandwich_mixer_rows(int i, int T, int p0, float* y, cudaStream_t s) 
         else if (o_tc) split_activations(pf_.ws, o, T, (int)(H * V), s, true);
     }
     NT_CHECK(cur <= sandwich_scratch_width() * (size_t)T, "sandwich_mixer_rows: scratch rows overrun");
-    (void)D; (void)G;
     spec_gemm(y, o, o_tc ? pf_.ws : nullptr, L.wo, T, DENSE_STORE, nullptr, 1.f, s);
 }
 
